@@ -51,6 +51,9 @@ def load_hf_config(model_path: str, trust_remote_code: bool = False, revision: s
         d = AutoConfig.from_pretrained(model_path, trust_remote_code=trust_remote_code, revision=revision).to_dict()
     if override:
         d.update(override)
+    if isinstance(d.get("architecture"), str) and "architectures" not in d:
+        from .native_formats import translate_native_config
+        d = translate_native_config(d)
     cfg = ConfigNS(**d)
     tc = d.get("text_config")
     if isinstance(tc, dict):
@@ -106,8 +109,9 @@ class ModelConfig:
         self.head_dim = getattr(c, "head_dim", None) or c.hidden_size // c.num_attention_heads
         self.vocab_size = c.vocab_size
         self.attention_arch = AttentionArch.MHA
-        if getattr(c, "kv_lora_rank", None) and any("Deepseek" in a or "DeepSeek" in a or "Kimi" in a or "Glm5" in a or "GlmMoeDsa" in a
-                                                    for a in self.architectures):
+        if getattr(c, "latent_kv_cache", False) or (
+                getattr(c, "kv_lora_rank", None) and any("Deepseek" in a or "DeepSeek" in a or "Kimi" in a or "Glm5" in a
+                                                         or "GlmMoeDsa" in a for a in self.architectures)):
             self.attention_arch = AttentionArch.MLA
             self.kv_lora_rank = c.kv_lora_rank
             self.qk_rope_head_dim = c.qk_rope_head_dim
@@ -120,7 +124,7 @@ class ModelConfig:
                 and rs.get("original_max_position_embeddings"):
             derived = max(derived, int(rs["original_max_position_embeddings"] * rs["factor"]))
         if context_length is not None:
-            if context_length > derived and not os.environ.get("SGLANG_ALLOW_OVERWRITE_LONGER_CONTEXT_LEN"):
+            if context_length > derived and not getattr(c, "unbounded_positions", False) and not os.environ.get("SGLANG_ALLOW_OVERWRITE_LONGER_CONTEXT_LEN"):
                 raise ValueError(f"context_length {context_length} exceeds the model's {derived}; set "
                                  f"SGLANG_ALLOW_OVERWRITE_LONGER_CONTEXT_LEN=1 to force")
             self.context_len = context_length

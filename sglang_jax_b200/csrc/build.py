@@ -21,10 +21,18 @@ OUT_DIR = os.path.join(os.path.dirname(HERE), "ops")
 # and skip the access.  It is a library of its own so the regular one stays as it is.
 CHECKED = os.environ.get("SGLB_BOUNDS_CHECK", "0") == "1"
 LIB_PATH = os.path.join(OUT_DIR, "libsglb200_checked.so" if CHECKED else "libsglb200.so")
-STAMP = LIB_PATH + ".stamp"
 
-NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
-              "--use_fast_math", "-Xcompiler", "-fPIC", "-shared"] + (["-DSGLB_BOUNDS_CHECK"] if CHECKED else [])
+NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++20",
+              "-Xcompiler", "-fPIC", "-shared"] + (["-DSGLB_BOUNDS_CHECK"] if CHECKED else [])
+# sources whose norms, exponentials and angles must be the accurate ones; the others take the fast-math substitutions
+ACCURATE = {"residual_stream.cu", "latent_attn.cu", "delta_scan.cu"}
+
+# what one model family launches outside sampling: enough for a library of its own, which a fresh checkout builds in a
+# few seconds (`ops/native.py: prefer_kernel_set`)
+KERNEL_SETS = {
+    "latent_delta": ["runtime.cu", "gemm_sm100.cu", "mla.cu", "latent_attn.cu", "latent_extend.cu", "delta_scan.cu",
+                     "residual_stream.cu"],
+}
 
 
 def _nvcc() -> str:
@@ -34,37 +42,52 @@ def _nvcc() -> str:
     raise RuntimeError("nvcc not found; set NVCC or add it to PATH")
 
 
-def sources() -> list[str]:
+def sources(kernel_set: str | None = None) -> list[str]:
+    if kernel_set is not None:
+        return [os.path.join(HERE, f) for f in KERNEL_SETS[kernel_set]]
     return sorted(glob.glob(os.path.join(HERE, "*.cu")))
 
 
-def _digest() -> str:
+def lib_path(kernel_set: str | None = None) -> str:
+    return LIB_PATH if kernel_set is None else LIB_PATH[:-3] + f"_{kernel_set}.so"
+
+
+def _flags(src: str) -> list[str]:
+    fast = [] if os.path.basename(src) in ACCURATE else ["--use_fast_math"]
+    return [f for f in NVCC_FLAGS if f != "-shared"] + fast
+
+
+def _digest(kernel_set: str | None = None) -> str:
     h = hashlib.sha256()
-    for f in sources() + sorted(glob.glob(os.path.join(HERE, "*.cuh"))) + sorted(glob.glob(os.path.join(HERE, "*.h"))):
-        h.update(f.encode())
+    headers = sorted(glob.glob(os.path.join(HERE, "*.cuh"))) + sorted(glob.glob(os.path.join(HERE, "*.h")))
+    for f in sources(kernel_set) + headers:
+        h.update(os.path.basename(f).encode())
         with open(f, "rb") as fh:
             h.update(fh.read())
-    h.update(" ".join(NVCC_FLAGS).encode())
+    h.update(" ".join(NVCC_FLAGS + sorted(ACCURATE)).encode())
     return h.hexdigest()
 
 
-def is_current() -> bool:
-    if not (os.path.exists(LIB_PATH) and os.path.exists(STAMP)):
+def is_current(kernel_set: str | None = None) -> bool:
+    path = lib_path(kernel_set)
+    if not (os.path.exists(path) and os.path.exists(path + ".stamp")):
         return False
-    with open(STAMP) as f:
-        return f.read().strip() == _digest()
+    with open(path + ".stamp") as f:
+        return f.read().strip() == _digest(kernel_set)
 
 
-def build(force: bool = False, verbose: bool = False) -> str:
-    if not force and is_current():
-        return LIB_PATH
+def build(force: bool = False, verbose: bool = False, kernel_set: str | None = None) -> str:
+    """Compile every source, or those of one kernel set, and link the library; returns its path."""
+    path = lib_path(kernel_set)
+    if not force and is_current(kernel_set):
+        return path
     objs = []
     tmp = os.path.join(HERE, "build_checked" if CHECKED else "build")
     os.makedirs(tmp, exist_ok=True)
     procs = []
-    for src in sources():
+    for src in sources(kernel_set):
         obj = os.path.join(tmp, os.path.basename(src)[:-3] + ".o")
-        cmd = [_nvcc(), *[f for f in NVCC_FLAGS if f != "-shared"], "-c", src, "-o", obj, "-I", HERE]
+        cmd = [_nvcc(), *_flags(src), "-c", src, "-o", obj, "-I", HERE]
         if verbose:
             cmd += ["-Xptxas", "-v"]
         procs.append((src, subprocess.Popen(cmd, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True)))
@@ -75,13 +98,15 @@ def build(force: bool = False, verbose: bool = False) -> str:
             print(out)
         if p.returncode != 0:
             raise RuntimeError(f"nvcc failed for {src}:\n{out}")
-    link = [_nvcc(), "-shared", "-o", LIB_PATH, *objs, "-gencode", "arch=compute_100a,code=sm_100a"]
+    part = f"{path}.{os.getpid()}"
+    link = [_nvcc(), "-shared", "-o", part, *objs, "-gencode", "arch=compute_100a,code=sm_100a"]
     r = subprocess.run(link, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True)
     if r.returncode != 0:
         raise RuntimeError(f"link failed:\n{r.stdout}")
-    with open(STAMP, "w") as f:
-        f.write(_digest())
-    return LIB_PATH
+    os.replace(part, path)
+    with open(path + ".stamp", "w") as f:
+        f.write(_digest(kernel_set))
+    return path
 
 
 if __name__ == "__main__":

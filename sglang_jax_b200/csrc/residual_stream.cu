@@ -1,0 +1,301 @@
+// Ops around a residual stream that is kept in 32-bit floats while the projections run in the model's type T (bf16, or
+// fp32 throughout).  A sublayer reads the stream itself, in T; its result is normalised, scaled per channel and added
+// back:
+//
+//   embed_scaled       x = table[id] * scale                          -> x (fp32), x in T
+//   postnorm_add       x <- x + s * y / sqrt(mean(y^2) + eps)         -> x (fp32, in place), x in T
+//                      (s, fp32 per channel, holds norm weight, layer scale and residual multiplier)
+//   rmsnorm_stream     y = x / sqrt(mean(x^2) + eps) * w              -> y in T
+//   gelu_mul           gelu_tanh(a) * b of a fused [a | b] projection
+//   sigmoid_gate       o * sigmoid(g), g a column range of a wider projection
+//
+// One CTA per row for the norms, the row in registers between its two passes.  This file is compiled without fast-math
+// substitutions: the statistics, exponentials and hyperbolic tangents are the accurate ones.
+#include "common.cuh"
+
+namespace sglb {
+namespace {
+
+// VEC consecutive elements (VEC = 4: 8 / 16 bytes, VEC = 1: any alignment)
+template <int VEC> __device__ __forceinline__ void load_v(const float* p, float (&f)[VEC]) {
+  if constexpr (VEC == 4) {
+    const float4 v = *reinterpret_cast<const float4*>(p);
+    f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+  } else {
+    f[0] = *p;
+  }
+}
+template <int VEC> __device__ __forceinline__ void load_v(const __nv_bfloat16* p, float (&f)[VEC]) {
+  if constexpr (VEC == 4) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.y));
+    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+  } else {
+    f[0] = __bfloat162float(*p);
+  }
+}
+template <int VEC> __device__ __forceinline__ void store_v(float* p, const float (&f)[VEC]) {
+  if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  else *p = f[0];
+}
+template <int VEC> __device__ __forceinline__ void store_v(__nv_bfloat16* p, const float (&f)[VEC]) {
+  if constexpr (VEC == 4) *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]));
+  else *p = __float2bfloat16(f[0]);
+}
+
+__device__ __forceinline__ float block_sum(float v, float* red) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  const int w = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  if ((threadIdx.x & 31) == 0) red[w] = v;
+  __syncthreads();
+  float t = 0.f;
+  for (int i = 0; i < nw; ++i) t += red[i];          // same order in every thread
+  return t;
+}
+
+template <typename T, int VEC>
+__global__ void embed_scaled_kernel(float* __restrict__ x, T* __restrict__ xt, const int* __restrict__ ids,
+                                    const T* __restrict__ table, int W, int rows, float scale) {
+  pdl_wait();
+  const size_t t = blockIdx.x;
+  const int id = min(max(ids[t], 0), rows - 1);
+  const T* src = table + static_cast<size_t>(id) * W;
+  for (int i = threadIdx.x * VEC; i < W; i += blockDim.x * VEC) {
+    float f[VEC];
+    load_v<VEC>(src + i, f);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) f[e] *= scale;
+    store_v<VEC>(x + t * W + i, f);
+    if (xt != nullptr) store_v<VEC>(xt + t * W + i, f);
+  }
+}
+
+template <typename T, int VEC, int VPT>
+__global__ void postnorm_add_kernel(float* __restrict__ x, T* __restrict__ xt, const T* __restrict__ y,
+                                    const float* __restrict__ s, int W, float eps) {
+  __shared__ float red[32];
+  pdl_wait();
+  const size_t row = static_cast<size_t>(blockIdx.x) * W;
+  float v[VPT][VEC];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * VEC;
+    if (c < W) {
+      load_v<VEC>(y + row + c, v[i]);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) ss += v[i][e] * v[i][e];
+    }
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / W + eps);
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * VEC;
+    if (c < W) {
+      float xv[VEC], sv[VEC];
+      load_v<VEC>(x + row + c, xv);
+      load_v<VEC>(s + c, sv);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) xv[e] += v[i][e] * inv * sv[e];
+      store_v<VEC>(x + row + c, xv);
+      if (xt != nullptr) store_v<VEC>(xt + row + c, xv);
+    }
+  }
+}
+
+template <typename T, int VEC, int VPT>
+__global__ void rmsnorm_stream_kernel(T* __restrict__ y, const float* __restrict__ x, const float* __restrict__ w, int W,
+                                      float eps) {
+  __shared__ float red[32];
+  pdl_wait();
+  const size_t row = static_cast<size_t>(blockIdx.x) * W;
+  float v[VPT][VEC];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * VEC;
+    if (c < W) {
+      load_v<VEC>(x + row + c, v[i]);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) ss += v[i][e] * v[i][e];
+    }
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / W + eps);
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * VEC;
+    if (c < W) {
+      float wv[VEC];
+      load_v<VEC>(w + c, wv);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v[i][e] *= inv * wv[e];
+      store_v<VEC>(y + row + c, v[i]);
+    }
+  }
+}
+
+__device__ __forceinline__ float gelu_tanh(float z) {
+  return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+
+template <typename T, int VEC>
+__global__ void gelu_mul_kernel(T* __restrict__ out, const T* __restrict__ in, long long rows, int F) {
+  pdl_wait();
+  const long long per = F / VEC, total = rows * per;
+  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < total;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long r = i / per;
+    const int c = static_cast<int>(i - r * per) * VEC;
+    float a[VEC], b[VEC];
+    load_v<VEC>(in + r * 2 * F + c, a);
+    load_v<VEC>(in + r * 2 * F + F + c, b);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) a[e] = gelu_tanh(a[e]) * b[e];
+    store_v<VEC>(out + r * F + c, a);
+  }
+}
+
+template <typename T, int VEC>
+__global__ void sigmoid_gate_kernel(T* __restrict__ out, const T* __restrict__ o, const T* __restrict__ g,
+                                    long long g_stride, long long rows, int F) {
+  pdl_wait();
+  const long long per = F / VEC, total = rows * per;
+  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < total;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long r = i / per;
+    const int c = static_cast<int>(i - r * per) * VEC;
+    float a[VEC], b[VEC];
+    load_v<VEC>(o + r * F + c, a);
+    load_v<VEC>(g + r * g_stride + c, b);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) a[e] = a[e] / (1.f + expf(-b[e]));
+    store_v<VEC>(out + r * F + c, a);
+  }
+}
+
+int row_threads(int groups) {
+  const int t = ((groups + 31) / 32) * 32;
+  return t > 1024 ? 1024 : t;
+}
+int grid_for(long long items) {
+  const long long b = (items + 255) / 256;
+  return static_cast<int>(b < 148LL * 16 ? b : 148LL * 16);
+}
+
+// Calls f.template operator()<VEC, VPT>() for a row of W elements; false when the row is too wide.
+template <typename F>
+bool for_row(int W, bool vec, int* threads, F&& f) {
+  const int groups = vec ? W / 4 : W;
+  *threads = row_threads(groups);
+  const int vpt = (groups + *threads - 1) / *threads;
+  if (vpt > 16) return false;
+  if (vec) {
+    if (vpt <= 1) f.template operator()<4, 1>();
+    else if (vpt <= 2) f.template operator()<4, 2>();
+    else if (vpt <= 4) f.template operator()<4, 4>();
+    else f.template operator()<4, 16>();
+  } else {
+    if (vpt <= 1) f.template operator()<1, 1>();
+    else if (vpt <= 4) f.template operator()<1, 4>();
+    else f.template operator()<1, 16>();
+  }
+  return true;
+}
+
+template <typename T>
+int embed_scaled(float* x, void* xt, const int* ids, const void* table, long long n, int W, int rows, float scale,
+                 cudaStream_t s) {
+  T* o = static_cast<T*>(xt);
+  const T* tb = static_cast<const T*>(table);
+  if (W % 4 == 0)
+    launch_pdl(embed_scaled_kernel<T, 4>, dim3(n), dim3(row_threads(W / 4) < 256 ? row_threads(W / 4) : 256), 0, s, x, o,
+               ids, tb, W, rows, scale);
+  else
+    launch_pdl(embed_scaled_kernel<T, 1>, dim3(n), dim3(row_threads(W) < 256 ? row_threads(W) : 256), 0, s, x, o, ids, tb,
+               W, rows, scale);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T>
+int postnorm_add(float* x, void* xt, const void* y, const float* sc, long long n, int W, float eps, cudaStream_t s) {
+  int threads = 0;
+  const bool ok = for_row(W, W % 4 == 0, &threads, [&]<int VEC, int VPT>() {
+    launch_pdl(postnorm_add_kernel<T, VEC, VPT>, dim3(n), dim3(threads), 0, s, x, static_cast<T*>(xt),
+               static_cast<const T*>(y), sc, W, eps);
+  });
+  return ok ? static_cast<int>(cudaGetLastError()) : -kBadArgument;
+}
+
+template <typename T>
+int rmsnorm_stream(void* y, const float* x, const float* w, long long n, int W, float eps, cudaStream_t s) {
+  int threads = 0;
+  const bool ok = for_row(W, W % 4 == 0, &threads, [&]<int VEC, int VPT>() {
+    launch_pdl(rmsnorm_stream_kernel<T, VEC, VPT>, dim3(n), dim3(threads), 0, s, static_cast<T*>(y), x, w, W, eps);
+  });
+  return ok ? static_cast<int>(cudaGetLastError()) : -kBadArgument;
+}
+
+template <typename T>
+int gelu_mul(void* out, const void* in, long long rows, int F, cudaStream_t s) {
+  T* o = static_cast<T*>(out);
+  const T* i = static_cast<const T*>(in);
+  if (F % 4 == 0) launch_pdl(gelu_mul_kernel<T, 4>, dim3(grid_for(rows * (F / 4))), dim3(256), 0, s, o, i, rows, F);
+  else launch_pdl(gelu_mul_kernel<T, 1>, dim3(grid_for(rows * F)), dim3(256), 0, s, o, i, rows, F);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T>
+int sigmoid_gate(void* out, const void* o, const void* g, long long g_stride, long long rows, int F, cudaStream_t s) {
+  T* d = static_cast<T*>(out);
+  const T* a = static_cast<const T*>(o);
+  const T* b = static_cast<const T*>(g);
+  const bool vec = F % 4 == 0 && g_stride % 4 == 0 && reinterpret_cast<uintptr_t>(g) % (4 * sizeof(T)) == 0;
+  if (vec)
+    launch_pdl(sigmoid_gate_kernel<T, 4>, dim3(grid_for(rows * (F / 4))), dim3(256), 0, s, d, a, b, g_stride, rows, F);
+  else
+    launch_pdl(sigmoid_gate_kernel<T, 1>, dim3(grid_for(rows * F)), dim3(256), 0, s, d, a, b, g_stride, rows, F);
+  return static_cast<int>(cudaGetLastError());
+}
+
+}  // namespace
+}  // namespace sglb
+
+extern "C" {
+
+// `is_f32`: T is fp32 (then `xt` is null, the fp32 stream itself is the projections' input), else bf16.
+int sglb_embed_scaled(float* x, void* xt, const int* ids, const void* table, long long n, int W, int rows, float scale,
+                      int is_f32, cudaStream_t s) {
+  if (n <= 0) return 0;
+  return is_f32 ? sglb::embed_scaled<float>(x, xt, ids, table, n, W, rows, scale, s)
+                : sglb::embed_scaled<__nv_bfloat16>(x, xt, ids, table, n, W, rows, scale, s);
+}
+
+int sglb_postnorm_add(float* x, void* xt, const void* y, const float* scale, long long n, int W, float eps, int is_f32,
+                      cudaStream_t s) {
+  if (n <= 0) return 0;
+  return is_f32 ? sglb::postnorm_add<float>(x, xt, y, scale, n, W, eps, s)
+                : sglb::postnorm_add<__nv_bfloat16>(x, xt, y, scale, n, W, eps, s);
+}
+
+int sglb_rmsnorm_stream(void* y, const float* x, const float* w, long long n, int W, float eps, int is_f32,
+                        cudaStream_t s) {
+  if (n <= 0) return 0;
+  return is_f32 ? sglb::rmsnorm_stream<float>(y, x, w, n, W, eps, s)
+                : sglb::rmsnorm_stream<__nv_bfloat16>(y, x, w, n, W, eps, s);
+}
+
+int sglb_gelu_tanh_and_mul(void* out, const void* in, long long rows, int F, int is_f32, cudaStream_t s) {
+  if (rows <= 0) return 0;
+  return is_f32 ? sglb::gelu_mul<float>(out, in, rows, F, s) : sglb::gelu_mul<__nv_bfloat16>(out, in, rows, F, s);
+}
+
+int sglb_sigmoid_gate(void* out, const void* o, const void* g, long long g_stride, long long rows, int F, int is_f32,
+                      cudaStream_t s) {
+  if (rows <= 0) return 0;
+  return is_f32 ? sglb::sigmoid_gate<float>(out, o, g, g_stride, rows, F, s)
+                : sglb::sigmoid_gate<__nv_bfloat16>(out, o, g, g_stride, rows, F, s);
+}
+
+}  // extern "C"

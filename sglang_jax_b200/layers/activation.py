@@ -2,7 +2,6 @@
 from torch import nn
 
 from .. import ops
-from ..ops import reference
 
 
 class SiluAndMul(nn.Module):
@@ -16,4 +15,4 @@ class GeluAndMul(nn.Module):
         self.approximate = approximate
 
     def forward(self, x):
-        return reference.gelu_and_mul(x, self.approximate)
+        return ops.gelu_and_mul(x, self.approximate)

@@ -247,7 +247,7 @@ def get_rope(head_size, rotary_dim, max_position, base, is_neox_style=True, rope
              dtype=torch.bfloat16, partial_rotary_factor: float = 1.0) -> RotaryEmbedding:
     if partial_rotary_factor < 1.0 and not (rope_scaling or {}).get("proportional"):
         rotary_dim = int(rotary_dim * partial_rotary_factor)
-    key = (head_size, rotary_dim, max_position, base, is_neox_style,
+    key = (str(torch.empty(0).device), head_size, rotary_dim, max_position, base, is_neox_style,
            tuple(sorted((k, str(v)) for k, v in (rope_scaling or {}).items())), partial_rotary_factor)
     if key in _ROPE_CACHE:
         return _ROPE_CACHE[key]

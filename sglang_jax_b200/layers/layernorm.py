@@ -68,3 +68,47 @@ class GatedRMSNorm(nn.Module):
         xf = x.float()
         y = xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + self.eps) * self.weight.float()
         return (y * torch.nn.functional.silu(gate.float())).to(x.dtype)
+
+
+class PostNormResidual(nn.Module):
+    """`x <- x + multiplier * layer_scale * rmsnorm(y) * weight` on an fp32 residual stream, y a sublayer's output.
+    Returns x in y's type, the input of the next projections.  The three factors are folded into one fp32 vector
+    (`fold()`, after loading)."""
+
+    def __init__(self, hidden_size: int, eps: float, multiplier: float = 1.0, layer_scale: bool = False,
+                 dtype=torch.bfloat16):
+        super().__init__()
+        self.weight = nn.Parameter(torch.ones(hidden_size, dtype=dtype), requires_grad=False)
+        self.layer_scale = nn.Parameter(torch.ones(hidden_size, dtype=dtype), requires_grad=False) if layer_scale else None
+        self.eps, self.multiplier = eps, multiplier
+        self.register_buffer("channel_scale", torch.ones(hidden_size, dtype=torch.float32), persistent=False)
+
+    def fold(self):
+        s = self.weight.float() * self.multiplier
+        self.channel_scale.copy_(s if self.layer_scale is None else s * self.layer_scale.float())
+
+    def weight_loader(self, param, w, shard_id=None):
+        param.data.copy_(w)
+
+    def forward(self, y: torch.Tensor, x: torch.Tensor) -> torch.Tensor:
+        return ops.postnorm_add(y, x, self.channel_scale, self.eps)
+
+
+class StreamRMSNorm(nn.Module):
+    """RMSNorm of an fp32 residual stream, result in the model's type.  `multiplier` scales the result (a logit scale
+    in front of a linear head)."""
+
+    def __init__(self, hidden_size: int, eps: float, multiplier: float = 1.0, dtype=torch.bfloat16):
+        super().__init__()
+        self.weight = nn.Parameter(torch.ones(hidden_size, dtype=dtype), requires_grad=False)
+        self.eps, self.multiplier = eps, multiplier
+        self.register_buffer("channel_scale", torch.ones(hidden_size, dtype=torch.float32), persistent=False)
+
+    def fold(self):
+        self.channel_scale.copy_(self.weight.float() * self.multiplier)
+
+    def weight_loader(self, param, w, shard_id=None):
+        param.data.copy_(w)
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        return ops.rmsnorm_stream(x, self.channel_scale, self.eps, self.weight.dtype)

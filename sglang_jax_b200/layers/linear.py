@@ -98,6 +98,39 @@ class MergedColumnParallelLinear(LinearBase):
         param.data.narrow(0, off, loc).copy_(w.narrow(0, self.tp_rank * loc, loc))
 
 
+class PackedColumnParallelLinear(LinearBase):
+    """Any number of projections of one input as a single GEMM.  `parts`: name -> (output rows, split over the tensor
+    ranks?); parts that are not split are replicated.  Every part starts on a multiple of `ALIGN` output columns (zero
+    rows in between), so that the parts of an output row keep 16-byte alignment whatever their sizes."""
+
+    ALIGN = 8
+
+    def __init__(self, in_features, parts: dict[str, tuple[int, bool]], dtype=torch.bfloat16, tp_size=None, tp_rank=None):
+        self.tp_size = tp_size if tp_size is not None else ps.tp_size()
+        self.tp_rank = tp_rank if tp_rank is not None else ps.tp_rank()
+        self.parts: dict[str, tuple[int, int, bool]] = {}            # name -> (first column, columns, split?)
+        off = 0
+        for name, (rows, split) in parts.items():
+            assert not split or rows % self.tp_size == 0, f"{name}: {rows} rows do not split over {self.tp_size} ranks"
+            n = rows // self.tp_size if split else rows
+            self.parts[name] = (off, n, split)
+            off += -(-n // self.ALIGN) * self.ALIGN
+        super().__init__(in_features, off, False, dtype)
+        self.weight.data.zero_()
+
+    def offset(self, name: str) -> int:
+        return self.parts[name][0]
+
+    def part(self, y: torch.Tensor, name: str) -> torch.Tensor:
+        """The columns of one part in an output of this layer (a view)."""
+        off, n, _ = self.parts[name]
+        return y[:, off:off + n]
+
+    def weight_loader(self, param, w, shard_id: str):
+        off, n, split = self.parts[shard_id]
+        param.data.narrow(0, off, n).copy_(w.narrow(0, self.tp_rank * n if split else 0, n))
+
+
 class QKVParallelLinear(LinearBase):
     """Fused q/k/v projection.  Query heads are split over ranks; KV heads are split
     when `tp <= kv_heads` and replicated otherwise (reference

@@ -11,9 +11,11 @@ from __future__ import annotations
 import torch
 from torch import nn
 
+from .. import ops
 from ..ops import linear_attention as la
+from ..parallel import state as ps
 from .layernorm import GatedRMSNorm
-from .linear import ReplicatedLinear
+from .linear import PackedColumnParallelLinear, ReplicatedLinear, RowParallelLinear
 
 
 def track_pieces(a0: int, a1: int, track):
@@ -139,6 +141,87 @@ class GatedDeltaNet(nn.Module):
                         rec_all[snap] = rec_all[sl[i]]
         out = self.norm(o.reshape(-1, self.dv), z.reshape(-1, self.dv)).reshape(T, self.value_dim)
         return self.out_proj(out)
+
+
+class GatedDeltaRule(nn.Module):
+    """Gated delta rule with separate query / key head and value head counts, all sizes as parameters: short causal
+    convolution + SiLU on q, k and v, unit q and k vectors, one scalar decay and write strength per value head, RMSNorm
+    and SiLU gate per head on the read-out.  Prefill and decode are the same kernels (`csrc/delta_scan.cu`); everything
+    from the convolution's output to the norm is fp32."""
+
+    def __init__(self, hidden_size: int, heads: int, kv_heads: int, dim: int, v_dim: int, conv_kernel: int, eps: float,
+                 linear_layer_index: int, dtype):
+        super().__init__()
+        tp = ps.tp_size()
+        assert heads % kv_heads == 0 and kv_heads % tp == 0, f"{kv_heads} query/key heads do not split over {tp} ranks"
+        self.layer_index = linear_layer_index
+        self.nv, self.nk, self.dk, self.dv = heads // tp, kv_heads // tp, dim, v_dim
+        self.conv_kernel, self.eps = conv_kernel, float(eps)
+        self.key_dim, self.value_dim = self.nk * dim, self.nv * v_dim
+        self.conv_dim = 2 * self.key_dim + self.value_dim
+        # q, k and v columns stay adjacent (the kernels take them as one run of channels), hence one part
+        self.proj = PackedColumnParallelLinear(hidden_size, {"qkv": (self.conv_dim, False), "g": (heads * v_dim, True),
+                                                             "b": (heads, True), "a": (heads, True)}, dtype)
+        self.conv_weight = nn.Parameter(torch.empty(self.conv_dim, conv_kernel, dtype=dtype), requires_grad=False)
+        self.A_log = nn.Parameter(torch.zeros(self.nv, dtype=torch.float32), requires_grad=False)
+        self.dt_bias = nn.Parameter(torch.zeros(self.nv, dtype=torch.float32), requires_grad=False)
+        self.norm_weight = nn.Parameter(torch.ones(v_dim, dtype=torch.float32), requires_grad=False)
+        self.o_proj = RowParallelLinear(heads * v_dim, hidden_size, False, dtype)
+
+    def state_spec(self) -> dict:
+        return dict(conv_dim=self.conv_dim, conv_kernel=self.conv_kernel, num_heads=self.nv, head_k_dim=self.dk,
+                    head_v_dim=self.dv)
+
+    def load(self, name: str, w: torch.Tensor):
+        """One checkpoint tensor: q, k, v (projections), their `.conv` kernels, g, b, a, A_log, dt_bias, norm, o."""
+        r = ps.tp_rank()
+        base, conv = (name[:-5], True) if name.endswith(".conv") else (name, False)
+        if base in ("q", "k", "v"):
+            off = {"q": 0, "k": self.key_dim, "v": 2 * self.key_dim}[base]
+            n = self.value_dim if base == "v" else self.key_dim
+            dst = self.conv_weight if conv else self.proj.weight
+            dst.data.narrow(0, off, n).copy_(w.narrow(0, r * n, n))
+        elif name in ("g", "b", "a"):
+            self.proj.weight_loader(self.proj.weight, w, name)
+        elif name == "o":
+            self.o_proj.weight_loader(self.o_proj.weight, w)
+        elif name == "norm":
+            self.norm_weight.data.copy_(w)
+        elif name in ("A_log", "dt_bias"):
+            getattr(self, name).data.copy_(w.narrow(0, r * self.nv, self.nv))
+        else:
+            raise KeyError(name)
+
+    def forward(self, h: torch.Tensor, fb) -> torch.Tensor:
+        pool = fb.extras["recurrent_pool"]
+        y = self.proj(h)
+        ragged = {}
+        if not fb.forward_mode.is_decode():
+            ragged = dict(cu=fb.cu_q_lens, prefix=fb.extend_prefix_lens)
+            track = checkpoint_tensors(fb)
+            if track is not None:
+                ragged.update(track_len=track[0], track_slot=track[1])
+        o = ops.delta_scan(y, self.proj.offset("g"), self.proj.offset("b"), self.proj.offset("a"), self.conv_weight,
+                           self.A_log, self.dt_bias, pool.conv_state[self.layer_index],
+                           pool.recurrent_state[self.layer_index], recurrent_slots(fb), self.nv, self.nk, self.dk, self.dv,
+                           **ragged)
+        return self.o_proj(ops.delta_gate(o, self.proj.part(y, "g"), self.norm_weight, self.eps))
+
+
+def checkpoint_tensors(fb):
+    """The step's prefix-cache checkpoints as `(tokens before it, slot)` int32 device tensors `[B]` (0 tokens: none);
+    None when no sequence has one."""
+    tracks = fb.extras.get("recurrent_tracks")
+    if not tracks:
+        return None
+    t = fb.extras.get("recurrent_track_tensors")
+    if t is None:
+        host = torch.zeros(2, fb.batch_size, dtype=torch.int32)
+        for i, (k, slot) in tracks.items():
+            host[0, i], host[1, i] = k, slot
+        dev = host.to(fb.positions.device)
+        t = fb.extras["recurrent_track_tensors"] = (dev[0], dev[1])
+    return t
 
 
 class _RecurrentMixer(nn.Module):

@@ -441,6 +441,8 @@ class ModelWorkerBatch:
     # (index of the sequence in the batch, tokens of this extend before the checkpoint, snapshot slot): the
     # linear-attention layers store their state after that many tokens of the sequence into the slot
     recurrent_tracks: list | None = None
+    # extend steps: rows of the flattened batch whose logits are wanted instead of every sequence's last row
+    logits_rows: np.ndarray | None = None
 
     @property
     def batch_size(self):

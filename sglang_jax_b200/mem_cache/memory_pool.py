@@ -285,18 +285,18 @@ class MLATokenToKVPool(KVCache):
     """Latent cache for absorbed MLA: per layer ``[num_pages, page_size, kv_lora_rank + rope_dim]``
     (reference `memory_pool.py:1209-1473`; there both parts are padded to 128 lanes
     for the TPU, here 512+64 = 576 bf16 = 1152 bytes per token is already 16-byte
-    aligned so no padding is needed)."""
+    aligned so no padding is needed).  `layer_dims`: `(kv_lora_rank, rope_dim)` of every layer for models whose
+    layers differ; their rows are padded to whole 16-byte units."""
 
     def __init__(self, size, page_size, dtype, kv_lora_rank, qk_rope_head_dim, layer_num, device,
-                 start_layer: int = 0, index_head_dim: int = 0):
+                 start_layer: int = 0, index_head_dim: int = 0, layer_dims: list[tuple[int, int]] | None = None):
         super().__init__(size, page_size, dtype, layer_num, device, start_layer)
         self.kv_lora_rank = kv_lora_rank
         self.qk_rope_head_dim = qk_rope_head_dim
         self.kv_dim = kv_lora_rank + qk_rope_head_dim
-        self.kv_buffer = [
-            torch.zeros((self.num_pages, page_size, self.kv_dim), dtype=dtype, device=device)
-            for _ in range(layer_num)
-        ]
+        self.layer_dims = list(layer_dims) if layer_dims is not None else [(kv_lora_rank, qk_rope_head_dim)] * layer_num
+        widths = [self.kv_dim] * layer_num if layer_dims is None else [self.row_width(r, p) for r, p in layer_dims]
+        self.kv_buffer = [torch.zeros((self.num_pages, page_size, w), dtype=dtype, device=device) for w in widths]
         # sparse-attention indexer keys (one `index_head_dim` row per token and layer), addressed
         # by the same slot ids as the latent rows
         self.index_head_dim = index_head_dim
@@ -306,7 +306,13 @@ class MLATokenToKVPool(KVCache):
         ] if index_head_dim else None
 
     @staticmethod
-    def cell_size(kv_lora_rank, qk_rope_head_dim, layer_num, dtype, index_head_dim: int = 0) -> int:
+    def row_width(kv_lora_rank, qk_rope_head_dim) -> int:
+        return -(-(kv_lora_rank + qk_rope_head_dim) // 8) * 8
+
+    @staticmethod
+    def cell_size(kv_lora_rank, qk_rope_head_dim, layer_num, dtype, index_head_dim: int = 0, layer_dims=None) -> int:
+        if layer_dims is not None:
+            return sum(MLATokenToKVPool.row_width(r, p) for r, p in layer_dims) * torch.finfo(dtype).bits // 8
         return (kv_lora_rank + qk_rope_head_dim + index_head_dim) * layer_num * torch.finfo(dtype).bits // 8
 
     def get_kv_size_bytes(self):
@@ -319,13 +325,14 @@ class MLATokenToKVPool(KVCache):
         return self.kv_buffer[layer_id - self.start_layer]
 
     def set_kv_buffer(self, layer_id, loc, kv_c: torch.Tensor, k_pe: torch.Tensor):
-        buf = self.get_kv_buffer(layer_id).view(-1, self.kv_dim)
-        buf[loc.long()] = torch.cat([kv_c, k_pe], dim=-1).to(self.dtype)
+        buf = self.get_kv_buffer(layer_id).flatten(0, 1)
+        rank, rope = self.layer_dims[layer_id - self.start_layer]
+        buf[loc.long(), :rank + rope] = torch.cat([kv_c, k_pe], dim=-1).to(self.dtype)
 
     def gather(self, layer_id, loc):
-        buf = self.get_kv_buffer(layer_id).view(-1, self.kv_dim)
-        rows = buf[loc.long()]
-        return rows[:, :self.kv_lora_rank], rows[:, self.kv_lora_rank:]
+        rows = self.get_kv_buffer(layer_id).flatten(0, 1)[loc.long()]
+        rank, rope = self.layer_dims[layer_id - self.start_layer]
+        return rows[:, :rank], rows[:, rank:rank + rope]
 
 
 class HybridLinearKVPool(KVCache):

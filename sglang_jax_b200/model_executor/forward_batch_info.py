@@ -163,5 +163,7 @@ class ForwardBatch:
             fb.extend_seq_lens_cpu = np.asarray(batch.extend_seq_lens)
             fb.max_extend_len = int(batch.extend_seq_lens.max()) if B else 0
             fb.last_token_indices = (fb.cu_q_lens[1:] - 1).long()
+            if batch.logits_rows is not None:
+                fb.last_token_indices = torch.from_numpy(np.asarray(batch.logits_rows, np.int64)).to(runner.device)
             fb.extend_logprob_start_lens_cpu = batch.extend_logprob_start_lens
         return fb

@@ -27,6 +27,11 @@ def use_native(x: torch.Tensor) -> bool:
     return (not _FORCE_REFERENCE) and x.is_cuda and x.dtype == torch.bfloat16
 
 
+def use_native_wide(x: torch.Tensor) -> bool:
+    """Ops whose kernels exist for bf16 and for fp32."""
+    return (not _FORCE_REFERENCE) and x.is_cuda and x.dtype in (torch.bfloat16, torch.float32)
+
+
 def varlen_attention(q, k, v, seq_lens, scale: float):
     """Bidirectional attention over packed sequences (encoders, diffusion transformers)."""
     if use_native(q) and q.shape[-1] <= 128 and q.shape[1] % k.shape[1] == 0 and q.shape[1] // k.shape[1] <= 16 \
@@ -61,6 +66,84 @@ def silu_and_mul(x):
     if use_native(x):
         return _native().silu_and_mul(x)
     return reference.silu_and_mul(x)
+
+
+def gelu_and_mul(x, approximate="tanh"):
+    if approximate == "tanh" and use_native_wide(x):
+        return _native().gelu_tanh_and_mul(x)
+    return reference.gelu_and_mul(x, approximate)
+
+
+def sigmoid_gate(o, gate):
+    """`o * sigmoid(gate)`, `[T, F]` each."""
+    return (_native() if use_native_wide(o) else reference).sigmoid_gate(o, gate)
+
+
+# ---- residual stream in fp32 (projections in the model's type)
+def embed_scaled(ids, table, scale):
+    """`table[ids] * scale` as `(fp32 stream, the same in the table's type)`."""
+    return (_native() if use_native_wide(table) else reference).embed_scaled(ids, table, scale)
+
+
+def postnorm_add(y, x, channel_scale, eps):
+    """`x += channel_scale * y / rms(y)` in place on the fp32 stream; returns x in y's type."""
+    return (_native() if use_native_wide(y) else reference).postnorm_add(y, x, channel_scale, eps)
+
+
+def rmsnorm_stream(x, weight, eps, dtype):
+    """`x / rms(x) * weight` of the fp32 stream, in `dtype`."""
+    return (_native() if use_native_wide(x) else reference).rmsnorm_stream(x, weight, eps, dtype)
+
+
+# ---- gated delta rule (see `native.delta_scan`)
+def delta_scan(proj, *a, **kw):
+    return (_native() if use_native_wide(proj) else reference).delta_scan(proj, *a, **kw)
+
+
+def delta_gate(o, gate, weight, eps):
+    return (_native() if use_native_wide(gate) else reference).delta_gate(o, gate, weight, eps)
+
+
+# ---- latent attention (see `native.latent_prep`)
+def latent_prep(proj, *a, **kw):
+    return (_native() if use_native_wide(proj) else reference).latent_prep(proj, *a, **kw)
+
+
+def latent_attention(q_lat, q_pe, cache, fb, scale, rows=None, lens=None):
+    """Absorbed attention of every query token over the cache rows it sees: `q_lat [T, H, R]`, `q_pe [T, H, rot]`,
+    `cache [pages, P, >= R + rot]` -> `[T, H, R]`.  `rows`, `lens` (int32 `[T]`): page-table row and number of visible
+    tokens of each query; None = the step's own tokens."""
+    R = q_lat.shape[-1]
+    if not use_native_wide(q_lat):
+        assert rows is None
+        decode = fb.forward_mode.is_decode()
+        return reference.mla_paged_attention(q_lat, q_pe, cache[..., :R + q_pe.shape[-1]], fb.page_table,
+                                             fb.req_pool_indices, fb.seq_lens, fb.page_size, scale, R,
+                                             None if decode else fb.cu_q_lens, None if decode else fb.extend_prefix_lens)
+    native = _native()
+    if rows is None:
+        if fb.forward_mode.is_decode():
+            rows, lens = fb.req_pool_indices, fb.seq_lens
+        else:
+            from ..layers.latent_attention import extend_plan
+            plan = extend_plan(fb, False)
+            rows, lens = plan.token_rows, plan.token_lens
+    if native.mla_decode_supported(q_lat, q_pe, cache, R, fb.page_size):
+        return native.mla_decode(q_lat, q_pe, cache, fb.page_table, rows, lens, fb.page_size, scale, fb.max_seq_len,
+                                 exact=True)
+    return native.latent_attn_any(q_lat, q_pe, cache, fb.page_table, rows, lens, fb.page_size, scale)
+
+
+def latent_extend_supported(q, dim, rot, v_dim, rank) -> bool:
+    return use_native(q) and _native().latent_extend_supported(q, dim, rot, v_dim, rank)
+
+
+def latent_gather(*a):
+    return _native().latent_gather(*a)
+
+
+def latent_extend(*a):
+    return _native().latent_extend(*a)
 
 
 def linear(x, w, bias=None):

@@ -21,74 +21,104 @@ _LIB_PATH = os.path.join(os.path.dirname(os.path.abspath(__file__)),
                          "libsglb200_checked.so" if os.environ.get("SGLB_BOUNDS_CHECK", "0") == "1"
                          else "libsglb200.so")
 LOADED = False
+_KERNEL_SET = None        # see `prefer_kernel_set`
+
+
+def prefer_kernel_set(name: str | None):
+    """When the library has not been built yet, let the first use build only the named kernel set of
+    `csrc/build.py: KERNEL_SETS` (what one model family launches) instead of everything."""
+    global _KERNEL_SET
+    _KERNEL_SET = name
 
 
 def lib():
     global _LIB, LOADED
     if _LIB is not None:
         return _LIB
-    if not os.path.exists(_LIB_PATH):
+    path = _LIB_PATH
+    if not os.path.exists(path):
         # source checkout on a box with nvcc: build on first use
         try:
             from ..csrc.build import build
-            build()
+            path = build(kernel_set=_KERNEL_SET)
         except Exception as e:
             raise RuntimeError(
                 f"native kernel library {_LIB_PATH} is missing and could not be built ({e}); "
                 f"run `python -m sglang_jax_b200.csrc.build`") from e
-    L = ctypes.CDLL(_LIB_PATH)
+    L = ctypes.CDLL(path)
+
+    def sig(name, argtypes):
+        f = getattr(L, name, None)            # a library with one kernel set lacks the other families' functions
+        if f is not None:
+            f.argtypes = argtypes
+
     L.sglb_version.restype = ctypes.c_char_p
-    L.sglb_gemm_decode_cluster.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]
-    L.sglb_gemm_decode_cluster_size.argtypes = [c_int, c_int, c_int]
-    L.sglb_enable_peer_access.argtypes = [c_int, c_int]
-    if hasattr(L, "sglb_debug_set_kv_pages"):
-        L.sglb_debug_set_kv_pages.argtypes = [c_int]
+    sig("sglb_gemm_decode_cluster", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p])
+    sig("sglb_gemm_decode_cluster_size", [c_int, c_int, c_int])
+    sig("sglb_enable_peer_access", [c_int, c_int])
+    sig("sglb_debug_set_kv_pages", [c_int])
     L.sglb_gemm_workspace_bytes.restype = c_size_t
-    L.sglb_gemm_workspace_bytes.argtypes = [c_int, c_int, c_int]
-    L.sglb_gemm_max_counters.argtypes = [c_int]
-    L.sglb_gemm_bf16.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_size_t,
-                                 c_void_p, c_int, c_int, c_void_p]
-    L.sglb_rmsnorm.argtypes = [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_float, c_int, c_void_p]
-    L.sglb_fused_add_rmsnorm.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_float, c_int,
-                                         c_void_p]
-    L.sglb_silu_and_mul.argtypes = [c_void_p, c_void_p, c_longlong, c_int, c_void_p]
-    L.sglb_embedding.argtypes = [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_void_p]
-    L.sglb_argmax.argtypes = [c_void_p, c_void_p, c_int, c_int, c_longlong, c_int, c_void_p]
-    L.sglb_rope_qknorm_kvwrite.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float,
+    sig("sglb_gemm_workspace_bytes", [c_int, c_int, c_int])
+    sig("sglb_gemm_max_counters", [c_int])
+    sig("sglb_gemm_bf16", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_size_t,
+                                 c_void_p, c_int, c_int, c_void_p])
+    sig("sglb_rmsnorm", [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_float, c_int, c_void_p])
+    sig("sglb_fused_add_rmsnorm", [c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_float, c_int,
+                                         c_void_p])
+    sig("sglb_silu_and_mul", [c_void_p, c_void_p, c_longlong, c_int, c_void_p])
+    sig("sglb_embedding", [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_void_p])
+    sig("sglb_argmax", [c_void_p, c_void_p, c_int, c_int, c_longlong, c_int, c_void_p])
+    sig("sglb_rope_qknorm_kvwrite", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float,
                                            c_longlong, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int,
-                                           c_void_p]
-    L.sglb_page_table_scatter.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p]
-    L.sglb_resolve_future.argtypes = [c_void_p, c_void_p, c_int, c_void_p]
-    L.sglb_decode_num_splits.argtypes = [c_int, c_int, c_int]
-    L.sglb_gemm_fp8.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p,
-                                c_size_t, c_void_p, c_void_p]
-    L.sglb_sample_filtered.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_longlong, c_int, c_void_p, c_void_p,
-                                       c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p]
-    L.sglb_quant_fp8_rows.argtypes = [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_void_p, c_void_p]
-    L.sglb_delta_rule_step.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                                       c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]
-    L.sglb_conv1d_update.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                                     c_void_p]
-    L.sglb_mla_decode.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p,
-                                  c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_void_p]
-    L.sglb_paged_decode.argtypes = [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p,
+                                           c_void_p])
+    sig("sglb_page_table_scatter", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p])
+    sig("sglb_resolve_future", [c_void_p, c_void_p, c_int, c_void_p])
+    sig("sglb_decode_num_splits", [c_int, c_int, c_int])
+    sig("sglb_gemm_fp8", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p,
+                                c_size_t, c_void_p, c_void_p])
+    sig("sglb_sample_filtered", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_longlong, c_int, c_void_p, c_void_p,
+                                       c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p])
+    sig("sglb_quant_fp8_rows", [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_void_p, c_void_p])
+    sig("sglb_delta_rule_step", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                       c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
+    sig("sglb_conv1d_update", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
+                                     c_void_p])
+    sig("sglb_mla_decode", [c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_longlong, c_int, c_void_p,
+                            c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p,
+                            c_void_p, c_int, c_void_p])
+    sig("sglb_mla_num_splits", [c_int, c_int, c_int])
+    sig("sglb_embed_scaled", [c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_float, c_int, c_void_p])
+    sig("sglb_postnorm_add", [c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_float, c_int, c_void_p])
+    sig("sglb_rmsnorm_stream", [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_float, c_int, c_void_p])
+    sig("sglb_gelu_tanh_and_mul", [c_void_p, c_void_p, c_longlong, c_int, c_int, c_void_p])
+    sig("sglb_sigmoid_gate", [c_void_p, c_void_p, c_void_p, c_longlong, c_longlong, c_int, c_int, c_void_p])
+    sig("sglb_latent_prep", [c_void_p, c_longlong] + [c_int] * 7 + [c_void_p, c_float, c_void_p, c_void_p, c_void_p,
+                                                                    c_void_p, c_int, c_int, c_void_p])
+    sig("sglb_latent_attn_any", [c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p,
+                                 c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p])
+    sig("sglb_latent_gather", [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int,
+                               c_int, c_int, c_int, c_void_p])
+    sig("sglb_delta_scan", [c_void_p, c_longlong, c_int, c_int, c_int] + [c_void_p] * 15 + [c_int] * 8 + [c_void_p])
+    sig("sglb_delta_gate", [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_int, c_int, c_float, c_int,
+                            c_void_p])
+    sig("sglb_paged_decode", [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p,
                                     c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_float, c_int, c_void_p,
-                                    c_void_p, c_void_p]
-    L.sglb_paged_extend.argtypes = [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p,
+                                    c_void_p, c_void_p])
+    sig("sglb_paged_extend", [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p,
                                     c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int,
-                                    c_float, c_void_p]
-    L.sglb_paged_extend_masked.argtypes = [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p,
+                                    c_float, c_void_p])
+    sig("sglb_paged_extend_masked", [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p,
                                            c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                                           c_float, c_int, c_float, c_void_p, c_int, c_int, c_void_p]
-    L.sglb_verify_tree_greedy.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
-                                          c_int, c_void_p]
-    L.sglb_tree_mask.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p]
-    L.sglb_lora_shrink.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]
-    L.sglb_lora_expand.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                                   c_int, c_int, c_void_p]
-    L.sglb_kv_page_copy.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_longlong, c_longlong,
-                                    c_longlong, c_void_p]
-    L.sglb_read_status.argtypes = [c_void_p]
+                                           c_float, c_int, c_float, c_void_p, c_int, c_int, c_void_p])
+    sig("sglb_verify_tree_greedy", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                                          c_int, c_void_p])
+    sig("sglb_tree_mask", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p])
+    sig("sglb_lora_shrink", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p])
+    sig("sglb_lora_expand", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
+                                   c_int, c_int, c_void_p])
+    sig("sglb_kv_page_copy", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_longlong, c_longlong,
+                                    c_longlong, c_void_p])
+    sig("sglb_read_status", [c_void_p])
     _LIB = L
     LOADED = True
     return L
@@ -518,27 +548,160 @@ def conv1d_update(x, state_pool, weight, slots, silu=True):
 
 
 def mla_decode_supported(q_latent, q_pe, kv_buffer, kv_lora_rank, page_size) -> bool:
-    return (q_latent.dtype == torch.bfloat16 and kv_buffer.dtype == torch.bfloat16 and kv_lora_rank == 512
-            and q_pe.shape[-1] == 64 and kv_buffer.shape[-1] == 576
+    return (q_latent.dtype == torch.bfloat16 and kv_buffer.dtype == torch.bfloat16 and kv_lora_rank <= 512
+            and q_pe.shape[-1] <= 64 and q_pe.stride(-1) == 1 and kv_buffer.shape[-1] % 8 == 0
+            and kv_buffer.data_ptr() % 16 == 0
             and ((64 % page_size == 0) if page_size < 64 else (page_size % 64 == 0)))
 
 
 def mla_decode(q_latent, q_pe, kv_buffer, page_table, req_pool_indices, seq_lens, page_size, scale, max_seq_len=0,
-               num_splits=None):
-    """Absorbed-MLA decode: `q_latent [B, H, 512]`, `q_pe [B, H, 64]`, latent cache
-    `[pages, P, 576]` -> latent output `[B, H, 512]` (the caller applies W_UV)."""
+               num_splits=None, exact=False):
+    """Absorbed-MLA decode: `q_latent [B, H, R]`, `q_pe [B, H, rotary lanes]` (any strides, unit innermost), latent
+    cache `[pages, P, row]` with `row >= R + rotary lanes` -> latent output `[B, H, R]` (the caller applies W_UV).
+    `exact`: the attention weights enter the value product unrounded."""
     B, H, R = q_latent.shape
-    q_latent, q_pe = q_latent.contiguous(), q_pe.contiguous()
+    q_latent = q_latent.contiguous()
     out = torch.empty_like(q_latent)
     if num_splits is None:
-        num_splits = decode_num_splits(B, (H + 15) // 16, max_seq_len or page_table.shape[1] * page_size)
+        num_splits = lib().sglb_mla_num_splits(B, (H + 15) // 16, max(max_seq_len or page_table.shape[1] * page_size, 1))
     part_o = part_lse = None
     if num_splits > 1:
         part_o = torch.empty((B, H, num_splits, R), dtype=torch.float32, device=q_latent.device)
         part_lse = torch.empty((B, H, num_splits), dtype=torch.float32, device=q_latent.device)
-    _check(lib().sglb_mla_decode(_p(q_latent), _p(q_pe), _p(out), _p(kv_buffer), kv_buffer.shape[0], _p(page_table),
-                                 page_table.shape[1], _p(req_pool_indices), _p(seq_lens), B, H, R, q_pe.shape[-1],
-                                 page_size, scale, num_splits, _p(part_o), _p(part_lse), _stream()), "mla_decode")
+    _check(lib().sglb_mla_decode(_p(q_latent), q_pe.data_ptr(), q_pe.stride(0), q_pe.stride(1), _p(out), _p(kv_buffer),
+                                 kv_buffer.shape[0], kv_buffer.shape[-1], _p(page_table), page_table.shape[1],
+                                 _p(req_pool_indices), _p(seq_lens), B, H, R, q_pe.shape[-1], page_size, scale,
+                                 num_splits, _p(part_o), _p(part_lse), int(exact), _stream()), "mla_decode")
+    return out
+
+
+# ---- fp32 residual stream (csrc/residual_stream.cu): T = bf16 or fp32 throughout
+def _f32(t) -> int:
+    assert t.dtype in (torch.float32, torch.bfloat16)
+    return int(t.dtype == torch.float32)
+
+
+def embed_scaled(ids, table, scale):
+    """`(x fp32 [T, W], x in the table's type)`; with an fp32 table both are the same tensor."""
+    ids = ids.contiguous()
+    assert ids.dtype == torch.int32 and table.is_contiguous()
+    n, W = ids.numel(), table.shape[1]
+    x = torch.empty((n, W), dtype=torch.float32, device=table.device)
+    f32 = _f32(table)
+    xt = None if f32 else torch.empty((n, W), dtype=table.dtype, device=table.device)
+    _check(lib().sglb_embed_scaled(_p(x), _p(xt), _p(ids), _p(table), n, W, table.shape[0], float(scale), f32, _stream()),
+           "embed_scaled")
+    return x, (x if f32 else xt)
+
+
+def postnorm_add(y, x, channel_scale, eps):
+    """`x += channel_scale * y / rms(y)` in place (x, channel_scale fp32); returns x in y's type."""
+    y = y.contiguous()
+    W = x.shape[-1]
+    assert x.dtype == channel_scale.dtype == torch.float32 and x.is_contiguous() and y.shape == x.shape
+    f32 = _f32(y)
+    xt = None if f32 else torch.empty_like(y)
+    _check(lib().sglb_postnorm_add(_p(x), _p(xt), _p(y), _p(channel_scale), x.numel() // W, W, float(eps), f32, _stream()),
+           "postnorm_add")
+    return x if f32 else xt
+
+
+def rmsnorm_stream(x, weight, eps, dtype):
+    """`x / rms(x) * weight` in `dtype`; x and weight fp32."""
+    assert x.dtype == weight.dtype == torch.float32 and x.is_contiguous()
+    n, W = x.shape
+    y = torch.empty((n, W), dtype=dtype, device=x.device)
+    _check(lib().sglb_rmsnorm_stream(_p(y), _p(x), _p(weight), n, W, float(eps), _f32(y), _stream()), "rmsnorm_stream")
+    return y
+
+
+def gelu_tanh_and_mul(x):
+    x = x.contiguous()
+    F = x.shape[-1] // 2
+    out = torch.empty((*x.shape[:-1], F), dtype=x.dtype, device=x.device)
+    _check(lib().sglb_gelu_tanh_and_mul(_p(out), _p(x), out.numel() // F, F, _f32(x), _stream()), "gelu_tanh_and_mul")
+    return out
+
+
+def sigmoid_gate(o, gate):
+    """`o * sigmoid(gate)`; `o [T, F]` contiguous, `gate [T, F]` with any row stride."""
+    assert o.is_contiguous() and gate.stride(-1) == 1 and gate.dtype == o.dtype
+    out = torch.empty_like(o)
+    _check(lib().sglb_sigmoid_gate(_p(out), _p(o), gate.data_ptr(), gate.stride(0), o.shape[0], o.shape[1], _f32(o),
+                                   _stream()), "sigmoid_gate")
+    return out
+
+
+# ---- latent attention of any sizes (csrc/latent_attn.cu, latent_extend.cu)
+def latent_prep(proj, q_off, dkv_off, heads, dim, rot, rank, norm_w, eps, cos_sin, positions, loc, cache):
+    """Rotates the queries of `proj [T, ld]` in place and writes the normalised latent and the rotated key part of its
+    rows into `cache [pages, P, row]` at slots `loc`."""
+    assert proj.stride(1) == 1 and cache.is_contiguous() and cache.dtype == proj.dtype
+    assert positions.dtype == loc.dtype == torch.int32 and norm_w.dtype == cos_sin.dtype == torch.float32
+    assert cos_sin.device == norm_w.device == cache.device == proj.device and cos_sin.is_contiguous()
+    _check(lib().sglb_latent_prep(_p(proj), proj.stride(0), q_off, dkv_off, proj.shape[0], heads, dim, rot, rank,
+                                  _p(norm_w), float(eps), _p(cos_sin), _p(positions), _p(loc), _p(cache),
+                                  cache.shape[-1], _f32(proj), _stream()), "latent_prep")
+
+
+def latent_attn_any(q_lat, q_pe, cache, page_table, rows, kv_lens, page_size, scale):
+    """Absorbed attention of single query tokens, fp32 arithmetic: `q_lat [N, H, R]`, query n sees the first
+    `kv_lens[n]` tokens of page-table row `rows[n]`."""
+    N, H, R = q_lat.shape
+    q_lat = q_lat.contiguous()
+    assert q_pe.stride(-1) == 1 and rows.dtype == kv_lens.dtype == torch.int32 and cache.dtype == q_lat.dtype
+    out = torch.empty_like(q_lat)
+    _check(lib().sglb_latent_attn_any(_p(q_lat), q_pe.data_ptr(), q_pe.stride(0), q_pe.stride(1), _p(cache),
+                                      cache.shape[-1], _p(page_table), page_table.shape[1], page_size, _p(rows),
+                                      _p(kv_lens), _p(out), N, H, R, q_pe.shape[-1], float(scale), _f32(q_lat),
+                                      _stream()), "latent_attn_any")
+    return out
+
+
+def latent_gather(cache, page_table, rows, ctx_start, total, rank, rot, page_size):
+    """Cache rows of whole sequences, laid end to end -> `(latents [total, rank], key parts [total, rot])`."""
+    lat = torch.empty((total, rank), dtype=cache.dtype, device=cache.device)
+    pe = torch.empty((total, rot), dtype=cache.dtype, device=cache.device)
+    _check(lib().sglb_latent_gather(_p(lat), _p(pe), _p(cache), cache.shape[-1], _p(page_table), page_table.shape[1],
+                                    page_size, _p(rows), _p(ctx_start), rows.numel(), total, rank, rot, _stream()),
+           "latent_gather")
+    return lat, pe
+
+
+def latent_extend_supported(q, dim, rot, v_dim, rank) -> bool:
+    return False
+
+
+# ---- gated delta rule over ragged batches (csrc/delta_scan.cu)
+def delta_scan(proj, g_off, b_off, a_off, conv_w, a_log, dt_bias, conv_state, state, slots, heads, kv_heads, dim, vdim,
+               cu=None, prefix=None, track_len=None, track_slot=None):
+    """Read-outs fp32 `[T, heads, vdim]` of the rows of `proj [T, ld]` (columns `q | k | v` first, gate / beta / decay
+    inputs at the given offsets); windows and states of `slots` are updated in place.  `cu [B + 1]` / `prefix [B]`:
+    ragged step (None: one row per request, all of them continuing)."""
+    T, dev = proj.shape[0], proj.device
+    f32 = dict(dtype=torch.float32, device=dev)
+    assert proj.stride(1) == 1 and conv_state.is_contiguous() and state.is_contiguous() and conv_w.is_contiguous()
+    assert conv_state.dtype == conv_w.dtype == proj.dtype and state.dtype == torch.float32 and slots.dtype == torch.int64
+    qk = torch.empty((T, kv_heads, 2, dim), **f32)
+    v = torch.empty((T, heads, vdim), **f32)
+    gb = torch.empty((T, heads, 2), **f32)
+    kq = torch.empty((T, kv_heads), **f32)
+    o = torch.empty((T, heads, vdim), **f32)
+    _check(lib().sglb_delta_scan(_p(proj), proj.stride(0), g_off, b_off, a_off, _p(conv_w), _p(a_log), _p(dt_bias),
+                                 _p(conv_state), _p(state), _p(slots), _p(cu), _p(prefix), _p(track_len), _p(track_slot),
+                                 _p(qk), _p(v), _p(gb), _p(kq), _p(o), slots.numel(), T, heads, kv_heads, dim, vdim,
+                                 conv_w.shape[1], _f32(proj), _stream()), "delta_scan")
+    return o
+
+
+def delta_gate(o, gate, weight, eps):
+    """`rmsnorm(o) * weight * silu(gate)` per head: `o [T, H, V]` fp32, `gate [T, H * V]` (any row stride) -> `[T, H * V]`
+    in the gate's type."""
+    T, H, V = o.shape
+    assert o.is_contiguous() and gate.stride(-1) == 1 and weight.dtype == torch.float32
+    out = torch.empty((T, H * V), dtype=gate.dtype, device=o.device)
+    _check(lib().sglb_delta_gate(_p(o), gate.data_ptr(), gate.stride(0), _p(weight), _p(out), T, H, V, float(eps),
+                                 _f32(gate), _stream()), "delta_gate")
     return out
 
 

@@ -346,3 +346,76 @@ def mla_paged_attention(q_nope_latent, q_pe, kv_buffer, page_table, req_pool_ind
         p = torch.softmax(logits, dim=-1)
         out[q0:q1] = torch.einsum("hns,sr->nhr", p, c).to(out.dtype)
     return out
+
+
+# ------------------------------------------------------------------ fp32 residual stream, delta rule, latent attention
+def sigmoid_gate(o, gate):
+    return (o.float() * torch.sigmoid(gate.float())).to(o.dtype)
+
+
+def embed_scaled(ids, table, scale):
+    x = F.embedding(ids.long(), table).float() * scale
+    return x, (x if table.dtype == torch.float32 else x.to(table.dtype))
+
+
+def postnorm_add(y, x, channel_scale, eps):
+    yf = y.float()
+    x += yf * torch.rsqrt(yf.pow(2).mean(-1, keepdim=True) + eps) * channel_scale
+    return x if y.dtype == torch.float32 else x.to(y.dtype)
+
+
+def rmsnorm_stream(x, weight, eps, dtype):
+    return (x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * weight).to(dtype)
+
+
+def delta_scan(proj, g_off, b_off, a_off, conv_w, a_log, dt_bias, conv_state, state, slots, heads, kv_heads, dim, vdim,
+               cu=None, prefix=None, track_len=None, track_slot=None):
+    """Statement of `native.delta_scan` through the primitives of `ops/linear_attention.py`."""
+    from . import linear_attention as la
+    B, T, r, kd = slots.numel(), proj.shape[0], heads // kv_heads, kv_heads * dim
+    o = torch.empty(T, heads, vdim, dtype=torch.float32, device=proj.device)
+    cu_l = cu.tolist() if cu is not None else list(range(B + 1))
+    pre = prefix.tolist() if prefix is not None else [1] * B
+    tr = track_len.tolist() if track_len is not None else [0] * B
+    win = conv_w.shape[1] - 1
+    for b, s in enumerate(slots.tolist()):
+        cuts = [cu_l[b], cu_l[b + 1]]
+        if cuts[0] == cuts[1]:
+            continue
+        if 0 < tr[b] < cuts[1] - cuts[0]:
+            cuts.insert(1, cuts[0] + tr[b])
+        fresh = pre[b] == 0
+        for a0, a1 in zip(cuts[:-1], cuts[1:]):
+            rows = proj[a0:a1].float()
+            x = rows[:, : 2 * kd + heads * vdim]
+            if win:
+                y, window = la.causal_conv1d_prefill(x, conv_w, None if fresh else conv_state[s])
+                conv_state[s] = window.to(conv_state.dtype)
+            else:
+                y = F.silu(x * conv_w.float()[:, 0])
+            q, k, v = y[:, :kd].view(-1, kv_heads, dim), y[:, kd:2 * kd].view(-1, kv_heads, dim), y[:, 2 * kd:]
+            g = -a_log.exp() * F.softplus(rows[:, a_off:a_off + heads] + dt_bias)
+            beta = torch.sigmoid(rows[:, b_off:b_off + heads])
+            o[a0:a1], state[s] = la.chunk_gated_delta_rule(
+                q.repeat_interleave(r, 1), k.repeat_interleave(r, 1), v.reshape(-1, heads, vdim), g, beta,
+                None if fresh else state[s])
+            fresh = False
+            if tr[b] and a1 - cuts[0] == tr[b]:
+                conv_state[int(track_slot[b])] = conv_state[s]
+                state[int(track_slot[b])] = state[s]
+    return o
+
+
+def delta_gate(o, gate, weight, eps):
+    T, H, V = o.shape
+    y = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * weight * F.silu(gate.float()).view(T, H, V)
+    return y.view(T, H * V).to(gate.dtype)
+
+
+def latent_prep(proj, q_off, dkv_off, heads, dim, rot, rank, norm_w, eps, cos_sin, positions, loc, cache):
+    q = proj[:, q_off:q_off + heads * (dim + rot)].unflatten(-1, (heads, dim + rot))[..., dim:]
+    q.copy_(apply_rope(q, positions, cos_sin, False))
+    c = proj[:, dkv_off:dkv_off + rank].float()
+    c = c * torch.rsqrt(c.pow(2).mean(-1, keepdim=True) + eps) * norm_w
+    pe = apply_rope(proj[:, dkv_off + rank:dkv_off + rank + rot].unsqueeze(1), positions, cos_sin, False).squeeze(1)
+    cache.view(-1, cache.shape[-1])[loc.long(), :rank + rot] = torch.cat([c, pe.float()], -1).to(cache.dtype)
