@@ -84,6 +84,22 @@ bool encode_tmap_2d(CUtensorMap* out, const void* base, uint64_t inner_elems, ui
   return r == CUDA_SUCCESS;
 }
 
+// 3-D bf16 tensor [d2][d1][d0] with byte strides `stride1`, `stride2` (multiples of 16), 128-byte swizzle; the box is
+// 64 x 1 x box_rows elements.  Elements outside the extents are read as zeros.
+bool encode_tmap_3d(CUtensorMap* out, const void* base, uint64_t d0, uint64_t d1, uint64_t d2, uint64_t stride1,
+                    uint64_t stride2, uint32_t box_rows) {
+  EncodeFn enc = get_encode();
+  if (!enc) return false;
+  if ((reinterpret_cast<uintptr_t>(base) & 15) || (stride1 & 15) || (stride2 & 15)) return false;
+  cuuint64_t dims[3] = {d0, d1, d2};
+  cuuint64_t strides[2] = {stride1, stride2};
+  cuuint32_t box[3] = {64, 1, box_rows};
+  cuuint32_t estr[3] = {1, 1, 1};
+  return enc(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr,
+             CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+             CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
+}
+
 }  // namespace sglb
 
 extern "C" {

@@ -116,6 +116,14 @@ class RotaryEmbedding(nn.Module):
                 reference.apply_rope(k, positions, self.cos_sin_cache, self.is_neox_style, self.rotary_dim))
 
 
+class ExactRotaryEmbedding(RotaryEmbedding):
+    """Frequencies evaluated in double precision and rounded once to fp32 (the powers of the base class are fp32)."""
+
+    def _compute_inv_freq(self, base):
+        e = torch.arange(0, self.rotary_dim, 2, dtype=torch.float64, device="cpu") / self.rotary_dim
+        return (float(base) ** -e).float()
+
+
 class Llama3RotaryEmbedding(RotaryEmbedding):
     def __init__(self, head_size, rotary_dim, max_pos, base, is_neox_style, dtype, scaling_factor,
                  low_freq_factor, high_freq_factor, orig_max_position):
@@ -262,6 +270,8 @@ def get_rope(head_size, rotary_dim, max_position, base, is_neox_style=True, rope
                                     bool(rs.get("mrope_interleaved", False)))
         else:
             rope = RotaryEmbedding(head_size, rotary_dim, max_position, base, is_neox_style, dtype)
+    elif kind == "exact":
+        rope = ExactRotaryEmbedding(head_size, rotary_dim, max_position, base, is_neox_style, dtype)
     elif kind == "llama3":
         rope = Llama3RotaryEmbedding(head_size, rotary_dim, max_position, base, is_neox_style, dtype,
                                      rs["factor"], rs["low_freq_factor"], rs["high_freq_factor"],

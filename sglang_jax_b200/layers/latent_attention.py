@@ -45,7 +45,7 @@ class LatentAttention(nn.Module):
         # per head: `dim` key rows, then `v_dim` value rows
         self.up = nn.Parameter(torch.empty(self.heads, dim + v_dim, kv_rank, dtype=dtype), requires_grad=False)
         self.o_proj = RowParallelLinear(num_heads * v_dim, hidden_size, False, dtype)
-        self.rotary_emb = get_rope(rot_dim, rot_dim, max_positions, rope_base, False, None, dtype)
+        self.rotary_emb = get_rope(rot_dim, rot_dim, max_positions, rope_base, False, {"rope_type": "exact"}, dtype)
 
     def load(self, name: str, w: torch.Tensor):
         """One checkpoint tensor: q, g, dkv (latent and key part), dkv.norm, uk / uv (key and value up-projection), o."""
@@ -132,7 +132,7 @@ class ExtendPlan:
             ctx = (pre + n)[long]
             ctx_start = np.concatenate([[0], np.cumsum(ctx)])
             self.ctx_total = int(ctx_start[-1])
-            tiles = (n[long] + 127) // 128
+            tiles = (n[long] + 255) // 256              # query rows per CTA of the prefill kernel
             self.num_tiles = int(tiles.sum())
             rows = fb.req_pool_indices[torch.from_numpy(long).to(dev)]
             meta = torch.from_numpy(np.concatenate([start[long], n[long], pre[long], ctx_start]).astype(np.int32)).to(dev)

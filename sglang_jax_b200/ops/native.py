@@ -98,6 +98,9 @@ def lib():
                                  c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p])
     sig("sglb_latent_gather", [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int,
                                c_int, c_int, c_int, c_void_p])
+    sig("sglb_latent_extend_supported", [c_int, c_int, c_int])
+    sig("sglb_latent_extend", [c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_int]
+        + [c_void_p] * 4 + [c_int] * 6 + [c_float, c_void_p])
     sig("sglb_delta_scan", [c_void_p, c_longlong, c_int, c_int, c_int] + [c_void_p] * 15 + [c_int] * 8 + [c_void_p])
     sig("sglb_delta_gate", [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_int, c_int, c_float, c_int,
                             c_void_p])
@@ -669,7 +672,21 @@ def latent_gather(cache, page_table, rows, ctx_start, total, rank, rot, page_siz
 
 
 def latent_extend_supported(q, dim, rot, v_dim, rank) -> bool:
-    return False
+    """Whether `latent_extend` takes these sizes and this (strided) query tensor `[T, H, dim + rot]`."""
+    return (q.dtype == torch.bfloat16 and rank % 8 == 0 and q.stride(2) == 1 and q.stride(1) == dim + rot
+            and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0
+            and bool(lib().sglb_latent_extend_supported(dim, rot, v_dim)))
+
+
+def latent_extend(q, kv, k_rot, out, plan, dim, v_dim, scale):
+    """Causal attention of the sequences of `plan` (`layers/latent_attention.ExtendPlan`) over expanded keys and values:
+    `q [T, H, dim + rot]` (strided view), `kv [ctx, H * (dim + v_dim)]`, `k_rot [ctx, rot]`, result into the rows of
+    those sequences of `out [T, H, v_dim]` (strided view)."""
+    assert kv.is_contiguous() and k_rot.is_contiguous() and out.stride(2) == 1 and out.dtype == q.dtype
+    _check(lib().sglb_latent_extend(q.data_ptr(), q.stride(0), q.shape[0], _p(kv), _p(k_rot), k_rot.shape[0],
+                                    out.data_ptr(), out.stride(0), out.stride(1), _p(plan.q_start), _p(plan.q_len),
+                                    _p(plan.prefix), _p(plan.ctx_start), plan.long, plan.num_tiles, q.shape[1], dim,
+                                    k_rot.shape[1], v_dim, float(scale), _stream()), "latent_extend")
 
 
 # ---- gated delta rule over ragged batches (csrc/delta_scan.cu)
