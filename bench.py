@@ -101,6 +101,11 @@ def parse_args():
     ap.add_argument("--disable-overlap", action="store_true")
     ap.add_argument("--device", default=None)
     ap.add_argument("--log-level", default="error")
+    ap.add_argument("--hybrid", action="store_true",
+                    help="instead of the headline workload: prefill / decode throughput of the hybrid recurrent / latent-"
+                         "attention decoders at equal sizes (sglang_jax_b200/bench_hybrid.py), one JSON line per size")
+    ap.add_argument("--hybrid-size", nargs="*", default=None)
+    ap.add_argument("--hybrid-models", nargs="*", default=None)
     ap.add_argument("--hang-timeout", type=float, default=float(os.environ.get("SGLB_BENCH_HANG_TIMEOUT", "300")),
                     help="seconds without progress after which every rank dumps its stacks and exits")
     a = ap.parse_args()
@@ -263,6 +268,9 @@ def percentile(xs, q):
 
 def main():
     args = parse_args()
+    if args.hybrid:
+        from sglang_jax_b200.bench_hybrid import main as hybrid_main
+        return hybrid_main(args.hybrid_size, args.hybrid_models)
     if args.impl == "reference":
         return reference_arm(args)
     if args.impl == "nccl":

@@ -1,0 +1,176 @@
+"""Prefill and decode throughput of hybrid recurrent / latent-attention decoders at equal sizes, random weights:
+Zozopel beside the framework's closest other models, Kimi-Linear (per-channel delta rule + latent attention) and
+Qwen3-Next (gated delta rule + grouped attention).  Runs on the model runner, decode through its CUDA graphs.
+
+    python bench.py --hybrid [--hybrid-size base large] [--hybrid-models zozopel kimi_linear qwen3_next]
+
+One JSON line per size.  Times are CUDA events around the forward, median over the repetitions; a step streams the
+weights of all layers, more than the L2 holds."""
+
+from __future__ import annotations
+
+import gc
+import json
+import os
+import tempfile
+
+import numpy as np
+
+SIZES = {
+    # width, feed-forward, heads of 128 (+ 64 rotary lanes), query/key heads of the delta rule, latent width, layers
+    "base": dict(width=2048, ff=6144, heads=16, kv_heads=8, rank=512, layers=8, vocab=32768),
+    "large": dict(width=4096, ff=12288, heads=32, kv_heads=16, rank=512, layers=8, vocab=32768),
+}
+PREFILL = [(1, 4096), (4, 2048), (16, 512)]        # (sequences, new tokens each)
+DECODE = [(1, 2048), (32, 2048), (128, 2048)]      # (sequences, cached tokens each)
+
+
+def model_config(name: str, s: dict) -> dict:
+    w, n = s["width"], s["layers"]
+    if name == "zozopel":
+        latent = {"type": "latent_attention", "mlp": {"kind": "dense", "ff": s["ff"]},
+                  "mixer": dict(heads=s["heads"], dim=128, rot_dim=64, vdim=128, kv_rank=s["rank"], scale=192 ** -0.5,
+                                rot={"base": 10000.0, "dims": 64})}
+        delta = {"type": "delta", "mlp": {"kind": "dense", "ff": s["ff"]},
+                 "mixer": dict(heads=s["heads"], kv_heads=s["kv_heads"], dim=128, vdim=128, conv=4)}
+        return dict(architecture="Zozopel", vocab=s["vocab"], width=w, embedding={"scale": 1.0}, norm={"eps": 1e-6},
+                    residual_mult=0.5, logit_scale=1.0, layers=[latent if i % 2 else delta for i in range(n)])
+    common = dict(hidden_size=w, intermediate_size=s["ff"], num_hidden_layers=n, rms_norm_eps=1e-6,
+                  vocab_size=s["vocab"], max_position_embeddings=32768, tie_word_embeddings=False,
+                  torch_dtype="bfloat16", num_attention_heads=s["heads"])
+    if name == "kimi_linear":
+        return dict(common, architectures=["KimiLinearForCausalLM"], model_type="kimi_linear",
+                    num_key_value_heads=s["heads"], kv_lora_rank=s["rank"], q_lora_rank=None, qk_nope_head_dim=128,
+                    qk_rope_head_dim=64, v_head_dim=128, mla_use_nope=True, num_experts=0,
+                    linear_attn_config={"kda_layers": [i + 1 for i in range(0, n, 2)], "num_heads": s["heads"],
+                                        "head_dim": 128, "short_conv_kernel_size": 4})
+    if name == "qwen3_next":
+        return dict(common, architectures=["Qwen3NextForCausalLM"], model_type="qwen3_next", head_dim=128,
+                    num_key_value_heads=max(s["heads"] // 4, 1), full_attention_interval=2, num_experts=0,
+                    linear_num_value_heads=s["heads"], linear_num_key_heads=s["kv_heads"], linear_key_head_dim=128,
+                    linear_value_head_dim=128, linear_conv_kernel_dim=4, rope_theta=10000.0, partial_rotary_factor=0.5)
+    raise ValueError(name)
+
+
+def build_runner(name: str, size: dict, max_reqs: int, max_tokens: int, device: str):
+    from .configs.model_config import ModelConfig
+    from .model_executor.model_runner import ModelRunner
+    from .server_args import ServerArgs
+    from .utils.tiny_models import write_config_only
+    path = write_config_only(os.path.join(tempfile.gettempdir(), f"sglb200_hybrid_{name}"), model_config(name, size))
+    sa = ServerArgs(model_path=path, load_format="dummy", device=device,
+                    dtype="bfloat16" if device == "cuda" else "float32", page_size=64, max_total_tokens=max_tokens,
+                    max_running_requests=max_reqs, context_length=8192, skip_tokenizer_init=True,
+                    disable_overlap_schedule=True, precompile_bs_paddings=sorted({b for b, _ in DECODE if b <= max_reqs}),
+                    cuda_graph_max_bs=max_reqs, disable_radix_cache=True, mem_fraction_static=0.9)
+    return ModelRunner(ModelConfig.from_server_args(sa), sa)
+
+
+class StaticBatch:
+    """`B` requests whose pages are laid out once, for timing single forwards."""
+
+    def __init__(self, runner, B: int, capacity: int):
+        from .managers.schedule_batch import ModelWorkerSamplingInfo
+        self.r, self.B, P = runner, B, runner.page_size
+        per = -(-capacity // P) * P
+        self.base = np.arange(B, dtype=np.int64) * per + P
+        for b in range(B):
+            runner.req_to_token_pool.write(b, 0, self.base[b] + np.arange(per))
+        self.deltas = runner.req_to_token_pool.take_page_deltas()
+        self.ids = np.random.RandomState(0).randint(1, runner.model_config.vocab_size, B * capacity).astype(np.int32)
+        self.info = lambda n: ModelWorkerSamplingInfo(np.ones(n, np.float32), np.ones(n, np.float32), np.ones(n, np.int32),
+                                                      np.zeros(n, np.float32), None, True, False, False, False)
+
+    def _deltas(self):
+        d = self.deltas
+        self.deltas = (np.empty(0, np.int32),) * 3
+        return dict(page_delta_rows=d[0], page_delta_pos=d[1], page_delta_ids=d[2])
+
+    def prefill(self, n: int):
+        from .managers.schedule_batch import ForwardMode, ModelWorkerBatch
+        B, f = self.B, lambda v: np.full(self.B, v, np.int32)
+        return self.r.forward(ModelWorkerBatch(
+            bid=0, forward_mode=ForwardMode.EXTEND, input_ids=self.ids[:B * n], req_pool_indices=np.arange(B, dtype=np.int32),
+            seq_lens=f(n), out_cache_loc=np.concatenate([b + np.arange(n) for b in self.base]).astype(np.int32),
+            positions=np.tile(np.arange(n, dtype=np.int32), B), extend_prefix_lens=f(0), extend_seq_lens=f(n),
+            extend_logprob_start_lens=f(0), sampling_info=self.info(B), **self._deltas()))
+
+    def decode(self, ctx: int):
+        from .managers.schedule_batch import ForwardMode, ModelWorkerBatch
+        B, f = self.B, lambda v: np.full(self.B, v, np.int32)
+        d = self._deltas()
+        if len(d["page_delta_rows"]):            # more entries than a graph takes: bring the device table up to date
+            import torch
+            t = lambda a: torch.from_numpy(np.asarray(a)).to(self.r.device)
+            self.r.req_to_token_pool.page_table[t(d["page_delta_rows"]).long(), t(d["page_delta_pos"]).long()] = \
+                t(d["page_delta_ids"])
+        return self.r.forward(ModelWorkerBatch(
+            bid=0, forward_mode=ForwardMode.DECODE, input_ids=self.ids[:B], req_pool_indices=np.arange(B, dtype=np.int32),
+            seq_lens=f(ctx + 1), out_cache_loc=(self.base + ctx).astype(np.int32), positions=f(ctx),
+            sampling_info=self.info(B)))
+
+
+def time_ms(fn, warmup: int = 3, reps: int = 7, budget_s: float = 20.0) -> float:
+    """Median CUDA-event time; a forward that would not fit the budget that often is measured fewer times."""
+    import time
+
+    import torch
+    t0 = time.perf_counter()
+    fn()
+    torch.cuda.synchronize()
+    one = time.perf_counter() - t0
+    if one * (warmup + reps) > budget_s:
+        warmup, reps = 0, 1
+    for _ in range(warmup):
+        fn()
+    torch.cuda.synchronize()
+    out = []
+    for _ in range(reps):
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        a.record()
+        fn()
+        b.record()
+        torch.cuda.synchronize()
+        out.append(a.elapsed_time(b))
+    return float(np.median(out))
+
+
+def run_model(name: str, size: dict, device: str = "cuda") -> dict:
+    import torch
+
+    from .ops import native
+    reqs = max(b for b, _ in PREFILL + DECODE)
+    tokens = max(b * (n + 64) for b, n in PREFILL + DECODE) + 64
+    runner = build_runner(name, size, reqs, tokens, device)
+    rec = {"weights_gib": round(runner.weight_bytes / 2 ** 30, 2), "prefill": {}, "decode": {}}
+    for B, n in PREFILL:
+        sb = StaticBatch(runner, B, n)
+        ms = time_ms(lambda: sb.prefill(n))
+        rec["prefill"][f"{B}x{n}"] = {"ms": round(ms, 3), "tok_s": round(B * n / ms * 1e3)}
+    for B, n in DECODE:
+        sb = StaticBatch(runner, B, n + 1)
+        ms = time_ms(lambda: sb.decode(n), reps=15)
+        rec["decode"][f"{B}x{n}"] = {"ms": round(ms, 3), "tok_s": round(B / ms * 1e3)}
+    native.check_status()
+    del runner, sb
+    gc.collect()
+    torch.cuda.empty_cache()
+    return rec
+
+
+def main(sizes=None, models=None) -> int:
+    import torch
+
+    from .parallel import state as ps
+    if not torch.cuda.is_available():
+        print(json.dumps({"metric": "hybrid decoders, prefill and decode tokens/s", "unavailable": "needs a CUDA device"}))
+        return 0
+    if not ps.get_state().initialized:
+        ps.init_distributed(0, 1, "cuda")
+    for s in sizes or list(SIZES):
+        out = {"metric": "hybrid decoders, prefill and decode tokens/s", "size": s, **SIZES[s], "dtype": "bf16",
+               "data": "synthetic token ids, random weights", "models": {}}
+        for m in models or ["zozopel", "kimi_linear", "qwen3_next"]:
+            out["models"][m] = run_model(m, SIZES[s])
+        print(json.dumps(out), flush=True)
+    return 0
