@@ -16,7 +16,7 @@
 namespace sglb {
 namespace {
 
-// VEC consecutive elements (VEC = 4: 8 / 16 bytes, VEC = 1: any alignment)
+// VEC consecutive elements: 8 (bf16 only, 16 bytes), 4 (8 / 16 bytes) or 1 (any alignment)
 template <int VEC> __device__ __forceinline__ void load_v(const float* p, float (&f)[VEC]) {
   if constexpr (VEC == 4) {
     const float4 v = *reinterpret_cast<const float4*>(p);
@@ -26,7 +26,15 @@ template <int VEC> __device__ __forceinline__ void load_v(const float* p, float 
   }
 }
 template <int VEC> __device__ __forceinline__ void load_v(const __nv_bfloat16* p, float (&f)[VEC]) {
-  if constexpr (VEC == 4) {
+  if constexpr (VEC == 8) {
+    const uint4 v = *reinterpret_cast<const uint4*>(p);
+    const uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      f[2 * i] = __uint_as_float(w[i] << 16);
+      f[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+    }
+  } else if constexpr (VEC == 4) {
     const uint2 v = *reinterpret_cast<const uint2*>(p);
     const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.x));
     const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.y));
@@ -40,7 +48,10 @@ template <int VEC> __device__ __forceinline__ void store_v(float* p, const float
   else *p = f[0];
 }
 template <int VEC> __device__ __forceinline__ void store_v(__nv_bfloat16* p, const float (&f)[VEC]) {
-  if constexpr (VEC == 4) *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]));
+  if constexpr (VEC == 8)
+    *reinterpret_cast<uint4*>(p) =
+        make_uint4(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]), pack_bf16(f[4], f[5]), pack_bf16(f[6], f[7]));
+  else if constexpr (VEC == 4) *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]));
   else *p = __float2bfloat16(f[0]);
 }
 
@@ -136,8 +147,9 @@ __global__ void rmsnorm_stream_kernel(T* __restrict__ y, const float* __restrict
   }
 }
 
+// 0.5 z (1 + tanh(y)) = z / (1 + exp(-2 y)), y = sqrt(2 / pi) (z + 0.044715 z^3)
 __device__ __forceinline__ float gelu_tanh(float z) {
-  return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+  return z / (1.f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
 }
 
 template <typename T, int VEC>
@@ -241,7 +253,10 @@ template <typename T>
 int gelu_mul(void* out, const void* in, long long rows, int F, cudaStream_t s) {
   T* o = static_cast<T*>(out);
   const T* i = static_cast<const T*>(in);
-  if (F % 4 == 0) launch_pdl(gelu_mul_kernel<T, 4>, dim3(grid_for(rows * (F / 4))), dim3(256), 0, s, o, i, rows, F);
+  constexpr int kWide = sizeof(T) == 2 ? 8 : 4;
+  if (F % kWide == 0)
+    launch_pdl(gelu_mul_kernel<T, kWide>, dim3(grid_for(rows * (F / kWide))), dim3(256), 0, s, o, i, rows, F);
+  else if (F % 4 == 0) launch_pdl(gelu_mul_kernel<T, 4>, dim3(grid_for(rows * (F / 4))), dim3(256), 0, s, o, i, rows, F);
   else launch_pdl(gelu_mul_kernel<T, 1>, dim3(grid_for(rows * F)), dim3(256), 0, s, o, i, rows, F);
   return static_cast<int>(cudaGetLastError());
 }
@@ -251,8 +266,12 @@ int sigmoid_gate(void* out, const void* o, const void* g, long long g_stride, lo
   T* d = static_cast<T*>(out);
   const T* a = static_cast<const T*>(o);
   const T* b = static_cast<const T*>(g);
+  constexpr int kWide = sizeof(T) == 2 ? 8 : 4;
   const bool vec = F % 4 == 0 && g_stride % 4 == 0 && reinterpret_cast<uintptr_t>(g) % (4 * sizeof(T)) == 0;
-  if (vec)
+  if (vec && F % kWide == 0 && g_stride % kWide == 0 && reinterpret_cast<uintptr_t>(g) % 16 == 0)
+    launch_pdl(sigmoid_gate_kernel<T, kWide>, dim3(grid_for(rows * (F / kWide))), dim3(256), 0, s, d, a, b, g_stride, rows,
+               F);
+  else if (vec)
     launch_pdl(sigmoid_gate_kernel<T, 4>, dim3(grid_for(rows * (F / 4))), dim3(256), 0, s, d, a, b, g_stride, rows, F);
   else
     launch_pdl(sigmoid_gate_kernel<T, 1>, dim3(grid_for(rows * F)), dim3(256), 0, s, d, a, b, g_stride, rows, F);
