@@ -3,12 +3,13 @@
 //   delta_prep    short causal convolution + SiLU of the q / k / v channels of a fused projection (window = this step's
 //                 rows, then the request's stored window, then zeros), unit q (times dim^-1/2) and k vectors, write
 //                 strength beta = sigmoid(b) and decay g = exp(-exp(A_log) softplus(a + dt_bias))
-//   delta_dots    scalar products of the k and q vectors inside blocks of four tokens (prefill)
-//   delta_scan    S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q   in blocks of four tokens; columns of S
-//                 are independent, so a CTA owns a few columns of one (sequence, head) and keeps them in registers from
-//                 the first token to the last.  The state is read once and written once per step, whatever the number
-//                 of tokens, and depends on how a prompt is cut by rounding only.  The convolution windows and the
-//                 optional checkpoint (state after `track` tokens, for prefix sharing) are written here too.
+//   delta_chunk   prefill: what a chunk of 32 tokens contributes independently of the state in front of it
+//   delta_scan    prefill: S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q   chunk by chunk as small matrix
+//                 products; columns of S are independent, so a CTA owns 32 columns of one (sequence, head) and keeps
+//                 them from the first token to the last.  The result depends on how a prompt is cut by rounding only
+//   delta_step    decode: the same for one token per request, the state streaming through once
+//                 The convolution windows and the optional checkpoint (state after `track` tokens, for prefix sharing)
+//                 are written by the last two.
 //   delta_gate    rmsnorm(o) * w * silu(gate) per head, in the projections' type
 //
 // Both state tensors belong to `RecurrentStatePool`: windows [slots, channels, taps - 1], states [slots, H, D, V].
@@ -49,7 +50,7 @@ struct DeltaParams {
   float* qk;                     // [T, Hk, 2, D] unit q * D^-1/2 | unit k
   float* v;                      // [T, H, V]
   float* gb;                     // [T, H, 2] decay, beta
-  float* dots;                   // [T, Hk, 8], see delta_dots_kernel
+  float* coef;                   // [T / 32 + 2 B, H, kCoefs], see delta_chunk_kernel
   float* o;                      // [T, H, V]
   int B, T, H, Hk, D, V, taps;
 };
@@ -220,340 +221,490 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const DeltaParams p) {
   }
 }
 
-// Scalar products inside a block of kBlock tokens (blocks are counted from the first row of a sequence):
-// dots[t][hk] = { k_j . k_t for the block's tokens j < t (kBlock - 1 places), k_j . q_t for j <= t (kBlock places) }.
-constexpr int kBlock = 4;
-
-__global__ void delta_dots_kernel(const DeltaParams p) {
-  pdl_wait();
-  const int lane = threadIdx.x & 31;
-  const long long wid = (blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x) >> 5;
-  if (wid >= static_cast<long long>(p.T) * p.Hk) return;
-  const int t = static_cast<int>(wid / p.Hk), hk = static_cast<int>(wid - static_cast<long long>(t) * p.Hk);
-  int local = 0;
-  if (p.cu != nullptr) {
-    int lo = 0, hi = p.B - 1;
-    while (lo < hi) {
-      const int mid = (lo + hi + 1) >> 1;
-      if (p.cu[mid] <= t) lo = mid;
-      else hi = mid - 1;
-    }
-    local = t - p.cu[lo];
-  }
-  const int at = local % kBlock;                       // place of t in its block
-  const long long stride = static_cast<long long>(p.Hk) * 2 * p.D;
-  const float* own = p.qk + wid * 2 * p.D;
-  float kk[kBlock], kq[kBlock];
-#pragma unroll
-  for (int j = 0; j < kBlock; ++j) kk[j] = kq[j] = 0.f;
-  for (int d = lane; d < p.D; d += 32) {
-    const float q = own[d], k = own[p.D + d];
-#pragma unroll
-    for (int j = 0; j < kBlock; ++j) {
-      if (j <= at) {
-        const float kj = j == at ? k : own[(j - at) * stride + p.D + d];
-        kk[j] += kj * k;
-        kq[j] += kj * q;
-      }
-    }
-  }
-#pragma unroll
-  for (int j = 0; j < kBlock; ++j) {
-    kk[j] = warp_sum(kk[j]);
-    kq[j] = warp_sum(kq[j]);
-  }
-  if (lane == 0) {
-    float4* dst = reinterpret_cast<float4*>(p.dots + wid * 2 * kBlock);
-    dst[0] = make_float4(kk[0], kk[1], kk[2], 0.f);
-    dst[1] = make_float4(kq[0], kq[1], kq[2], kq[3]);
-  }
-}
-
 // ---------------------------------------------------------------------------------------------
-constexpr int kScanThreads = 128;
-constexpr int kChunk = 16;        // tokens staged in shared memory at a time (two buffers)
-constexpr int kLanes = 8;         // lanes that share a column of the state
+// Prefill works in chunks of kC tokens.  With S the state in front of a chunk, G_t the product of its decays up to and
+// including t, and g_tj the product over j + 1 .. t, the recurrence unrolls to
+//
+//   u_t + sum_{j<t} beta_t g_tj (k_t . k_j) u_j = beta_t (v_t - G_t S^T k_t)
+//   o_t = G_t S^T q_t + sum_{j<=t} g_tj (q_t . k_j) u_j          S <- G S + sum_j g_Cj k_j u_j^T
+//
+// delta_chunk solves the unit lower-triangular system once per (chunk, head), independently of the state, so that the
+// sequential part (delta_scan) is matrix products only.  All in fp32; decays are products of decays, never quotients.
+constexpr int kC = 32;
+constexpr int kCoefRow = kC;                           // coefficient block of a (chunk, head):
+constexpr int kCoefB = kC * kC;                        //   [0]      (I + A)^-1 diag(beta), rows t
+constexpr int kCoefVec = 2 * kC * kC;                  //   [kCoefB] g_tj (q_t . k_j), rows t
+constexpr int kCoefs = 2 * kC * kC + 2 * kC;           //   [kCoefVec] G_t | g_Cj
 
-__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+// Chunks of one sequence: they start anew after `track` tokens (a checkpoint falls on a chunk boundary).
+struct Chunks {
+  int n, track;
+  __device__ __forceinline__ Chunks(int n_, int track_) : n(n_), track(track_ > 0 && track_ < n_ ? track_ : 0) {}
+  __device__ __forceinline__ int count() const { return (track + kC - 1) / kC + (n - track + kC - 1) / kC; }
+  __device__ __forceinline__ int first(int i) const {
+    const int head = (track + kC - 1) / kC;
+    return i < head ? i * kC : track + (i - head) * kC;
+  }
+  __device__ __forceinline__ int len(int i) const {
+    const int f = first(i);
+    return min(kC, (f < track ? track : n) - f);
+  }
+};
+// place of a sequence's first chunk in the coefficient array: sequences never overlap there
+__host__ __device__ __forceinline__ int chunk_base(int start, int b) { return start / kC + 2 * b; }
+
+__device__ __forceinline__ void cp_async16(void* dst, const void* src, int bytes = 16) {      // bytes 0: zero fill
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(bytes) : "memory");
 }
-__device__ __forceinline__ void cp_async4(void* dst, const void* src) {
-  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+__device__ __forceinline__ void cp_async4(void* dst, const void* src, int bytes = 4) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(bytes) : "memory");
 }
 __device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-// RPL rows and CPL adjacent columns of the state per lane: D <= 8 * RPL, a CTA owns 16 * CPL columns.  CHUNK tokens are
-// staged at a time; they are worked off in blocks of BLK: with S the state in front of a block, G_t the product of the
-// block's decays up to and including t, and g_jt = G_t / G_j (again a product of decays),
-//
-//   u_t = beta_t (v_t - G_t S^T k_t - sum_{j<t} g_jt (k_j . k_t) u_j)
-//   o_t = G_t S^T q_t + sum_{j<=t} g_jt (k_j . q_t) u_j          S <- G_n S + sum_j g_jn k_j u_j^T
-//
-// which is the recurrence with the block's read-outs taken from S at once: their reductions overlap.
-template <int RPL, int CPL, int CHUNK>
+// kC rows of unit q (which = 0) or k (1) vectors into smem rows of `ld` floats; rows past m become zeros.  Lanes past D
+// of a row are left alone.
+template <int THREADS>
+__device__ __forceinline__ void stage_rows(float* dst, int ld, const DeltaParams& p, int row0, int hk, int which, int m) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, D = p.D;
+  const long long tok = static_cast<long long>(p.Hk) * 2 * D;
+  const float* src = p.qk + row0 * tok + (static_cast<long long>(hk) * 2 + which) * D;
+  for (int r = warp; r < kC; r += THREADS / 32) {
+    const bool in = r < m;
+    const float* s = src + (in ? r : 0) * tok;
+    if (D % 4 == 0)
+      for (int e = lane * 4; e < D; e += 128) cp_async16(dst + r * ld + e, s + e, in ? 16 : 0);
+    else
+      for (int e = lane; e < D; e += 32) cp_async4(dst + r * ld + e, s + e, in ? 4 : 0);
+  }
+}
+
+// One CTA per (chunk, q / k head): products of the chunk's vectors, then the coefficients of every value head that uses
+// them (one warp per head).
+constexpr int kChunkThreads = 128;
+constexpr int kGramLd = kC + 4;
+
+__global__ void __launch_bounds__(kChunkThreads) delta_chunk_kernel(const DeltaParams p, int Dp) {
+  extern __shared__ float4 sm4[];
+  float* rows = reinterpret_cast<float*>(sm4);         // [k 0..kC-1 | q 0..kC-1][ld]
+  const int ld = Dp + 4;
+  float* gram = rows + 2 * kC * ld;                    // [k . k | q . k][kC][kGramLd]
+  float* line = gram + 2 * kC * kGramLd;               // [warp][kC]
+  pdl_wait();
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, hk = blockIdx.y;
+  const int idx = blockIdx.x;
+  int b = 0;
+  {
+    int lo = 0, hi = p.B - 1;
+    while (lo < hi) {                                  // last sequence whose chunks begin at or before idx
+      const int mid = (lo + hi + 1) >> 1;
+      if (chunk_base(p.cu[mid], mid) <= idx) lo = mid;
+      else hi = mid - 1;
+    }
+    b = lo;
+  }
+  const int start = p.cu[b];
+  const Chunks ch(p.cu[b + 1] - start, p.track_len != nullptr ? p.track_len[b] : 0);
+  const int ci = idx - chunk_base(start, b);
+  if (ch.n <= 0 || ci >= ch.count()) return;
+  const int row0 = start + ch.first(ci), m = ch.len(ci);
+  for (int i = tid; i < 2 * kC * (ld - p.D); i += kChunkThreads) rows[(i / (ld - p.D)) * ld + p.D + i % (ld - p.D)] = 0.f;
+  stage_rows<kChunkThreads>(rows, ld, p, row0, hk, 1, m);
+  stage_rows<kChunkThreads>(rows + kC * ld, ld, p, row0, hk, 0, m);
+  cp_commit();
+  cp_wait<0>();
+  __syncthreads();
+  {
+    // 64 x 32 products, four rows by four columns per thread
+    const int r0 = (tid >> 3) * 4, j0 = tid & 7;       // columns j0, j0 + 8, ...: neighbouring lanes, neighbouring rows
+    float acc[4][4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+    for (int d = 0; d < Dp; d += 4) {
+      float4 a[4], c[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        a[i] = *reinterpret_cast<const float4*>(rows + (r0 + i) * ld + d);
+        c[i] = *reinterpret_cast<const float4*>(rows + (j0 + 8 * i) * ld + d);
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] += a[i].x * c[j].x + a[i].y * c[j].y + a[i].z * c[j].z + a[i].w * c[j].w;
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) gram[(r0 + i) * kGramLd + j0 + 8 * j] = acc[i][j];
+  }
+  __syncthreads();
+  const int r = p.H / p.Hk;
+  for (int hh = warp; hh < r; hh += kChunkThreads / 32) {
+    const int h = hk * r + hh;
+    const float* gb = p.gb + (static_cast<long long>(row0 + lane) * p.H + h) * 2;
+    const float g = lane < m ? gb[0] : 1.f, beta = lane < m ? gb[1] : 0.f;
+    float* out = p.coef + (static_cast<long long>(idx) * p.H + h) * kCoefs;
+    float* a = line + warp * kC;
+    float from = 1.f, G = 1.f;                         // lane j: product of the decays j + 1 .. t; product up to t
+    float X[kC];                                       // lane c: column c of (I + A)^-1
+#pragma unroll
+    for (int t = 0; t < kC; ++t) {
+      const float gt = __shfl_sync(0xffffffffu, g, t), bt = __shfl_sync(0xffffffffu, beta, t);
+      G *= gt;
+      if (lane < t) from *= gt;
+      __syncwarp();
+      a[lane] = lane < t ? bt * from * gram[t * kGramLd + lane] : 0.f;
+      out[kCoefB + t * kCoefRow + lane] = lane <= t ? from * gram[(kC + t) * kGramLd + lane] : 0.f;
+      if (lane == t) out[kCoefVec + t] = G;
+      __syncwarp();
+      float x = lane == t ? 1.f : 0.f;
+#pragma unroll
+      for (int j = 0; j < t; j += 4) {
+        const float4 c = *reinterpret_cast<const float4*>(a + j);
+        x -= c.x * X[j];
+        if (j + 1 < t) x -= c.y * X[j + 1];
+        if (j + 2 < t) x -= c.z * X[j + 2];
+        if (j + 3 < t) x -= c.w * X[j + 3];
+      }
+      X[t] = x;
+      out[t * kCoefRow + lane] = x * beta;
+    }
+    out[kCoefVec + kC + lane] = from;
+  }
+}
+
+// ---------------------------------------------------------------------------------------------
+constexpr int kScanThreads = 256;
+constexpr int kCols = 32;          // columns of the state per CTA
+
+// Convolution windows of one head's channels after a step of n rows (the q / k channels are written by the first value
+// head that uses them), and after its first `track` rows in the checkpoint's slot.
+template <typename T>
+__device__ __forceinline__ void write_windows(const DeltaParams& p, int b, int h, int start, int n, bool fresh, int track,
+                                              int threads) {
+  const int D = p.D, V = p.V, win = p.taps - 1, channels = 2 * p.Hk * D + p.H * V, hk = h / (p.H / p.Hk);
+  const T* proj = static_cast<const T*>(p.proj) + start * p.ld;
+  T* cs = static_cast<T*>(p.conv_state);
+  T* own = cs + p.slots[b] * channels * win;
+  auto window = [&](int c) {
+    T* w = own + static_cast<long long>(c) * win;
+    auto input = [&](int i) {                          // input number i of this step (negative: before it)
+      return i >= 0 ? proj[i * p.ld + c] : (fresh ? from_f<T>(0.f) : w[win + i]);
+    };
+    if (track > 0 && track <= n) {
+      T* sw = cs + (static_cast<long long>(p.track_slot[b]) * channels + c) * win;
+      for (int j = 0; j < win; ++j) sw[j] = input(track - win + j);
+    }
+    for (int j = 0; j < win; ++j) w[j] = input(n - win + j);          // reads w[j + n] before w[j + n] is overwritten
+  };
+  for (int i = threadIdx.x; i < V; i += threads) window(2 * p.Hk * D + h * V + i);
+  if (h % (p.H / p.Hk) == 0)
+    for (int i = threadIdx.x; i < D; i += threads) {
+      window(hk * D + i);
+      window(p.Hk * D + hk * D + i);
+    }
+}
+
+// Prefill: one CTA per (sequence, head, 32 columns of the state).  Thread (rg, cp) of 16 x 16 owns RPT rows and the two
+// columns 2 cp, 2 cp + 1 of the state (registers, mirrored in shared memory as the operand of the next chunk).  Per chunk:
+//   Y = [K; Q] S                    rows 4 rg .. of the 64: warps 0-3 turn K S into the right-hand side, 4-7 keep G Q S
+//   U = (I + A)^-1 diag(beta) (V - G K S)
+//   O = G Q S + B U                 warps 4-7;         S <- G S + K^T diag(g_C) U   all warps
+template <int RPT>
 struct ScanShape {
-  static constexpr int kBlk = CHUNK < kBlock ? CHUNK : kBlock;
-  static constexpr int kBufs = CHUNK == 1 ? 1 : 2;
-  static constexpr int kDp = kLanes * RPL;
-  static constexpr int kCols = (kScanThreads / kLanes) * CPL;
-  static constexpr int kScal = 4 + 2 * kBlock;         // decay, beta, -, - | dots
-  static constexpr int kStageFloats = CHUNK * (2 * kDp + kCols + kScal);
-  static constexpr int kSmem = kBufs * kStageFloats * 4;
+  static constexpr int kDp = 16 * RPT, kLd = kDp + 4;
+  static constexpr int kK = kC * kLd;                  // one buffer of k (two of them), and the one of q
+  static constexpr int kCo = kC * kGramLd;             // T', B
+  static constexpr int kFloats = 3 * kK + kC * kCols + 2 * kCo + 2 * 2 * kC + kDp * kCols + 2 * kC * kCols;
+  static constexpr int kSmem = kFloats * 4;
 };
 
-template <typename T, int RPL, int CPL, int CHUNK>
-__global__ void __launch_bounds__(kScanThreads)
-delta_scan_kernel(const DeltaParams p) {
-  using Sh = ScanShape<RPL, CPL, CHUNK>;
-  constexpr int BLK = Sh::kBlk;
+template <typename T, int RPT>
+__global__ void __launch_bounds__(kScanThreads, RPT <= 8 ? 2 : 1) delta_scan_kernel(const DeltaParams p) {
+  using Sh = ScanShape<RPT>;
+  constexpr int ld = Sh::kLd;
   extern __shared__ float4 sm4[];
-  float* sm = reinterpret_cast<float*>(sm4);
+  float* ks = reinterpret_cast<float*>(sm4);           // [2][kC][ld]
+  float* qs = ks + 2 * Sh::kK;                         // [kC][ld]
+  float* vs = qs + Sh::kK;                             // [kC][kCols]
+  float* ts = vs + kC * kCols;                         // [kC][kGramLd]  (I + A)^-1 diag(beta)
+  float* bs = ts + Sh::kCo;                            // [kC][kGramLd]
+  float* vec = bs + Sh::kCo;                           // [2][G_t | g_Cj]
+  float* ss = vec + 4 * kC;                            // [kDp][kCols]
+  float* us = ss + Sh::kDp * kCols;                    // [kC][kCols]
+  float* rs = us + kC * kCols;                         // [kC][kCols]    right-hand side, then diag(g_C) U
   pdl_wait();
-  const int tid = threadIdx.x, lane = tid & 31, rl = lane & (kLanes - 1);
-  const int b = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * Sh::kCols;
-  const int hk = h / (p.H / p.Hk);
-  const int start = p.cu != nullptr ? p.cu[b] : b;
-  const int n = p.cu != nullptr ? p.cu[b + 1] - start : 1;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, cp = (lane & 15) * 2, rg = warp * 2 + (lane >> 4);
+  const int b = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * kCols, hk = h / (p.H / p.Hk);
+  const int start = p.cu[b], n = p.cu[b + 1] - start, D = p.D, V = p.V;
   if (n <= 0) return;
-  const bool fresh = p.prefix != nullptr && p.prefix[b] == 0;
-  const long long slot = p.slots[b];
+  const bool fresh = p.prefix[b] == 0;
   const int track = p.track_len != nullptr ? p.track_len[b] : 0;
-  const int D = p.D, V = p.V;
-  const int col = ((tid >> 5) * (32 / kLanes) + (lane / kLanes)) * CPL;      // first of this lane's columns in the CTA
+  const Chunks ch(n, track);
+  const int nch = ch.count();
   const long long plane = static_cast<long long>(D) * V;
-  float* st = p.state + (slot * p.H + h) * plane;
-  const int gc = c0 + col;                             // the same in the head
-  const bool vec = CPL > 1 && V % CPL == 0;            // whole column groups: wide accesses
+  float* st = p.state + (p.slots[b] * p.H + h) * plane;
+  const float* coef = p.coef + (static_cast<long long>(chunk_base(start, b)) * p.H + h) * kCoefs;
 
-  // rows of this lane: groups of four, row = 4 * (i * kLanes + rl) + e
-  auto row_of = [&](int i) { return 4 * ((i >> 2) * kLanes + rl) + (i & 3); };
-  float S[RPL][CPL];
-  auto store_state = [&](float* dst, const float (&M)[RPL][CPL]) {
+  float S[RPT][2];
 #pragma unroll
-    for (int i = 0; i < RPL; ++i) {
-      const int r = row_of(i);
-      float* d = dst + static_cast<long long>(r) * V + gc;
-      if (r >= D || gc >= V) continue;
-      if constexpr (CPL == 4) {
-        if (vec) { *reinterpret_cast<float4*>(d) = make_float4(M[i][0], M[i][1], M[i][2], M[i][3]); continue; }
-      }
-      if constexpr (CPL == 2) {
-        if (vec) { *reinterpret_cast<float2*>(d) = make_float2(M[i][0], M[i][1]); continue; }
-      }
+  for (int i = 0; i < RPT; ++i) {
+    const int r = rg * RPT + i;
 #pragma unroll
-      for (int c = 0; c < CPL; ++c)
-        if (gc + c < V) d[c] = M[i][c];
+    for (int c = 0; c < 2; ++c)
+      S[i][c] = (!fresh && r < D && c0 + cp + c < V) ? st[static_cast<long long>(r) * V + c0 + cp + c] : 0.f;
+    *reinterpret_cast<float2*>(ss + r * kCols + cp) = make_float2(S[i][0], S[i][1]);
+  }
+  auto store = [&](float* dst) {
+#pragma unroll
+    for (int i = 0; i < RPT; ++i) {
+      const int r = rg * RPT + i;
+#pragma unroll
+      for (int c = 0; c < 2; ++c)
+        if (r < D && c0 + cp + c < V) dst[static_cast<long long>(r) * V + c0 + cp + c] = S[i][c];
     }
   };
+  for (int i = tid; i < 3 * kC * (ld - D); i += kScanThreads) ks[(i / (ld - D)) * ld + D + i % (ld - D)] = 0.f;
+
+  auto stage_tokens = [&](int ci) {                    // k, q, v and the decays of chunk ci
+    const int row0 = start + ch.first(ci), m = ch.len(ci);
+    stage_rows<kScanThreads>(ks + (ci & 1) * Sh::kK, ld, p, row0, hk, 1, m);
+    stage_rows<kScanThreads>(qs, ld, p, row0, hk, 0, m);
+    for (int i = tid; i < kC * kCols; i += kScanThreads) {
+      const int t = i / kCols, e = i % kCols;
+      const bool in = t < m && c0 + e < V;
+      cp_async4(vs + i, p.v + (static_cast<long long>(row0 + (in ? t : 0)) * p.H + h) * V + (in ? c0 + e : 0), in ? 4 : 0);
+    }
+    const float* src = coef + static_cast<long long>(ci) * p.H * kCoefs + kCoefVec;
+    if (tid < 2 * kC / 4) cp_async16(vec + (ci & 1) * 2 * kC + tid * 4, src + tid * 4);
+    cp_commit();
+  };
+  auto stage_coefs = [&](int ci) {
+    const float* src = coef + static_cast<long long>(ci) * p.H * kCoefs;
+    for (int i = tid; i < 2 * kC * kC / 4; i += kScanThreads) {
+      const int row = i / (kC / 4), e = (i % (kC / 4)) * 4;              // rows 0..kC-1 of T', then of B
+      cp_async16(ts + row * kGramLd + e, src + row * kC + e);
+    }
+    cp_commit();
+  };
+
+  stage_tokens(0);
+  stage_coefs(0);
+  for (int ci = 0; ci < nch; ++ci) {
+    const float* kb = ks + (ci & 1) * Sh::kK;
+    const float* gv = vec + (ci & 1) * 2 * kC;
+    cp_wait<1>();                                      // the tokens; the coefficients may still be on their way
+    __syncthreads();
+    float y[4][2];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) y[i][0] = y[i][1] = 0.f;
+    {
+      const float* a = (rg < 8 ? kb + rg * 4 * ld : qs + (rg - 8) * 4 * ld);
+#pragma unroll 4
+      for (int d = 0; d < Sh::kDp; d += 4) {
+        float4 x[4];
+        float2 z[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          x[i] = *reinterpret_cast<const float4*>(a + i * ld + d);
+          z[i] = *reinterpret_cast<const float2*>(ss + (d + i) * kCols + cp);
+        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          y[i][0] += x[i].x * z[0].x + x[i].y * z[1].x + x[i].z * z[2].x + x[i].w * z[3].x;
+          y[i][1] += x[i].x * z[0].y + x[i].y * z[1].y + x[i].z * z[2].y + x[i].w * z[3].y;
+        }
+      }
+    }
+    const int t4 = (rg & 7) * 4;                       // first of this thread's four tokens
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float G = gv[t4 + i];
+      y[i][0] *= G;
+      y[i][1] *= G;
+      if (rg < 8) {
+        const float2 v = *reinterpret_cast<const float2*>(vs + (t4 + i) * kCols + cp);
+        *reinterpret_cast<float2*>(rs + (t4 + i) * kCols + cp) = make_float2(v.x - y[i][0], v.y - y[i][1]);
+      }
+    }
+    cp_wait<0>();
+    __syncthreads();
+    if (ci + 1 < nch) stage_tokens(ci + 1);            // q, v and the other k buffer are free
+    {
+      float u[2][2] = {{0.f, 0.f}, {0.f, 0.f}};
+      const int t2 = rg * 2;
+      for (int j = 0; j <= 4 * warp; j += 4) {         // T' is lower triangular; this warp's rows end at 4 warp + 3
+        float4 x[2];
+        float2 z[4];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) x[i] = *reinterpret_cast<const float4*>(ts + (t2 + i) * kGramLd + j);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) z[i] = *reinterpret_cast<const float2*>(rs + (j + i) * kCols + cp);
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          u[i][0] += x[i].x * z[0].x + x[i].y * z[1].x + x[i].z * z[2].x + x[i].w * z[3].x;
+          u[i][1] += x[i].x * z[0].y + x[i].y * z[1].y + x[i].z * z[2].y + x[i].w * z[3].y;
+        }
+      }
+      __syncthreads();                                 // everyone is done with the right-hand side
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const float w = gv[kC + t2 + i];
+        *reinterpret_cast<float2*>(us + (t2 + i) * kCols + cp) = make_float2(u[i][0], u[i][1]);
+        *reinterpret_cast<float2*>(rs + (t2 + i) * kCols + cp) = make_float2(w * u[i][0], w * u[i][1]);
+      }
+    }
+    __syncthreads();
+    if (warp >= 4) {
+      for (int j = 0; j < 8 * (warp - 3); j += 4) {    // B is lower triangular; this warp's tokens end at 8 (warp - 3) - 1
+        float4 x[4];
+        float2 z[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          x[i] = *reinterpret_cast<const float4*>(bs + (t4 + i) * kGramLd + j);
+          z[i] = *reinterpret_cast<const float2*>(us + (j + i) * kCols + cp);
+        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          y[i][0] += x[i].x * z[0].x + x[i].y * z[1].x + x[i].z * z[2].x + x[i].w * z[3].x;
+          y[i][1] += x[i].x * z[0].y + x[i].y * z[1].y + x[i].z * z[2].y + x[i].w * z[3].y;
+        }
+      }
+      const int row0 = start + ch.first(ci), m = ch.len(ci);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        if (t4 + i >= m) continue;
+        float* o = p.o + (static_cast<long long>(row0 + t4 + i) * p.H + h) * V + c0 + cp;
+        if (c0 + cp < V) o[0] = y[i][0];
+        if (c0 + cp + 1 < V) o[1] = y[i][1];
+      }
+    }
+    const float G = gv[kC - 1];
+#pragma unroll
+    for (int i = 0; i < RPT; ++i) {
+      S[i][0] *= G;
+      S[i][1] *= G;
+    }
+#pragma unroll 4
+    for (int j = 0; j < kC; ++j) {
+      const float2 w = *reinterpret_cast<const float2*>(rs + j * kCols + cp);
+#pragma unroll
+      for (int i = 0; i < RPT; i += 4) {
+        const float4 k = *reinterpret_cast<const float4*>(kb + j * ld + rg * RPT + i);
+        S[i][0] += k.x * w.x;
+        S[i][1] += k.x * w.y;
+        S[i + 1][0] += k.y * w.x;
+        S[i + 1][1] += k.y * w.y;
+        S[i + 2][0] += k.z * w.x;
+        S[i + 2][1] += k.z * w.y;
+        S[i + 3][0] += k.w * w.x;
+        S[i + 3][1] += k.w * w.y;
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < RPT; ++i)
+      *reinterpret_cast<float2*>(ss + (rg * RPT + i) * kCols + cp) = make_float2(S[i][0], S[i][1]);
+    if (track > 0 && ch.first(ci) + ch.len(ci) == track)
+      store(p.state + (static_cast<long long>(p.track_slot[b]) * p.H + h) * plane);
+    __syncthreads();
+    if (ci + 1 < nch) stage_coefs(ci + 1);
+  }
+  store(st);
+  if (blockIdx.z == 0) write_windows<T>(p, b, h, start, n, fresh, track, kScanThreads);
+}
+
+// Decode: one token per request.  Eight lanes share a column group, RPL rows and CPL adjacent columns of the state per
+// lane (D <= 8 * RPL); a CTA owns 16 * CPL columns of one (request, head).  The state streams through once.
+constexpr int kLanes = 8;
+constexpr int kStepThreads = 128;
+
+template <typename T, int RPL, int CPL>
+__global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaParams p) {
+  __shared__ __align__(16) float qk[2][kLanes * RPL];
+  pdl_wait();
+  const int tid = threadIdx.x, lane = tid & 31, rl = lane & (kLanes - 1);
+  const int b = blockIdx.x, h = blockIdx.y, hk = h / (p.H / p.Hk), D = p.D, V = p.V;
+  const int gc = blockIdx.z * (kStepThreads / kLanes) * CPL + ((tid >> 5) * (32 / kLanes) + lane / kLanes) * CPL;
+  const bool vec = V % CPL == 0;                       // whole column groups: wide accesses
+  float* st = p.state + (p.slots[b] * p.H + h) * static_cast<long long>(D) * V;
+  float S[RPL][CPL];
+  auto row_of = [&](int i) { return 4 * ((i >> 2) * kLanes + rl) + (i & 3); };
 #pragma unroll
   for (int i = 0; i < RPL; ++i) {
     const int r = row_of(i);
     const float* d = st + static_cast<long long>(r) * V + gc;
 #pragma unroll
     for (int c = 0; c < CPL; ++c) S[i][c] = 0.f;
-    if (fresh || r >= D || gc >= V) continue;
-    if constexpr (CPL == 4) {
-      if (vec) {
-        const float4 v = *reinterpret_cast<const float4*>(d);
-        S[i][0] = v.x; S[i][1] = v.y; S[i][2] = v.z; S[i][3] = v.w;
-        continue;
-      }
-    }
-    if constexpr (CPL == 2) {
-      if (vec) {
-        const float2 v = *reinterpret_cast<const float2*>(d);
-        S[i][0] = v.x; S[i][1] = v.y;
-        continue;
-      }
-    }
-#pragma unroll
-    for (int c = 0; c < CPL; ++c)
-      if (gc + c < V) S[i][c] = d[c];
-  }
-  // padding rows and columns, and the places of missing tokens, stay zero
-  for (int i = tid; i < Sh::kBufs * Sh::kStageFloats; i += kScanThreads) sm[i] = 0.f;
-  __syncthreads();
-
-  auto stage = [&](int buf, int t0) {
-    float* base = sm + buf * Sh::kStageFloats;
-    const int m = min(CHUNK, n - t0);
-    float* vs = base + CHUNK * 2 * Sh::kDp;
-    float* ss = vs + CHUNK * Sh::kCols;
-    const long long tok = static_cast<long long>(p.Hk) * 2 * D;
-    const float* qk = p.qk + (start + t0) * tok + static_cast<long long>(hk) * 2 * D;
-    // a warp per (token, q | k) vector
-    for (int x = tid >> 5; x < 2 * m; x += kScanThreads / 32) {
-      const float* src = qk + (x >> 1) * tok + (x & 1) * D;
-      float* dst = base + x * Sh::kDp;
-      if (D % 4 == 0)
-        for (int e = lane * 4; e < D; e += 128) cp_async16(dst + e, src + e);
-      else
-        for (int e = lane; e < D; e += 32) cp_async4(dst + e, src + e);
-    }
-    for (int i = tid; i < m * Sh::kCols; i += kScanThreads) {
-      const int tk = i / Sh::kCols, e = i % Sh::kCols;
-      if (c0 + e < V) cp_async4(vs + i, p.v + (static_cast<long long>(start + t0 + tk) * p.H + h) * V + c0 + e);
-    }
-    if (tid < m) {
-      const long long th = start + t0 + tid;
-      cp_async4(ss + tid * Sh::kScal, p.gb + (th * p.H + h) * 2);
-      cp_async4(ss + tid * Sh::kScal + 1, p.gb + (th * p.H + h) * 2 + 1);
-      if (BLK > 1) {
-        cp_async16(ss + tid * Sh::kScal + 4, p.dots + (th * p.Hk + hk) * 2 * kBlock);
-        cp_async16(ss + tid * Sh::kScal + 8, p.dots + (th * p.Hk + hk) * 2 * kBlock + 4);
-      }
-    }
-    cp_commit();
-  };
-
-  stage(0, 0);
-  for (int t0 = 0, buf = 0; t0 < n; t0 += CHUNK, buf ^= (Sh::kBufs - 1)) {
-    if (Sh::kBufs == 2 && t0 + CHUNK < n) {
-      stage(buf ^ 1, t0 + CHUNK);
-      cp_wait<1>();
+    if (r >= D || gc >= V) continue;
+    if (CPL == 4 && vec) {
+      const float4 v = *reinterpret_cast<const float4*>(d);
+      S[i][0] = v.x; S[i][1 % CPL] = v.y; S[i][2 % CPL] = v.z; S[i][3 % CPL] = v.w;
+    } else if (CPL == 2 && vec) {
+      const float2 v = *reinterpret_cast<const float2*>(d);
+      S[i][0] = v.x; S[i][1 % CPL] = v.y;
     } else {
-      cp_wait<0>();
-    }
-    __syncthreads();
-    const float* base = sm + buf * Sh::kStageFloats;
-    const float* vs = base + CHUNK * 2 * Sh::kDp;
-    const float* ss = vs + CHUNK * Sh::kCols;
-    const int m = min(CHUNK, n - t0);
-#pragma unroll 1
-    for (int t = 0; t < m; t += BLK) {
-      const int nb = min(BLK, m - t);                  // tokens of this block
-      float kd[BLK][CPL], qd[BLK][CPL];
-      float self = 0.f;                                // k . q of a single token
 #pragma unroll
-      for (int j = 0; j < BLK; ++j) {
-#pragma unroll
-        for (int c = 0; c < CPL; ++c) kd[j][c] = qd[j][c] = 0.f;
-        const float4* qv = reinterpret_cast<const float4*>(base + (t + j) * 2 * Sh::kDp) + rl;
-        const float4* kv = reinterpret_cast<const float4*>(base + (t + j) * 2 * Sh::kDp + Sh::kDp) + rl;
-#pragma unroll
-        for (int i = 0; i < RPL; i += 4) {
-          const float4 k4 = kv[(i >> 2) * kLanes], q4 = qv[(i >> 2) * kLanes];
-#pragma unroll
-          for (int c = 0; c < CPL; ++c) {
-            kd[j][c] += S[i][c] * k4.x + S[i + 1][c] * k4.y + S[i + 2][c] * k4.z + S[i + 3][c] * k4.w;
-            qd[j][c] += S[i][c] * q4.x + S[i + 1][c] * q4.y + S[i + 2][c] * q4.z + S[i + 3][c] * q4.w;
-          }
-          if (BLK == 1) self += k4.x * q4.x + k4.y * q4.y + k4.z * q4.z + k4.w * q4.w;
-        }
-      }
-#pragma unroll
-      for (int o = kLanes / 2; o > 0; o >>= 1) {
-#pragma unroll
-        for (int j = 0; j < BLK; ++j)
-#pragma unroll
-          for (int c = 0; c < CPL; ++c) {
-            kd[j][c] += __shfl_xor_sync(0xffffffffu, kd[j][c], o);
-            qd[j][c] += __shfl_xor_sync(0xffffffffu, qd[j][c], o);
-          }
-        if (BLK == 1) self += __shfl_xor_sync(0xffffffffu, self, o);
-      }
-      float u[BLK][CPL], g[BLK];
-#pragma unroll
-      for (int j = 0; j < BLK; ++j) {
-        const float* sc = ss + (t + j) * Sh::kScal;
-        g[j] = j < nb ? sc[0] : 1.f;
-        const float beta = j < nb ? sc[1] : 0.f;
-        // decay[i] = product of g over tokens i + 1 .. j, decay of the state itself in front of them
-        float from[BLK], G = g[j];
-        from[j] = 1.f;
-#pragma unroll
-        for (int i = j - 1; i >= 0; --i) {
-          from[i] = G;
-          G *= g[i];
-        }
-        float out[CPL];
-#pragma unroll
-        for (int c = 0; c < CPL; ++c) {
-          float a = G * kd[j][c];
-          out[c] = G * qd[j][c];
-#pragma unroll
-          for (int i = 0; i < j; ++i) {
-            a += from[i] * sc[4 + i] * u[i][c];
-            out[c] += from[i] * sc[4 + kBlock + i] * u[i][c];
-          }
-          u[j][c] = beta * (vs[(t + j) * Sh::kCols + col + c] - a);
-          out[c] += (BLK == 1 ? self : sc[4 + kBlock + j]) * u[j][c];
-        }
-        if (rl == 0 && j < nb) {
-          float* d = p.o + (static_cast<long long>(start + t0 + t + j) * p.H + h) * V + gc;
-#pragma unroll
-          for (int c = 0; c < CPL; ++c)
-            if (gc + c < V) d[c] = out[c];
-        }
-      }
-      // the state after the block's first `upto` tokens
-      auto advance = [&](int upto, float (&M)[RPL][CPL]) {
-        float w[BLK], G = 1.f;
-#pragma unroll
-        for (int j = BLK - 1; j >= 0; --j) {
-          w[j] = j < upto ? G : 0.f;
-          if (j < upto) G *= g[j];
-        }
-#pragma unroll
-        for (int i = 0; i < RPL; ++i)
-#pragma unroll
-          for (int c = 0; c < CPL; ++c) M[i][c] = G * S[i][c];
-#pragma unroll
-        for (int j = 0; j < BLK; ++j) {
-          const float4* kv = reinterpret_cast<const float4*>(base + (t + j) * 2 * Sh::kDp + Sh::kDp) + rl;
-          float wu[CPL];
-#pragma unroll
-          for (int c = 0; c < CPL; ++c) wu[c] = w[j] * u[j][c];
-#pragma unroll
-          for (int i = 0; i < RPL; i += 4) {
-            const float4 k4 = kv[(i >> 2) * kLanes];
-#pragma unroll
-            for (int c = 0; c < CPL; ++c) {
-              M[i][c] += k4.x * wu[c];
-              M[i + 1][c] += k4.y * wu[c];
-              M[i + 2][c] += k4.z * wu[c];
-              M[i + 3][c] += k4.w * wu[c];
-            }
-          }
-        }
-      };
-      if (track > t0 + t && track <= t0 + t + nb) {
-        float M[RPL][CPL];
-        advance(track - t0 - t, M);
-        store_state(p.state + (static_cast<long long>(p.track_slot[b]) * p.H + h) * plane, M);
-      }
-      advance(nb, S);
-    }
-    __syncthreads();                                   // this buffer is refilled in the next round
-  }
-  store_state(st, S);
-
-  // convolution windows of this head's channels (the q / k channels by the first value head that uses them)
-  if (blockIdx.z == 0) {
-    const int win = p.taps - 1, channels = 2 * p.Hk * D + p.H * V;
-    const T* proj = static_cast<const T*>(p.proj) + start * p.ld;
-    T* cs = static_cast<T*>(p.conv_state);
-    T* own = cs + slot * channels * win;
-    auto window = [&](int c) {
-      T* w = own + static_cast<long long>(c) * win;
-      auto input = [&](int i) {                        // input number i of this step (negative: before it)
-        return i >= 0 ? proj[i * p.ld + c] : (fresh ? from_f<T>(0.f) : w[win + i]);
-      };
-      if (track > 0 && track <= n) {
-        T* sw = cs + (static_cast<long long>(p.track_slot[b]) * channels + c) * win;
-        for (int j = 0; j < win; ++j) sw[j] = input(track - win + j);
-      }
-      for (int j = 0; j < win; ++j) w[j] = input(n - win + j);      // reads w[j + n] before w[j + n] is overwritten
-    };
-    for (int i = tid; i < V; i += kScanThreads) window(2 * p.Hk * D + h * V + i);
-    if (h % (p.H / p.Hk) == 0) {
-      for (int i = tid; i < D; i += kScanThreads) {
-        window(hk * D + i);
-        window(p.Hk * D + hk * D + i);
-      }
+      for (int c = 0; c < CPL; ++c)
+        if (gc + c < V) S[i][c] = d[c];
     }
   }
+  for (int i = tid; i < 2 * kLanes * RPL; i += kStepThreads) {
+    const int which = i / (kLanes * RPL), e = i - which * kLanes * RPL;
+    qk[which][e] = e < D ? p.qk[((static_cast<long long>(b) * p.Hk + hk) * 2 + which) * D + e] : 0.f;
+  }
+  __syncthreads();
+  const long long bh = static_cast<long long>(b) * p.H + h;
+  const float g = p.gb[bh * 2], beta = p.gb[bh * 2 + 1];
+  float kd[CPL], qd[CPL], kq = 0.f, kr[RPL];
+#pragma unroll
+  for (int c = 0; c < CPL; ++c) kd[c] = qd[c] = 0.f;
+#pragma unroll
+  for (int i = 0; i < RPL; i += 4) {
+    const float4 q = *reinterpret_cast<const float4*>(&qk[0][row_of(i)]), k = *reinterpret_cast<const float4*>(&qk[1][row_of(i)]);
+    kr[i] = k.x; kr[i + 1] = k.y; kr[i + 2] = k.z; kr[i + 3] = k.w;
+    kq += k.x * q.x + k.y * q.y + k.z * q.z + k.w * q.w;
+#pragma unroll
+    for (int c = 0; c < CPL; ++c) {
+      kd[c] += S[i][c] * k.x + S[i + 1][c] * k.y + S[i + 2][c] * k.z + S[i + 3][c] * k.w;
+      qd[c] += S[i][c] * q.x + S[i + 1][c] * q.y + S[i + 2][c] * q.z + S[i + 3][c] * q.w;
+    }
+  }
+#pragma unroll
+  for (int o = kLanes / 2; o > 0; o >>= 1) {
+    kq += __shfl_xor_sync(0xffffffffu, kq, o);
+#pragma unroll
+    for (int c = 0; c < CPL; ++c) {
+      kd[c] += __shfl_xor_sync(0xffffffffu, kd[c], o);
+      qd[c] += __shfl_xor_sync(0xffffffffu, qd[c], o);
+    }
+  }
+#pragma unroll
+  for (int c = 0; c < CPL; ++c) {
+    const float v = gc + c < V ? p.v[bh * V + gc + c] : 0.f;
+    const float u = beta * (v - g * kd[c]);
+    // o = S'^T q with S' = g S + k u^T, that is g (S^T q) + u (k . q)
+    if (rl == 0 && gc + c < V) p.o[bh * V + gc + c] = g * qd[c] + u * kq;
+#pragma unroll
+    for (int i = 0; i < RPL; ++i) S[i][c] = g * S[i][c] + kr[i] * u;
+  }
+#pragma unroll
+  for (int i = 0; i < RPL; ++i) {
+    const int r = row_of(i);
+    float* d = st + static_cast<long long>(r) * V + gc;
+    if (r >= D || gc >= V) continue;
+    if (CPL == 4 && vec) {
+      *reinterpret_cast<float4*>(d) = make_float4(S[i][0], S[i][1 % CPL], S[i][2 % CPL], S[i][3 % CPL]);
+    } else if (CPL == 2 && vec) {
+      *reinterpret_cast<float2*>(d) = make_float2(S[i][0], S[i][1 % CPL]);
+    } else {
+#pragma unroll
+      for (int c = 0; c < CPL; ++c)
+        if (gc + c < V) d[c] = S[i][c];
+    }
+  }
+  if (blockIdx.z == 0) write_windows<T>(p, b, h, b, 1, false, 0, kStepThreads);
 }
 
 // One warp per (token, head); a lane holds NV groups of four adjacent columns (V <= 128 * NV, V % 4 == 0), or takes single
@@ -634,32 +785,45 @@ int launch_prep(const DeltaParams& p, cudaStream_t s) {
   return static_cast<int>(cudaGetLastError());
 }
 
-template <typename T, int RPL, int CPL, int CHUNK>
+template <typename K>
+int set_smem(K kernel, int smem, bool* done) {
+  if (*done) return 0;
+  const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  if (e == cudaSuccess) *done = true;
+  return static_cast<int>(e);
+}
+
+template <typename T, int RPT>
 int launch_scan(const DeltaParams& p, cudaStream_t s) {
-  using Sh = ScanShape<RPL, CPL, CHUNK>;
-  static bool cfg = false;
-  if (!cfg) {
-    const cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<T, RPL, CPL, CHUNK>,
-                                               cudaFuncAttributeMaxDynamicSharedMemorySize, Sh::kSmem);
-    if (e != cudaSuccess) return static_cast<int>(e);
-    cfg = true;
-  }
-  launch_pdl(delta_scan_kernel<T, RPL, CPL, CHUNK>, dim3(p.B, p.H, (p.V + Sh::kCols - 1) / Sh::kCols),
-             dim3(kScanThreads), Sh::kSmem, s, p);
+  using Sh = ScanShape<RPT>;
+  static bool cfg = false, cfg_chunk = false;
+  const int chunk_smem = (2 * kC * Sh::kLd + 2 * kC * kGramLd + kChunkThreads) * 4;
+  int e = set_smem(delta_chunk_kernel, (2 * kC * ScanShape<16>::kLd + 2 * kC * kGramLd + kChunkThreads) * 4, &cfg_chunk);
+  if (e == 0) e = set_smem(delta_scan_kernel<T, RPT>, Sh::kSmem, &cfg);
+  if (e != 0) return e;
+  launch_pdl(delta_chunk_kernel, dim3(chunk_base(p.T, p.B), p.Hk), dim3(kChunkThreads), chunk_smem, s, p,
+             static_cast<int>(Sh::kDp));
+  e = static_cast<int>(cudaGetLastError());
+  if (e != 0) return e;
+  launch_pdl(delta_scan_kernel<T, RPT>, dim3(p.B, p.H, (p.V + kCols - 1) / kCols), dim3(kScanThreads), Sh::kSmem, s, p);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T, int RPL, int CPL>
+int launch_step(const DeltaParams& p, cudaStream_t s) {
+  constexpr int cols = (kStepThreads / kLanes) * CPL;
+  launch_pdl(delta_step_kernel<T, RPL, CPL>, dim3(p.B, p.H, (p.V + cols - 1) / cols), dim3(kStepThreads), 0, s, p);
   return static_cast<int>(cudaGetLastError());
 }
 
 template <typename T, int RPL>
-int launch_rows(const DeltaParams& p, cudaStream_t s) {
-  const long long groups = static_cast<long long>(p.B) * p.H * ((p.V + 15) / 16);      // 16-column slices of all states
-  if (p.cu == nullptr) {                               // one token each: the state streams through once
-    if (RPL <= 16 && groups >= 148 * 32) return launch_scan<T, RPL, (RPL <= 16 ? 4 : 1), 1>(p, s);
-    if (RPL <= 16 && groups >= 148 * 8) return launch_scan<T, RPL, (RPL <= 16 ? 2 : 1), 1>(p, s);
-    return launch_scan<T, RPL, 1, 1>(p, s);
-  }
-  // two columns per lane once that still leaves the machine full: fewer shared-memory reads per state element
-  if (RPL <= 16 && groups >= 148 * 8) return launch_scan<T, RPL, (RPL <= 16 ? 2 : 1), 16>(p, s);
-  return launch_scan<T, RPL, 1, 16>(p, s);
+int launch_step_rows(const DeltaParams& p, cudaStream_t s) {
+  // wide accesses once there are states enough to fill the machine with the fewer threads
+  const long long groups = static_cast<long long>(p.B) * p.H * ((p.V + 15) / 16);
+  constexpr int kMost = RPL <= 16 ? 4 : 2;
+  if (groups >= 148 * 32) return launch_step<T, RPL, kMost>(p, s);
+  if (groups >= 148 * 8) return launch_step<T, RPL, 2>(p, s);
+  return launch_step<T, RPL, 1>(p, s);
 }
 
 template <typename T>
@@ -671,17 +835,15 @@ int run_delta(const DeltaParams& p, cudaStream_t s) {
   else
     e = wide <= 128 ? launch_prep<T, 4, 16>(p, s) : launch_prep<T, 8, 16>(p, s);
   if (e != 0) return e;
-  if (p.cu != nullptr) {
-    const long long warps = static_cast<long long>(p.T) * p.Hk;
-    launch_pdl(delta_dots_kernel, dim3(static_cast<unsigned>((warps + 3) / 4)), dim3(128), 0, s, p);
-    e = static_cast<int>(cudaGetLastError());
-    if (e != 0) return e;
+  if (p.cu == nullptr) {
+    if (p.D <= 32) return launch_step_rows<T, 4>(p, s);
+    if (p.D <= 64) return launch_step_rows<T, 8>(p, s);
+    if (p.D <= 128) return launch_step_rows<T, 16>(p, s);
+    return launch_step_rows<T, 32>(p, s);
   }
-  const int rows = (p.D + kLanes - 1) / kLanes;
-  if (rows <= 4) return launch_rows<T, 4>(p, s);
-  if (rows <= 8) return launch_rows<T, 8>(p, s);
-  if (rows <= 16) return launch_rows<T, 16>(p, s);
-  return launch_rows<T, 32>(p, s);
+  if (p.D <= 64) return launch_scan<T, 4>(p, s);
+  if (p.D <= 128) return launch_scan<T, 8>(p, s);
+  return launch_scan<T, 16>(p, s);
 }
 
 }  // namespace
@@ -693,13 +855,14 @@ extern "C" {
 int sglb_delta_scan(const void* proj, long long ld, int g_off, int b_off, int a_off, const void* conv_w,
                     const float* a_log, const float* dt_bias, void* conv_state, float* state, const long long* slots,
                     const int* cu, const int* prefix, const int* track_len, const int* track_slot, float* qk, float* v,
-                    float* gb, float* dots, float* o, int B, int T, int H, int Hk, int D, int V, int taps, int is_f32,
+                    float* gb, float* coef, float* o, int B, int T, int H, int Hk, int D, int V, int taps, int is_f32,
                     cudaStream_t s) {
   using namespace sglb;
   if (B <= 0 || T <= 0) return 0;
-  if (D < 1 || D > 32 * kLanes || V < 1 || Hk < 1 || H % Hk != 0 || taps < 1 || taps > 16 || H > 65535) return -kBadArgument;
+  if (cu != nullptr && (prefix == nullptr || coef == nullptr)) return -kBadArgument;
+  if (D < 1 || D > 256 || V < 1 || Hk < 1 || H % Hk != 0 || taps < 1 || taps > 16 || H > 65535) return -kBadArgument;
   DeltaParams p{proj, ld, g_off, b_off, a_off, conv_w, a_log, dt_bias, conv_state, state, slots, cu, prefix, track_len,
-                track_slot, qk, v, gb, dots, o, B, T, H, Hk, D, V, taps};
+                track_slot, qk, v, gb, coef, o, B, T, H, Hk, D, V, taps};
   return is_f32 ? run_delta<float>(p, s) : run_delta<__nv_bfloat16>(p, s);
 }
 

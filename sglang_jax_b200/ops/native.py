@@ -702,11 +702,12 @@ def delta_scan(proj, g_off, b_off, a_off, conv_w, a_log, dt_bias, conv_state, st
     qk = torch.empty((T, kv_heads, 2, dim), **f32)
     v = torch.empty((T, heads, vdim), **f32)
     gb = torch.empty((T, heads, 2), **f32)
-    dots = torch.empty((T, kv_heads, 8), **f32) if cu is not None else None
+    # coefficients of the chunks of 32 tokens: two 32 x 32 blocks and two vectors (sizes in csrc/delta_scan.cu)
+    coef = torch.empty((T // 32 + 2 * slots.numel(), heads, 2112), **f32) if cu is not None else None
     o = torch.empty((T, heads, vdim), **f32)
     _check(lib().sglb_delta_scan(_p(proj), proj.stride(0), g_off, b_off, a_off, _p(conv_w), _p(a_log), _p(dt_bias),
                                  _p(conv_state), _p(state), _p(slots), _p(cu), _p(prefix), _p(track_len), _p(track_slot),
-                                 _p(qk), _p(v), _p(gb), _p(dots), _p(o), slots.numel(), T, heads, kv_heads, dim, vdim,
+                                 _p(qk), _p(v), _p(gb), _p(coef), _p(o), slots.numel(), T, heads, kv_heads, dim, vdim,
                                  conv_w.shape[1], _f32(proj), _stream()), "delta_scan")
     return o
 
