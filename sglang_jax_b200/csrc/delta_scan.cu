@@ -53,6 +53,7 @@ struct DeltaParams {
   float* coef;                   // [T / 32 + 2 B, H, kCoefs], see delta_chunk_kernel
   float* o;                      // [T, H, V]
   int B, T, H, Hk, D, V, taps;
+  int singles;                   // ragged step: how many sequences bring exactly one token (-1: not known)
 };
 
 // One warp per (run of RUN consecutive rows, head): the convolution window slides through registers.  A lane owns the
@@ -157,17 +158,22 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const DeltaParams p) {
     cq.load_kernel(kernel, q0, p.D, taps, lane);
     ck.load_kernel(kernel, k0, p.D, taps, lane);
     const float scale = 1.f / sqrtf(static_cast<float>(p.D));
+    float in_q[NPL], in_k[NPL];
+    rows(t0, q0, p.D, in_q);
+    rows(t0, k0, p.D, in_k);
     walk(
         [&](const T* stored, bool fresh, int start, int local) {
           cq.load_window(proj, p.ld, stored, fresh, start, local, q0, p.D, taps, lane);
           ck.load_window(proj, p.ld, stored, fresh, start, local, k0, p.D, taps, lane);
         },
         [&](int t) {
-          float in[NPL], q[NPL], k[NPL];
-          rows(t, q0, p.D, in);
-          cq.step(in, q);
-          rows(t, k0, p.D, in);
-          ck.step(in, k);
+          float q[NPL], k[NPL];
+          cq.step(in_q, q);
+          ck.step(in_k, k);
+          if (t + 1 < t1) {                            // the next row is on its way while this one is worked on
+            rows(t + 1, q0, p.D, in_q);
+            rows(t + 1, k0, p.D, in_k);
+          }
           float qq = 0.f, kk = 0.f;
 #pragma unroll
           for (int i = 0; i < NPL; ++i) {
@@ -196,14 +202,16 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const DeltaParams p) {
       const int v0 = 2 * p.Hk * p.D + h * p.V + vb, width = min(32 * NPL, p.V - vb);
       Conv<T, NPL, TAPS> cv;
       cv.load_kernel(kernel, v0, width, taps, lane);
+      float in[NPL];
+      rows(t0, v0, width, in);
       walk(
           [&](const T* stored, bool fresh, int start, int local) {
             cv.load_window(proj, p.ld, stored, fresh, start, local, v0, width, taps, lane);
           },
           [&](int t) {
-            float in[NPL], v[NPL];
-            rows(t, v0, width, in);
+            float v[NPL];
             cv.step(in, v);
+            if (t + 1 < t1) rows(t + 1, v0, width, in);
             float* dst = p.v + (static_cast<long long>(t) * p.H + h) * p.V + vb;
 #pragma unroll
             for (int i = 0; i < NPL; ++i)
@@ -306,7 +314,7 @@ __global__ void __launch_bounds__(kChunkThreads) delta_chunk_kernel(const DeltaP
   const int start = p.cu[b];
   const Chunks ch(p.cu[b + 1] - start, p.track_len != nullptr ? p.track_len[b] : 0);
   const int ci = idx - chunk_base(start, b);
-  if (ch.n <= 0 || ci >= ch.count()) return;
+  if (ch.n <= 1 || ci >= ch.count()) return;         // single tokens: delta_step
   const int row0 = start + ch.first(ci), m = ch.len(ci);
   for (int i = tid; i < 2 * kC * (ld - p.D); i += kChunkThreads) rows[(i / (ld - p.D)) * ld + p.D + i % (ld - p.D)] = 0.f;
   stage_rows<kChunkThreads>(rows, ld, p, row0, hk, 1, m);
@@ -439,7 +447,7 @@ __global__ void __launch_bounds__(kScanThreads, RPT <= 8 ? 2 : 1) delta_scan_ker
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, cp = (lane & 15) * 2, rg = warp * 2 + (lane >> 4);
   const int b = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * kCols, hk = h / (p.H / p.Hk);
   const int start = p.cu[b], n = p.cu[b + 1] - start, D = p.D, V = p.V;
-  if (n <= 0) return;
+  if (n <= 1) return;                                  // single tokens: delta_step
   const bool fresh = p.prefix[b] == 0;
   const int track = p.track_len != nullptr ? p.track_len[b] : 0;
   const Chunks ch(n, track);
@@ -615,7 +623,7 @@ __global__ void __launch_bounds__(kScanThreads, RPT <= 8 ? 2 : 1) delta_scan_ker
   if (blockIdx.z == 0) write_windows<T>(p, b, h, start, n, fresh, track, kScanThreads);
 }
 
-// Decode: one token per request.  Eight lanes share a column group, RPL rows and CPL adjacent columns of the state per
+// Decode, and the sequences of a ragged step that bring one token.  Eight lanes share a column group, RPL rows and CPL adjacent columns of the state per
 // lane (D <= 8 * RPL); a CTA owns 16 * CPL columns of one (request, head).  The state streams through once.
 constexpr int kLanes = 8;
 constexpr int kStepThreads = 128;
@@ -626,6 +634,12 @@ __global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaPar
   pdl_wait();
   const int tid = threadIdx.x, lane = tid & 31, rl = lane & (kLanes - 1);
   const int b = blockIdx.x, h = blockIdx.y, hk = h / (p.H / p.Hk), D = p.D, V = p.V;
+  int t = b;
+  if (p.cu != nullptr) {
+    t = p.cu[b];
+    if (p.cu[b + 1] - t != 1) return;
+  }
+  const bool fresh = p.prefix != nullptr && p.prefix[b] == 0;
   const int gc = blockIdx.z * (kStepThreads / kLanes) * CPL + ((tid >> 5) * (32 / kLanes) + lane / kLanes) * CPL;
   const bool vec = V % CPL == 0;                       // whole column groups: wide accesses
   float* st = p.state + (p.slots[b] * p.H + h) * static_cast<long long>(D) * V;
@@ -637,7 +651,7 @@ __global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaPar
     const float* d = st + static_cast<long long>(r) * V + gc;
 #pragma unroll
     for (int c = 0; c < CPL; ++c) S[i][c] = 0.f;
-    if (r >= D || gc >= V) continue;
+    if (fresh || r >= D || gc >= V) continue;
     if (CPL == 4 && vec) {
       const float4 v = *reinterpret_cast<const float4*>(d);
       S[i][0] = v.x; S[i][1 % CPL] = v.y; S[i][2 % CPL] = v.z; S[i][3 % CPL] = v.w;
@@ -652,10 +666,10 @@ __global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaPar
   }
   for (int i = tid; i < 2 * kLanes * RPL; i += kStepThreads) {
     const int which = i / (kLanes * RPL), e = i - which * kLanes * RPL;
-    qk[which][e] = e < D ? p.qk[((static_cast<long long>(b) * p.Hk + hk) * 2 + which) * D + e] : 0.f;
+    qk[which][e] = e < D ? p.qk[((static_cast<long long>(t) * p.Hk + hk) * 2 + which) * D + e] : 0.f;
   }
   __syncthreads();
-  const long long bh = static_cast<long long>(b) * p.H + h;
+  const long long bh = static_cast<long long>(t) * p.H + h;
   const float g = p.gb[bh * 2], beta = p.gb[bh * 2 + 1];
   float kd[CPL], qd[CPL], kq = 0.f, kr[RPL];
 #pragma unroll
@@ -689,22 +703,27 @@ __global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaPar
 #pragma unroll
     for (int i = 0; i < RPL; ++i) S[i][c] = g * S[i][c] + kr[i] * u;
   }
+  auto store = [&](float* dst) {
 #pragma unroll
-  for (int i = 0; i < RPL; ++i) {
-    const int r = row_of(i);
-    float* d = st + static_cast<long long>(r) * V + gc;
-    if (r >= D || gc >= V) continue;
-    if (CPL == 4 && vec) {
-      *reinterpret_cast<float4*>(d) = make_float4(S[i][0], S[i][1 % CPL], S[i][2 % CPL], S[i][3 % CPL]);
-    } else if (CPL == 2 && vec) {
-      *reinterpret_cast<float2*>(d) = make_float2(S[i][0], S[i][1 % CPL]);
-    } else {
+    for (int i = 0; i < RPL; ++i) {
+      const int r = row_of(i);
+      float* d = dst + static_cast<long long>(r) * V + gc;
+      if (r >= D || gc >= V) continue;
+      if (CPL == 4 && vec) {
+        *reinterpret_cast<float4*>(d) = make_float4(S[i][0], S[i][1 % CPL], S[i][2 % CPL], S[i][3 % CPL]);
+      } else if (CPL == 2 && vec) {
+        *reinterpret_cast<float2*>(d) = make_float2(S[i][0], S[i][1 % CPL]);
+      } else {
 #pragma unroll
-      for (int c = 0; c < CPL; ++c)
-        if (gc + c < V) d[c] = S[i][c];
+        for (int c = 0; c < CPL; ++c)
+          if (gc + c < V) d[c] = S[i][c];
+      }
     }
-  }
-  if (blockIdx.z == 0) write_windows<T>(p, b, h, b, 1, false, 0, kStepThreads);
+  };
+  store(st);
+  const int track = p.cu != nullptr && p.track_len != nullptr ? p.track_len[b] : 0;
+  if (track == 1) store(p.state + (static_cast<long long>(p.track_slot[b]) * p.H + h) * static_cast<long long>(D) * V);
+  if (blockIdx.z == 0) write_windows<T>(p, b, h, t, 1, fresh, track, kStepThreads);
 }
 
 // One warp per (token, head); a lane holds NV groups of four adjacent columns (V <= 128 * NV, V % 4 == 0), or takes single
@@ -835,11 +854,10 @@ int run_delta(const DeltaParams& p, cudaStream_t s) {
   else
     e = wide <= 128 ? launch_prep<T, 4, 16>(p, s) : launch_prep<T, 8, 16>(p, s);
   if (e != 0) return e;
-  if (p.cu == nullptr) {
-    if (p.D <= 32) return launch_step_rows<T, 4>(p, s);
-    if (p.D <= 64) return launch_step_rows<T, 8>(p, s);
-    if (p.D <= 128) return launch_step_rows<T, 16>(p, s);
-    return launch_step_rows<T, 32>(p, s);
+  if (p.cu == nullptr || p.singles) {
+    const int r = p.D <= 32 ? launch_step_rows<T, 4>(p, s) : p.D <= 64 ? launch_step_rows<T, 8>(p, s)
+                  : p.D <= 128 ? launch_step_rows<T, 16>(p, s) : launch_step_rows<T, 32>(p, s);
+    if (r != 0 || p.cu == nullptr || p.singles == p.B) return r;
   }
   if (p.D <= 64) return launch_scan<T, 4>(p, s);
   if (p.D <= 128) return launch_scan<T, 8>(p, s);
@@ -855,14 +873,15 @@ extern "C" {
 int sglb_delta_scan(const void* proj, long long ld, int g_off, int b_off, int a_off, const void* conv_w,
                     const float* a_log, const float* dt_bias, void* conv_state, float* state, const long long* slots,
                     const int* cu, const int* prefix, const int* track_len, const int* track_slot, float* qk, float* v,
-                    float* gb, float* coef, float* o, int B, int T, int H, int Hk, int D, int V, int taps, int is_f32,
+                    float* gb, float* coef, float* o, int B, int T, int H, int Hk, int D, int V, int taps, int singles,
+                    int is_f32,
                     cudaStream_t s) {
   using namespace sglb;
   if (B <= 0 || T <= 0) return 0;
-  if (cu != nullptr && (prefix == nullptr || coef == nullptr)) return -kBadArgument;
+  if (cu != nullptr && (prefix == nullptr || (coef == nullptr && singles != B))) return -kBadArgument;
   if (D < 1 || D > 256 || V < 1 || Hk < 1 || H % Hk != 0 || taps < 1 || taps > 16 || H > 65535) return -kBadArgument;
   DeltaParams p{proj, ld, g_off, b_off, a_off, conv_w, a_log, dt_bias, conv_state, state, slots, cu, prefix, track_len,
-                track_slot, qk, v, gb, coef, o, B, T, H, Hk, D, V, taps};
+                track_slot, qk, v, gb, coef, o, B, T, H, Hk, D, V, taps, singles};
   return is_f32 ? run_delta<float>(p, s) : run_delta<__nv_bfloat16>(p, s);
 }
 

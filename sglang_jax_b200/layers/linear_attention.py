@@ -197,7 +197,7 @@ class GatedDeltaRule(nn.Module):
         y = self.proj(h)
         ragged = {}
         if not fb.forward_mode.is_decode():
-            ragged = dict(cu=fb.cu_q_lens, prefix=fb.extend_prefix_lens)
+            ragged = dict(cu=fb.cu_q_lens, prefix=fb.extend_prefix_lens, lens=fb.extend_seq_lens_cpu)
             track = checkpoint_tensors(fb)
             if track is not None:
                 ragged.update(track_len=track[0], track_slot=track[1])

@@ -101,7 +101,7 @@ def lib():
     sig("sglb_latent_extend_supported", [c_int, c_int, c_int])
     sig("sglb_latent_extend", [c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_int]
         + [c_void_p] * 4 + [c_int] * 6 + [c_float, c_void_p])
-    sig("sglb_delta_scan", [c_void_p, c_longlong, c_int, c_int, c_int] + [c_void_p] * 15 + [c_int] * 8 + [c_void_p])
+    sig("sglb_delta_scan", [c_void_p, c_longlong, c_int, c_int, c_int] + [c_void_p] * 15 + [c_int] * 9 + [c_void_p])
     sig("sglb_delta_gate", [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_int, c_int, c_float, c_int,
                             c_void_p])
     sig("sglb_paged_decode", [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p,
@@ -691,11 +691,13 @@ def latent_extend(q, kv, k_rot, out, plan, dim, v_dim, scale):
 
 # ---- gated delta rule over ragged batches (csrc/delta_scan.cu)
 def delta_scan(proj, g_off, b_off, a_off, conv_w, a_log, dt_bias, conv_state, state, slots, heads, kv_heads, dim, vdim,
-               cu=None, prefix=None, track_len=None, track_slot=None):
+               cu=None, prefix=None, track_len=None, track_slot=None, lens=None):
     """Read-outs fp32 `[T, heads, vdim]` of the rows of `proj [T, ld]` (columns `q | k | v` first, gate / beta / decay
     inputs at the given offsets); windows and states of `slots` are updated in place.  `cu [B + 1]` / `prefix [B]`:
-    ragged step (None: one row per request, all of them continuing)."""
-    T, dev = proj.shape[0], proj.device
+    ragged step (None: one row per request, all of them continuing); `lens`: its sequence lengths on the host, if known
+    (without them the kernel for single tokens is launched on the chance that there are some)."""
+    T, dev, B = proj.shape[0], proj.device, slots.numel()
+    singles = 0 if cu is None else (int((lens == 1).sum()) if lens is not None else -1)
     f32 = dict(dtype=torch.float32, device=dev)
     assert proj.stride(1) == 1 and conv_state.is_contiguous() and state.is_contiguous() and conv_w.is_contiguous()
     assert conv_state.dtype == conv_w.dtype == proj.dtype and state.dtype == torch.float32 and slots.dtype == torch.int64
@@ -703,12 +705,12 @@ def delta_scan(proj, g_off, b_off, a_off, conv_w, a_log, dt_bias, conv_state, st
     v = torch.empty((T, heads, vdim), **f32)
     gb = torch.empty((T, heads, 2), **f32)
     # coefficients of the chunks of 32 tokens: two 32 x 32 blocks and two vectors (sizes in csrc/delta_scan.cu)
-    coef = torch.empty((T // 32 + 2 * slots.numel(), heads, 2112), **f32) if cu is not None else None
+    coef = torch.empty((T // 32 + 2 * B, heads, 2112), **f32) if cu is not None else None
     o = torch.empty((T, heads, vdim), **f32)
     _check(lib().sglb_delta_scan(_p(proj), proj.stride(0), g_off, b_off, a_off, _p(conv_w), _p(a_log), _p(dt_bias),
                                  _p(conv_state), _p(state), _p(slots), _p(cu), _p(prefix), _p(track_len), _p(track_slot),
-                                 _p(qk), _p(v), _p(gb), _p(coef), _p(o), slots.numel(), T, heads, kv_heads, dim, vdim,
-                                 conv_w.shape[1], _f32(proj), _stream()), "delta_scan")
+                                 _p(qk), _p(v), _p(gb), _p(coef), _p(o), B, T, heads, kv_heads, dim, vdim,
+                                 conv_w.shape[1], singles, _f32(proj), _stream()), "delta_scan")
     return o
 
 

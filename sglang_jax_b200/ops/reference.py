@@ -369,7 +369,7 @@ def rmsnorm_stream(x, weight, eps, dtype):
 
 
 def delta_scan(proj, g_off, b_off, a_off, conv_w, a_log, dt_bias, conv_state, state, slots, heads, kv_heads, dim, vdim,
-               cu=None, prefix=None, track_len=None, track_slot=None):
+               cu=None, prefix=None, track_len=None, track_slot=None, lens=None):
     """Statement of `native.delta_scan` through the primitives of `ops/linear_attention.py`."""
     from . import linear_attention as la
     B, T, r, kd = slots.numel(), proj.shape[0], heads // kv_heads, kv_heads * dim
