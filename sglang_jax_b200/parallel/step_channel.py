@@ -40,7 +40,8 @@ def _plain(batch) -> bool:
             and not batch.return_output_logprob_only and not any(batch.lora_ids or [])
             and batch.spec_info is None and batch.spec_algorithm is None and batch.input_embeds is None
             and batch.input_embeds_rows is None and batch.mrope_positions is None and batch.deepstack_embeds is None
-            and not batch.recurrent_copies and not batch.recurrent_tracks and batch.extend_logprob_start_lens is None
+            and not batch.recurrent_copies and not batch.recurrent_tracks and batch.logits_rows is None
+            and batch.extend_logprob_start_lens is None
             and batch.launch_done is None
             and (si is None or (si.linear_penalty is None and si.vocab_mask is None and si.logit_bias is None
                                 and getattr(si, "penalties", None) is None)))
