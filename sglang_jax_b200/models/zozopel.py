@@ -55,6 +55,8 @@ class ZozopelForCausalLM(nn.Module):
         super().__init__()
         self.config = config
         self.dtype = dtype
+        # library products (up-projections of single tokens, widths that are not multiples of 8) reduce in fp32, too
+        torch.backends.cuda.matmul.allow_bf16_reduced_precision_reduction = False
         self.embed_tokens = VocabParallelEmbedding(config.vocab_size, config.hidden_size, dtype)
         self.layers = nn.ModuleList()
         kv = lin = 0
@@ -94,7 +96,11 @@ class ZozopelForCausalLM(nn.Module):
     # ------------------------------------------------------------------ loading
     def load_weights(self, weights):
         expected = self._expected_tensors()
+        # a layer without a feed-forward has no use for the second norm, should the file carry one
+        unused = {f"l{i}.{n}" for i, l in enumerate(self.layers) if l.mlp is None for n in ("norm2", "ls2")}
         for name, w in weights:
+            if name in unused:
+                continue
             if name not in expected:
                 raise RuntimeError(f"unexpected tensor {name} in the checkpoint")
             self._load_one(name, w)
