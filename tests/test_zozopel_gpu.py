@@ -89,7 +89,7 @@ def _delta_case(H, Hk, D, V, K, lens, dtype, seed=0):
 
 @pytest.mark.parametrize("dtype", [torch.bfloat16, torch.float32])
 @pytest.mark.parametrize("H,Hk,D,V,K,lens", [
-    (4, 2, 64, 64, 4, [70, 1, 33]), (6, 3, 24, 40, 3, [50, 9, 4]), (2, 1, 128, 128, 4, [130]), (3, 3, 100, 36, 2, [41, 2]),
+    (6, 2, 64, 48, 4, [70, 1, 33]), (6, 3, 24, 40, 3, [50, 9, 4]), (2, 1, 128, 128, 4, [130]), (3, 3, 100, 36, 2, [41, 2]),
     (2, 1, 16, 200, 6, [23]), (2, 2, 256, 64, 1, [20]), (3, 1, 13, 9, 4, [18, 5]), (32, 16, 128, 128, 4, [9] * 40),
     (16, 4, 32, 32, 4, [6] * 150)])
 def test_delta_scan_whole_in_portions_and_token_by_token(native, H, Hk, D, V, K, lens, dtype):
@@ -154,7 +154,7 @@ def _latent_cache(lens, R, rot, P, dtype, seed):
 
 
 @pytest.mark.parametrize("P", [16, 64, 128])
-@pytest.mark.parametrize("R,rot,H", [(512, 64, 16), (64, 32, 6), (128, 32, 17), (48, 8, 3), (320, 64, 4), (21, 6, 3),
+@pytest.mark.parametrize("R,rot,H", [(512, 64, 16), (64, 32, 6), (128, 24, 17), (48, 8, 3), (320, 64, 4), (21, 6, 3),
                                      (256, 16, 33)])
 def test_absorbed_latent_attention_of_any_size(native, R, rot, H, P):
     """bf16 on the tensor cores and fp32 on the CUDA cores; in fp32, and with `exact` weights, far beyond bf16 steps."""
@@ -184,7 +184,7 @@ def test_absorbed_latent_attention_of_any_size(native, R, rot, H, P):
 
 
 @pytest.mark.parametrize("H,dim,rot,v,lens,pres,gain", [
-    (2, 64, 32, 64, [256], [0], 1), (2, 64, 32, 64, [32], [0], 1), (3, 64, 32, 64, [300, 77, 1000], [0, 5, 900], 1),
+    (2, 64, 40, 72, [256], [0], 1), (2, 64, 40, 72, [32], [0], 1), (3, 64, 40, 72, [300, 77, 1000], [0, 5, 900], 1),
     (2, 128, 64, 128, [513, 33], [64, 0], 1), (2, 96, 16, 80, [129], [1], 6), (4, 128, 64, 128, [1024], [0], 8),
     (1, 40, 8, 24, [700], [13], 1), (2, 192, 64, 128, [300], [10], 3)])
 def test_expanded_latent_prefill(native, H, dim, rot, v, lens, pres, gain):

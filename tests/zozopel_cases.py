@@ -36,7 +36,7 @@ CONFIGS = {
     # sizes without any alignment
     "odd": config([latent(3, 10, 6, 11, 21, ff=37), delta(3, 1, 13, 9, 4, ff=37)], 51, 77),
     "delta_only": config([delta(4, 4, 16, 16, 4, ff=64), delta(2, 1, 16, 32, 4)], 64, 96),
-    "latent_only": config([latent(2, 64, 32, 64, 128, base=50.0, ff=64), latent(17, 8, 8, 8, 32)], 64, 96),
+    "latent_only": config([latent(2, 64, 48, 56, 112, base=50.0, ff=64), latent(17, 8, 8, 8, 32)], 64, 96),
 }
 
 
