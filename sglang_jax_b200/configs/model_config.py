@@ -53,7 +53,7 @@ def load_hf_config(model_path: str, trust_remote_code: bool = False, revision: s
         d.update(override)
     if isinstance(d.get("architecture"), str) and "architectures" not in d:
         from .native_formats import translate_native_config
-        d = translate_native_config(d)
+        d = translate_native_config(d, model_path)
     cfg = ConfigNS(**d)
     tc = d.get("text_config")
     if isinstance(tc, dict):

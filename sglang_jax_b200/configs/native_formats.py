@@ -4,9 +4,12 @@ own description (layer list, constants) in place for the model class."""
 
 from __future__ import annotations
 
+import glob
+import json
+import os
 from typing import Callable
 
-_TRANSLATORS: dict[str, Callable[[dict], dict]] = {}
+_TRANSLATORS: dict[str, Callable[[dict, dict], dict]] = {}
 
 
 def native_format(name: str):
@@ -16,11 +19,22 @@ def native_format(name: str):
     return register
 
 
-def translate_native_config(d: dict) -> dict:
+def translate_native_config(d: dict, model_path: str | None = None) -> dict:
+    """`model_path`: the folder of the file; sizes that a design leaves to its tensors are read off the headers there."""
     name = d["architecture"]
     if name not in _TRANSLATORS:
         raise ValueError(f"unknown architecture {name!r} in config.json; known: {sorted(_TRANSLATORS)}")
-    return _TRANSLATORS[name](d)
+    return _TRANSLATORS[name](d, tensor_shapes(model_path) if model_path else {})
+
+
+def tensor_shapes(model_path: str) -> dict[str, list[int]]:
+    """Name -> shape of every tensor in the folder's safetensors files (headers only)."""
+    out = {}
+    for fn in sorted(glob.glob(os.path.join(model_path, "*.safetensors"))):
+        with open(fn, "rb") as f:
+            header = json.loads(f.read(int.from_bytes(f.read(8), "little")))
+        out.update((n, t["shape"]) for n, t in header.items() if n != "__metadata__")
+    return out
 
 
 # positions are computed, not learned, and the file states no limit: the context length used unless one is asked for
@@ -28,7 +42,7 @@ DEFAULT_CONTEXT = 32768
 
 
 @native_format("Zozopel")
-def _zozopel(d: dict) -> dict:
+def _zozopel(d: dict, shapes: dict) -> dict:
     layers = d["layers"]
     known = {"delta": "linear_attention", "latent_attention": "full_attention"}
     for i, e in enumerate(layers):
@@ -46,3 +60,37 @@ def _zozopel(d: dict) -> dict:
         norm_eps=d["norm"]["eps"], embedding_scale=d["embedding"]["scale"], residual_multiplier=d["residual_mult"],
         logit_scale=d["logit_scale"], max_position_embeddings=DEFAULT_CONTEXT, unbounded_positions=True,
         tie_word_embeddings=False, torch_dtype="bfloat16", eos_token_id=None, bos_token_id=None)
+
+
+@native_format("Zidivik")
+def _zidivik(d: dict, shapes: dict) -> dict:
+    known = {"channel_delta": "linear_attention", "attention": "full_attention"}
+    layers = []
+    for i, e in enumerate(d["layers"]):
+        if e["type"] not in known:
+            raise ValueError(f"layer {i}: unknown mixer {e['type']!r}; known: {sorted(known)}")
+        if e.get("mlp") is not None and e["mlp"]["kind"] != "moe":
+            raise ValueError(f"layer {i}: unknown feed-forward {e['mlp']['kind']!r}")
+        m = dict(e["mixer"])
+        if e["type"] == "channel_delta":
+            # widths of the low-rank pairs: only the tensors tell; without any (dummy weights) the key / value width
+            for key, name, default in (("decay_rank", "a1", m["dim"]), ("gate_rank", "g1", m["vdim"])):
+                shape = shapes.get(f"l{i}.mix.{name}")
+                m[key] = shape[0] if shape else m.get(key) or default
+        elif m.get("kv_from") is not None:
+            j = m["kv_from"]
+            if not (0 <= j < i and d["layers"][j]["type"] == "attention" and d["layers"][j]["mixer"].get("kv_from") is None):
+                raise ValueError(f"layer {i}: layer {j} has no keys and values of its own to share")
+        layers.append(dict(e, mixer=m))
+    attn = [e["mixer"] for e in layers if e["type"] == "attention"]
+    first = attn[0] if attn else dict(layers[0]["mixer"])
+    routers = [e["mlp"]["router"] for e in layers if e.get("mlp") is not None]
+    moe = dict(num_experts=max(r["experts"] for r in routers), num_experts_per_tok=max(r["top"] for r in routers)) \
+        if routers else {}
+    return dict(
+        architectures=["ZidivikForCausalLM"], model_type="zidivik", hidden_size=d["width"], vocab_size=d["vocab"],
+        num_hidden_layers=len(layers), num_attention_heads=first["heads"], num_key_value_heads=first["kv_heads"],
+        head_dim=first["dim"], layers=layers, layer_types=[known[e["type"]] for e in layers], norm_eps=d["norm"]["eps"],
+        token_side_dim=(d.get("token_side") or {}).get("dim", 0), max_position_embeddings=DEFAULT_CONTEXT,
+        unbounded_positions=True, tie_word_embeddings=False, torch_dtype="bfloat16", eos_token_id=None, bos_token_id=None,
+        **moe)

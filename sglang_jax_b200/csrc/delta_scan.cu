@@ -2,7 +2,8 @@
 //
 //   delta_prep    short causal convolution + SiLU of the q / k / v channels of a fused projection (window = this step's
 //                 rows, then the request's stored window, then zeros), unit q (times dim^-1/2) and k vectors, write
-//                 strength beta = sigmoid(b) and decay g = exp(-exp(A_log) softplus(a + dt_bias))
+//                 strength beta = sigmoid(b) and decay g = exp(-exp(A_log) softplus(a + dt_bias)), one per head or one
+//                 per head and key channel (then the next two kernels compute it, the only readers of its input)
 //   delta_chunk   prefill: what a chunk of 32 tokens contributes independently of the state in front of it
 //   delta_scan    prefill: S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q   chunk by chunk as small matrix
 //                 products; columns of S are independent, so a CTA owns 32 columns of one (sequence, head) and keeps
@@ -10,7 +11,7 @@
 //   delta_step    decode: the same for one token per request, the state streaming through once
 //                 The convolution windows and the optional checkpoint (state after `track` tokens, for prefix sharing)
 //                 are written by the last two.
-//   delta_gate    rmsnorm(o) * w * silu(gate) per head, in the projections' type
+//   delta_gate    rmsnorm(o) * w * silu(gate) (or sigmoid(gate)) per head, in the projections' type
 //
 // Both state tensors belong to `RecurrentStatePool`: windows [slots, channels, taps - 1], states [slots, H, D, V].
 // Compiled without fast-math substitutions.
@@ -39,7 +40,8 @@ struct DeltaParams {
   int g_off, b_off, a_off;
   const void* conv_w;            // [channels, taps], channels = q | k | v
   const float* a_log;            // [H]
-  const float* dt_bias;          // [H]
+  const float* dt_bias;          // [H]; per channel: [H, D]
+  const void* chan_a;            // [T, H, D] inputs of the decays per channel; null: one decay per head, from proj
   void* conv_state;              // [slots, channels, taps - 1]
   float* state;                  // [slots, H, D, V]
   const long long* slots;        // [B]
@@ -51,10 +53,14 @@ struct DeltaParams {
   float* v;                      // [T, H, V]
   float* gb;                     // [T, H, 2] decay, beta
   float* coef;                   // [T / 32 + 2 B, H, kCoefs], see delta_chunk_kernel
+  float* kq;                     // per channel: [T, H, 3, D], see delta_chunk_channel_kernel
+  float* gc;                     // per channel: [T / 32 + 2 B, H, D] decay over a whole chunk
   float* o;                      // [T, H, V]
   int B, T, H, Hk, D, V, taps;
   int singles;                   // ragged step: how many sequences bring exactly one token (-1: not known)
 };
+
+__device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
 // One warp per (run of RUN consecutive rows, head): the convolution window slides through registers.  A lane owns the
 // channels lane, lane + 32, ... (NPL of them); TAPS >= taps, the kernel and the window are padded in front with zeros.
@@ -220,10 +226,8 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const DeltaParams p) {
     }
     for (int t = t0 + lane; t < t1; t += 32) {
       const T* row = proj + static_cast<long long>(t) * p.ld;
-      const float z = to_f(row[p.a_off + h]) + p.dt_bias[h];
-      const float sp = fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
       float* gb = p.gb + (static_cast<long long>(t) * p.H + h) * 2;
-      gb[0] = expf(-expf(p.a_log[h]) * sp);
+      if (p.chan_a == nullptr) gb[0] = expf(-expf(p.a_log[h]) * softplus(to_f(row[p.a_off + h]) + p.dt_bias[h]));
       gb[1] = 1.f / (1.f + expf(-to_f(row[p.b_off + h])));
     }
   }
@@ -270,13 +274,12 @@ __device__ __forceinline__ void cp_async4(void* dst, const void* src, int bytes 
 __device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-// kC rows of unit q (which = 0) or k (1) vectors into smem rows of `ld` floats; rows past m become zeros.  Lanes past D
+// kC rows (of D floats, `tok` floats apart) into smem rows of `ld` floats; rows past m become zeros; below, those of the unit
+// q (which = 0) or k (1) vectors.  Lanes past D
 // of a row are left alone.
 template <int THREADS>
-__device__ __forceinline__ void stage_rows(float* dst, int ld, const DeltaParams& p, int row0, int hk, int which, int m) {
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, D = p.D;
-  const long long tok = static_cast<long long>(p.Hk) * 2 * D;
-  const float* src = p.qk + row0 * tok + (static_cast<long long>(hk) * 2 + which) * D;
+__device__ __forceinline__ void stage_rows(float* dst, int ld, const float* src, long long tok, int D, int m) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   for (int r = warp; r < kC; r += THREADS / 32) {
     const bool in = r < m;
     const float* s = src + (in ? r : 0) * tok;
@@ -285,6 +288,32 @@ __device__ __forceinline__ void stage_rows(float* dst, int ld, const DeltaParams
     else
       for (int e = lane; e < D; e += 32) cp_async4(dst + r * ld + e, s + e, in ? 4 : 0);
   }
+}
+
+// Where chunk `idx` of the launch lies: sequence, first row, rows; none of them for places no sequence uses and for single
+// tokens (delta_step).
+struct ChunkPlace {
+  int row0, m;
+  __device__ __forceinline__ ChunkPlace(const DeltaParams& p, int idx) : row0(0), m(0) {
+    int lo = 0, hi = p.B - 1;
+    while (lo < hi) {                                  // last sequence whose chunks begin at or before idx
+      const int mid = (lo + hi + 1) >> 1;
+      if (chunk_base(p.cu[mid], mid) <= idx) lo = mid;
+      else hi = mid - 1;
+    }
+    const int start = p.cu[lo];
+    const Chunks ch(p.cu[lo + 1] - start, p.track_len != nullptr ? p.track_len[lo] : 0);
+    const int ci = idx - chunk_base(start, lo);
+    if (ch.n <= 1 || ci >= ch.count()) return;
+    row0 = start + ch.first(ci);
+    m = ch.len(ci);
+  }
+};
+
+template <int THREADS>
+__device__ __forceinline__ void stage_rows(float* dst, int ld, const DeltaParams& p, int row0, int hk, int which, int m) {
+  const long long tok = static_cast<long long>(p.Hk) * 2 * p.D;
+  stage_rows<THREADS>(dst, ld, p.qk + row0 * tok + (static_cast<long long>(hk) * 2 + which) * p.D, tok, p.D, m);
 }
 
 // One CTA per (chunk, q / k head): products of the chunk's vectors, then the coefficients of every value head that uses
@@ -301,21 +330,9 @@ __global__ void __launch_bounds__(kChunkThreads) delta_chunk_kernel(const DeltaP
   pdl_wait();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, hk = blockIdx.y;
   const int idx = blockIdx.x;
-  int b = 0;
-  {
-    int lo = 0, hi = p.B - 1;
-    while (lo < hi) {                                  // last sequence whose chunks begin at or before idx
-      const int mid = (lo + hi + 1) >> 1;
-      if (chunk_base(p.cu[mid], mid) <= idx) lo = mid;
-      else hi = mid - 1;
-    }
-    b = lo;
-  }
-  const int start = p.cu[b];
-  const Chunks ch(p.cu[b + 1] - start, p.track_len != nullptr ? p.track_len[b] : 0);
-  const int ci = idx - chunk_base(start, b);
-  if (ch.n <= 1 || ci >= ch.count()) return;         // single tokens: delta_step
-  const int row0 = start + ch.first(ci), m = ch.len(ci);
+  const ChunkPlace place(p, idx);
+  if (place.m == 0) return;
+  const int row0 = place.row0, m = place.m;
   for (int i = tid; i < 2 * kC * (ld - p.D); i += kChunkThreads) rows[(i / (ld - p.D)) * ld + p.D + i % (ld - p.D)] = 0.f;
   stage_rows<kChunkThreads>(rows, ld, p, row0, hk, 1, m);
   stage_rows<kChunkThreads>(rows + kC * ld, ld, p, row0, hk, 0, m);
@@ -383,6 +400,188 @@ __global__ void __launch_bounds__(kChunkThreads) delta_chunk_kernel(const DeltaP
   }
 }
 
+// The same with one decay per head and key channel, one CTA per (chunk, head).  The products need the decay between two
+// tokens inside the sum over channels.  A block of tokens is halved down to blocks of four: between the halves the decay is
+// split at the last token of the first half, so neither factor exceeds one, and the products are plain ones of scaled
+// vectors; inside four tokens the decays are taken pair by pair.  Every exponent is a sum over just the tokens in between,
+// never a difference of longer sums, so that strong decays earlier in the chunk do not cost precision.  Scaled vectors for
+// delta_scan: k and q times the decay from the chunk's start (what meets the state in front of it), and k times the decay to
+// its end (what it leaves behind).
+struct ChannelShape {
+  static constexpr int kRows = 3 * kC + kC + kC / 2;   // k, q, c; scaled k, scaled q of second halves
+  static int smem(int Dp) { return (kRows * (Dp + 4) + 2 * kC * kGramLd + kC) * 4; }
+};
+
+template <typename T>
+__global__ void __launch_bounds__(kChunkThreads) delta_chunk_channel_kernel(const DeltaParams p, int Dp) {
+  extern __shared__ float4 sm4[];
+  const int ld = Dp + 4;
+  float* ks = reinterpret_cast<float*>(sm4);           // [kC][ld]
+  float* qs = ks + kC * ld;                            // [kC][ld]
+  float* cs = qs + kC * ld;                            // [kC][ld]  logarithms of the tokens' decays
+  float* sk = cs + kC * ld;                            // [kC][ld]
+  float* sq = sk + kC * ld;                            // [kC / 2][ld]
+  float* gram = sq + kC / 2 * ld;                      // [k . k | q . k][kC][kGramLd]
+  float* line = gram + 2 * kC * kGramLd;               // [kC]
+  pdl_wait();
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.y, hk = h / (p.H / p.Hk), D = p.D;
+  const int idx = blockIdx.x;
+  const ChunkPlace place(p, idx);
+  if (place.m == 0) return;
+  const int row0 = place.row0, m = place.m;
+  for (int i = tid; i < 3 * kC * (ld - D); i += kChunkThreads) ks[(i / (ld - D)) * ld + D + i % (ld - D)] = 0.f;
+  stage_rows<kChunkThreads>(ks, ld, p, row0, hk, 1, m);
+  stage_rows<kChunkThreads>(qs, ld, p, row0, hk, 0, m);
+  cp_commit();
+  const float rate = -expf(p.a_log[h]);
+  float* gc = p.gc + (static_cast<long long>(idx) * p.H + h) * D;
+  for (int d = tid; d < D; d += kChunkThreads) {
+    const T* a = static_cast<const T*>(p.chan_a) + (static_cast<long long>(row0) * p.H + h) * D + d;
+    const float bias = p.dt_bias[h * D + d];
+    float c = 0.f;
+#pragma unroll 8
+    for (int t = 0; t < kC; ++t) {
+      const float lg = t < m ? rate * softplus(to_f(a[static_cast<long long>(t) * p.H * D]) + bias) : 0.f;
+      c += lg;
+      cs[t * ld + d] = lg;
+    }
+    gc[d] = expf(c);
+  }
+  for (int i = tid; i < 2 * kC * kGramLd; i += kChunkThreads) gram[i] = 0.f;
+  cp_wait<0>();
+  __syncthreads();
+  for (int d = tid; d < D; d += kChunkThreads) {
+    float* dst = p.kq + (static_cast<long long>(row0) * p.H + h) * 3 * D + d;
+    const long long tok = static_cast<long long>(p.H) * 3 * D;
+    float c = 0.f, e = 0.f;                            // from the start up to t; after the t'th last to the end
+#pragma unroll 4
+    for (int t = 0; t < m; ++t) {
+      c += cs[t * ld + d];
+      const float f = expf(c);
+      dst[t * tok] = ks[t * ld + d] * f;
+      dst[t * tok + D] = qs[t * ld + d] * f;
+    }
+#pragma unroll 4
+    for (int t = m - 1; t >= 0; --t) {
+      dst[t * tok + 2 * D] = ks[t * ld + d] * expf(e);
+      e += cs[t * ld + d];
+    }
+  }
+#pragma unroll
+  for (int half = kC / 2; half >= 4; half >>= 1) {
+    // scaled vectors: first halves backwards from their last token, second halves forwards from there
+    for (int d = tid; d < Dp; d += kChunkThreads)
+      for (int blk = 0; blk < kC; blk += 2 * half) {
+        float c = 0.f;
+#pragma unroll 4
+        for (int t = blk + half - 1; t >= blk; --t) {
+          sk[t * ld + d] = ks[t * ld + d] * expf(c);
+          c += cs[t * ld + d];
+        }
+        c = 0.f;
+#pragma unroll 4
+        for (int t = blk + half; t < blk + 2 * half; ++t) {
+          c += cs[t * ld + d];
+          const float f = expf(c);
+          sk[t * ld + d] = ks[t * ld + d] * f;
+          sq[(t - half - blk / 2) * ld + d] = qs[t * ld + d] * f;
+        }
+      }
+    __syncthreads();
+    // kC / 2 second-half rows times `half` columns of their first half, for k and q; two rows per thread at the top
+    const int rows = half == kC / 2 ? 2 : 1, items = kC / 2 * half / rows;
+    if (tid < items) {
+      const int j = tid % half, r = tid / half * rows;           // r: place among the second-half rows
+      const int blk = r / half * 2 * half, t = blk + half + r % half;
+      const float* col = sk + (blk + j) * ld;
+      float kk[2] = {0.f, 0.f}, qk[2] = {0.f, 0.f};
+      for (int d = 0; d < Dp; d += 4) {
+        const float4 c = *reinterpret_cast<const float4*>(col + d);
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          if (i >= rows) break;
+          const float4 a = *reinterpret_cast<const float4*>(sk + (t + i) * ld + d);
+          const float4 b = *reinterpret_cast<const float4*>(sq + (r + i) * ld + d);
+          kk[i] += a.x * c.x + a.y * c.y + a.z * c.z + a.w * c.w;
+          qk[i] += b.x * c.x + b.y * c.y + b.z * c.z + b.w * c.w;
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        if (i >= rows) break;
+        gram[(t + i) * kGramLd + blk + j] = kk[i];
+        gram[(kC + t + i) * kGramLd + blk + j] = qk[i];
+      }
+    }
+    __syncthreads();
+  }
+  // blocks of four tokens: one warp each, lanes share the channels
+  for (int blk = warp * 4; blk < kC; blk += kChunkThreads / 32 * 4) {
+    float kk[6], qk[10];
+#pragma unroll
+    for (int i = 0; i < 6; ++i) kk[i] = 0.f;
+#pragma unroll
+    for (int i = 0; i < 10; ++i) qk[i] = 0.f;
+    for (int d = lane; d < Dp; d += 32) {
+      float k[4], q[4], c[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        k[i] = ks[(blk + i) * ld + d];
+        q[i] = qs[(blk + i) * ld + d];
+        c[i] = cs[(blk + i) * ld + d];
+      }
+#pragma unroll
+      for (int t = 0; t < 4; ++t) {
+        float e = 0.f;
+#pragma unroll
+        for (int j = t - 1; j >= 0; --j) {
+          e += c[j + 1];
+          const float f = expf(e) * k[j];
+          kk[t * (t - 1) / 2 + j] += k[t] * f;
+          qk[t * (t + 1) / 2 + j] += q[t] * f;
+        }
+        qk[t * (t + 1) / 2 + t] += q[t] * k[t];
+      }
+    }
+#pragma unroll
+    for (int t = 0; t < 4; ++t)
+#pragma unroll
+      for (int j = 0; j <= t; ++j) {
+        const float b = warp_sum(qk[t * (t + 1) / 2 + j]);
+        const float a = j < t ? warp_sum(kk[t > 0 ? t * (t - 1) / 2 + (j < t ? j : 0) : 0]) : 0.f;
+        if (lane == 0) {
+          gram[(blk + t) * kGramLd + blk + j] = a;
+          gram[(kC + blk + t) * kGramLd + blk + j] = b;
+        }
+      }
+  }
+  __syncthreads();
+  if (warp == 0) {
+    const float beta = lane < m ? p.gb[(static_cast<long long>(row0 + lane) * p.H + h) * 2 + 1] : 0.f;
+    float* out = p.coef + (static_cast<long long>(idx) * p.H + h) * kCoefs;
+    float X[kC];                                       // lane c: column c of (I + A)^-1
+#pragma unroll
+    for (int t = 0; t < kC; ++t) {
+      const float bt = __shfl_sync(0xffffffffu, beta, t);
+      __syncwarp();
+      line[lane] = lane < t ? bt * gram[t * kGramLd + lane] : 0.f;
+      out[kCoefB + t * kCoefRow + lane] = lane <= t ? gram[(kC + t) * kGramLd + lane] : 0.f;
+      __syncwarp();
+      float x = lane == t ? 1.f : 0.f;
+#pragma unroll
+      for (int j = 0; j < t; j += 4) {
+        const float4 c = *reinterpret_cast<const float4*>(line + j);
+        x -= c.x * X[j];
+        if (j + 1 < t) x -= c.y * X[j + 1];
+        if (j + 2 < t) x -= c.z * X[j + 2];
+        if (j + 3 < t) x -= c.w * X[j + 3];
+      }
+      X[t] = x;
+      out[t * kCoefRow + lane] = x * beta;
+    }
+  }
+}
+
 // ---------------------------------------------------------------------------------------------
 constexpr int kScanThreads = 256;
 constexpr int kCols = 32;          // columns of the state per CTA
@@ -420,16 +619,17 @@ __device__ __forceinline__ void write_windows(const DeltaParams& p, int b, int h
 //   Y = [K; Q] S                    rows 4 rg .. of the 64: warps 0-3 turn K S into the right-hand side, 4-7 keep G Q S
 //   U = (I + A)^-1 diag(beta) (V - G K S)
 //   O = G Q S + B U                 warps 4-7;         S <- G S + K^T diag(g_C) U   all warps
+// With decays per channel (CHAN) the factors sit in three scaled copies of K and Q instead (delta_chunk_channel_kernel).
 template <int RPT>
 struct ScanShape {
   static constexpr int kDp = 16 * RPT, kLd = kDp + 4;
   static constexpr int kK = kC * kLd;                  // one buffer of k (two of them), and the one of q
   static constexpr int kCo = kC * kGramLd;             // T', B
-  static constexpr int kFloats = 3 * kK + kC * kCols + 2 * kCo + 2 * 2 * kC + kDp * kCols + 2 * kC * kCols;
+  static constexpr int kFloats = 3 * kK + kC * kCols + 2 * kCo + 2 * 2 * kC + kDp * kCols + 2 * kC * kCols + kDp;
   static constexpr int kSmem = kFloats * 4;
 };
 
-template <typename T, int RPT>
+template <typename T, int RPT, bool CHAN>
 __global__ void __launch_bounds__(kScanThreads, RPT <= 8 ? 2 : 1) delta_scan_kernel(const DeltaParams p) {
   using Sh = ScanShape<RPT>;
   constexpr int ld = Sh::kLd;
@@ -443,6 +643,7 @@ __global__ void __launch_bounds__(kScanThreads, RPT <= 8 ? 2 : 1) delta_scan_ker
   float* ss = vec + 4 * kC;                            // [kDp][kCols]
   float* us = ss + Sh::kDp * kCols;                    // [kC][kCols]
   float* rs = us + kC * kCols;                         // [kC][kCols]    right-hand side, then diag(g_C) U
+  float* gcs = rs + kC * kCols;                        // [kDp]          CHAN: decays over the chunk
   pdl_wait();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, cp = (lane & 15) * 2, rg = warp * 2 + (lane >> 4);
   const int b = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * kCols, hk = h / (p.H / p.Hk);
@@ -476,17 +677,30 @@ __global__ void __launch_bounds__(kScanThreads, RPT <= 8 ? 2 : 1) delta_scan_ker
   };
   for (int i = tid; i < 3 * kC * (ld - D); i += kScanThreads) ks[(i / (ld - D)) * ld + D + i % (ld - D)] = 0.f;
 
+  if (CHAN)
+    for (int i = tid; i < Sh::kDp - D; i += kScanThreads) gcs[D + i] = 0.f;
+  auto scaled = [&](float* dst, int ci, int which) {   // CHAN: one of the three copies of chunk ci
+    const long long tok = static_cast<long long>(p.H) * 3 * D;
+    stage_rows<kScanThreads>(dst, ld, p.kq + (start + ch.first(ci)) * tok + (static_cast<long long>(h) * 3 + which) * D, tok,
+                             D, ch.len(ci));
+  };
+
   auto stage_tokens = [&](int ci) {                    // k, q, v and the decays of chunk ci
     const int row0 = start + ch.first(ci), m = ch.len(ci);
-    stage_rows<kScanThreads>(ks + (ci & 1) * Sh::kK, ld, p, row0, hk, 1, m);
-    stage_rows<kScanThreads>(qs, ld, p, row0, hk, 0, m);
+    if constexpr (CHAN) {
+      scaled(ks, ci, 0);
+      scaled(qs, ci, 1);
+    } else {
+      stage_rows<kScanThreads>(ks + (ci & 1) * Sh::kK, ld, p, row0, hk, 1, m);
+      stage_rows<kScanThreads>(qs, ld, p, row0, hk, 0, m);
+    }
     for (int i = tid; i < kC * kCols; i += kScanThreads) {
       const int t = i / kCols, e = i % kCols;
       const bool in = t < m && c0 + e < V;
       cp_async4(vs + i, p.v + (static_cast<long long>(row0 + (in ? t : 0)) * p.H + h) * V + (in ? c0 + e : 0), in ? 4 : 0);
     }
     const float* src = coef + static_cast<long long>(ci) * p.H * kCoefs + kCoefVec;
-    if (tid < 2 * kC / 4) cp_async16(vec + (ci & 1) * 2 * kC + tid * 4, src + tid * 4);
+    if (!CHAN && tid < 2 * kC / 4) cp_async16(vec + (ci & 1) * 2 * kC + tid * 4, src + tid * 4);
     cp_commit();
   };
   auto stage_coefs = [&](int ci) {
@@ -495,13 +709,19 @@ __global__ void __launch_bounds__(kScanThreads, RPT <= 8 ? 2 : 1) delta_scan_ker
       const int row = i / (kC / 4), e = (i % (kC / 4)) * 4;              // rows 0..kC-1 of T', then of B
       cp_async16(ts + row * kGramLd + e, src + row * kC + e);
     }
+    if constexpr (CHAN) {
+      scaled(ks + Sh::kK, ci, 2);
+      const float* g = p.gc + (static_cast<long long>(chunk_base(start, b) + ci) * p.H + h) * D;
+      for (int i = tid; i < D; i += kScanThreads) cp_async4(gcs + i, g + i);
+    }
     cp_commit();
   };
 
   stage_tokens(0);
   stage_coefs(0);
   for (int ci = 0; ci < nch; ++ci) {
-    const float* kb = ks + (ci & 1) * Sh::kK;
+    const float* kb = ks + (CHAN ? 0 : (ci & 1) * Sh::kK);
+    const float* ku = CHAN ? ks + Sh::kK : kb;         // what the state's update reads
     const float* gv = vec + (ci & 1) * 2 * kC;
     cp_wait<1>();                                      // the tokens; the coefficients may still be on their way
     __syncthreads();
@@ -529,9 +749,11 @@ __global__ void __launch_bounds__(kScanThreads, RPT <= 8 ? 2 : 1) delta_scan_ker
     const int t4 = (rg & 7) * 4;                       // first of this thread's four tokens
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
-      const float G = gv[t4 + i];
-      y[i][0] *= G;
-      y[i][1] *= G;
+      if constexpr (!CHAN) {
+        const float G = gv[t4 + i];
+        y[i][0] *= G;
+        y[i][1] *= G;
+      }
       if (rg < 8) {
         const float2 v = *reinterpret_cast<const float2*>(vs + (t4 + i) * kCols + cp);
         *reinterpret_cast<float2*>(rs + (t4 + i) * kCols + cp) = make_float2(v.x - y[i][0], v.y - y[i][1]);
@@ -559,7 +781,7 @@ __global__ void __launch_bounds__(kScanThreads, RPT <= 8 ? 2 : 1) delta_scan_ker
       __syncthreads();                                 // everyone is done with the right-hand side
 #pragma unroll
       for (int i = 0; i < 2; ++i) {
-        const float w = gv[kC + t2 + i];
+        const float w = CHAN ? 1.f : gv[kC + t2 + i];
         *reinterpret_cast<float2*>(us + (t2 + i) * kCols + cp) = make_float2(u[i][0], u[i][1]);
         *reinterpret_cast<float2*>(rs + (t2 + i) * kCols + cp) = make_float2(w * u[i][0], w * u[i][1]);
       }
@@ -589,9 +811,9 @@ __global__ void __launch_bounds__(kScanThreads, RPT <= 8 ? 2 : 1) delta_scan_ker
         if (c0 + cp + 1 < V) o[1] = y[i][1];
       }
     }
-    const float G = gv[kC - 1];
 #pragma unroll
     for (int i = 0; i < RPT; ++i) {
+      const float G = CHAN ? gcs[rg * RPT + i] : gv[kC - 1];
       S[i][0] *= G;
       S[i][1] *= G;
     }
@@ -600,7 +822,7 @@ __global__ void __launch_bounds__(kScanThreads, RPT <= 8 ? 2 : 1) delta_scan_ker
       const float2 w = *reinterpret_cast<const float2*>(rs + j * kCols + cp);
 #pragma unroll
       for (int i = 0; i < RPT; i += 4) {
-        const float4 k = *reinterpret_cast<const float4*>(kb + j * ld + rg * RPT + i);
+        const float4 k = *reinterpret_cast<const float4*>(ku + j * ld + rg * RPT + i);
         S[i][0] += k.x * w.x;
         S[i][1] += k.x * w.y;
         S[i + 1][0] += k.y * w.x;
@@ -628,9 +850,9 @@ __global__ void __launch_bounds__(kScanThreads, RPT <= 8 ? 2 : 1) delta_scan_ker
 constexpr int kLanes = 8;
 constexpr int kStepThreads = 128;
 
-template <typename T, int RPL, int CPL>
+template <typename T, int RPL, int CPL, bool CHAN>
 __global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaParams p) {
-  __shared__ __align__(16) float qk[2][kLanes * RPL];
+  __shared__ __align__(16) float qk[CHAN ? 3 : 2][kLanes * RPL];       // q, k, decays per channel
   pdl_wait();
   const int tid = threadIdx.x, lane = tid & 31, rl = lane & (kLanes - 1);
   const int b = blockIdx.x, h = blockIdx.y, hk = h / (p.H / p.Hk), D = p.D, V = p.V;
@@ -668,9 +890,27 @@ __global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaPar
     const int which = i / (kLanes * RPL), e = i - which * kLanes * RPL;
     qk[which][e] = e < D ? p.qk[((static_cast<long long>(t) * p.Hk + hk) * 2 + which) * D + e] : 0.f;
   }
-  __syncthreads();
   const long long bh = static_cast<long long>(t) * p.H + h;
-  const float g = p.gb[bh * 2], beta = p.gb[bh * 2 + 1];
+  if constexpr (CHAN) {
+    const float rate = -expf(p.a_log[h]);
+    for (int e = tid; e < kLanes * RPL; e += kStepThreads)
+      qk[CHAN ? 2 : 0][e] = e < D ? expf(rate * softplus(to_f(static_cast<const T*>(p.chan_a)[bh * D + e]) + p.dt_bias[h * D + e]))
+                                  : 0.f;
+  }
+  __syncthreads();
+  const float g = CHAN ? 1.f : p.gb[bh * 2], beta = p.gb[bh * 2 + 1];
+  if constexpr (CHAN)
+#pragma unroll
+    for (int i = 0; i < RPL; i += 4) {
+      const float4 d = *reinterpret_cast<const float4*>(&qk[CHAN ? 2 : 0][row_of(i)]);
+#pragma unroll
+      for (int c = 0; c < CPL; ++c) {
+        S[i][c] *= d.x;
+        S[i + 1][c] *= d.y;
+        S[i + 2][c] *= d.z;
+        S[i + 3][c] *= d.w;
+      }
+    }
   float kd[CPL], qd[CPL], kq = 0.f, kr[RPL];
 #pragma unroll
   for (int c = 0; c < CPL; ++c) kd[c] = qd[c] = 0.f;
@@ -728,7 +968,7 @@ __global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaPar
 
 // One warp per (token, head); a lane holds NV groups of four adjacent columns (V <= 128 * NV, V % 4 == 0), or takes single
 // columns (NV = 0, any V).
-template <typename T, int NV>
+template <typename T, int NV, bool SIGMOID>
 __global__ void delta_gate_kernel(const float* __restrict__ o, const T* __restrict__ gate, long long ld,
                                   const float* __restrict__ w, T* __restrict__ out, long long T_, int H, int V, float eps) {
   pdl_wait();
@@ -740,7 +980,7 @@ __global__ void delta_gate_kernel(const float* __restrict__ o, const T* __restri
   const float* src = o + wid * V;
   const T* g = gate + t * ld + static_cast<long long>(h) * V;
   T* dst = out + wid * V;
-  auto gated = [](float x, float gv) { return x * (gv / (1.f + expf(-gv))); };
+  auto gated = [](float x, float gv) { return x * ((SIGMOID ? 1.f : gv) / (1.f + expf(-gv))); };
   float ss = 0.f;
   if constexpr (NV > 0) {
     float4 v[NV];
@@ -777,16 +1017,16 @@ __global__ void delta_gate_kernel(const float* __restrict__ o, const T* __restri
   }
 }
 
-template <typename T>
+template <typename T, bool SIGMOID>
 int run_gate(const float* o, const void* gate, long long ld, const float* w, void* out, long long n, int H, int V,
              float eps, cudaStream_t s) {
   const dim3 grid(static_cast<unsigned>((n * H + 3) / 4));
   const T* g = static_cast<const T*>(gate);
   T* d = static_cast<T*>(out);
   const bool vec = V % 4 == 0 && ld % 4 == 0 && reinterpret_cast<uintptr_t>(gate) % (4 * sizeof(T)) == 0;
-  if (vec && V <= 128) launch_pdl(delta_gate_kernel<T, 1>, grid, dim3(128), 0, s, o, g, ld, w, d, n, H, V, eps);
-  else if (vec && V <= 256) launch_pdl(delta_gate_kernel<T, 2>, grid, dim3(128), 0, s, o, g, ld, w, d, n, H, V, eps);
-  else launch_pdl(delta_gate_kernel<T, 0>, grid, dim3(128), 0, s, o, g, ld, w, d, n, H, V, eps);
+  if (vec && V <= 128) launch_pdl(delta_gate_kernel<T, 1, SIGMOID>, grid, dim3(128), 0, s, o, g, ld, w, d, n, H, V, eps);
+  else if (vec && V <= 256) launch_pdl(delta_gate_kernel<T, 2, SIGMOID>, grid, dim3(128), 0, s, o, g, ld, w, d, n, H, V, eps);
+  else launch_pdl(delta_gate_kernel<T, 0, SIGMOID>, grid, dim3(128), 0, s, o, g, ld, w, d, n, H, V, eps);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -813,25 +1053,43 @@ int set_smem(K kernel, int smem, bool* done) {
 }
 
 template <typename T, int RPT>
+int launch_scan_channel(const DeltaParams& p, cudaStream_t s) {
+  using Sh = ScanShape<RPT>;
+  static bool cfg = false, cfg_chunk = false;
+  const int chunk_smem = ChannelShape::smem(Sh::kDp);
+  int e = set_smem(delta_chunk_channel_kernel<T>, ChannelShape::smem(ScanShape<16>::kDp), &cfg_chunk);
+  if (e == 0) e = set_smem(delta_scan_kernel<T, RPT, true>, Sh::kSmem, &cfg);
+  if (e != 0) return e;
+  launch_pdl(delta_chunk_channel_kernel<T>, dim3(chunk_base(p.T, p.B), p.H), dim3(kChunkThreads), chunk_smem, s, p,
+             static_cast<int>(Sh::kDp));
+  e = static_cast<int>(cudaGetLastError());
+  if (e != 0) return e;
+  launch_pdl(delta_scan_kernel<T, RPT, true>, dim3(p.B, p.H, (p.V + kCols - 1) / kCols), dim3(kScanThreads), Sh::kSmem, s, p);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T, int RPT>
 int launch_scan(const DeltaParams& p, cudaStream_t s) {
   using Sh = ScanShape<RPT>;
+  if (p.chan_a != nullptr) return launch_scan_channel<T, RPT>(p, s);
   static bool cfg = false, cfg_chunk = false;
   const int chunk_smem = (2 * kC * Sh::kLd + 2 * kC * kGramLd + kChunkThreads) * 4;
   int e = set_smem(delta_chunk_kernel, (2 * kC * ScanShape<16>::kLd + 2 * kC * kGramLd + kChunkThreads) * 4, &cfg_chunk);
-  if (e == 0) e = set_smem(delta_scan_kernel<T, RPT>, Sh::kSmem, &cfg);
+  if (e == 0) e = set_smem(delta_scan_kernel<T, RPT, false>, Sh::kSmem, &cfg);
   if (e != 0) return e;
   launch_pdl(delta_chunk_kernel, dim3(chunk_base(p.T, p.B), p.Hk), dim3(kChunkThreads), chunk_smem, s, p,
              static_cast<int>(Sh::kDp));
   e = static_cast<int>(cudaGetLastError());
   if (e != 0) return e;
-  launch_pdl(delta_scan_kernel<T, RPT>, dim3(p.B, p.H, (p.V + kCols - 1) / kCols), dim3(kScanThreads), Sh::kSmem, s, p);
+  launch_pdl(delta_scan_kernel<T, RPT, false>, dim3(p.B, p.H, (p.V + kCols - 1) / kCols), dim3(kScanThreads), Sh::kSmem, s, p);
   return static_cast<int>(cudaGetLastError());
 }
 
 template <typename T, int RPL, int CPL>
 int launch_step(const DeltaParams& p, cudaStream_t s) {
   constexpr int cols = (kStepThreads / kLanes) * CPL;
-  launch_pdl(delta_step_kernel<T, RPL, CPL>, dim3(p.B, p.H, (p.V + cols - 1) / cols), dim3(kStepThreads), 0, s, p);
+  const auto kernel = p.chan_a != nullptr ? delta_step_kernel<T, RPL, CPL, true> : delta_step_kernel<T, RPL, CPL, false>;
+  launch_pdl(kernel, dim3(p.B, p.H, (p.V + cols - 1) / cols), dim3(kStepThreads), 0, s, p);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -871,27 +1129,30 @@ extern "C" {
 
 // Shapes in DeltaParams; T = bf16 or fp32 (`is_f32`) is the type of `proj`, `conv_w` and `conv_state`.
 int sglb_delta_scan(const void* proj, long long ld, int g_off, int b_off, int a_off, const void* conv_w,
-                    const float* a_log, const float* dt_bias, void* conv_state, float* state, const long long* slots,
-                    const int* cu, const int* prefix, const int* track_len, const int* track_slot, float* qk, float* v,
-                    float* gb, float* coef, float* o, int B, int T, int H, int Hk, int D, int V, int taps, int singles,
-                    int is_f32,
-                    cudaStream_t s) {
+                    const float* a_log, const float* dt_bias, const void* chan_a, void* conv_state, float* state,
+                    const long long* slots, const int* cu, const int* prefix, const int* track_len, const int* track_slot,
+                    float* qk, float* v, float* gb, float* coef, float* kq, float* gc, float* o, int B, int T, int H, int Hk,
+                    int D, int V, int taps, int singles, int is_f32, cudaStream_t s) {
   using namespace sglb;
   if (B <= 0 || T <= 0) return 0;
   if (cu != nullptr && (prefix == nullptr || (coef == nullptr && singles != B))) return -kBadArgument;
+  if (chan_a != nullptr && coef != nullptr && (kq == nullptr || gc == nullptr)) return -kBadArgument;
   if (D < 1 || D > 256 || V < 1 || Hk < 1 || H % Hk != 0 || taps < 1 || taps > 16 || H > 65535) return -kBadArgument;
-  DeltaParams p{proj, ld, g_off, b_off, a_off, conv_w, a_log, dt_bias, conv_state, state, slots, cu, prefix, track_len,
-                track_slot, qk, v, gb, coef, o, B, T, H, Hk, D, V, taps, singles};
+  DeltaParams p{proj, ld, g_off, b_off, a_off, conv_w, a_log, dt_bias, chan_a, conv_state, state, slots, cu, prefix,
+                track_len, track_slot, qk, v, gb, coef, kq, gc, o, B, T, H, Hk, D, V, taps, singles};
   return is_f32 ? run_delta<float>(p, s) : run_delta<__nv_bfloat16>(p, s);
 }
 
-// out [T, H * V] = rmsnorm(o [T, H, V], over V) * w [V] * silu(gate), gate at row stride `ld`.
+// out [T, H * V] = rmsnorm(o [T, H, V], over V) * w [V] * silu(gate) (or sigmoid(gate)), gate at row stride `ld`.
 int sglb_delta_gate(const float* o, const void* gate, long long ld, const float* w, void* out, long long T, int H, int V,
-                    float eps, int is_f32, cudaStream_t s) {
+                    float eps, int sigmoid, int is_f32, cudaStream_t s) {
   using namespace sglb;
   if (T <= 0) return 0;
-  return is_f32 ? run_gate<float>(o, gate, ld, w, out, T, H, V, eps, s)
-                : run_gate<__nv_bfloat16>(o, gate, ld, w, out, T, H, V, eps, s);
+  if (sigmoid)
+    return is_f32 ? run_gate<float, true>(o, gate, ld, w, out, T, H, V, eps, s)
+                  : run_gate<__nv_bfloat16, true>(o, gate, ld, w, out, T, H, V, eps, s);
+  return is_f32 ? run_gate<float, false>(o, gate, ld, w, out, T, H, V, eps, s)
+                : run_gate<__nv_bfloat16, false>(o, gate, ld, w, out, T, H, V, eps, s);
 }
 
 }  // extern "C"

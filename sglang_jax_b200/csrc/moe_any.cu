@@ -1,0 +1,242 @@
+// Routed experts beside the tensor-core kernels of moe.cu / gemm_sm100.cu, in bf16 or fp32, any sizes:
+//
+//   route_by_logit     z = W x + b in fp32 (or z given), the k largest, weights = softmax over those
+//   grouped_gemm_any   out[r] = x[row(r)] . w[group of r]^T on the CUDA cores with fp32 accumulation: the fp32 mode, and
+//                      bf16 sizes whose rows are not whole 16-byte units
+//
+// Compiled without fast-math substitutions.
+#include <float.h>
+#include <math.h>
+
+#include "common.cuh"
+
+namespace sglb {
+namespace {
+
+constexpr int kMaxExperts = 512, kMaxTop = 16;
+constexpr int kRouteThreads = 256;
+
+__device__ __forceinline__ float to_f(float v) { return v; }
+__device__ __forceinline__ float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <typename T> __device__ __forceinline__ T from_f(float v);
+template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
+
+// dot product of one row pair over a warp's lanes
+template <typename T>
+__device__ __forceinline__ float warp_dot(const T* __restrict__ w, const float* __restrict__ x, int K, int lane, bool wide) {
+  float a = 0.f;
+  if (sizeof(T) == 2 && wide) {
+    for (int i = lane * 8; i < K; i += 256) {
+      const uint4 v = *reinterpret_cast<const uint4*>(w + i);
+      const uint32_t u[4] = {v.x, v.y, v.z, v.w};
+      const float4 p = *reinterpret_cast<const float4*>(x + i), q = *reinterpret_cast<const float4*>(x + i + 4);
+      const float f[8] = {p.x, p.y, p.z, p.w, q.x, q.y, q.z, q.w};
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        a += __uint_as_float(u[e] << 16) * f[2 * e] + __uint_as_float(u[e] & 0xffff0000u) * f[2 * e + 1];
+    }
+  } else {
+    for (int i = lane; i < K; i += 32) a += to_f(w[i]) * x[i];
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) a += __shfl_xor_sync(0xffffffffu, a, o);
+  return a;
+}
+
+// The k largest of z[0 .. E) by one warp (ties: the lower index), and their softmax.
+__device__ __forceinline__ void choose(float* z, int E, int k, float* __restrict__ out_w, int* __restrict__ out_ids,
+                                       int lane) {
+  float mine = -INFINITY;
+  int my_id = 0;
+  for (int j = 0; j < k; ++j) {
+    float best = -INFINITY;
+    int bi = 0x7fffffff;
+    for (int e = lane; e < E; e += 32) {
+      const float v = z[e];
+      if (v > best || (v == best && e < bi)) {
+        best = v;
+        bi = e;
+      }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+      if (ov > best || (ov == best && oi < bi)) {
+        best = ov;
+        bi = oi;
+      }
+    }
+    if (bi >= E) bi = 0;                               // logits that are not numbers: some expert all the same
+    if (lane == j) {
+      mine = best;
+      my_id = bi;
+    }
+    __syncwarp();
+    if (lane == 0) z[bi] = -INFINITY;
+    __syncwarp();
+  }
+  const float top = __shfl_sync(0xffffffffu, mine, 0);
+  float p = lane < k ? expf(mine - top) : 0.f, sum = p;
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+  if (lane < k) {
+    out_w[lane] = p / sum;
+    out_ids[lane] = my_id;
+  }
+}
+
+// One CTA per token: the warps share the experts' dot products, the first one chooses.
+template <typename T>
+__global__ void __launch_bounds__(kRouteThreads)
+route_token_kernel(const T* __restrict__ x, const T* __restrict__ w, const T* __restrict__ bias, float* __restrict__ out_w,
+                   int* __restrict__ out_ids, int E, int K, int k, int wide) {
+  extern __shared__ float4 sm4[];
+  float* xs = reinterpret_cast<float*>(sm4);           // [K]
+  float* z = xs + (K + 3) / 4 * 4;                     // [E]
+  pdl_wait();
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const size_t t = blockIdx.x;
+  for (int i = tid; i < K; i += kRouteThreads) xs[i] = to_f(x[t * K + i]);
+  __syncthreads();
+  for (int e = warp; e < E; e += kRouteThreads / 32) {
+    const float a = warp_dot(w + static_cast<size_t>(e) * K, xs, K, lane, wide != 0);
+    if (lane == 0) z[e] = a + (bias != nullptr ? to_f(bias[e]) : 0.f);
+  }
+  __syncthreads();
+  if (warp == 0) choose(z, E, k, out_w + t * k, out_ids + t * k, lane);
+}
+
+// Logits given: one warp per token.
+template <typename T>
+__global__ void __launch_bounds__(128)
+route_logits_kernel(const float* __restrict__ logits, const T* __restrict__ bias, float* __restrict__ out_w,
+                    int* __restrict__ out_ids, int T_, int E, int k) {
+  extern __shared__ float4 sm4[];
+  pdl_wait();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const size_t t = blockIdx.x * 4ull + warp;
+  if (t >= T_) return;
+  float* z = reinterpret_cast<float*>(sm4) + warp * E;
+  for (int e = lane; e < E; e += 32) z[e] = logits[t * E + e] + (bias != nullptr ? to_f(bias[e]) : 0.f);
+  __syncwarp();
+  choose(z, E, k, out_w + t * k, out_ids + t * k, lane);
+}
+
+// ---------------------------------------------------------------------------------------------
+// CTA tile 64 rows x 64 outputs, 4 x 4 per thread, K in steps of 16.  Token tiles come from moe_align's list (128 rows
+// each, two CTAs share one).
+constexpr int kGM = 64, kGN = 64, kGK = 16;
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+grouped_gemm_any_kernel(const T* __restrict__ x, const int* __restrict__ row_token, const T* __restrict__ w,
+                        T* __restrict__ out, const int* __restrict__ offsets, const int* __restrict__ tile_group,
+                        const int* __restrict__ tile_row0, const int* __restrict__ num_tiles, int N, int K) {
+  __shared__ float as[kGK][kGM + 4], bs[kGK][kGN + 4];
+  __shared__ int src[kGM];
+  pdl_wait();
+  const int tile = blockIdx.x >> 1, tid = threadIdx.x;
+  if (tile >= *num_tiles) return;
+  const int g = tile_group[tile], r0 = tile_row0[tile] + (blockIdx.x & 1) * kGM;
+  const int r1 = min(offsets[g + 1], tile_row0[tile] + 128), n0 = blockIdx.y * kGN;
+  if (r0 >= r1) return;
+  if (tid < kGM) {
+    const int r = min(r0 + tid, r1 - 1);
+    src[tid] = row_token != nullptr ? row_token[r] : r;
+  }
+  __syncthreads();
+  const T* wg = w + static_cast<size_t>(g) * N * K;
+  const int tr = (tid >> 4) * 4, tc = (tid & 15) * 4;
+  float acc[4][4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+  for (int k0 = 0; k0 < K; k0 += kGK) {
+#pragma unroll
+    for (int i = 0; i < kGM * kGK / 256; ++i) {
+      const int e = tid + i * 256, r = e / kGK, k = e % kGK, n = n0 + r;
+      as[k][r] = k0 + k < K ? to_f(x[static_cast<size_t>(src[r]) * K + k0 + k]) : 0.f;
+      bs[k][r] = (k0 + k < K && n < N) ? to_f(wg[static_cast<size_t>(n) * K + k0 + k]) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < kGK; ++k) {
+      const float4 a = *reinterpret_cast<const float4*>(&as[k][tr]), b = *reinterpret_cast<const float4*>(&bs[k][tc]);
+      const float av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] += av[i] * bv[j];
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+      if (r0 + tr + i < r1 && n0 + tc + j < N)
+        out[static_cast<size_t>(r0 + tr + i) * N + n0 + tc + j] = from_f<T>(acc[i][j]);
+}
+
+template <typename T>
+int route(const float* z, const void* x, const void* w, const void* bias, float* out_w, int* out_ids, int T_, int E, int K,
+          int k, cudaStream_t s) {
+  const T* b = static_cast<const T*>(bias);
+  if (z != nullptr) {
+    launch_pdl(route_logits_kernel<T>, dim3((T_ + 3) / 4), dim3(128), 4 * E * sizeof(float), s, z, b, out_w, out_ids, T_, E,
+               k);
+  } else {
+    const size_t smem = ((K + 3) / 4 * 4 + E) * sizeof(float);
+    if (smem > 48 * 1024) {
+      static size_t cfg = 0;
+      if (cfg < smem) {
+        const cudaError_t e = cudaFuncSetAttribute(route_token_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                                   static_cast<int>(smem));
+        if (e != cudaSuccess) return static_cast<int>(e);
+        cfg = smem;
+      }
+    }
+    const int wide = K % 8 == 0 && reinterpret_cast<uintptr_t>(w) % 16 == 0;
+    launch_pdl(route_token_kernel<T>, dim3(T_), dim3(kRouteThreads), smem, s, static_cast<const T*>(x),
+               static_cast<const T*>(w), b, out_w, out_ids, E, K, k, wide);
+  }
+  return static_cast<int>(cudaGetLastError());
+}
+
+}  // namespace
+}  // namespace sglb
+
+extern "C" {
+
+// x [T, K], w [E, K], bias [E] or null (bf16 or fp32); z [T, E] fp32: logits without the bias, if computed elsewhere.
+int sglb_route_by_logit(const float* z, const void* x, const void* w, const void* bias, float* out_w, int* out_ids, int T,
+                        int E, int K, int k, int is_f32, cudaStream_t s) {
+  using namespace sglb;
+  if (T <= 0) return 0;
+  if (E < 1 || E > kMaxExperts || k < 1 || k > kMaxTop || k > E || K < 1 || K > 32768) return -kBadArgument;
+  return is_f32 ? route<float>(z, x, w, bias, out_w, out_ids, T, E, K, k, s)
+                : route<__nv_bfloat16>(z, x, w, bias, out_w, out_ids, T, E, K, k, s);
+}
+
+// x rows of K, row_token [rows] or null (row r reads x row r), w [groups, N, K], out [rows, N]; lists from sglb_moe_align.
+int sglb_grouped_gemm_any(const void* x, const int* row_token, const void* w, void* out, const int* offsets,
+                          const int* tile_group, const int* tile_row0, const int* num_tiles, int rows, int N, int K,
+                          int groups, int is_f32, cudaStream_t s) {
+  using namespace sglb;
+  if (rows <= 0 || groups <= 0) return 0;
+  const dim3 grid(2 * (rows / 128 + groups), (N + kGN - 1) / kGN);
+  if (grid.y > 65535) return -kBadArgument;
+  if (is_f32)
+    launch_pdl(grouped_gemm_any_kernel<float>, grid, dim3(256), 0, s, static_cast<const float*>(x), row_token,
+               static_cast<const float*>(w), static_cast<float*>(out), offsets, tile_group, tile_row0, num_tiles, N, K);
+  else
+    launch_pdl(grouped_gemm_any_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, static_cast<const __nv_bfloat16*>(x),
+               row_token, static_cast<const __nv_bfloat16*>(w), static_cast<__nv_bfloat16*>(out), offsets, tile_group,
+               tile_row0, num_tiles, N, K);
+  return static_cast<int>(cudaGetLastError());
+}
+
+}  // extern "C"

@@ -2,11 +2,15 @@
 // fp32 throughout).  A sublayer reads the stream itself, in T; its result is normalised, scaled per channel and added
 // back:
 //
-//   embed_scaled       x = table[id] * scale                          -> x (fp32), x in T
+//   embed_scaled       x = table[id] * scale (+ sinusoidal position)  -> x (fp32), x in T
 //   postnorm_add       x <- x + s * y / sqrt(mean(y^2) + eps)         -> x (fp32, in place), x in T
-//                      (s, fp32 per channel, holds norm weight, layer scale and residual multiplier)
+//                      (s, fp32 per channel, holds norm weight, layer scale and residual multiplier), or, instead of x in
+//                      T, the next sublayer's input x / sqrt(mean(x^2) + eps') * w
+//   stream_add         x <- x + y (+ weighted rows of routed experts) -> x (fp32, in place), x in T
 //   rmsnorm_stream     y = x / sqrt(mean(x^2) + eps) * w              -> y in T
 //   gelu_mul           gelu_tanh(a) * b of a fused [a | b] projection
+//   clipped_swiglu     g sigmoid(alpha g) (u + 1) of a fused [a | b] projection, g = min(a, limit), u = clamp(b, +-limit)
+//   side_gate          gelu_tanh(z) * a column range of table[id]
 //   sigmoid_gate       o * sigmoid(g), g a column range of a wider projection
 //
 // One CTA per row for the norms, the row in registers between its two passes.  This file is compiled without fast-math
@@ -66,9 +70,22 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
   return t;
 }
 
+// Adds sin / cos of `pos` times the channel pair's turns per position.  The angle is reduced to less than half a turn in
+// double precision, so that it is as exact at the millionth position as at the first.
+template <int VEC> __device__ __forceinline__ void add_position(float (&f)[VEC], const double* __restrict__ turns, int c,
+                                                                int pos) {
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) {
+    const double a = turns[(c + e) >> 1] * pos;
+    const float h = 2.f * static_cast<float>(a - rint(a));            // in half turns
+    f[e] += ((c + e) & 1) ? cospif(h) : sinpif(h);
+  }
+}
+
 template <typename T, int VEC>
 __global__ void embed_scaled_kernel(float* __restrict__ x, T* __restrict__ xt, const int* __restrict__ ids,
-                                    const T* __restrict__ table, int W, int rows, float scale) {
+                                    const T* __restrict__ table, int W, int rows, float scale,
+                                    const int* __restrict__ positions, const double* __restrict__ turns) {
   pdl_wait();
   const size_t t = blockIdx.x;
   const int id = min(max(ids[t], 0), rows - 1);
@@ -78,15 +95,17 @@ __global__ void embed_scaled_kernel(float* __restrict__ x, T* __restrict__ xt, c
     load_v<VEC>(src + i, f);
 #pragma unroll
     for (int e = 0; e < VEC; ++e) f[e] *= scale;
+    if (turns != nullptr) add_position<VEC>(f, turns, i, positions[t]);
     store_v<VEC>(x + t * W + i, f);
     if (xt != nullptr) store_v<VEC>(xt + t * W + i, f);
   }
 }
 
-template <typename T, int VEC, int VPT>
+template <typename T, int VEC, int VPT, bool NEXT>
 __global__ void postnorm_add_kernel(float* __restrict__ x, T* __restrict__ xt, const T* __restrict__ y,
-                                    const float* __restrict__ s, int W, float eps) {
-  __shared__ float red[32];
+                                    const float* __restrict__ s, int W, float eps, const float* __restrict__ next_s,
+                                    float next_eps) {
+  __shared__ float red[64];
   pdl_wait();
   const size_t row = static_cast<size_t>(blockIdx.x) * W;
   float v[VPT][VEC];
@@ -111,8 +130,60 @@ __global__ void postnorm_add_kernel(float* __restrict__ x, T* __restrict__ xt, c
 #pragma unroll
       for (int e = 0; e < VEC; ++e) xv[e] += v[i][e] * inv * sv[e];
       store_v<VEC>(x + row + c, xv);
-      if (xt != nullptr) store_v<VEC>(xt + row + c, xv);
+      if constexpr (NEXT) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) v[i][e] = xv[e];
+      } else {
+        if (xt != nullptr) store_v<VEC>(xt + row + c, xv);
+      }
     }
+  }
+  if constexpr (NEXT) {
+    ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i)
+      if ((threadIdx.x + i * blockDim.x) * VEC < W)
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) ss += v[i][e] * v[i][e];
+    const float next_inv = 1.f / sqrtf(block_sum(ss, red + 32) / W + next_eps);
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = (threadIdx.x + i * blockDim.x) * VEC;
+      if (c < W) {
+        float w[VEC];
+        load_v<VEC>(next_s + c, w);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) v[i][e] *= next_inv * w[e];
+        store_v<VEC>(xt + row + c, v[i]);
+      }
+    }
+  }
+}
+
+// One row per CTA.  `rows` (null: none) holds k result rows per token, negative where a result lives on another rank.
+template <typename T, int VEC>
+__global__ void stream_add_kernel(float* __restrict__ x, T* __restrict__ xt, const T* __restrict__ y,
+                                  const T* __restrict__ expert, const float* __restrict__ weights,
+                                  const int* __restrict__ rows, int k, int W) {
+  pdl_wait();
+  const size_t t = blockIdx.x, row = t * W;
+  for (int c = threadIdx.x * VEC; c < W; c += blockDim.x * VEC) {
+    float f[VEC], xv[VEC];
+    load_v<VEC>(y + row + c, f);
+    for (int j = 0; j < k; ++j) {
+      const int r = rows[t * k + j];
+      if (r < 0) continue;
+      const float w = weights[t * k + j];
+      float g[VEC];
+      load_v<VEC>(expert + static_cast<size_t>(r) * W + c, g);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) f[e] += w * g[e];
+    }
+    load_v<VEC>(x + row + c, xv);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) xv[e] += f[e];
+    store_v<VEC>(x + row + c, xv);
+    if (xt != nullptr) store_v<VEC>(xt + row + c, xv);
   }
 }
 
@@ -170,6 +241,47 @@ __global__ void gelu_mul_kernel(T* __restrict__ out, const T* __restrict__ in, l
 }
 
 template <typename T, int VEC>
+__global__ void clipped_swiglu_kernel(T* __restrict__ out, const T* __restrict__ in, long long rows, int F, float limit,
+                                      float alpha) {
+  pdl_wait();
+  const long long per = F / VEC, total = rows * per;
+  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < total;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long r = i / per;
+    const int c = static_cast<int>(i - r * per) * VEC;
+    float a[VEC], b[VEC];
+    load_v<VEC>(in + r * 2 * F + c, a);
+    load_v<VEC>(in + r * 2 * F + F + c, b);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) {
+      const float g = fminf(a[e], limit), u = fminf(fmaxf(b[e], -limit), limit);
+      a[e] = g / (1.f + expf(-alpha * g)) * (u + 1.f);
+    }
+    store_v<VEC>(out + r * F + c, a);
+  }
+}
+
+template <typename T, int VEC>
+__global__ void side_gate_kernel(T* __restrict__ out, const T* __restrict__ z, const T* __restrict__ table,
+                                 long long table_ld, int offset, const int* __restrict__ ids, int table_rows,
+                                 long long rows, int F) {
+  pdl_wait();
+  const long long per = F / VEC, total = rows * per;
+  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < total;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long r = i / per;
+    const int c = static_cast<int>(i - r * per) * VEC;
+    const int id = min(max(ids[r], 0), table_rows - 1);
+    float a[VEC], b[VEC];
+    load_v<VEC>(z + r * F + c, a);
+    load_v<VEC>(table + id * table_ld + offset + c, b);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) a[e] = gelu_tanh(a[e]) * b[e];
+    store_v<VEC>(out + r * F + c, a);
+  }
+}
+
+template <typename T, int VEC>
 __global__ void sigmoid_gate_kernel(T* __restrict__ out, const T* __restrict__ o, const T* __restrict__ g,
                                     long long g_stride, long long rows, int F) {
   pdl_wait();
@@ -218,24 +330,26 @@ bool for_row(int W, bool vec, int* threads, F&& f) {
 
 template <typename T>
 int embed_scaled(float* x, void* xt, const int* ids, const void* table, long long n, int W, int rows, float scale,
-                 cudaStream_t s) {
+                 const int* positions, const double* turns, cudaStream_t s) {
   T* o = static_cast<T*>(xt);
   const T* tb = static_cast<const T*>(table);
   if (W % 4 == 0)
     launch_pdl(embed_scaled_kernel<T, 4>, dim3(n), dim3(row_threads(W / 4) < 256 ? row_threads(W / 4) : 256), 0, s, x, o,
-               ids, tb, W, rows, scale);
+               ids, tb, W, rows, scale, positions, turns);
   else
     launch_pdl(embed_scaled_kernel<T, 1>, dim3(n), dim3(row_threads(W) < 256 ? row_threads(W) : 256), 0, s, x, o, ids, tb,
-               W, rows, scale);
+               W, rows, scale, positions, turns);
   return static_cast<int>(cudaGetLastError());
 }
 
 template <typename T>
-int postnorm_add(float* x, void* xt, const void* y, const float* sc, long long n, int W, float eps, cudaStream_t s) {
+int postnorm_add(float* x, void* xt, const void* y, const float* sc, long long n, int W, float eps, const float* next_s,
+                 float next_eps, cudaStream_t s) {
   int threads = 0;
   const bool ok = for_row(W, W % 4 == 0, &threads, [&]<int VEC, int VPT>() {
-    launch_pdl(postnorm_add_kernel<T, VEC, VPT>, dim3(n), dim3(threads), 0, s, x, static_cast<T*>(xt),
-               static_cast<const T*>(y), sc, W, eps);
+    const auto kernel = next_s != nullptr ? postnorm_add_kernel<T, VEC, VPT, true> : postnorm_add_kernel<T, VEC, VPT, false>;
+    launch_pdl(kernel, dim3(n), dim3(threads), 0, s, x, static_cast<T*>(xt), static_cast<const T*>(y), sc, W, eps, next_s,
+               next_eps);
   });
   return ok ? static_cast<int>(cudaGetLastError()) : -kBadArgument;
 }
@@ -262,6 +376,48 @@ int gelu_mul(void* out, const void* in, long long rows, int F, cudaStream_t s) {
 }
 
 template <typename T>
+int stream_add(float* x, void* xt, const void* y, const void* expert, const float* weights, const int* rows, int k,
+               long long n, int W, cudaStream_t s) {
+  T* o = static_cast<T*>(xt);
+  const T* a = static_cast<const T*>(y);
+  const T* b = static_cast<const T*>(expert);
+  auto threads = [](int groups) { return dim3(row_threads(groups) < 256 ? row_threads(groups) : 256); };
+  if (W % 4 == 0)
+    launch_pdl(stream_add_kernel<T, 4>, dim3(n), threads(W / 4), 0, s, x, o, a, b, weights, rows, k, W);
+  else
+    launch_pdl(stream_add_kernel<T, 1>, dim3(n), threads(W), 0, s, x, o, a, b, weights, rows, k, W);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T>
+int clipped_swiglu(void* out, const void* in, long long rows, int F, float limit, float alpha, cudaStream_t s) {
+  T* o = static_cast<T*>(out);
+  const T* i = static_cast<const T*>(in);
+  constexpr int kWide = sizeof(T) == 2 ? 8 : 4;
+  if (F % kWide == 0)
+    launch_pdl(clipped_swiglu_kernel<T, kWide>, dim3(grid_for(rows * (F / kWide))), dim3(256), 0, s, o, i, rows, F, limit,
+               alpha);
+  else
+    launch_pdl(clipped_swiglu_kernel<T, 1>, dim3(grid_for(rows * F)), dim3(256), 0, s, o, i, rows, F, limit, alpha);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T>
+int side_gate(void* out, const void* z, const void* table, long long ld, int offset, const int* ids, int table_rows,
+              long long rows, int F, cudaStream_t s) {
+  T* o = static_cast<T*>(out);
+  const T* a = static_cast<const T*>(z);
+  const T* b = static_cast<const T*>(table);
+  if (F % 4 == 0 && ld % 4 == 0 && offset % 4 == 0)
+    launch_pdl(side_gate_kernel<T, 4>, dim3(grid_for(rows * (F / 4))), dim3(256), 0, s, o, a, b, ld, offset, ids,
+               table_rows, rows, F);
+  else
+    launch_pdl(side_gate_kernel<T, 1>, dim3(grid_for(rows * F)), dim3(256), 0, s, o, a, b, ld, offset, ids, table_rows,
+               rows, F);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T>
 int sigmoid_gate(void* out, const void* o, const void* g, long long g_stride, long long rows, int F, cudaStream_t s) {
   T* d = static_cast<T*>(out);
   const T* a = static_cast<const T*>(o);
@@ -284,18 +440,45 @@ int sigmoid_gate(void* out, const void* o, const void* g, long long g_stride, lo
 extern "C" {
 
 // `is_f32`: T is fp32 (then `xt` is null, the fp32 stream itself is the projections' input), else bf16.
+// `turns` (null: no positions) [ceil(W / 2)]: turns per position of channels 2i (sine) and 2i + 1 (cosine).
 int sglb_embed_scaled(float* x, void* xt, const int* ids, const void* table, long long n, int W, int rows, float scale,
-                      int is_f32, cudaStream_t s) {
+                      const int* positions, const double* turns, int is_f32, cudaStream_t s) {
   if (n <= 0) return 0;
-  return is_f32 ? sglb::embed_scaled<float>(x, xt, ids, table, n, W, rows, scale, s)
-                : sglb::embed_scaled<__nv_bfloat16>(x, xt, ids, table, n, W, rows, scale, s);
+  if (turns != nullptr && positions == nullptr) return -sglb::kBadArgument;
+  return is_f32 ? sglb::embed_scaled<float>(x, xt, ids, table, n, W, rows, scale, positions, turns, s)
+                : sglb::embed_scaled<__nv_bfloat16>(x, xt, ids, table, n, W, rows, scale, positions, turns, s);
 }
 
-int sglb_postnorm_add(float* x, void* xt, const void* y, const float* scale, long long n, int W, float eps, int is_f32,
-                      cudaStream_t s) {
+// With `next_scale`, `xt` (then required in either type) receives next_scale * x / sqrt(mean(x^2) + next_eps).
+int sglb_postnorm_add(float* x, void* xt, const void* y, const float* scale, long long n, int W, float eps,
+                      const float* next_scale, float next_eps, int is_f32, cudaStream_t s) {
   if (n <= 0) return 0;
-  return is_f32 ? sglb::postnorm_add<float>(x, xt, y, scale, n, W, eps, s)
-                : sglb::postnorm_add<__nv_bfloat16>(x, xt, y, scale, n, W, eps, s);
+  if (next_scale != nullptr && xt == nullptr) return -sglb::kBadArgument;
+  return is_f32 ? sglb::postnorm_add<float>(x, xt, y, scale, n, W, eps, next_scale, next_eps, s)
+                : sglb::postnorm_add<__nv_bfloat16>(x, xt, y, scale, n, W, eps, next_scale, next_eps, s);
+}
+
+// x += y + sum_j weights[t, j] * expert[rows[t, j]] (k = 0: no experts).
+int sglb_stream_add(float* x, void* xt, const void* y, const void* expert, const float* weights, const int* rows, int k,
+                    long long n, int W, int is_f32, cudaStream_t s) {
+  if (n <= 0) return 0;
+  return is_f32 ? sglb::stream_add<float>(x, xt, y, expert, weights, rows, k, n, W, s)
+                : sglb::stream_add<__nv_bfloat16>(x, xt, y, expert, weights, rows, k, n, W, s);
+}
+
+int sglb_clipped_swiglu(void* out, const void* in, long long rows, int F, float limit, float alpha, int is_f32,
+                        cudaStream_t s) {
+  if (rows <= 0) return 0;
+  return is_f32 ? sglb::clipped_swiglu<float>(out, in, rows, F, limit, alpha, s)
+                : sglb::clipped_swiglu<__nv_bfloat16>(out, in, rows, F, limit, alpha, s);
+}
+
+// out [rows, F] = gelu_tanh(z) * table[ids, offset : offset + F], table rows of `ld` elements.
+int sglb_side_gate(void* out, const void* z, const void* table, long long ld, int offset, const int* ids, int table_rows,
+                   long long rows, int F, int is_f32, cudaStream_t s) {
+  if (rows <= 0) return 0;
+  return is_f32 ? sglb::side_gate<float>(out, z, table, ld, offset, ids, table_rows, rows, F, s)
+                : sglb::side_gate<__nv_bfloat16>(out, z, table, ld, offset, ids, table_rows, rows, F, s);
 }
 
 int sglb_rmsnorm_stream(void* y, const float* x, const float* w, long long n, int W, float eps, int is_f32,

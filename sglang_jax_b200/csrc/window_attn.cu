@@ -1,0 +1,560 @@
+// Windowed grouped-query attention that keeps a sequence's first tokens (window_mask.cuh), any sizes, in bf16 or fp32,
+// over the paged cache  [pages, kv heads, P, row],  row = [key | value], both parts padded to 16-byte units:
+//
+//   attn_prep          one pass over a step's fused projection: divides queries and keys by their root mean square per head,
+//                      writes queries (padded with zeros) and cache rows
+//   window_decode      every query token on its own (bf16): the heads of one KV head fill the 16 rows of an MMA, 64-key
+//                      tiles stream through a TMA ring straight out of the pages, KV split over CTAs + combine.  The
+//                      attention weights enter the value product as two bf16 terms (rounding and remainder)
+//   window_attn_any    the same on the CUDA cores in fp32: the fp32 mode and sizes the above does not take
+//
+// Both finish with the gate per head, if there is one: out * sigmoid(gate).  Waits are bounded, no multicast.  Compiled
+// without fast-math substitutions.
+#include <math.h>
+
+#include "common.cuh"
+#include "window_mask.cuh"
+
+namespace sglb {
+namespace {
+
+__device__ __forceinline__ float to_f(float v) { return v; }
+__device__ __forceinline__ float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <typename T> __device__ __forceinline__ T from_f(float v);
+template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
+
+constexpr float kLog2e = 1.4426950408889634f;
+
+// ------------------------------------------------------------------------------------------- prep
+template <typename T, int VEC> struct Pack { T v[VEC]; };
+template <> struct alignas(8) Pack<__nv_bfloat16, 4> { __nv_bfloat16 v[4]; };
+template <> struct alignas(16) Pack<float, 4> { float v[4]; };
+
+struct PrepParams {
+  long long ld;
+  int q_off, k_off, v_off, H, G, D, V, Dp, Vp, P, norm;
+  float eps;
+};
+
+// One warp per (token, head): query heads, then KV heads (key and value).
+template <typename T, int VEC>
+__global__ void __launch_bounds__(128)
+attn_prep_kernel(const T* __restrict__ proj, T* __restrict__ q, T* __restrict__ cache, const int* __restrict__ loc,
+                 long long tokens, const PrepParams p) {
+  pdl_wait();
+  const int lane = threadIdx.x & 31, units = p.H + (p.k_off >= 0 ? p.G : 0);
+  const long long wid = (blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x) >> 5;
+  if (wid >= tokens * units) return;
+  const long long t = wid / units;
+  const int u = static_cast<int>(wid - t * units);
+  const T* row = proj + t * p.ld;
+  auto normed = [&](const T* src, T* dst) {             // D values, zeros up to Dp
+    float inv = 1.f;
+    if (p.norm) {
+      float ss = 0.f;
+      for (int i = lane * VEC; i < p.D; i += 32 * VEC) {
+        const Pack<T, VEC> a = *reinterpret_cast<const Pack<T, VEC>*>(src + i);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) ss += to_f(a.v[e]) * to_f(a.v[e]);
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      inv = 1.f / sqrtf(ss / p.D + p.eps);
+    }
+    for (int i = lane * VEC; i < p.Dp; i += 32 * VEC) {
+      Pack<T, VEC> a;
+      if (i < p.D) a = *reinterpret_cast<const Pack<T, VEC>*>(src + i);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) a.v[e] = i < p.D ? from_f<T>(to_f(a.v[e]) * inv) : from_f<T>(0.f);
+      *reinterpret_cast<Pack<T, VEC>*>(dst + i) = a;
+    }
+  };
+  if (u < p.H) {
+    normed(row + p.q_off + static_cast<long long>(u) * p.D, q + (t * p.H + u) * p.Dp);
+    return;
+  }
+  const int g = u - p.H, slot = loc[t], page = slot / p.P;
+  T* dst = cache + ((static_cast<long long>(page) * p.G + g) * p.P + (slot - page * p.P)) * (p.Dp + p.Vp);
+  normed(row + p.k_off + static_cast<long long>(g) * p.D, dst);
+  const T* v = row + p.v_off + static_cast<long long>(g) * p.V;
+  for (int i = lane * VEC; i < p.Vp; i += 32 * VEC) {
+    Pack<T, VEC> a;
+    if (i < p.V) a = *reinterpret_cast<const Pack<T, VEC>*>(v + i);
+    else
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) a.v[e] = from_f<T>(0.f);
+    *reinterpret_cast<Pack<T, VEC>*>(dst + p.Dp + i) = a;
+  }
+}
+
+// ------------------------------------------------------------------------------------------- decode
+constexpr int kTile = 64;                    // keys per tile
+constexpr int kConsumers = 4;                // warps, 16 keys of a tile each
+constexpr int kThreads = (kConsumers + 1) * 32;
+constexpr int kBlock = kTile * 128;          // [64 keys][64 bf16], swizzled
+constexpr int kStages = 3;
+
+struct DecodeParams {
+  const __nv_bfloat16* q;                    // [N, H, Dp]
+  __nv_bfloat16* out;                        // [N, H, V]
+  const __nv_bfloat16* gate;                 // [N, H] with row stride gate_ld, or null
+  long long gate_ld;
+  float* part_o;                             // splits: [N, H, S, V]
+  float* part_lse;                           // [N, H, S]
+  const int *page_table, *rows, *lens;
+  Status* status;
+  int H, G, Dp, V, max_pages, page_size, splits, m_blocks;
+  Window win;
+  float scale_log2;
+};
+
+__device__ __forceinline__ void ldsm_x4(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ldsm_x4_t(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// byte offset of (row, 16-byte chunk) inside a swizzled block
+__device__ __forceinline__ uint32_t sw_off(int row, int chunk) { return row * 128 + ((chunk ^ (row & 7)) << 4); }
+
+__device__ __forceinline__ float gate_of(const __nv_bfloat16* gate, long long ld, long long n, int h) {
+  return gate == nullptr ? 1.f : 1.f / (1.f + expf(-__bfloat162float(gate[n * ld + h])));
+}
+
+// NK / NV: 64-lane blocks of a key / value
+template <int NK, int NV>
+__global__ void __launch_bounds__(kThreads)
+window_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
+                     const DecodeParams p) {
+  constexpr int kStage = (NK + NV) * kBlock;
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  uint64_t* full_bar = reinterpret_cast<uint64_t*>(smem + kStages * kStage);
+  uint64_t* empty_bar = full_bar + kStages;
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(empty_bar + kStages);
+  float* merge = reinterpret_cast<float*>(smem);       // used after the main loop
+
+  const int n = blockIdx.x, g = blockIdx.y / p.m_blocks, mb = blockIdx.y - g * p.m_blocks, split = blockIdx.z;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int share = p.H / p.G, h0 = g * share + mb * 16, nh = min(16, share - mb * 16);
+  if (threadIdx.x == 0) {
+    for (int s = 0; s < kStages; ++s) {
+      mbar_init(smem_u32(&full_bar[s]), 1);
+      mbar_init(smem_u32(&empty_bar[s]), kConsumers);
+    }
+    *abort_flag = 0;
+    fence_barrier_init();
+  }
+  pdl_wait();
+  const int pos = p.lens[n] - 1;
+  const int* pt = p.page_table + static_cast<size_t>(p.rows[n]) * p.max_pages;
+  const int lo = p.win.first(pos);
+  const KeyTiles<kTile> tiles(p.win, pos, pos);
+  const int per = (tiles.count + p.splits - 1) / p.splits, i0 = split * per, i1 = min(i0 + per, tiles.count);
+  __syncthreads();
+
+  float o[NV * 8][4];
+  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};    // rows lane / 4 and lane / 4 + 8, log2 domain
+#pragma unroll
+  for (int i = 0; i < NV * 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+
+  if (warp == kConsumers) {
+    if (lane == 0) {
+      prefetch_tmap(&map_k);
+      prefetch_tmap(&map_v);
+      const int run = p.page_size < kTile ? p.page_size : kTile;
+      const uint64_t pol = l2_policy_evict_first();
+      for (int i = i0, c = 0; i < i1 && !*abort_flag; ++i, ++c) {
+        const int st = c % kStages;
+        if (!mbar_wait(smem_u32(&empty_bar[st]), ((c / kStages) & 1) ^ 1)) {
+          report(p.status, kTimeoutEmptyBarrier, n, i);
+          *abort_flag = 1;
+          break;
+        }
+        const uint32_t bar = smem_u32(&full_bar[st]), dst = smem_u32(smem + st * kStage);
+        mbar_expect_tx(bar, kStage);
+        const int tok0 = tiles.tile(i) * kTile;
+        for (int r = 0; r < kTile / run; ++r) {
+          const int tok = tok0 + r * run, pg = min(tok / p.page_size, p.max_pages - 1);
+          const int row = (pt[pg] * p.G + g) * p.page_size + tok % p.page_size;
+#pragma unroll
+          for (int b = 0; b < NK; ++b) tma_load_2d_hint(dst + b * kBlock + r * run * 128, &map_k, bar, b * 64, row, pol);
+#pragma unroll
+          for (int b = 0; b < NV; ++b)
+            tma_load_2d_hint(dst + (NK + b) * kBlock + r * run * 128, &map_v, bar, b * 64, row, pol);
+        }
+      }
+    }
+  } else {
+    const int gr = lane >> 2, t4 = lane & 3;
+    uint32_t qf[NK * 4][4];
+    const __nv_bfloat16* qa = p.q + (static_cast<size_t>(n) * p.H + h0 + gr) * p.Dp;
+    const __nv_bfloat16* qb = qa + 8 * p.Dp;
+#pragma unroll
+    for (int kk = 0; kk < NK * 4; ++kk) {
+      const int c = kk * 16 + t4 * 2;
+      qf[kk][0] = gr < nh && c < p.Dp ? *reinterpret_cast<const uint32_t*>(qa + c) : 0u;
+      qf[kk][1] = gr + 8 < nh && c < p.Dp ? *reinterpret_cast<const uint32_t*>(qb + c) : 0u;
+      qf[kk][2] = gr < nh && c + 8 < p.Dp ? *reinterpret_cast<const uint32_t*>(qa + c + 8) : 0u;
+      qf[kk][3] = gr + 8 < nh && c + 8 < p.Dp ? *reinterpret_cast<const uint32_t*>(qb + c + 8) : 0u;
+    }
+    for (int i = i0, c = 0; i < i1 && !*abort_flag; ++i, ++c) {
+      const int st = c % kStages;
+      if (!mbar_wait(smem_u32(&full_bar[st]), (c / kStages) & 1)) {
+        report(p.status, kTimeoutFullBarrier, n, i);
+        *abort_flag = 1;
+        break;
+      }
+      const uint32_t ks = smem_u32(smem + st * kStage), vs = ks + NK * kBlock;
+      const int tok0 = tiles.tile(i) * kTile + warp * 16;      // this warp's 16 keys
+      if (tok0 <= pos && (tok0 + 15 >= lo || tok0 < p.win.keep)) {
+        float s[2][4] = {};
+#pragma unroll
+        for (int kk = 0; kk < NK * 4; ++kk) {
+          if (kk * 16 >= p.Dp) break;
+          uint32_t b[4];
+          ldsm_x4(ks + (kk >> 2) * kBlock +
+                      sw_off(warp * 16 + (lane & 7) + ((lane >> 4) << 3), (kk & 3) * 2 + ((lane >> 3) & 1)),
+                  b);
+          mma16816(s[0], qf[kk], b[0], b[1]);
+          mma16816(s[1], qf[kk], b[2], b[3]);
+        }
+        float mx[2] = {m[0], m[1]};
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int key = tok0 + j * 8 + t4 * 2 + (e & 1);
+            s[j][e] = key <= pos && (key >= lo || key < p.win.keep) ? s[j][e] * p.scale_log2 : -INFINITY;
+            mx[e >> 1] = fmaxf(mx[e >> 1], s[j][e]);
+          }
+        float corr[2], ref[2], sum[2] = {0.f, 0.f};
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
+          mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
+          ref[r] = mx[r] == -INFINITY ? 0.f : mx[r];
+          corr[r] = exp2f(m[r] - ref[r]);
+          m[r] = mx[r];
+        }
+        uint32_t hi[4], lw[4];
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+          for (int r = 0; r < 2; ++r) {
+            const float x = exp2f(s[j][2 * r] - ref[r]), y = exp2f(s[j][2 * r + 1] - ref[r]);
+            sum[r] += x + y;
+            const uint32_t h = pack_bf16(x, y);
+            hi[2 * j + r] = h;
+            lw[2 * j + r] = pack_bf16(x - __uint_as_float(h << 16), y - __uint_as_float(h & 0xffff0000u));
+          }
+#pragma unroll
+        for (int r = 0; r < 2; ++r) l[r] = l[r] * corr[r] + sum[r];
+#pragma unroll
+        for (int np = 0; np < NV * 4; ++np) {
+          if (np * 16 >= p.V) break;
+          uint32_t b[4];
+          const int dcol = np * 16 + ((lane >> 4) << 3);
+          ldsm_x4_t(vs + (dcol >> 6) * kBlock +
+                        sw_off(warp * 16 + (lane & 7) + (((lane >> 3) & 1) << 3), (dcol & 63) >> 3),
+                    b);
+#pragma unroll
+          for (int half = 0; half < 2; ++half) {
+            float(&acc)[4] = o[2 * np + half];
+            acc[0] *= corr[0];
+            acc[1] *= corr[0];
+            acc[2] *= corr[1];
+            acc[3] *= corr[1];
+            mma16816(acc, hi, b[2 * half], b[2 * half + 1]);
+            mma16816(acc, lw, b[2 * half], b[2 * half + 1]);
+          }
+        }
+      }
+      __syncwarp();
+      if (lane == 0) mbar_arrive(smem_u32(&empty_bar[st]));
+    }
+  }
+  __syncthreads();                                     // the ring is idle: it serves the merge of the four warps now
+  constexpr int kW = NV * 64;
+  float* m_s = merge;                                  // [4][16]
+  float* l_s = merge + 64;                             // [4][16]
+  float* o_s = merge + 128;                            // [4][16][kW]
+  if (warp < kConsumers) {
+    const int gr = lane >> 2, t4 = lane & 3;
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      float s = l[r];
+      s += __shfl_xor_sync(0xffffffffu, s, 1);
+      s += __shfl_xor_sync(0xffffffffu, s, 2);
+      if (t4 == 0) {
+        m_s[warp * 16 + gr + 8 * r] = m[r];
+        l_s[warp * 16 + gr + 8 * r] = s;
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < NV * 8; ++i) {
+      float* a = o_s + (warp * 16 + gr) * kW + i * 8 + t4 * 2;
+      a[0] = o[i][0];
+      a[1] = o[i][1];
+      a[8 * kW] = o[i][2];
+      a[8 * kW + 1] = o[i][3];
+    }
+  }
+  __syncthreads();
+  for (int idx = threadIdx.x; idx < nh * p.V; idx += kThreads) {
+    const int r = idx / p.V, d = idx - r * p.V;
+    float mm = -INFINITY;
+#pragma unroll
+    for (int w = 0; w < kConsumers; ++w) mm = fmaxf(mm, m_s[w * 16 + r]);
+    float ls = 0.f, acc = 0.f;
+#pragma unroll
+    for (int w = 0; w < kConsumers; ++w) {
+      const float f = m_s[w * 16 + r] == -INFINITY ? 0.f : exp2f(m_s[w * 16 + r] - mm);
+      ls += l_s[w * 16 + r] * f;
+      acc += o_s[(w * 16 + r) * kW + d] * f;
+    }
+    const float inv = ls > 0.f ? 1.f / ls : 0.f;
+    const size_t nh_ = static_cast<size_t>(n) * p.H + h0 + r;
+    if (p.splits == 1) {
+      p.out[nh_ * p.V + d] = __float2bfloat16(acc * inv * gate_of(p.gate, p.gate_ld, n, h0 + r));
+    } else {
+      p.part_o[(nh_ * p.splits + split) * p.V + d] = acc * inv;
+      if (d == 0) p.part_lse[nh_ * p.splits + split] = ls > 0.f ? mm + log2f(ls) : -INFINITY;
+    }
+  }
+}
+
+__global__ void window_combine_kernel(const DecodeParams p) {
+  pdl_wait();
+  const long long row = blockIdx.x;                    // n * H + h
+  const float* lse = p.part_lse + row * p.splits;
+  float mm = -INFINITY;
+  for (int s = 0; s < p.splits; ++s) mm = fmaxf(mm, lse[s]);
+  float ws = 0.f;
+  for (int s = 0; s < p.splits; ++s) ws += lse[s] == -INFINITY ? 0.f : exp2f(lse[s] - mm);
+  const float f = (ws > 0.f ? 1.f / ws : 0.f) * gate_of(p.gate, p.gate_ld, row / p.H, static_cast<int>(row % p.H));
+  for (int d = threadIdx.x; d < p.V; d += blockDim.x) {
+    float acc = 0.f;
+    for (int s = 0; s < p.splits; ++s)
+      if (lse[s] != -INFINITY) acc += exp2f(lse[s] - mm) * p.part_o[(row * p.splits + s) * p.V + d];
+    p.out[row * p.V + d] = __float2bfloat16(acc * f);
+  }
+}
+
+template <int NK, int NV>
+int launch_decode(const CUtensorMap& mk, const CUtensorMap& mv, const DecodeParams& p, int N, cudaStream_t s) {
+  constexpr int smem = kStages * (NK + NV) * kBlock + 2 * kStages * 8 + 16 + 1024;
+  static_assert((128 + 4 * 16 * NV * 64) * 4 <= kStages * (NK + NV) * kBlock, "the merge fits into the ring");
+  static bool cfg = false;
+  if (!cfg) {
+    const cudaError_t e = cudaFuncSetAttribute(window_decode_kernel<NK, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    cfg = true;
+  }
+  launch_pdl(window_decode_kernel<NK, NV>, dim3(N, p.G * p.m_blocks, p.splits), dim3(kThreads), smem, s, mk, mv, p);
+  int e = static_cast<int>(cudaGetLastError());
+  if (e != 0 || p.splits == 1) return e;
+  launch_pdl(window_combine_kernel, dim3(N * p.H), dim3(p.V < 128 ? 64 : 128), 0, s, p);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <int NK>
+int launch_decode_v(int nv, const CUtensorMap& mk, const CUtensorMap& mv, const DecodeParams& p, int N, cudaStream_t s) {
+  switch (nv) {
+    case 1: return launch_decode<NK, 1>(mk, mv, p, N, s);
+    case 2: return launch_decode<NK, 2>(mk, mv, p, N, s);
+    case 3: return launch_decode<NK, 3>(mk, mv, p, N, s);
+    default: return launch_decode<NK, 4>(mk, mv, p, N, s);
+  }
+}
+
+// ------------------------------------------------------------------------------------------- any size
+// One CTA per (query token, head): online softmax over tiles of 64 keys.
+constexpr int kAnyThreads = 128;
+constexpr int kAnyMaxAcc = 8;                          // value width up to 8 * 128
+
+struct AnyParams {
+  long long gate_ld;
+  const int *page_table, *rows, *lens;
+  int H, G, D, V, Dp, Vp, max_pages, page_size;
+  Window win;
+  float scale;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(kAnyThreads)
+window_attn_any_kernel(const T* __restrict__ q, const T* __restrict__ gate, const T* __restrict__ cache,
+                       T* __restrict__ out, const AnyParams p) {
+  extern __shared__ float sm[];
+  float* qs = sm;                                      // [D]
+  float* sc = sm + p.D;                                // [kTile]
+  int* slot = reinterpret_cast<int*>(sc + kTile);      // [kTile] row of the cache
+  pdl_wait();
+  const int h = blockIdx.y, g = h / (p.H / p.G), tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const long long n = blockIdx.x, nh = n * p.H + h;
+  const int pos = p.lens[n] - 1, width = p.Dp + p.Vp;
+  const int* pt = p.page_table + static_cast<long long>(p.rows[n]) * p.max_pages;
+  for (int i = tid; i < p.D; i += kAnyThreads) qs[i] = to_f(q[nh * p.Dp + i]);
+  float acc[kAnyMaxAcc];
+#pragma unroll
+  for (int i = 0; i < kAnyMaxAcc; ++i) acc[i] = 0.f;
+  float m = -INFINITY, l = 0.f;
+  const KeyTiles<kTile> tiles(p.win, pos, pos);
+  for (int t = 0; t < tiles.count; ++t) {
+    const int k0 = tiles.tile(t) * kTile, nk = min(kTile, pos + 1 - k0);
+    __syncthreads();                                   // qs written / the previous tile's scores and slots read
+    if (tid < nk) {
+      const int pg = (k0 + tid) / p.page_size;
+      slot[tid] = (pt[pg] * p.G + g) * p.page_size + (k0 + tid - pg * p.page_size);
+    }
+    __syncthreads();
+    for (int j = warp; j < nk; j += kAnyThreads / 32) {
+      const T* kr = cache + static_cast<long long>(slot[j]) * width;
+      float a = 0.f;
+      for (int i = lane; i < p.D; i += 32) a += qs[i] * to_f(kr[i]);
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) a += __shfl_xor_sync(0xffffffffu, a, o);
+      if (lane == 0) sc[j] = p.win.sees(pos, k0 + j) ? a * p.scale : -INFINITY;
+    }
+    __syncthreads();
+    float mx = m;
+    for (int j = 0; j < nk; ++j) mx = fmaxf(mx, sc[j]);
+    if (mx == -INFINITY) continue;                     // nothing of this tile is visible (uniform for the CTA)
+    const float corr = expf(m - mx);
+    l *= corr;
+#pragma unroll
+    for (int i = 0; i < kAnyMaxAcc; ++i) acc[i] *= corr;
+    for (int j = 0; j < nk; ++j) {
+      const float w = expf(sc[j] - mx);
+      l += w;
+      const T* vr = cache + static_cast<long long>(slot[j]) * width + p.Dp;
+#pragma unroll
+      for (int i = 0; i < kAnyMaxAcc; ++i) {
+        const int d = tid + i * kAnyThreads;
+        if (d < p.V) acc[i] += w * to_f(vr[d]);
+      }
+    }
+    m = mx;
+  }
+  float f = l > 0.f ? 1.f / l : 0.f;
+  if (gate != nullptr) f *= 1.f / (1.f + expf(-to_f(gate[n * p.gate_ld + h])));
+#pragma unroll
+  for (int i = 0; i < kAnyMaxAcc; ++i) {
+    const int d = tid + i * kAnyThreads;
+    if (d < p.V) out[nh * p.V + d] = from_f<T>(acc[i] * f);
+  }
+}
+
+template <typename T>
+int prep(const void* proj, void* q, void* cache, const int* loc, long long tokens, const PrepParams& p, cudaStream_t s) {
+  const int units = p.H + (p.k_off >= 0 ? p.G : 0);
+  const dim3 grid(static_cast<unsigned>((tokens * units + 3) / 4));
+  const bool vec = p.D % 4 == 0 && p.V % 4 == 0 && p.ld % 4 == 0 && p.q_off % 4 == 0 &&
+                   (p.k_off < 0 || (p.k_off % 4 == 0 && p.v_off % 4 == 0)) &&
+                   reinterpret_cast<uintptr_t>(proj) % (4 * sizeof(T)) == 0;
+  const auto kernel = vec ? attn_prep_kernel<T, 4> : attn_prep_kernel<T, 1>;
+  launch_pdl(kernel, grid, dim3(128), 0, s, static_cast<const T*>(proj), static_cast<T*>(q), static_cast<T*>(cache), loc,
+             tokens, p);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T>
+int attn_any(const void* q, const void* gate, const void* cache, void* out, int N, const AnyParams& p, cudaStream_t s) {
+  launch_pdl(window_attn_any_kernel<T>, dim3(N, p.H), dim3(kAnyThreads), (p.D + 2 * kTile) * sizeof(float), s,
+             static_cast<const T*>(q), static_cast<const T*>(gate), static_cast<const T*>(cache), static_cast<T*>(out), p);
+  return static_cast<int>(cudaGetLastError());
+}
+
+int pad8(int n) { return (n + 7) / 8 * 8; }
+
+}  // namespace
+}  // namespace sglb
+
+extern "C" {
+
+// proj [T, ld]: query heads at column q_off, KV heads' keys / values at k_off / v_off (k_off < 0: the layer writes no
+// cache); q [T, H, pad8(D)], cache [pages, G, P, pad8(D) + pad8(V)], token t goes to slot loc[t].
+int sglb_attn_prep(const void* proj, long long ld, int q_off, int k_off, int v_off, void* q, void* cache, const int* loc,
+                   long long T, int H, int G, int D, int V, int P, int norm, float eps, int is_f32, cudaStream_t s) {
+  using namespace sglb;
+  if (T <= 0) return 0;
+  if (H < 1 || G < 1 || D < 1 || P < 1) return -kBadArgument;
+  const PrepParams p{ld, q_off, k_off, v_off, H, G, D, V, pad8(D), pad8(V), P, norm, eps};
+  return is_f32 ? prep<float>(proj, q, cache, loc, T, p, s) : prep<__nv_bfloat16>(proj, q, cache, loc, T, p, s);
+}
+
+// Whether window_decode takes these sizes.
+int sglb_window_decode_supported(int D, int V, int page_size) {
+  return D > 0 && V > 0 && D <= 256 && V <= 256 && (page_size < 64 ? page_size >= 8 && 64 % page_size == 0 : page_size % 64 == 0);
+}
+
+int sglb_window_num_splits(int N, int groups, int visible) {
+  const int sms = sglb::sm_count(), ctas = N * groups, tiles = (visible + 63) / 64 + 1;
+  int splits = (2 * sms + ctas - 1) / ctas;
+  if (splits > tiles / 2) splits = tiles / 2;
+  return splits < 1 ? 1 : (splits > 32 ? 32 : splits);
+}
+
+// Query n sees, of the first lens[n] tokens of table row rows[n], the last `window` (0: all) and the first `keep`.
+int sglb_window_decode(const void* q, const void* gate, long long gate_ld, const void* cache, long long num_pages,
+                       const int* page_table, int max_pages, int page_size, const int* rows, const int* lens, void* out,
+                       int N, int H, int G, int D, int V, float scale, int window, int keep, int splits, float* part_o,
+                       float* part_lse, cudaStream_t s) {
+  using namespace sglb;
+  if (N <= 0) return 0;
+  if (!sglb_window_decode_supported(D, V, page_size) || H % G != 0 || (splits > 1 && (!part_o || !part_lse)))
+    return -kBadArgument;
+  const int Dp = pad8(D), Vp = pad8(V);
+  const uint64_t n_rows = static_cast<uint64_t>(num_pages) * G * page_size, stride = static_cast<uint64_t>(Dp + Vp) * 2;
+  const __nv_bfloat16* c = static_cast<const __nv_bfloat16*>(cache);
+  const int run = page_size < 64 ? page_size : 64;
+  CUtensorMap mk, mv;
+  if (!encode_tmap_2d(&mk, c, Dp, n_rows, stride, 64, run, 2) || !encode_tmap_2d(&mv, c + Dp, Vp, n_rows, stride, 64, run, 2))
+    return -100;
+  DecodeParams p{};
+  p.q = static_cast<const __nv_bfloat16*>(q);
+  p.out = static_cast<__nv_bfloat16*>(out);
+  p.gate = static_cast<const __nv_bfloat16*>(gate);
+  p.gate_ld = gate_ld;
+  p.part_o = part_o;
+  p.part_lse = part_lse;
+  p.page_table = page_table;
+  p.rows = rows;
+  p.lens = lens;
+  p.status = device_status();
+  p.H = H; p.G = G; p.Dp = Dp; p.V = V; p.max_pages = max_pages; p.page_size = page_size;
+  p.splits = splits < 1 ? 1 : splits;
+  p.m_blocks = (H / G + 15) / 16;
+  if (static_cast<long long>(G) * p.m_blocks > 65535) return -kBadArgument;
+  p.win = Window{window, keep};
+  p.scale_log2 = scale * kLog2e;
+  const int nv = (Vp + 63) / 64;
+  switch ((Dp + 63) / 64) {
+    case 1: return launch_decode_v<1>(nv, mk, mv, p, N, s);
+    case 2: return launch_decode_v<2>(nv, mk, mv, p, N, s);
+    case 3: return launch_decode_v<3>(nv, mk, mv, p, N, s);
+    default: return launch_decode_v<4>(nv, mk, mv, p, N, s);
+  }
+}
+
+int sglb_window_attn_any(const void* q, const void* gate, long long gate_ld, const void* cache, const int* page_table,
+                         int max_pages, int page_size, const int* rows, const int* lens, void* out, int N, int H, int G,
+                         int D, int V, float scale, int window, int keep, int is_f32, cudaStream_t s) {
+  using namespace sglb;
+  if (N <= 0) return 0;
+  if (V > kAnyMaxAcc * kAnyThreads || D > 8192 || H > 65535 || H % G != 0) return -kBadArgument;
+  const AnyParams p{gate_ld, page_table, rows, lens, H, G, D, V, pad8(D), pad8(V), max_pages, page_size,
+                    Window{window, keep}, scale};
+  return is_f32 ? attn_any<float>(q, gate, cache, out, N, p, s) : attn_any<__nv_bfloat16>(q, gate, cache, out, N, p, s);
+}
+
+}  // extern "C"

@@ -1,0 +1,466 @@
+// Prefill of windowed grouped-query attention that keeps a sequence's first tokens (window_mask.cuh), on the 5th-generation
+// tensor cores (bf16 operands, fp32 softmax), over the paged cache  [pages, kv heads, P, row],  row = [key | value].
+//
+// One CTA per (256 query rows of one sequence, query head): two 128-row tiles that share every K / V tile of 64 keys.  The
+// key tiles are those of the kept first tokens and those from the first row's window on; a query tile leaves out the ones
+// that only the other needs.  Warp 0 drives TMA (page gathers, two-stage ring), warp 1 issues tcgen05.mma, warps 2..5 and
+// 6..9 do the softmax of the two tiles, one thread per row:
+//
+//   S_j = Q K_j^T      128 x 64, two accumulator buffers per tile in tensor memory
+//   P_j = exp2(S_j-m)  read with tcgen05.ld, written back over S_j as two bf16 terms (rounding and remainder, so that
+//                      the weights keep 16 bits of mantissa in the product) in the A-operand layout
+//   O  += P_j V_j      A from tensor memory, V the MN-major B operand in shared memory
+//
+// While one tile's exponentials run, the tensor pipe works on the other tile.  The running maximum is only raised when it
+// grows by more than 2^8.  Lanes past the widths arrive as zeros and whole zero steps are skipped.  The result is
+// multiplied by sigmoid(gate) per head, if there is one.  All waits are bounded; a timeout unwinds through the normal
+// teardown.  No multicast.
+#include <math.h>
+
+#include "common.cuh"
+#include "window_mask.cuh"
+
+namespace sglb {
+namespace {
+
+constexpr int kTileQ = 128, kTiles = 2, kTileK = 64;
+constexpr int kBlkQ = kTileQ * 128;                 // [128 rows][64 bf16], swizzled
+constexpr int kBlkK = kTileK * 128;                 // [64 keys][64 bf16]
+constexpr int kThreads = 64 + kTiles * 128;
+constexpr int kTmemCols = 512;                      // per tile: S 2 x 64 (P in place), O 128
+constexpr int kTmemTile = 256, kTmemO = 128;
+constexpr float kRescale = 8.f;
+constexpr float kLog2e = 1.4426950408889634f;
+constexpr int kMinSmem = 120 * 1024;                // one CTA per SM: it takes all of tensor memory
+
+struct Bars {
+  uint64_t q_full, k_full[2], k_empty[2], v_full[2], v_empty[2];
+  uint64_t s_full[kTiles][2], p_ready[kTiles][2], pv_done[kTiles][2];
+  uint32_t tmem_slot;
+  int abort_flag;
+};
+
+struct Params {
+  __nv_bfloat16* out;            // [T, H, V]
+  const __nv_bfloat16* gate;     // [T, H] with row stride gate_ld, or null
+  long long gate_ld;
+  const int *q_start, *q_len, *prefix, *rows;        // [B]
+  const int* page_table;
+  Status* status;
+  int B, H, G, Dp, V, max_pages, page_size;
+  int nb_k, nb_v;                // 64-lane blocks of a key / value
+  Window win;
+  float scale_log2;
+};
+
+// The key tiles of one CTA, and of each of its query tiles.  Tiles are numbered as KeyTiles orders them.  Query tile t
+// leaves out [gap, gap + skip) and everything from n on; local(j) counts the tiles it takes.
+struct QueryTile {
+  int n, gap, skip;
+  __device__ __forceinline__ bool takes(int j) const { return j < n && (j < gap || j >= gap + skip); }
+  __device__ __forceinline__ int local(int j) const { return j < gap ? j : j - skip; }
+  __device__ __forceinline__ int count() const { return n > 0 ? n - skip : 0; }
+};
+
+__device__ __forceinline__ float ex2_approx(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+__global__ void __launch_bounds__(kThreads, 1)
+window_extend_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
+                     const __grid_constant__ CUtensorMap map_v, const Params p) {
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  const int nb_q = p.nb_k;
+  const int stage_bytes = (nb_q + p.nb_v) * kBlkK;
+  uint8_t* q_s = smem;                                            // [tile][block]
+  uint8_t* kv_s = smem + kTiles * nb_q * kBlkQ;
+  Bars* bars = reinterpret_cast<Bars*>(kv_s + 2 * stage_bytes);
+  volatile int* abort_flag = &bars->abort_flag;
+
+  // (sequence, 256-row query tile); long rows of keys first
+  int b = 0, tile = -1;
+  {
+    int acc = 0;
+    const int want = gridDim.x - 1 - blockIdx.x;
+    for (int i = 0; i < p.B; ++i) {
+      const int nt = (p.q_len[i] + kTiles * kTileQ - 1) / (kTiles * kTileQ);
+      if (want < acc + nt) {
+        b = i;
+        tile = want - acc;
+        break;
+      }
+      acc += nt;
+    }
+    if (tile < 0) return;
+  }
+  const int head = blockIdx.y, kv_head = head / (p.H / p.G);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int q_len = p.q_len[b], prefix = p.prefix[b], seq = prefix + q_len;
+  const int q0 = tile * kTiles * kTileQ;
+  const int* pt_row = p.page_table + static_cast<size_t>(p.rows[b]) * p.max_pages;
+  const KeyTiles<kTileK> keys(p.win, prefix + q0, prefix + min(q0 + kTiles * kTileQ, q_len) - 1);
+  QueryTile qt[kTiles];
+  {
+    // tiles of kept tokens reach this far; beyond, a query tile starts at its own window
+    const int kept_end = keys.kept + max(0, (p.win.keep + kTileK - 1) / kTileK - keys.begin);
+#pragma unroll
+    for (int t = 0; t < kTiles; ++t) {
+      const int first = q0 + t * kTileQ;
+      if (first >= q_len) {
+        qt[t] = {0, 0, 0};
+        continue;
+      }
+      const int own = keys.kept + p.win.first(prefix + first) / kTileK - keys.begin;
+      qt[t] = {keys.kept + (prefix + min(first + kTileQ, q_len) - 1) / kTileK + 1 - keys.begin, kept_end,
+               max(0, own - kept_end)};
+    }
+  }
+  const int n = max(qt[0].n, qt[1].n);
+
+  if (threadIdx.x == 0) {
+    prefetch_tmap(&map_q);
+    prefetch_tmap(&map_k);
+    prefetch_tmap(&map_v);
+    mbar_init(smem_u32(&bars->q_full), 1);
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(smem_u32(&bars->k_full[i]), 1);
+      mbar_init(smem_u32(&bars->k_empty[i]), 1);
+      mbar_init(smem_u32(&bars->v_full[i]), 1);
+      mbar_init(smem_u32(&bars->v_empty[i]), 1);
+      for (int t = 0; t < kTiles; ++t) {
+        mbar_init(smem_u32(&bars->s_full[t][i]), 1);
+        mbar_init(smem_u32(&bars->p_ready[t][i]), 4);             // one arrival per softmax warp of the tile
+        mbar_init(smem_u32(&bars->pv_done[t][i]), 1);
+      }
+    }
+    bars->abort_flag = 0;
+    fence_barrier_init();
+  }
+  if (warp == 1) {
+    tmem_alloc(smem_u32(&bars->tmem_slot), kTmemCols);
+    tmem_relinquish();
+  }
+  tc_fence_before_sync();
+  __syncthreads();
+  tc_fence_after_sync();
+  const uint32_t tmem = bars->tmem_slot;
+
+  if (warp == 0) {
+    // ------------------------------------------------------------------ TMA producer
+    if (lane == 0) {
+      const uint32_t qb = smem_u32(&bars->q_full);
+      mbar_expect_tx(qb, kTiles * nb_q * kBlkQ);
+      for (int t = 0; t < kTiles; ++t) {
+        const int row = p.q_start[b] + q0 + t * kTileQ;           // rows past the projection read as zeros
+        for (int c = 0; c < nb_q; ++c) {
+          const uint32_t dst = smem_u32(q_s + (t * nb_q + c) * kBlkQ);
+          tma_load_3d(dst, &map_q, qb, c * 64, head, row);
+        }
+      }
+      auto load = [&](int j, bool values) -> bool {
+        const int st = j & 1;
+        uint64_t* empty = values ? &bars->v_empty[st] : &bars->k_empty[st];
+        if (!mbar_wait(smem_u32(empty), ((j >> 1) & 1) ^ 1)) {
+          report(p.status, kTimeoutEmptyBarrier, b, j);
+          *abort_flag = 1;
+          return false;
+        }
+        const uint32_t fb = smem_u32(values ? &bars->v_full[st] : &bars->k_full[st]);
+        const uint32_t dst = smem_u32(kv_s + st * stage_bytes) + (values ? nb_q * kBlkK : 0);
+        const int run = p.page_size < kTileK ? p.page_size : kTileK, nb = values ? p.nb_v : nb_q;
+        mbar_expect_tx(fb, nb * kBlkK);
+        for (int r = 0; r < kTileK / run; ++r) {
+          const int tok = keys.tile(j) * kTileK + r * run, pg = min(tok / p.page_size, p.max_pages - 1);
+          const int row = (pt_row[pg] * p.G + kv_head) * p.page_size + tok % p.page_size;
+          for (int c = 0; c < nb; ++c) tma_load_2d(dst + c * kBlkK + r * run * 128, values ? &map_v : &map_k, fb, c * 64, row);
+        }
+        return true;
+      };
+      bool fed = load(0, false);
+      for (int j = 0; fed && j < n && !*abort_flag; ++j) {
+        if (j + 1 < n) fed = load(j + 1, false);
+        if (fed) fed = load(j, true);
+      }
+    }
+  } else if (warp == 1) {
+    // ------------------------------------------------------------------ MMA issuer
+    if (lane == 0) {
+      constexpr uint32_t idesc_s = make_idesc(kTileQ, kTileK, 1, 1);
+      const uint32_t idesc_pv = make_idesc(kTileQ, 64 * p.nb_v, 1, 1) | (1u << 16);      // B (values) is MN-major
+      const int steps = (p.Dp + 15) / 16;
+      bool ok = mbar_wait(smem_u32(&bars->q_full), 0);
+      if (!ok) report(p.status, kTimeoutFullBarrier, b, -1);
+      tc_fence_after_sync();
+      auto issue_pv = [&](int i) -> bool {
+        if (!mbar_wait(smem_u32(&bars->v_full[i & 1]), (i >> 1) & 1)) {
+          report(p.status, kTimeoutFullBarrier, b, 5000 + i);
+          return false;
+        }
+        const uint32_t v_addr = smem_u32(kv_s + (i & 1) * stage_bytes) + nb_q * kBlkK;
+        for (int t = 0; t < kTiles; ++t) {
+          if (!qt[t].takes(i)) continue;
+          const int li = qt[t].local(i);
+          if (!mbar_wait(smem_u32(&bars->p_ready[t][li & 1]), (li >> 1) & 1)) {
+            report(p.status, kTimeoutTmemFull, b, 1000 + i);
+            return false;
+          }
+          tc_fence_after_sync();
+          const uint32_t p_tm = tmem + t * kTmemTile + (li & 1) * kTileK, o_tm = tmem + t * kTmemTile + kTmemO;
+#pragma unroll
+          for (int term = 0; term < 2; ++term)
+#pragma unroll
+            for (int kk = 0; kk < kTileK / 16; ++kk)
+              umma_bf16_ts(o_tm, p_tm + term * (kTileK / 2) + kk * 8,
+                           make_smem_desc_sw128_mn(v_addr + kk * 16 * 128, kBlkK), idesc_pv,
+                           (li > 0 || term > 0 || kk > 0) ? 1u : 0u);
+          umma_commit(smem_u32(&bars->pv_done[t][li & 1]));
+        }
+        umma_commit(smem_u32(&bars->v_empty[i & 1]));
+        return true;
+      };
+      for (int j = 0; ok && j < n && !*abort_flag; ++j) {
+        const int st = j & 1;
+        if (!mbar_wait(smem_u32(&bars->k_full[st]), (j >> 1) & 1)) {
+          report(p.status, kTimeoutFullBarrier, b, j);
+          ok = false;
+          break;
+        }
+        const uint32_t k_addr = smem_u32(kv_s + st * stage_bytes);
+        for (int t = 0; ok && t < kTiles; ++t) {
+          if (!qt[t].takes(j)) continue;
+          const int lj = qt[t].local(j), sb = lj & 1;
+          // this S buffer holds P of the tile before last until its product is done
+          if (lj >= 2 && !mbar_wait(smem_u32(&bars->pv_done[t][sb]), ((lj - 2) >> 1) & 1)) {
+            report(p.status, kTimeoutTmemEmpty, b, j);
+            ok = false;
+            break;
+          }
+          tc_fence_after_sync();
+          const uint32_t q_addr = smem_u32(q_s + t * nb_q * kBlkQ), s_tm = tmem + t * kTmemTile + sb * kTileK;
+          for (int s = 0; s < steps; ++s)
+            umma_bf16(s_tm, make_smem_desc_sw128(q_addr + (s >> 2) * kBlkQ) + 2 * (s & 3),
+                      make_smem_desc_sw128(k_addr + (s >> 2) * kBlkK) + 2 * (s & 3), idesc_s, s > 0 ? 1u : 0u);
+          umma_commit(smem_u32(&bars->s_full[t][sb]));
+        }
+        if (!ok) break;
+        umma_commit(smem_u32(&bars->k_empty[st]));
+        if (j >= 1) ok = issue_pv(j - 1);
+      }
+      if (ok && !*abort_flag) ok = issue_pv(n - 1);
+      if (!ok) *abort_flag = 1;
+    }
+  } else {
+    // ------------------------------------------------------------------ softmax (one thread per query row)
+    const int t = (warp - 2) >> 2, qd = warp & 3;
+    const int row = qd * 32 + lane;
+    const uint32_t tm = tmem + t * kTmemTile + (static_cast<uint32_t>(qd * 32) << 16);
+    const int r_seq = q0 + t * kTileQ + row;                        // row within the sequence's new tokens
+    const int pos = min(prefix + r_seq, seq - 1);                   // rows past the end: anything finite
+    const int kmin = p.win.first(pos);
+    const float scale_log2 = p.scale_log2;
+    const int nt = qt[t].count();
+    float m_used = -INFINITY, l = 0.f;
+    bool ok = nt > 0;
+    for (int j = 0, lj = 0; ok && j < qt[t].n; ++j) {
+      if (!qt[t].takes(j)) continue;
+      const int st = lj & 1;
+      // (votes keep the warp's control flow uniform: one lane per warp arrives on the barriers below)
+      if (!__all_sync(0xffffffffu, mbar_wait(smem_u32(&bars->s_full[t][st]), (lj >> 1) & 1))) {
+        report(p.status, kTimeoutTmemFull, b, j);
+        *abort_flag = 1;
+        ok = false;
+        break;
+      }
+      tc_fence_after_sync();
+      uint32_t v0[32], v1[32];
+      const uint32_t s_addr = tm + st * kTileK;
+      tmem_ld32(s_addr, v0);
+      tmem_ld32(s_addr + 32, v1);
+      tmem_ld_wait();
+      // bit e: key e of this tile is visible
+      const int k0 = keys.tile(j) * kTileK;
+      auto below = [](int c) -> uint64_t { return c <= 0 ? 0ull : (c >= 64 ? ~0ull : (1ull << c) - 1); };
+      const uint64_t seen = below(pos - k0 + 1) & (~below(kmin - k0) | below(p.win.keep - k0));
+      const bool full = seen == ~0ull;
+      const uint32_t see0 = static_cast<uint32_t>(seen), see1 = static_cast<uint32_t>(seen >> 32);
+      float mx = -INFINITY;
+      if (full) {
+#pragma unroll
+        for (int e = 0; e < 32; ++e) mx = fmaxf(mx, fmaxf(__uint_as_float(v0[e]), __uint_as_float(v1[e])));
+      } else {
+#pragma unroll
+        for (int e = 0; e < 32; ++e) {
+          if ((see0 >> e) & 1) mx = fmaxf(mx, __uint_as_float(v0[e]));
+          if ((see1 >> e) & 1) mx = fmaxf(mx, __uint_as_float(v1[e]));
+        }
+      }
+      mx *= scale_log2;
+      const bool raise = lj > 0 && mx > m_used + kRescale;
+      if (lj == 0) {
+        m_used = mx;
+      } else if (__any_sync(0xffffffffu, raise)) {
+        // rare: bring O and the row sum to the new maximum, after the product in flight; tcgen05.ld / .st are
+        // warp-collective, rows that do not need it take part with a factor of one
+        if (!__all_sync(0xffffffffu, mbar_wait(smem_u32(&bars->pv_done[t][(lj - 1) & 1]), ((lj - 1) >> 1) & 1))) {
+          report(p.status, kTimeoutTmemFull, b, 2000 + j);
+          *abort_flag = 1;
+          ok = false;
+          break;
+        }
+        tc_fence_after_sync();
+        const float f = raise ? exp2f(m_used - mx) : 1.f;
+        l *= f;
+#pragma unroll 1
+        for (int c0 = 0; c0 < 64 * p.nb_v; c0 += 32) {
+          uint32_t o[32];
+          tmem_ld32(tm + kTmemO + c0, o);
+          tmem_ld_wait();
+#pragma unroll
+          for (int e = 0; e < 32; ++e) o[e] = __float_as_uint(__uint_as_float(o[e]) * f);
+          tmem_st32(tm + kTmemO + c0, o);
+        }
+        tmem_st_wait();
+        if (raise) m_used = mx;
+      }
+      float sum = 0.f;
+      const float ref = m_used == -INFINITY ? 0.f : m_used;         // (nothing seen so far)
+      uint32_t hi[32], lo[32];
+#pragma unroll
+      for (int c = 0; c < 32; ++c) {
+        const uint32_t a = c < 16 ? v0[2 * c] : v1[2 * c - 32], bb = c < 16 ? v0[2 * c + 1] : v1[2 * c - 31];
+        float x = ex2_approx(fmaf(__uint_as_float(a), scale_log2, -ref));
+        float y = ex2_approx(fmaf(__uint_as_float(bb), scale_log2, -ref));
+        if (!full) {
+          const uint32_t see = c < 16 ? see0 >> (2 * c) : see1 >> (2 * c - 32);
+          if (!(see & 1)) x = 0.f;
+          if (!(see & 2)) y = 0.f;
+        }
+        sum += x + y;
+        hi[c] = pack_bf16(x, y);
+        lo[c] = pack_bf16(x - __uint_as_float(hi[c] << 16), y - __uint_as_float(hi[c] & 0xffff0000u));
+      }
+      l += sum;
+      tmem_st32(s_addr, hi);
+      tmem_st32(s_addr + 32, lo);
+      tmem_st_wait();
+      tc_fence_before_sync();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(smem_u32(&bars->p_ready[t][st]));
+      ++lj;
+    }
+    if (ok) {
+      if (!__all_sync(0xffffffffu, mbar_wait(smem_u32(&bars->pv_done[t][(nt - 1) & 1]), ((nt - 1) >> 1) & 1))) {
+        report(p.status, kTimeoutTmemFull, b, 3000);
+        *abort_flag = 1;
+      } else {
+        tc_fence_after_sync();
+        const long long tok = p.q_start[b] + r_seq;
+        float inv = l > 0.f ? 1.f / l : 0.f;
+        if (p.gate != nullptr && r_seq < q_len)
+          inv *= 1.f / (1.f + expf(-__bfloat162float(p.gate[tok * p.gate_ld + head])));
+        __nv_bfloat16* orow = p.out + (tok * p.H + head) * p.V;
+        const bool wide = p.V % 8 == 0;
+#pragma unroll 1
+        for (int c0 = 0; c0 < p.V; c0 += 32) {
+          uint32_t o[32];
+          tmem_ld32(tm + kTmemO + c0, o);
+          tmem_ld_wait();
+          if (r_seq < q_len && wide) {
+#pragma unroll
+            for (int e = 0; e < 32; e += 8)
+              if (c0 + e < p.V)
+                *reinterpret_cast<uint4*>(orow + c0 + e) =
+                    make_uint4(pack_bf16(__uint_as_float(o[e]) * inv, __uint_as_float(o[e + 1]) * inv),
+                               pack_bf16(__uint_as_float(o[e + 2]) * inv, __uint_as_float(o[e + 3]) * inv),
+                               pack_bf16(__uint_as_float(o[e + 4]) * inv, __uint_as_float(o[e + 5]) * inv),
+                               pack_bf16(__uint_as_float(o[e + 6]) * inv, __uint_as_float(o[e + 7]) * inv));
+          } else if (r_seq < q_len) {
+#pragma unroll
+            for (int e = 0; e < 32; ++e)
+              if (c0 + e < p.V) orow[c0 + e] = __float2bfloat16(__uint_as_float(o[e]) * inv);
+          }
+          __syncwarp();
+        }
+      }
+    }
+  }
+
+  tc_fence_before_sync();
+  __syncthreads();
+  if (*abort_flag) {
+    // give copies and products that are still in flight time to land before shared and tensor memory are released
+    const uint64_t t0 = global_timer_ns();
+    while (global_timer_ns() - t0 < 200000ull) __nanosleep(1000);
+    __syncthreads();
+  }
+  if (warp == 1) {
+    tc_fence_after_sync();
+    tmem_dealloc(tmem, kTmemCols);
+  }
+}
+
+int extend_smem(int nb_k, int nb_v) {
+  const int need = kTiles * nb_k * kBlkQ + 2 * (nb_k + nb_v) * kBlkK + 256 + 1024;
+  return need > kMinSmem ? need : kMinSmem;
+}
+
+int pad8(int n) { return (n + 7) / 8 * 8; }
+
+}  // namespace
+}  // namespace sglb
+
+extern "C" {
+
+// Whether the prefill kernel takes these sizes.
+int sglb_window_extend_supported(int D, int V, int page_size) {
+  return D > 0 && V > 0 && V <= 128 && D <= 256 && (page_size < 64 ? page_size >= 8 && 64 % page_size == 0 : page_size % 64 == 0) &&
+         sglb::extend_smem((D + 63) / 64, (V + 63) / 64) <= 227 * 1024;
+}
+
+// q [total_q, H, pad8(D)]; cache [num_pages, G, page_size, pad8(D) + pad8(V)]; out [total_q, H, V].  B sequences: rows
+// q_start .. q_start + q_len of q, `prefix` tokens before them, page-table row `rows`.  num_tiles = sum_b ceil(q_len / 256).
+int sglb_window_extend(const void* q, int total_q, const void* gate, long long gate_ld, const void* cache,
+                       long long num_pages, const int* page_table, int max_pages, int page_size, const int* rows,
+                       const int* q_start, const int* q_len, const int* prefix, int B, int num_tiles, void* out, int H,
+                       int G, int D, int V, float scale, int window, int keep, cudaStream_t stream) {
+  using namespace sglb;
+  if (B <= 0 || num_tiles <= 0 || total_q <= 0) return 0;
+  if (!sglb_window_extend_supported(D, V, page_size) || H < 1 || H > 65535 || H % G != 0) return -kBadArgument;
+  const int Dp = pad8(D), Vp = pad8(V);
+  const __nv_bfloat16* c = static_cast<const __nv_bfloat16*>(cache);
+  const uint64_t n_rows = static_cast<uint64_t>(num_pages) * G * page_size, stride = static_cast<uint64_t>(Dp + Vp) * 2;
+  const int run = page_size < kTileK ? page_size : kTileK;
+  CUtensorMap mq, mk, mv;
+  if (!encode_tmap_3d(&mq, q, Dp, H, total_q, static_cast<uint64_t>(Dp) * 2, static_cast<uint64_t>(H) * Dp * 2, kTileQ) ||
+      !encode_tmap_2d(&mk, c, Dp, n_rows, stride, 64, run, 2) || !encode_tmap_2d(&mv, c + Dp, Vp, n_rows, stride, 64, run, 2))
+    return -100;
+  Params p{};
+  p.out = static_cast<__nv_bfloat16*>(out);
+  p.gate = static_cast<const __nv_bfloat16*>(gate);
+  p.gate_ld = gate_ld;
+  p.q_start = q_start;
+  p.q_len = q_len;
+  p.prefix = prefix;
+  p.rows = rows;
+  p.page_table = page_table;
+  p.status = device_status();
+  p.B = B; p.H = H; p.G = G; p.Dp = Dp; p.V = V; p.max_pages = max_pages; p.page_size = page_size;
+  p.nb_k = (Dp + 63) / 64;
+  p.nb_v = (Vp + 63) / 64;
+  p.win = Window{window, keep};
+  p.scale_log2 = scale * kLog2e;
+  const int smem = extend_smem(p.nb_k, p.nb_v);
+  static int cfg = 0;
+  if (cfg < smem) {
+    const cudaError_t e = cudaFuncSetAttribute(window_extend_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    cfg = smem;
+  }
+  window_extend_kernel<<<dim3(num_tiles, H), kThreads, smem, stream>>>(mq, mk, mv, p);
+  return static_cast<int>(cudaGetLastError());
+}
+
+}  // extern "C"

@@ -30,6 +30,11 @@ class GateLogit(nn.Module):
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         return F.linear(x.float(), self.weight.float(), self.bias.float() if self.bias is not None else None)
 
+    def route_by_logit(self, x: torch.Tensor, top_k: int):
+        """The experts with the largest logits, weights the softmax over the chosen logits only: `(weights fp32, ids int32)`,
+        `[T, top_k]` each."""
+        return ops.route_by_logit(x, self.weight, self.bias, top_k)
+
 
 class TopK(nn.Module):
     def __init__(self, top_k: int, renormalize: bool = True, num_expert_group: int = 0, topk_group: int = 0,

@@ -13,17 +13,14 @@ A step may mix both: the choice is made per sequence from the number of its new 
 
 from __future__ import annotations
 
-import numpy as np
 import torch
 from torch import nn
 
 from .. import ops
 from ..parallel import state as ps
 from .embeddings import get_rope
+from .extend_plan import extend_plan
 from .linear import PackedColumnParallelLinear, RowParallelLinear
-
-# a sequence with at least this many new tokens takes the expanded route
-EXPAND_MIN_TOKENS = 32
 
 
 class LatentAttention(nn.Module):
@@ -112,44 +109,3 @@ class LatentAttention(nn.Module):
             h1 = min(h0 + step, self.heads)
             kv = ops.linear(lat, self.up[h0:h1].reshape(-1, self.rank))
             ops.latent_extend(q[:, h0:h1], kv, pe, out[:, h0:h1], plan, self.dim, self.v_dim, self.scale)
-
-
-class ExtendPlan:
-    """How the sequences of an extend step are split between the two routes, as device tensors; one per forward."""
-
-    def __init__(self, fb, expand: bool):
-        n = np.asarray(fb.extend_seq_lens_cpu, np.int64)
-        pre = np.asarray(fb.extend_prefix_lens_cpu, np.int64)
-        start = np.concatenate([[0], np.cumsum(n)[:-1]])
-        long = np.nonzero(n >= EXPAND_MIN_TOKENS)[0] if expand else np.empty(0, np.int64)
-        dev = fb.positions.device
-        self.long = len(long)
-        # every token as a query of its own: its sequence's row, and the tokens up to and including itself
-        self.token_rows = torch.repeat_interleave(fb.req_pool_indices, fb.extend_seq_lens.long(), output_size=fb.num_tokens)
-        self.token_lens = fb.positions + 1
-        self.short_tokens = None
-        if self.long:
-            ctx = (pre + n)[long]
-            ctx_start = np.concatenate([[0], np.cumsum(ctx)])
-            self.ctx_total = int(ctx_start[-1])
-            tiles = (n[long] + 255) // 256              # query rows per CTA of the prefill kernel
-            self.num_tiles = int(tiles.sum())
-            rows = fb.req_pool_indices[torch.from_numpy(long).to(dev)]
-            meta = torch.from_numpy(np.concatenate([start[long], n[long], pre[long], ctx_start]).astype(np.int32)).to(dev)
-            L = self.long
-            self.q_start, self.q_len, self.prefix, self.ctx_start = meta[:L], meta[L:2 * L], meta[2 * L:3 * L], meta[3 * L:]
-            self.rows = rows
-            if L < len(n):
-                keep = np.ones(len(n), bool)
-                keep[long] = False
-                short = np.concatenate([np.arange(start[i], start[i] + n[i]) for i in np.nonzero(keep)[0]])
-                if len(short):
-                    self.short_tokens = torch.from_numpy(short).to(dev)
-
-
-def extend_plan(fb, expand: bool) -> ExtendPlan:
-    key = ("latent_extend_plan", expand)
-    plan = fb.extras.get(key)
-    if plan is None:
-        plan = fb.extras[key] = ExtendPlan(fb, expand)
-    return plan

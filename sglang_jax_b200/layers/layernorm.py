@@ -93,6 +93,10 @@ class PostNormResidual(nn.Module):
     def forward(self, y: torch.Tensor, x: torch.Tensor) -> torch.Tensor:
         return ops.postnorm_add(y, x, self.channel_scale, self.eps)
 
+    def then(self, y: torch.Tensor, x: torch.Tensor, norm: "StreamRMSNorm") -> torch.Tensor:
+        """The same step, but what is returned is `norm(x)`."""
+        return ops.postnorm_add_norm(y, x, self.channel_scale, self.eps, norm.channel_scale, norm.eps)
+
 
 class StreamRMSNorm(nn.Module):
     """RMSNorm of an fp32 residual stream, result in the model's type.  `multiplier` scales the result (a logit scale

@@ -100,19 +100,22 @@ class MergedColumnParallelLinear(LinearBase):
 
 class PackedColumnParallelLinear(LinearBase):
     """Any number of projections of one input as a single GEMM.  `parts`: name -> (output rows, split over the tensor
-    ranks?); parts that are not split are replicated.  Every part starts on a multiple of `ALIGN` output columns (zero
+    ranks?); parts that are not split are replicated, and a split of n > 1 shares each piece among n neighbouring ranks
+    (fewer key heads than ranks).  Every part starts on a multiple of `ALIGN` output columns (zero
     rows in between), so that the parts of an output row keep 16-byte alignment whatever their sizes."""
 
     ALIGN = 8
 
-    def __init__(self, in_features, parts: dict[str, tuple[int, bool]], dtype=torch.bfloat16, tp_size=None, tp_rank=None):
+    def __init__(self, in_features, parts: dict[str, tuple[int, bool | int]], dtype=torch.bfloat16, tp_size=None,
+                 tp_rank=None):
         self.tp_size = tp_size if tp_size is not None else ps.tp_size()
         self.tp_rank = tp_rank if tp_rank is not None else ps.tp_rank()
-        self.parts: dict[str, tuple[int, int, bool]] = {}            # name -> (first column, columns, split?)
+        self.parts: dict[str, tuple[int, int, bool | int]] = {}      # name -> (first column, columns, split?)
         off = 0
         for name, (rows, split) in parts.items():
-            assert not split or rows % self.tp_size == 0, f"{name}: {rows} rows do not split over {self.tp_size} ranks"
-            n = rows // self.tp_size if split else rows
+            pieces = self.tp_size // int(split) if split else 1
+            assert rows % pieces == 0, f"{name}: {rows} rows do not split over {self.tp_size} ranks"
+            n = rows // pieces
             self.parts[name] = (off, n, split)
             off += -(-n // self.ALIGN) * self.ALIGN
         super().__init__(in_features, off, False, dtype)
@@ -128,7 +131,7 @@ class PackedColumnParallelLinear(LinearBase):
 
     def weight_loader(self, param, w, shard_id: str):
         off, n, split = self.parts[shard_id]
-        param.data.narrow(0, off, n).copy_(w.narrow(0, self.tp_rank * n if split else 0, n))
+        param.data.narrow(0, off, n).copy_(w.narrow(0, self.tp_rank // int(split) * n if split else 0, n))
 
 
 class QKVParallelLinear(LinearBase):

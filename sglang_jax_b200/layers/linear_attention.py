@@ -195,17 +195,88 @@ class GatedDeltaRule(nn.Module):
     def forward(self, h: torch.Tensor, fb) -> torch.Tensor:
         pool = fb.extras["recurrent_pool"]
         y = self.proj(h)
-        ragged = {}
-        if not fb.forward_mode.is_decode():
-            ragged = dict(cu=fb.cu_q_lens, prefix=fb.extend_prefix_lens, lens=fb.extend_seq_lens_cpu)
-            track = checkpoint_tensors(fb)
-            if track is not None:
-                ragged.update(track_len=track[0], track_slot=track[1])
         o = ops.delta_scan(y, self.proj.offset("g"), self.proj.offset("b"), self.proj.offset("a"), self.conv_weight,
                            self.A_log, self.dt_bias, pool.conv_state[self.layer_index],
                            pool.recurrent_state[self.layer_index], recurrent_slots(fb), self.nv, self.nk, self.dk, self.dv,
-                           **ragged)
+                           **ragged_step(fb))
         return self.o_proj(ops.delta_gate(o, self.proj.part(y, "g"), self.norm_weight, self.eps))
+
+
+class ChannelDeltaRule(nn.Module):
+    """Delta rule whose state decays per key channel: as `GatedDeltaRule`, but the decay is one number per head and key
+    channel and comes from a low-rank pair of projections, and so does the gate of the read-out, a sigmoid.  Same kernels
+    (`csrc/delta_scan.cu`); everything from the convolution's output to the norm is fp32."""
+
+    def __init__(self, hidden_size: int, heads: int, kv_heads: int, dim: int, v_dim: int, conv_kernel: int, decay_rank: int,
+                 gate_rank: int, eps: float, linear_layer_index: int, dtype, reduce_results: bool = True):
+        super().__init__()
+        tp = ps.tp_size()
+        assert heads % kv_heads == 0 and kv_heads % tp == 0, f"{kv_heads} query/key heads do not split over {tp} ranks"
+        self.layer_index = linear_layer_index
+        self.nv, self.nk, self.dk, self.dv = heads // tp, kv_heads // tp, dim, v_dim
+        self.conv_kernel, self.eps = conv_kernel, float(eps)
+        self.key_dim, self.value_dim = self.nk * dim, self.nv * v_dim
+        self.conv_dim = 2 * self.key_dim + self.value_dim
+        # q, k and v columns stay adjacent (the kernels take them as one run of channels), hence one part
+        self.proj = PackedColumnParallelLinear(hidden_size, {"qkv": (self.conv_dim * tp, True), "b": (heads, True),
+                                                             "a1": (decay_rank, False), "g1": (gate_rank, False)}, dtype)
+        self.decay_up = nn.Parameter(torch.empty(self.nv * dim, decay_rank, dtype=dtype), requires_grad=False)
+        self.gate_up = nn.Parameter(torch.empty(self.value_dim, gate_rank, dtype=dtype), requires_grad=False)
+        self.conv_weight = nn.Parameter(torch.empty(self.conv_dim, conv_kernel, dtype=dtype), requires_grad=False)
+        self.A_log = nn.Parameter(torch.zeros(self.nv, dtype=torch.float32), requires_grad=False)
+        self.dt_bias = nn.Parameter(torch.zeros(self.nv * dim, dtype=torch.float32), requires_grad=False)
+        self.norm_weight = nn.Parameter(torch.ones(v_dim, dtype=torch.float32), requires_grad=False)
+        self.o_proj = RowParallelLinear(heads * v_dim, hidden_size, False, dtype, reduce_results=reduce_results)
+
+    def state_spec(self) -> dict:
+        return dict(conv_dim=self.conv_dim, conv_kernel=self.conv_kernel, num_heads=self.nv, head_k_dim=self.dk,
+                    head_v_dim=self.dv)
+
+    def load(self, name: str, w: torch.Tensor):
+        """One checkpoint tensor: q, k, v (projections), their `.conv` kernels, b, a1, a2, g1, g2, A_log, dt_bias, norm, o."""
+        r = ps.tp_rank()
+
+        def mine(n):                                   # this rank's rows of a tensor that splits by heads
+            return w.narrow(0, r * n, n)
+
+        base, conv = (name[:-5], True) if name.endswith(".conv") else (name, False)
+        if base in ("q", "k", "v"):
+            off = {"q": 0, "k": self.key_dim, "v": 2 * self.key_dim}[base]
+            n = self.value_dim if base == "v" else self.key_dim
+            (self.conv_weight if conv else self.proj.weight).data.narrow(0, off, n).copy_(mine(n))
+        elif name in ("b", "a1", "g1"):
+            self.proj.weight_loader(self.proj.weight, w, name)
+        elif name == "o":
+            self.o_proj.weight_loader(self.o_proj.weight, w)
+        elif name == "norm":
+            self.norm_weight.data.copy_(w)
+        elif name in ("a2", "g2", "A_log", "dt_bias"):
+            p = {"a2": self.decay_up, "g2": self.gate_up}.get(name)
+            p = getattr(self, name) if p is None else p
+            p.data.copy_(mine(p.shape[0]))
+        else:
+            raise KeyError(name)
+
+    def forward(self, h: torch.Tensor, fb) -> torch.Tensor:
+        pool = fb.extras["recurrent_pool"]
+        y = self.proj(h)
+        a = ops.low_rank_up(self.proj.part(y, "a1"), self.decay_up)
+        o = ops.delta_scan(y, -1, self.proj.offset("b"), -1, self.conv_weight, self.A_log, self.dt_bias,
+                           pool.conv_state[self.layer_index], pool.recurrent_state[self.layer_index], recurrent_slots(fb),
+                           self.nv, self.nk, self.dk, self.dv, channel_a=a, **ragged_step(fb))
+        gate = ops.low_rank_up(self.proj.part(y, "g1"), self.gate_up)
+        return self.o_proj(ops.delta_gate(o, gate, self.norm_weight, self.eps, "sigmoid"))
+
+
+def ragged_step(fb) -> dict:
+    """Arguments of `ops.delta_scan` that describe a step which is not a plain decode step."""
+    if fb.forward_mode.is_decode():
+        return {}
+    ragged = dict(cu=fb.cu_q_lens, prefix=fb.extend_prefix_lens, lens=fb.extend_seq_lens_cpu)
+    track = checkpoint_tensors(fb)
+    if track is not None:
+        ragged.update(track_len=track[0], track_slot=track[1])
+    return ragged
 
 
 def checkpoint_tensors(fb):

@@ -75,9 +75,12 @@ def configure_moe_runtime(num_redundant: int = 0, init_expert_location: str | No
 class FusedMoE(nn.Module):
     def __init__(self, num_experts: int, hidden_size: int, intermediate_size: int, dtype=torch.bfloat16,
                  ep_size: int | None = None, tp_size=None, tp_rank=None, layer_id: int = 0,
-                 activation: str = "silu"):
+                 activation: str = "silu", act_limit: float = 0.0, act_alpha: float = 1.702):
+        """`activation`: "silu", "gelu", or "clipped_swiglu" with its `act_limit` and `act_alpha`
+        (`ops.clipped_swiglu`)."""
         super().__init__()
         self.activation = activation
+        self.act_limit, self.act_alpha = float(act_limit), float(act_alpha)
         self.tp_size = tp_size if tp_size is not None else ps.tp_size()
         self.tp_rank = tp_rank if tp_rank is not None else ps.tp_rank()
         ep = ep_size if ep_size is not None else ps.ep_size()
@@ -113,6 +116,7 @@ class FusedMoE(nn.Module):
             self.local_intermediate = intermediate_size // self.tp_size
         I = self.local_intermediate
         self.workspace = None
+        self._outgrown = []              # workspaces that captured graphs may still point into
         self.routed_experts_capturer = None
         self.dtype = dtype
         # e4m3 storage from the start (set by the loader for W8A8 per-channel recipes): the bf16 experts of a large
@@ -251,21 +255,49 @@ class FusedMoE(nn.Module):
         return ((self.w13_weight.float() * self.w13_scale[..., None]).to(self.dtype),
                 (self.w2_weight.float() * self.w2_scale[..., None]).to(self.dtype))
 
-    def forward(self, x: torch.Tensor, topk_weights: torch.Tensor, topk_ids: torch.Tensor,
-                add: torch.Tensor | None = None, out: torch.Tensor | None = None) -> torch.Tensor:
-        """Partial sum over this rank's experts / intermediate slice (`add` is folded in, e.g. the
-        shared expert's partial output)."""
+    def _observe(self, topk_ids):
+        """Report the chosen experts to whoever listens; physical ids where experts have replicas."""
         if self.routed_experts_capturer is not None:
             self.routed_experts_capturer.capture(self.layer_id, topk_ids)
         if self.recorder is not None:
             self.recorder.record(self.layer_id, topk_ids)
-        if self.expert_location is not None:
-            topk_ids = self.expert_location.logical_to_physical(topk_ids)
+        return topk_ids if self.expert_location is None else self.expert_location.logical_to_physical(topk_ids)
+
+    def _workspace(self, pairs: int, device):
+        from ..ops import moe_native
+        if self.workspace is None or self.workspace.max_pairs < pairs:
+            if self.workspace is not None:
+                self._outgrown.append(self.workspace)
+            self.workspace = moe_native.MoeWorkspace(max(pairs, 2048), self.num_local_experts, device)
+        return self.workspace
+
+    def _act(self, h):
+        """Gated activation of `[gate | up]` rows by this layer's kind."""
+        if self.activation == "clipped_swiglu":
+            return ops.clipped_swiglu(h, self.act_limit, self.act_alpha)
+        return ops.silu_and_mul(h) if self.activation == "silu" else ops.gelu_and_mul(h)
+
+    def forward_stream(self, x: torch.Tensor, topk_weights: torch.Tensor, topk_ids: torch.Tensor, mixed: torch.Tensor,
+                       stream: torch.Tensor) -> torch.Tensor:
+        """`stream += mixed + sum of the chosen experts' outputs` on an fp32 residual stream, `mixed` another sublayer's
+        output (a partial sum, like the experts', under tensor parallelism); returns the stream in x's type."""
+        if ops.use_native_wide(x) and self.tp_size == 1 and not self.fp8:
+            from ..ops import moe_native
+            topk_ids = self._observe(topk_ids)
+            ws = self._workspace(topk_ids.numel(), x.device)
+            y = moe_native.sorted_experts(x, self.w13_weight, self.w2_weight, topk_ids, self.expert_start, ws, self._act)
+            return ops.stream_add(mixed, stream, y, topk_weights, ws.pair_row)
+        y = self.forward(x, topk_weights, topk_ids, add=mixed)
+        return ops.stream_add(ps.all_reduce(y) if self.tp_size > 1 else y, stream)
+
+    def forward(self, x: torch.Tensor, topk_weights: torch.Tensor, topk_ids: torch.Tensor,
+                add: torch.Tensor | None = None, out: torch.Tensor | None = None) -> torch.Tensor:
+        """Partial sum over this rank's experts / intermediate slice (`add` is folded in, e.g. the
+        shared expert's partial output)."""
+        topk_ids = self._observe(topk_ids)
         if ops.use_native(x) and self.activation == "silu":
             from ..ops import moe_native
-            pairs = x.shape[0] * topk_ids.shape[1]
-            if self.workspace is None or self.workspace.max_pairs < pairs:
-                self.workspace = moe_native.MoeWorkspace(max(pairs, 2048), self.num_local_experts, x.device)
+            self._workspace(x.shape[0] * topk_ids.shape[1], x.device)
             if self.fp8_block:
                 return moe_native.fused_experts_fp8_block(x, self.w13_weight, self.w13_scale, self.w2_weight,
                                                           self.w2_scale, topk_weights, topk_ids, self.expert_start,
@@ -276,6 +308,11 @@ class FusedMoE(nn.Module):
                                                     out)
             return moe_native.fused_experts(x, self.w13_weight, self.w2_weight, topk_weights, topk_ids,
                                             self.expert_start, self.workspace, add, out)
+        if self.activation == "clipped_swiglu" and not self.fp8 and ops.use_native(x) and x.shape[1] % 8 == 0:
+            from ..ops import moe_native
+            ws = self._workspace(topk_ids.numel(), x.device)
+            y = moe_native.sorted_experts(x, self.w13_weight, self.w2_weight, topk_ids, self.expert_start, ws, self._act)
+            return moe_native.moe_combine(y, topk_weights, ws, x.shape[0], add=add, out=out)
         if self.fp8:
             y = _fp8_reference_experts(x, self, topk_weights, topk_ids)
             if add is not None:
@@ -285,7 +322,8 @@ class FusedMoE(nn.Module):
                                   add)
         else:
             from ..ops import reference
-            y = reference.moe_forward(x, self.w13_weight, self.w2_weight, topk_weights, topk_ids, self.expert_start, act=self.activation)
+            act = self._act if self.activation == "clipped_swiglu" else self.activation
+            y = reference.moe_forward(x, self.w13_weight, self.w2_weight, topk_weights, topk_ids, self.expert_start, act=act)
             if add is not None:
                 y = (y.float() + add.float()).to(y.dtype)
         if out is not None:
@@ -330,6 +368,34 @@ def _fp8_reference_experts(x, moe: "FusedMoE", topk_weights, topk_ids):
         y = y.to(x.dtype).float()
         out.index_add_(0, tok, y * topk_weights[tok, slot].float()[:, None])
     return out.to(x.dtype)
+
+
+class RoutedFeedForward(nn.Module):
+    """Feed-forward of experts chosen by their router logits (bias included), weighted by the softmax over the chosen logits,
+    in a layer whose other sublayer reads the same input: both are added to the residual stream at once."""
+
+    def __init__(self, hidden_size: int, num_experts: int, top_k: int, intermediate_size: int, dtype, layer_id: int = 0,
+                 activation: str = "clipped_swiglu", act_limit: float = 0.0):
+        super().__init__()
+        from .gate import GateLogit
+        self.top_k = top_k
+        self.gate = GateLogit(hidden_size, num_experts, dtype, use_bias=True)
+        self.experts = FusedMoE(num_experts, hidden_size, intermediate_size, dtype, layer_id=layer_id,
+                                activation=activation, act_limit=act_limit)
+
+    def load(self, name: str, w: torch.Tensor):
+        """One checkpoint tensor: `router`, `router.b`, or `e<i>.gate` / `.up` / `.down`."""
+        if name == "router":
+            return self.gate.weight.data.copy_(w)
+        if name == "router.b":
+            return self.gate.bias.data.copy_(w)
+        expert, shard = name.split(".")
+        param = self.experts.w2_weight if shard == "down" else self.experts.w13_weight
+        self.experts.weight_loader(param, w, shard, int(expert[1:]))
+
+    def forward(self, h: torch.Tensor, mixed: torch.Tensor, stream: torch.Tensor) -> torch.Tensor:
+        weights, ids = self.gate.route_by_logit(h, self.top_k)
+        return self.experts.forward_stream(h, weights, ids, mixed, stream)
 
 
 EPMoE = FusedMoE

@@ -335,6 +335,46 @@ class MLATokenToKVPool(KVCache):
         return rows[:, :rank], rows[:, rank:rank + rope]
 
 
+class PackedKVPool(KVCache):
+    """Keys and values of unequal widths, every layer with sizes of its own: per layer `[num_pages, heads, page_size, row]`,
+    a row being `[key | value]` of one head and token, both parts padded to whole 16-byte units (of bf16), so that either
+    part of a page is a strided 2-D block that a tensor copy can fetch.  `layer_shapes`: `(heads, key width, value width)`."""
+
+    def __init__(self, size, page_size, dtype, layer_shapes: list[tuple[int, int, int]], device, start_layer: int = 0):
+        super().__init__(size, page_size, dtype, len(layer_shapes), device, start_layer)
+        self.layer_shapes = list(layer_shapes)
+        self.kv_buffer = [torch.zeros((self.num_pages, h, page_size, self.padded(k) + self.padded(v)), dtype=dtype,
+                                      device=device) for h, k, v in layer_shapes]
+
+    @staticmethod
+    def padded(width: int) -> int:
+        return -(-width // 8) * 8
+
+    @staticmethod
+    def cell_size(layer_shapes, dtype) -> int:
+        return sum(h * (PackedKVPool.padded(k) + PackedKVPool.padded(v)) for h, k, v in layer_shapes) * \
+            torch.finfo(dtype).bits // 8
+
+    def get_kv_size_bytes(self):
+        return sum(b.numel() * b.element_size() for b in self.kv_buffer)
+
+    def get_kv_buffer(self, layer_id):
+        return self.kv_buffer[layer_id - self.start_layer]
+
+    def set_kv_buffer(self, layer_id, loc, k: torch.Tensor, v: torch.Tensor):
+        """`k [T, heads, key width]`, `v [T, heads, value width]` into slots `loc [T]`."""
+        buf, at = self.get_kv_buffer(layer_id), self.padded(k.shape[-1])
+        page, off = (loc // self.page_size).long(), (loc % self.page_size).long()
+        buf[page, :, off, :k.shape[-1]] = k.to(self.dtype)
+        buf[page, :, off, at:at + v.shape[-1]] = v.to(self.dtype)
+
+    def gather(self, layer_id, loc):
+        _, kd, vd = self.layer_shapes[layer_id - self.start_layer]
+        rows = self.get_kv_buffer(layer_id)[(loc // self.page_size).long(), :, (loc % self.page_size).long()]
+        at = self.padded(kd)
+        return rows[..., :kd], rows[..., at:at + vd]
+
+
 class HybridLinearKVPool(KVCache):
     """KV pool for hybrid models: only the full-attention layers own KV pages; the
     layer id is remapped to the dense index (reference `memory_pool.py:1475`)."""

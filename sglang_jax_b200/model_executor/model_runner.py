@@ -21,7 +21,7 @@ from ..configs.model_config import AttentionArch, ModelConfig
 from ..layers.radix_attention import AttentionBackend
 from ..layers.sampler import Sampler, SamplingMetadata
 from ..managers.schedule_batch import ForwardMode, ModelWorkerBatch
-from ..mem_cache.memory_pool import MHATokenToKVPool, MLATokenToKVPool, ReqToTokenPool, SWAKVPool
+from ..mem_cache.memory_pool import MHATokenToKVPool, MLATokenToKVPool, PackedKVPool, ReqToTokenPool, SWAKVPool
 from ..model_loader.loader import get_model_loader
 from ..parallel import state as ps
 from .forward_batch_info import ForwardBatch, _PinnedRing
@@ -169,6 +169,8 @@ class ModelRunner:
         mc = self.model_config
         kv_dtype = self.kv_cache_dtype
         n_layers = getattr(self.model, "num_kv_layers", None) or mc.num_hidden_layers
+        if getattr(self.model, "kv_layer_shapes", None):
+            return PackedKVPool.cell_size(self.model.kv_layer_shapes, kv_dtype)
         if mc.attention_arch == AttentionArch.MLA:
             return MLATokenToKVPool.cell_size(mc.kv_lora_rank, mc.qk_rope_head_dim, n_layers, kv_dtype,
                                               getattr(self.model, "index_head_dim", 0),
@@ -250,7 +252,10 @@ class ModelRunner:
             self.recurrent_pool = RecurrentStatePool(req_to_token_pool.size, device=str(self.device),
                                                      conv_dtype=self.dtype, snapshot_slots=snap, **spec)
         n_layers = getattr(self.model, "num_kv_layers", None) or mc.num_hidden_layers
-        if mc.attention_arch == AttentionArch.MLA:
+        if getattr(self.model, "kv_layer_shapes", None):
+            self.token_to_kv_pool = PackedKVPool(self.max_total_num_tokens, self.page_size, self.kv_cache_dtype,
+                                                 self.model.kv_layer_shapes, str(self.device))
+        elif mc.attention_arch == AttentionArch.MLA:
             self.token_to_kv_pool = MLATokenToKVPool(self.max_total_num_tokens, self.page_size, self.kv_cache_dtype,
                                                      mc.kv_lora_rank, mc.qk_rope_head_dim, n_layers, str(self.device),
                                                      index_head_dim=getattr(self.model, "index_head_dim", 0),

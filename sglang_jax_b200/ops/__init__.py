@@ -79,10 +79,32 @@ def sigmoid_gate(o, gate):
     return (_native() if use_native_wide(o) else reference).sigmoid_gate(o, gate)
 
 
+def clipped_swiglu(x, limit: float, alpha: float = 1.702):
+    """`g * sigmoid(alpha g) * (u + 1)` of `x = [gate | up]`, `g = min(gate, limit)`, `u = clamp(up, -limit, limit)`."""
+    return (_native() if use_native_wide(x) else reference).clipped_swiglu(x, limit, alpha)
+
+
+def token_side_gate(z, table, ids, offset: int):
+    """`gelu_tanh(z) * table[ids, offset : offset + dim]`, `z [T, dim]`."""
+    return (_native() if use_native_wide(z) else reference).token_side_gate(z, table, ids, offset)
+
+
 # ---- residual stream in fp32 (projections in the model's type)
-def embed_scaled(ids, table, scale):
-    """`table[ids] * scale` as `(fp32 stream, the same in the table's type)`."""
-    return (_native() if use_native_wide(table) else reference).embed_scaled(ids, table, scale)
+def embed_scaled(ids, table, scale, positions=None, turns=None):
+    """`table[ids] * scale` as `(fp32 stream, the same in the table's type)`.  `turns` (double, `[ceil(width / 2)]`): adds
+    the sinusoidal vector of `positions`, channels 2i and 2i + 1 being sine and cosine of `turns[i]` turns a position."""
+    return (_native() if use_native_wide(table) else reference).embed_scaled(ids, table, scale, positions, turns)
+
+
+def stream_add(y, x, expert_out=None, weights=None, pair_row=None):
+    """`x += y` in place on the fp32 stream, with `expert_out` also `sum_j weights[t, j] * expert_out[pair_row[t, j]]`
+    (negative rows: nothing); returns x in y's type."""
+    return (_native() if use_native_wide(y) else reference).stream_add(y, x, expert_out, weights, pair_row)
+
+
+def postnorm_add_norm(y, x, channel_scale, eps, next_scale, next_eps):
+    """`x += channel_scale * y / rms(y)` in place on the fp32 stream; returns `next_scale * x / rms(x)` in y's type."""
+    return (_native() if use_native_wide(y) else reference).postnorm_add_norm(y, x, channel_scale, eps, next_scale, next_eps)
 
 
 def postnorm_add(y, x, channel_scale, eps):
@@ -100,8 +122,45 @@ def delta_scan(proj, *a, **kw):
     return (_native() if use_native_wide(proj) else reference).delta_scan(proj, *a, **kw)
 
 
-def delta_gate(o, gate, weight, eps):
-    return (_native() if use_native_wide(gate) else reference).delta_gate(o, gate, weight, eps)
+def delta_gate(o, gate, weight, eps, act: str = "silu"):
+    """`rmsnorm(o) * weight * act(gate)` per head, act silu or sigmoid."""
+    return (_native() if use_native_wide(gate) else reference).delta_gate(o, gate, weight, eps, act)
+
+
+# ---- windowed attention over `PackedKVPool` rows (see `native.attn_prep`)
+def attn_prep(proj, *a, **kw):
+    return (_native() if use_native_wide(proj) else reference).attn_prep(proj, *a, **kw)
+
+
+def window_attention(q, gate, cache, fb, rows, lens, dim, v_dim, scale, window, keep_first):
+    """Every query token on its own: query n sees the first `lens[n]` tokens of page-table row `rows[n]`, of those the last
+    `window` (0: all) and the first `keep_first`."""
+    n = _native()
+    args = (q, gate, cache, fb.page_table, rows, lens, dim, v_dim, fb.page_size, scale, window, keep_first)
+    if n.window_decode_supported(q, cache, dim, v_dim, fb.page_size):
+        return n.window_decode(*args, max_seq_len=fb.max_seq_len)
+    return n.window_attn_any(*args)
+
+
+def window_extend_supported(q, cache, dim, v_dim) -> bool:
+    return use_native(q) and _native().window_extend_supported(q, cache, dim, v_dim)
+
+
+def window_extend(q, gate, cache, fb, plan, out, dim, v_dim, scale, window, keep_first):
+    return _native().window_extend(q, gate, cache, fb.page_table, plan, out, dim, v_dim, scale, window, keep_first)
+
+
+def low_rank_up(x, w):
+    """Second product of a low-rank pair; `x` may be a column range of a wider output.  A library GEMM on the GPU."""
+    return reference.linear(x, w)
+
+
+def route_by_logit(x, weight, bias, top_k):
+    """The `top_k` experts with the largest logits `x weight^T + bias` (fp32) and the softmax over them."""
+    if use_native_wide(x) and weight.shape[0] <= 512 and top_k <= 16 and weight.dtype == x.dtype:
+        from . import moe_native
+        return moe_native.route_by_logit(x, weight, bias, top_k)
+    return reference.route_by_logit(x, weight, bias, top_k)
 
 
 # ---- latent attention (see `native.latent_prep`)
@@ -125,7 +184,7 @@ def latent_attention(q_lat, q_pe, cache, fb, scale, rows=None, lens=None):
         if fb.forward_mode.is_decode():
             rows, lens = fb.req_pool_indices, fb.seq_lens
         else:
-            from ..layers.latent_attention import extend_plan
+            from ..layers.extend_plan import extend_plan
             plan = extend_plan(fb, False)
             rows, lens = plan.token_rows, plan.token_lens
     if native.mla_decode_supported(q_lat, q_pe, cache, R, fb.page_size):

@@ -23,6 +23,10 @@ def _lib():
         L.sglb_moe_combine.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p]
         L.sglb_grouped_gemm_bf16.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                              c_int, c_int, c_int, c_int, c_void_p, c_size_t, c_void_p, c_void_p]
+        L.sglb_route_by_logit.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
+                                          c_int, c_int, c_void_p]
+        L.sglb_grouped_gemm_any.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                            c_int, c_int, c_int, c_int, c_int, c_void_p]
         L.sglb_grouped_gemm_fp8.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                             c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_size_t,
                                             c_void_p, c_void_p]
@@ -196,3 +200,46 @@ def fused_experts(x, w13, w2, topk_weights, topk_ids, expert_start: int = 0, ws:
     a = native.silu_and_mul(h)
     y = grouped_gemm(a, w2, ws, pairs)
     return moe_combine(y, topk_weights, ws, T, add=add, out=out)
+
+
+# tokens up to which the router is one launch; above, its product is a library GEMM with fp32 results
+ROUTE_FUSED_TOKENS = 256
+
+
+def route_by_logit(x, weight, bias, top_k):
+    """`z = x weight^T + bias` in fp32, the `top_k` largest (ties: the lower index) and their softmax."""
+    T, K = x.shape
+    E = weight.shape[0]
+    x = x.contiguous()
+    assert weight.is_contiguous() and weight.dtype == x.dtype and (bias is None or bias.dtype == x.dtype)
+    w = torch.empty((T, top_k), dtype=torch.float32, device=x.device)
+    ids = torch.empty((T, top_k), dtype=torch.int32, device=x.device)
+    z = None
+    if T > ROUTE_FUSED_TOKENS:
+        z = torch.mm(x, weight.t()) if x.dtype == torch.float32 else torch.mm(x, weight.t(), out_dtype=torch.float32)
+    p = native._p
+    native._check(_lib().sglb_route_by_logit(p(z), p(x), p(weight), p(bias), p(w), p(ids), T, E, K, top_k, native._f32(x),
+                                             native._stream()), "route_by_logit")
+    return w, ids
+
+
+def grouped_gemm_any(x, row_token, w, ws: MoeWorkspace, rows: int):
+    """Grouped product of any sizes in bf16 or fp32 on the CUDA cores, fp32 accumulation: row r of the result is row
+    `row_token[r]` (None: r) of `x` times its expert's `w [E_local, N, K]`."""
+    E, N, K = w.shape
+    assert x.is_contiguous() and w.is_contiguous() and x.dtype == w.dtype and x.shape[1] == K
+    out = torch.empty((rows, N), dtype=x.dtype, device=x.device)
+    native._check(_lib().sglb_grouped_gemm_any(x.data_ptr(), native._p(row_token), w.data_ptr(), out.data_ptr(),
+                                               ws.offsets.data_ptr(), ws.tile_group.data_ptr(), ws.tile_row0.data_ptr(),
+                                               ws.counts.data_ptr() + 4, rows, N, K, E, native._f32(x), native._stream()),
+                  "grouped_gemm_any")
+    return out
+
+
+def sorted_experts(x, w13, w2, topk_ids, expert_start, ws: MoeWorkspace, act):
+    """Outputs of the routed experts, one row per (token, choice) pair in the workspace's order (`ws.pair_row`)."""
+    pairs, E_local = topk_ids.numel(), w13.shape[0]
+    moe_align(topk_ids, expert_start, E_local, ws)
+    if x.dtype == torch.bfloat16 and x.shape[1] % 8 == 0 and w2.shape[2] % 8 == 0:
+        return grouped_gemm(act(grouped_gemm(moe_gather(x, ws, pairs), w13, ws, pairs)), w2, ws, pairs)
+    return grouped_gemm_any(act(grouped_gemm_any(x.contiguous(), ws.row_token, w13, ws, pairs)), None, w2, ws, pairs)

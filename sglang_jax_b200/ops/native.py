@@ -87,8 +87,14 @@ def lib():
                             c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p,
                             c_void_p, c_int, c_void_p])
     sig("sglb_mla_num_splits", [c_int, c_int, c_int])
-    sig("sglb_embed_scaled", [c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_float, c_int, c_void_p])
-    sig("sglb_postnorm_add", [c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_float, c_int, c_void_p])
+    sig("sglb_embed_scaled", [c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_float, c_void_p,
+                              c_void_p, c_int, c_void_p])
+    sig("sglb_postnorm_add", [c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_float, c_void_p, c_float, c_int,
+                              c_void_p])
+    sig("sglb_stream_add", [c_void_p] * 6 + [c_int, c_longlong, c_int, c_int, c_void_p])
+    sig("sglb_clipped_swiglu", [c_void_p, c_void_p, c_longlong, c_int, c_float, c_float, c_int, c_void_p])
+    sig("sglb_side_gate", [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_int, c_longlong, c_int, c_int,
+                           c_void_p])
     sig("sglb_rmsnorm_stream", [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_float, c_int, c_void_p])
     sig("sglb_gelu_tanh_and_mul", [c_void_p, c_void_p, c_longlong, c_int, c_int, c_void_p])
     sig("sglb_sigmoid_gate", [c_void_p, c_void_p, c_void_p, c_longlong, c_longlong, c_int, c_int, c_void_p])
@@ -101,9 +107,20 @@ def lib():
     sig("sglb_latent_extend_supported", [c_int, c_int, c_int])
     sig("sglb_latent_extend", [c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_int]
         + [c_void_p] * 4 + [c_int] * 6 + [c_float, c_void_p])
-    sig("sglb_delta_scan", [c_void_p, c_longlong, c_int, c_int, c_int] + [c_void_p] * 15 + [c_int] * 9 + [c_void_p])
+    sig("sglb_delta_scan", [c_void_p, c_longlong, c_int, c_int, c_int] + [c_void_p] * 18 + [c_int] * 9 + [c_void_p])
     sig("sglb_delta_gate", [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_int, c_int, c_float, c_int,
-                            c_void_p])
+                            c_int, c_void_p])
+    sig("sglb_attn_prep", [c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_longlong]
+        + [c_int] * 6 + [c_float, c_int, c_void_p])
+    sig("sglb_window_decode_supported", [c_int, c_int, c_int])
+    sig("sglb_window_num_splits", [c_int, c_int, c_int])
+    sig("sglb_window_decode", [c_void_p, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_int, c_int, c_void_p,
+                               c_void_p, c_void_p] + [c_int] * 5 + [c_float, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p])
+    sig("sglb_window_attn_any", [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p,
+                                 c_void_p] + [c_int] * 5 + [c_float, c_int, c_int, c_int, c_void_p])
+    sig("sglb_window_extend_supported", [c_int, c_int, c_int])
+    sig("sglb_window_extend", [c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_int, c_int]
+        + [c_void_p] * 4 + [c_int, c_int, c_void_p] + [c_int] * 4 + [c_float, c_int, c_int, c_void_p])
     sig("sglb_paged_decode", [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p,
                                     c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_float, c_int, c_void_p,
                                     c_void_p, c_void_p])
@@ -584,16 +601,20 @@ def _f32(t) -> int:
     return int(t.dtype == torch.float32)
 
 
-def embed_scaled(ids, table, scale):
-    """`(x fp32 [T, W], x in the table's type)`; with an fp32 table both are the same tensor."""
+def embed_scaled(ids, table, scale, positions=None, turns=None):
+    """`(x fp32 [T, W], x in the table's type)`; with an fp32 table both are the same tensor.  `turns`: see
+    `ops.embed_scaled`."""
     ids = ids.contiguous()
     assert ids.dtype == torch.int32 and table.is_contiguous()
+    if turns is not None:
+        assert turns.dtype == torch.float64 and turns.numel() == (table.shape[1] + 1) // 2
+        assert positions.dtype == torch.int32 and positions.is_contiguous() and positions.numel() == ids.numel()
     n, W = ids.numel(), table.shape[1]
     x = torch.empty((n, W), dtype=torch.float32, device=table.device)
     f32 = _f32(table)
     xt = None if f32 else torch.empty((n, W), dtype=table.dtype, device=table.device)
-    _check(lib().sglb_embed_scaled(_p(x), _p(xt), _p(ids), _p(table), n, W, table.shape[0], float(scale), f32, _stream()),
-           "embed_scaled")
+    _check(lib().sglb_embed_scaled(_p(x), _p(xt), _p(ids), _p(table), n, W, table.shape[0], float(scale), _p(positions),
+                                   _p(turns), f32, _stream()), "embed_scaled")
     return x, (x if f32 else xt)
 
 
@@ -604,9 +625,57 @@ def postnorm_add(y, x, channel_scale, eps):
     assert x.dtype == channel_scale.dtype == torch.float32 and x.is_contiguous() and y.shape == x.shape
     f32 = _f32(y)
     xt = None if f32 else torch.empty_like(y)
-    _check(lib().sglb_postnorm_add(_p(x), _p(xt), _p(y), _p(channel_scale), x.numel() // W, W, float(eps), f32, _stream()),
-           "postnorm_add")
+    _check(lib().sglb_postnorm_add(_p(x), _p(xt), _p(y), _p(channel_scale), x.numel() // W, W, float(eps), None, 0.0, f32,
+                                   _stream()), "postnorm_add")
     return x if f32 else xt
+
+
+def postnorm_add_norm(y, x, channel_scale, eps, next_scale, next_eps):
+    """`x += channel_scale * y / rms(y)` in place; returns `next_scale * x / rms(x)` in y's type."""
+    y = y.contiguous()
+    W = x.shape[-1]
+    assert x.dtype == channel_scale.dtype == next_scale.dtype == torch.float32 and x.is_contiguous() and y.shape == x.shape
+    h = torch.empty_like(y)
+    _check(lib().sglb_postnorm_add(_p(x), _p(h), _p(y), _p(channel_scale), x.numel() // W, W, float(eps), _p(next_scale),
+                                   float(next_eps), _f32(y), _stream()), "postnorm_add_norm")
+    return h
+
+
+def stream_add(y, x, expert_out=None, weights=None, pair_row=None):
+    """`x += y` (+ the weighted expert rows of `weights [T, k]`, `pair_row [>= T k]`) in place; returns x in y's type."""
+    y = y.contiguous()
+    n, W = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and y.shape == x.shape
+    k = 0
+    if expert_out is not None:
+        k = weights.shape[1]
+        assert expert_out.is_contiguous() and expert_out.dtype == y.dtype and expert_out.shape[1] == W
+        assert weights.dtype == torch.float32 and weights.is_contiguous() and pair_row.dtype == torch.int32
+    f32 = _f32(y)
+    xt = None if f32 else torch.empty_like(y)
+    _check(lib().sglb_stream_add(_p(x), _p(xt), _p(y), _p(expert_out), _p(weights), _p(pair_row), k, n, W, f32, _stream()),
+           "stream_add")
+    return x if f32 else xt
+
+
+def clipped_swiglu(x, limit, alpha=1.702):
+    x = x.contiguous()
+    F = x.shape[-1] // 2
+    out = torch.empty((*x.shape[:-1], F), dtype=x.dtype, device=x.device)
+    _check(lib().sglb_clipped_swiglu(_p(out), _p(x), out.numel() // F, F, float(limit), float(alpha), _f32(x), _stream()),
+           "clipped_swiglu")
+    return out
+
+
+def token_side_gate(z, table, ids, offset):
+    """`gelu_tanh(z) * table[ids, offset : offset + dim]`, `z [T, dim]` in the table's type."""
+    z, ids = z.contiguous(), ids.contiguous()
+    assert table.dtype == z.dtype and table.stride(1) == 1 and ids.dtype == torch.int32
+    assert 0 <= offset and offset + z.shape[1] <= table.shape[1]
+    out = torch.empty_like(z)
+    _check(lib().sglb_side_gate(_p(out), _p(z), table.data_ptr(), table.stride(0), offset, _p(ids), table.shape[0],
+                                z.shape[0], z.shape[1], _f32(z), _stream()), "token_side_gate")
+    return out
 
 
 def rmsnorm_stream(x, weight, eps, dtype):
@@ -679,7 +748,7 @@ def latent_extend_supported(q, dim, rot, v_dim, rank) -> bool:
 
 
 def latent_extend(q, kv, k_rot, out, plan, dim, v_dim, scale):
-    """Causal attention of the sequences of `plan` (`layers/latent_attention.ExtendPlan`) over expanded keys and values:
+    """Causal attention of the sequences of `plan` (`layers/extend_plan.ExtendPlan`) over expanded keys and values:
     `q [T, H, dim + rot]` (strided view), `kv [ctx, H * (dim + v_dim)]`, `k_rot [ctx, rot]`, result into the rows of
     those sequences of `out [T, H, v_dim]` (strided view)."""
     assert kv.is_contiguous() and k_rot.is_contiguous() and out.stride(2) == 1 and out.dtype == q.dtype
@@ -691,11 +760,12 @@ def latent_extend(q, kv, k_rot, out, plan, dim, v_dim, scale):
 
 # ---- gated delta rule over ragged batches (csrc/delta_scan.cu)
 def delta_scan(proj, g_off, b_off, a_off, conv_w, a_log, dt_bias, conv_state, state, slots, heads, kv_heads, dim, vdim,
-               cu=None, prefix=None, track_len=None, track_slot=None, lens=None):
+               cu=None, prefix=None, track_len=None, track_slot=None, lens=None, channel_a=None):
     """Read-outs fp32 `[T, heads, vdim]` of the rows of `proj [T, ld]` (columns `q | k | v` first, gate / beta / decay
     inputs at the given offsets); windows and states of `slots` are updated in place.  `cu [B + 1]` / `prefix [B]`:
     ragged step (None: one row per request, all of them continuing); `lens`: its sequence lengths on the host, if known
-    (without them the kernel for single tokens is launched on the chance that there are some)."""
+    (without them the kernel for single tokens is launched on the chance that there are some).  `channel_a [T, heads * dim]`:
+    one decay per head and key channel from these inputs, `dt_bias [heads * dim]` (`a_off` is not used then)."""
     T, dev, B = proj.shape[0], proj.device, slots.numel()
     singles = 0 if cu is None else (int((lens == 1).sum()) if lens is not None else -1)
     f32 = dict(dtype=torch.float32, device=dev)
@@ -705,24 +775,112 @@ def delta_scan(proj, g_off, b_off, a_off, conv_w, a_log, dt_bias, conv_state, st
     v = torch.empty((T, heads, vdim), **f32)
     gb = torch.empty((T, heads, 2), **f32)
     # coefficients of the chunks of 32 tokens: two 32 x 32 blocks and two vectors (sizes in csrc/delta_scan.cu)
-    coef = torch.empty((T // 32 + 2 * B, heads, 2112), **f32) if cu is not None else None
+    coef = torch.empty((T // 32 + 2 * B, heads, 2112), **f32) if cu is not None and singles != B else None
+    kq = gc = None
+    if channel_a is not None:
+        assert channel_a.is_contiguous() and channel_a.dtype == proj.dtype and channel_a.shape == (T, heads * dim)
+        assert dt_bias.numel() == heads * dim
+        if cu is not None and singles != B:
+            kq = torch.empty((T, heads, 3, dim), **f32)
+            gc = torch.empty((T // 32 + 2 * B, heads, dim), **f32)
     o = torch.empty((T, heads, vdim), **f32)
     _check(lib().sglb_delta_scan(_p(proj), proj.stride(0), g_off, b_off, a_off, _p(conv_w), _p(a_log), _p(dt_bias),
-                                 _p(conv_state), _p(state), _p(slots), _p(cu), _p(prefix), _p(track_len), _p(track_slot),
-                                 _p(qk), _p(v), _p(gb), _p(coef), _p(o), B, T, heads, kv_heads, dim, vdim,
-                                 conv_w.shape[1], singles, _f32(proj), _stream()), "delta_scan")
+                                 _p(channel_a), _p(conv_state), _p(state), _p(slots), _p(cu), _p(prefix), _p(track_len),
+                                 _p(track_slot), _p(qk), _p(v), _p(gb), _p(coef), _p(kq), _p(gc), _p(o), B, T, heads,
+                                 kv_heads, dim, vdim, conv_w.shape[1], singles, _f32(proj), _stream()), "delta_scan")
     return o
 
 
-def delta_gate(o, gate, weight, eps):
-    """`rmsnorm(o) * weight * silu(gate)` per head: `o [T, H, V]` fp32, `gate [T, H * V]` (any row stride) -> `[T, H * V]`
+def delta_gate(o, gate, weight, eps, act="silu"):
+    """`rmsnorm(o) * weight * act(gate)` per head, act silu or sigmoid: `o [T, H, V]` fp32, `gate [T, H * V]` (any row stride) -> `[T, H * V]`
     in the gate's type."""
     T, H, V = o.shape
     assert o.is_contiguous() and gate.stride(-1) == 1 and weight.dtype == torch.float32
     out = torch.empty((T, H * V), dtype=gate.dtype, device=o.device)
     _check(lib().sglb_delta_gate(_p(o), gate.data_ptr(), gate.stride(0), _p(weight), _p(out), T, H, V, float(eps),
-                                 _f32(gate), _stream()), "delta_gate")
+                                 int(act == "sigmoid"), _f32(gate), _stream()), "delta_gate")
     return out
+
+
+# ---- windowed attention over [key | value] rows (csrc/window_attn.cu, window_extend.cu); sizes padded to 16-byte units
+def _pad8(n: int) -> int:
+    return -(-n // 8) * 8
+
+
+def attn_prep(proj, q_off, k_off, v_off, heads, kv_heads, dim, v_dim, eps, qk_norm, loc, cache):
+    """Queries `[T, heads, dim padded]` of a fused projection `[T, ld]`, divided by their root mean square (`qk_norm`); with
+    `k_off >= 0` also writes keys (likewise) and values into `cache [pages, kv heads, P, row]` at slots `loc`."""
+    T = proj.shape[0]
+    assert proj.stride(1) == 1 and cache.is_contiguous() and cache.dtype == proj.dtype and loc.dtype == torch.int32
+    assert cache.shape[1] == kv_heads and cache.shape[3] == _pad8(dim) + _pad8(v_dim)
+    q = torch.empty((T, heads, _pad8(dim)), dtype=proj.dtype, device=proj.device)
+    _check(lib().sglb_attn_prep(_p(proj), proj.stride(0), q_off, k_off, v_off, _p(q), _p(cache), _p(loc), T, heads, kv_heads,
+                                dim, v_dim, cache.shape[2], int(qk_norm), float(eps), _f32(proj), _stream()), "attn_prep")
+    return q
+
+
+def _check_window_args(q, gate, cache, rows, lens, dim, v_dim):
+    assert q.is_contiguous() and q.shape[2] == _pad8(dim) and cache.is_contiguous() and cache.dtype == q.dtype
+    assert cache.shape[3] == _pad8(dim) + _pad8(v_dim) and q.shape[1] % cache.shape[1] == 0
+    assert rows.dtype == lens.dtype == torch.int32 and rows.is_contiguous() and lens.is_contiguous()
+    assert gate is None or (gate.stride(1) == 1 and gate.dtype == q.dtype and gate.shape == q.shape[:2])
+
+
+def window_decode_supported(q, cache, dim, v_dim, page_size) -> bool:
+    return q.dtype == torch.bfloat16 and cache.dtype == torch.bfloat16 and \
+        bool(lib().sglb_window_decode_supported(dim, v_dim, page_size))
+
+
+def window_decode(q, gate, cache, page_table, rows, lens, dim, v_dim, page_size, scale, window, keep_first, max_seq_len=0,
+                  num_splits=None):
+    """Attention of single query tokens (`ops.window_attention`), times `sigmoid(gate)` per head -> `[N, heads, v_dim]`."""
+    _check_window_args(q, gate, cache, rows, lens, dim, v_dim)
+    N, H, _ = q.shape
+    G = cache.shape[1]
+    out = torch.empty((N, H, v_dim), dtype=q.dtype, device=q.device)
+    if num_splits is None:
+        seen = max_seq_len or page_table.shape[1] * page_size
+        if window:
+            seen = min(seen, window + keep_first)
+        num_splits = lib().sglb_window_num_splits(N, G * -(-(H // G) // 16), max(seen, 1))
+    part_o = part_lse = None
+    if num_splits > 1:
+        part_o = torch.empty((N, H, num_splits, v_dim), dtype=torch.float32, device=q.device)
+        part_lse = torch.empty((N, H, num_splits), dtype=torch.float32, device=q.device)
+    _check(lib().sglb_window_decode(_p(q), None if gate is None else gate.data_ptr(), 0 if gate is None else gate.stride(0),
+                                    _p(cache), cache.shape[0], _p(page_table), page_table.shape[1], page_size, _p(rows),
+                                    _p(lens), _p(out), N, H, G, dim, v_dim, float(scale), int(window), int(keep_first),
+                                    num_splits, _p(part_o), _p(part_lse), _stream()), "window_decode")
+    return out
+
+
+def window_attn_any(q, gate, cache, page_table, rows, lens, dim, v_dim, page_size, scale, window, keep_first):
+    """The same in fp32 arithmetic for any sizes, bf16 or fp32."""
+    _check_window_args(q, gate, cache, rows, lens, dim, v_dim)
+    N, H, _ = q.shape
+    out = torch.empty((N, H, v_dim), dtype=q.dtype, device=q.device)
+    _check(lib().sglb_window_attn_any(_p(q), None if gate is None else gate.data_ptr(), 0 if gate is None else gate.stride(0),
+                                      _p(cache), _p(page_table), page_table.shape[1], page_size, _p(rows), _p(lens), _p(out),
+                                      N, H, cache.shape[1], dim, v_dim, float(scale), int(window), int(keep_first), _f32(q),
+                                      _stream()), "window_attn_any")
+    return out
+
+
+def window_extend_supported(q, cache, dim, v_dim) -> bool:
+    return q.dtype == torch.bfloat16 and cache.dtype == torch.bfloat16 and \
+        bool(lib().sglb_window_extend_supported(dim, v_dim, cache.shape[2]))
+
+
+def window_extend(q, gate, cache, page_table, plan, out, dim, v_dim, scale, window, keep_first):
+    """Prefill attention of the sequences of `plan` (`layers/extend_plan.ExtendPlan`) into their rows of
+    `out [T, heads, v_dim]`."""
+    _check_window_args(q, gate, cache, plan.rows, plan.prefix, dim, v_dim)
+    assert out.is_contiguous() and out.dtype == q.dtype and out.shape == (*q.shape[:2], v_dim)
+    _check(lib().sglb_window_extend(_p(q), q.shape[0], None if gate is None else gate.data_ptr(),
+                                    0 if gate is None else gate.stride(0), _p(cache), cache.shape[0], _p(page_table),
+                                    page_table.shape[1], cache.shape[2], _p(plan.rows), _p(plan.q_start), _p(plan.q_len),
+                                    _p(plan.prefix), plan.long, plan.num_tiles, _p(out), q.shape[1], cache.shape[1], dim,
+                                    v_dim, float(scale), int(window), int(keep_first), _stream()), "window_extend")
 
 
 def lora_bgmv(x, y, a_buf, b_bufs, out_offsets, token_slots, scalings):

@@ -296,7 +296,7 @@ def moe_forward(x, w13, w2, topk_weights, topk_ids, expert_start: int = 0, act="
         if tok.numel() == 0:
             continue
         h = F.linear(x[tok], w13[e])
-        h = silu_and_mul(h) if act == "silu" else gelu_and_mul(h)
+        h = act(h) if callable(act) else silu_and_mul(h) if act == "silu" else gelu_and_mul(h)
         y = F.linear(h, w2[e]).float()
         out.index_add_(0, tok, y * topk_weights[tok, slot].unsqueeze(-1).float())
     return out.to(x.dtype)
@@ -353,8 +353,86 @@ def sigmoid_gate(o, gate):
     return (o.float() * torch.sigmoid(gate.float())).to(o.dtype)
 
 
-def embed_scaled(ids, table, scale):
+def clipped_swiglu(x, limit, alpha=1.702):
+    g, u = x.float().chunk(2, -1)
+    g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+    return (g * torch.sigmoid(alpha * g) * (u + 1)).to(x.dtype)
+
+
+def token_side_gate(z, table, ids, offset):
+    e = table[ids.long(), offset:offset + z.shape[-1]].float()
+    return (F.gelu(z.float(), approximate="tanh") * e).to(z.dtype)
+
+
+def stream_add(y, x, expert_out=None, weights=None, pair_row=None):
+    x += y.float()
+    if expert_out is not None:
+        rows = pair_row[:weights.numel()].view(weights.shape).long()
+        x += ((weights * (rows >= 0)).unsqueeze(-1) * expert_out[rows.clamp_min(0)].float()).sum(1)
+    return x if y.dtype == torch.float32 else x.to(y.dtype)
+
+
+def postnorm_add_norm(y, x, channel_scale, eps, next_scale, next_eps):
+    postnorm_add(y, x, channel_scale, eps)
+    return rmsnorm_stream(x, next_scale, next_eps, y.dtype)
+
+
+def route_by_logit(x, weight, bias, top_k):
+    z = F.linear(x.float(), weight.float(), bias.float() if bias is not None else None)
+    best = z.topk(top_k, dim=-1)
+    return torch.softmax(best.values, -1), best.indices.to(torch.int32)
+
+
+def attn_prep(proj, q_off, k_off, v_off, heads, kv_heads, dim, v_dim, eps, qk_norm, loc, cache):
+    def part(off, n, d):
+        return proj[:, off:off + n * d].unflatten(-1, (n, d)).float()
+
+    def unit(t):
+        return t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps) if qk_norm else t
+
+    if k_off >= 0:
+        P, at = cache.shape[2], -(-dim // 8) * 8
+        page, off = (loc // P).long(), (loc % P).long()
+        cache[page, :, off, :dim] = unit(part(k_off, kv_heads, dim)).to(cache.dtype)
+        cache[page, :, off, at:at + v_dim] = part(v_off, kv_heads, v_dim).to(cache.dtype)
+    return unit(part(q_off, heads, dim)).to(proj.dtype)
+
+
+def window_attention(q, gate, cache, fb, dim, v_dim, scale, window, keep_first):
+    """Statement of the windowed attention of a whole step; `q [T, heads, >= dim]`, `cache [pages, kv heads, P, row]`."""
+    decode = fb.forward_mode.is_decode()
+    B, at = fb.batch_size, -(-dim // 8) * 8
+    cu = list(range(B + 1)) if decode else fb.cu_q_lens.tolist()
+    lens = fb.seq_lens.tolist()
+    out = torch.empty(q.shape[0], q.shape[1], v_dim, dtype=q.dtype, device=q.device)
+    for b, row in enumerate(fb.req_pool_indices.tolist()):
+        n, S = cu[b + 1] - cu[b], lens[b]
+        if n == 0:
+            continue
+        pages = fb.page_table[row, :-(-S // fb.page_size)].long()
+        kv = cache[pages].transpose(1, 2).flatten(0, 1)[:S].float()                  # [S, kv heads, row]
+        k, v = kv[..., :dim], kv[..., at:at + v_dim]
+        qb = q[cu[b]:cu[b + 1], :, :dim].float().unflatten(1, (k.shape[1], -1))
+        i = torch.arange(S - n, S, device=q.device)[:, None]
+        j = torch.arange(S, device=q.device)[None]
+        see = j <= i
+        if window > 0:
+            see &= (i - j < window) | (j < keep_first)
+        s = torch.einsum("nghd,sgd->ghns", qb, k) * scale
+        p = torch.softmax(s.masked_fill(~see, float("-inf")), -1)
+        o = torch.einsum("ghns,sgd->nghd", p, v).flatten(1, 2)
+        if gate is not None:
+            o = o * torch.sigmoid(gate[cu[b]:cu[b + 1]].float())[..., None]
+        out[cu[b]:cu[b + 1]] = o.to(q.dtype)
+    return out
+
+
+def embed_scaled(ids, table, scale, positions=None, turns=None):
     x = F.embedding(ids.long(), table).float() * scale
+    if turns is not None:
+        a = positions.double()[:, None] * turns
+        a = (2 * math.pi * (a - a.round())).float()
+        x += torch.stack([torch.sin(a), torch.cos(a)], -1).flatten(1)[:, :x.shape[1]]
     return x, (x if table.dtype == torch.float32 else x.to(table.dtype))
 
 
@@ -369,7 +447,7 @@ def rmsnorm_stream(x, weight, eps, dtype):
 
 
 def delta_scan(proj, g_off, b_off, a_off, conv_w, a_log, dt_bias, conv_state, state, slots, heads, kv_heads, dim, vdim,
-               cu=None, prefix=None, track_len=None, track_slot=None, lens=None):
+               cu=None, prefix=None, track_len=None, track_slot=None, lens=None, channel_a=None):
     """Statement of `native.delta_scan` through the primitives of `ops/linear_attention.py`."""
     from . import linear_attention as la
     B, T, r, kd = slots.numel(), proj.shape[0], heads // kv_heads, kv_heads * dim
@@ -394,11 +472,18 @@ def delta_scan(proj, g_off, b_off, a_off, conv_w, a_log, dt_bias, conv_state, st
             else:
                 y = F.silu(x * conv_w.float()[:, 0])
             q, k, v = y[:, :kd].view(-1, kv_heads, dim), y[:, kd:2 * kd].view(-1, kv_heads, dim), y[:, 2 * kd:]
-            g = -a_log.exp() * F.softplus(rows[:, a_off:a_off + heads] + dt_bias)
             beta = torch.sigmoid(rows[:, b_off:b_off + heads])
-            o[a0:a1], state[s] = la.chunk_gated_delta_rule(
-                q.repeat_interleave(r, 1), k.repeat_interleave(r, 1), v.reshape(-1, heads, vdim), g, beta,
-                None if fresh else state[s])
+            if channel_a is not None:
+                g = F.softplus((channel_a[a0:a1].float() + dt_bias).view(-1, heads, dim)) * -a_log.exp().view(heads, 1)
+                out, last = la.kda_recurrent(q.repeat_interleave(r, 1)[None], k.repeat_interleave(r, 1)[None],
+                                             v.reshape(1, -1, heads, vdim), g[None], beta[None],
+                                             torch.zeros_like(state[s:s + 1]) if fresh else state[s:s + 1])
+                o[a0:a1], state[s] = out[0], last[0]
+            else:
+                g = -a_log.exp() * F.softplus(rows[:, a_off:a_off + heads] + dt_bias)
+                o[a0:a1], state[s] = la.chunk_gated_delta_rule(
+                    q.repeat_interleave(r, 1), k.repeat_interleave(r, 1), v.reshape(-1, heads, vdim), g, beta,
+                    None if fresh else state[s])
             fresh = False
             if tr[b] and a1 - cuts[0] == tr[b]:
                 conv_state[int(track_slot[b])] = conv_state[s]
@@ -406,9 +491,10 @@ def delta_scan(proj, g_off, b_off, a_off, conv_w, a_log, dt_bias, conv_state, st
     return o
 
 
-def delta_gate(o, gate, weight, eps):
+def delta_gate(o, gate, weight, eps, act="silu"):
     T, H, V = o.shape
-    y = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * weight * F.silu(gate.float()).view(T, H, V)
+    g = F.silu(gate.float()) if act == "silu" else torch.sigmoid(gate.float())
+    y = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * weight * g.view(T, H, V)
     return y.view(T, H * V).to(gate.dtype)
 
 
