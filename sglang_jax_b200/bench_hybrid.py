@@ -1,8 +1,9 @@
-"""Prefill and decode throughput of hybrid recurrent / latent-attention decoders at equal sizes, random weights:
-Zozopel beside the framework's closest other models, Kimi-Linear (per-channel delta rule + latent attention) and
-Qwen3-Next (gated delta rule + grouped attention).  Runs on the model runner, decode through its CUDA graphs.
+"""Prefill and decode throughput of hybrid recurrent decoders at equal sizes, random weights: Zozopel (dense feed-forward)
+and Zidivik (routed experts) beside the framework's closest other models, Kimi-Linear (per-channel delta rule + latent
+attention) and Qwen3-Next (gated delta rule + grouped attention), with the feed-forward of the size.  Runs on the model
+runner, decode through its CUDA graphs.
 
-    python bench.py --hybrid [--hybrid-size base large] [--hybrid-models zozopel kimi_linear qwen3_next]
+    python bench.py --hybrid [--hybrid-size base large moe moe-large] [--hybrid-models zozopel zidivik kimi_linear ...]
 
 One JSON line per size.  Times are CUDA events around the forward, median over the repetitions; a step streams the
 weights of all layers, more than the L2 holds."""
@@ -20,7 +21,12 @@ SIZES = {
     # width, feed-forward, heads of 128 (+ 64 rotary lanes), query/key heads of the delta rule, latent width, layers
     "base": dict(width=2048, ff=6144, heads=16, kv_heads=8, rank=512, layers=8, vocab=32768),
     "large": dict(width=4096, ff=12288, heads=32, kv_heads=16, rank=512, layers=8, vocab=32768),
+    # routed experts instead of a dense feed-forward; attention sees the whole context (the window is as long)
+    "moe": dict(width=2048, ff=768, experts=64, top=8, heads=16, kv_heads=8, rank=512, side=128, layers=8, vocab=32768),
+    "moe-large": dict(width=4096, ff=1536, experts=64, top=4, heads=32, kv_heads=16, rank=512, side=256, layers=8,
+                      vocab=32768),
 }
+MODELS = {False: ["zozopel", "kimi_linear", "qwen3_next"], True: ["zidivik", "kimi_linear", "qwen3_next"]}
 PREFILL = [(1, 4096), (4, 2048), (16, 512)]        # (sequences, new tokens each)
 DECODE = [(1, 2048), (32, 2048), (128, 2048)]      # (sequences, cached tokens each)
 
@@ -35,18 +41,29 @@ def model_config(name: str, s: dict) -> dict:
                  "mixer": dict(heads=s["heads"], kv_heads=s["kv_heads"], dim=128, vdim=128, conv=4)}
         return dict(architecture="Zozopel", vocab=s["vocab"], width=w, embedding={"scale": 1.0}, norm={"eps": 1e-6},
                     residual_mult=0.5, logit_scale=1.0, layers=[latent if i % 2 else delta for i in range(n)])
+    if name == "zidivik":
+        mlp = {"kind": "moe", "expert": {"ff": s["ff"], "limit": 7.0}, "router": {"experts": s["experts"], "top": s["top"]}}
+        attn = {"type": "attention", "mlp": mlp,
+                "mixer": dict(heads=s["heads"], kv_heads=max(s["heads"] // 4, 1), dim=128, vdim=128, scale=128 ** -0.5,
+                              mask={"size": 8192, "keep_first": 4})}
+        delta = {"type": "channel_delta", "mlp": mlp,
+                 "mixer": dict(heads=s["heads"], kv_heads=s["kv_heads"], dim=128, vdim=128, conv=4)}
+        return dict(architecture="Zidivik", vocab=s["vocab"], width=w, norm={"eps": 1e-6}, token_side={"dim": s["side"]},
+                    layers=[attn if i % 2 else delta for i in range(n)])
+    experts = dict(num_experts=s["experts"], num_experts_per_tok=s["top"], moe_intermediate_size=s["ff"],
+                   norm_topk_prob=True) if "experts" in s else dict(num_experts=0)
     common = dict(hidden_size=w, intermediate_size=s["ff"], num_hidden_layers=n, rms_norm_eps=1e-6,
                   vocab_size=s["vocab"], max_position_embeddings=32768, tie_word_embeddings=False,
                   torch_dtype="bfloat16", num_attention_heads=s["heads"])
     if name == "kimi_linear":
         return dict(common, architectures=["KimiLinearForCausalLM"], model_type="kimi_linear",
                     num_key_value_heads=s["heads"], kv_lora_rank=s["rank"], q_lora_rank=None, qk_nope_head_dim=128,
-                    qk_rope_head_dim=64, v_head_dim=128, mla_use_nope=True, num_experts=0,
+                    qk_rope_head_dim=64, v_head_dim=128, mla_use_nope=True, n_shared_experts=0, **experts,
                     linear_attn_config={"kda_layers": [i + 1 for i in range(0, n, 2)], "num_heads": s["heads"],
                                         "head_dim": 128, "short_conv_kernel_size": 4})
     if name == "qwen3_next":
         return dict(common, architectures=["Qwen3NextForCausalLM"], model_type="qwen3_next", head_dim=128,
-                    num_key_value_heads=max(s["heads"] // 4, 1), full_attention_interval=2, num_experts=0,
+                    num_key_value_heads=max(s["heads"] // 4, 1), full_attention_interval=2, **experts,
                     linear_num_value_heads=s["heads"], linear_num_key_heads=s["kv_heads"], linear_key_head_dim=128,
                     linear_value_head_dim=128, linear_conv_kernel_dim=4, rope_theta=10000.0, partial_rotary_factor=0.5)
     raise ValueError(name)
@@ -170,7 +187,7 @@ def main(sizes=None, models=None) -> int:
     for s in sizes or list(SIZES):
         out = {"metric": "hybrid decoders, prefill and decode tokens/s", "size": s, **SIZES[s], "dtype": "bf16",
                "data": "synthetic token ids, random weights", "models": {}}
-        for m in models or ["zozopel", "kimi_linear", "qwen3_next"]:
+        for m in models or MODELS["experts" in SIZES[s]]:
             out["models"][m] = run_model(m, SIZES[s])
         print(json.dumps(out), flush=True)
     return 0

@@ -407,116 +407,111 @@ __global__ void __launch_bounds__(kChunkThreads) delta_chunk_kernel(const DeltaP
 // never a difference of longer sums, so that strong decays earlier in the chunk do not cost precision.  Scaled vectors for
 // delta_scan: k and q times the decay from the chunk's start (what meets the state in front of it), and k times the decay to
 // its end (what it leaves behind).
+constexpr int kChannelThreads = 256;
+
 struct ChannelShape {
-  static constexpr int kRows = 3 * kC + kC + kC / 2;   // k, q, c; scaled k, scaled q of second halves
-  static int smem(int Dp) { return (kRows * (Dp + 4) + 2 * kC * kGramLd + kC) * 4; }
+  static constexpr int kRows = 3 * kC + kC + kC / 2;   // k, q, logs of the decays; scaled k, scaled q of second halves
+  static int smem(int Dp) { return (kRows * (Dp + 4) + 2 * kC * kGramLd) * 4; }
 };
 
+__device__ __forceinline__ float ex2_approx(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
 template <typename T>
-__global__ void __launch_bounds__(kChunkThreads) delta_chunk_channel_kernel(const DeltaParams p, int Dp) {
+__global__ void __launch_bounds__(kChannelThreads, 2) delta_chunk_channel_kernel(const DeltaParams p, int Dp) {
   extern __shared__ float4 sm4[];
   const int ld = Dp + 4;
   float* ks = reinterpret_cast<float*>(sm4);           // [kC][ld]
   float* qs = ks + kC * ld;                            // [kC][ld]
-  float* cs = qs + kC * ld;                            // [kC][ld]  logarithms of the tokens' decays
+  float* cs = qs + kC * ld;                            // [kC][ld]  binary logarithms of the tokens' decays
   float* sk = cs + kC * ld;                            // [kC][ld]
   float* sq = sk + kC * ld;                            // [kC / 2][ld]
-  float* gram = sq + kC / 2 * ld;                      // [k . k | q . k][kC][kGramLd]
-  float* line = gram + 2 * kC * kGramLd;               // [kC]
+  float* gram = sq + kC / 2 * ld;                      // [beta k . k | q . k][kC][kGramLd]
   pdl_wait();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.y, hk = h / (p.H / p.Hk), D = p.D;
   const int idx = blockIdx.x;
   const ChunkPlace place(p, idx);
   if (place.m == 0) return;
   const int row0 = place.row0, m = place.m;
-  for (int i = tid; i < 3 * kC * (ld - D); i += kChunkThreads) ks[(i / (ld - D)) * ld + D + i % (ld - D)] = 0.f;
-  stage_rows<kChunkThreads>(ks, ld, p, row0, hk, 1, m);
-  stage_rows<kChunkThreads>(qs, ld, p, row0, hk, 0, m);
+  for (int i = tid; i < 3 * kC * (ld - D); i += kChannelThreads) ks[(i / (ld - D)) * ld + D + i % (ld - D)] = 0.f;
+  stage_rows<kChannelThreads>(ks, ld, p, row0, hk, 1, m);
+  stage_rows<kChannelThreads>(qs, ld, p, row0, hk, 0, m);
   cp_commit();
-  const float rate = -expf(p.a_log[h]);
-  float* gc = p.gc + (static_cast<long long>(idx) * p.H + h) * D;
-  for (int d = tid; d < D; d += kChunkThreads) {
+  // a channel's 32 tokens are shared by two threads, one for each half
+  const int shift = 31 - __clz(Dp);
+  const float rate = -1.4426950408889634f * expf(p.a_log[h]);
+  for (int i = tid; i < 2 * Dp; i += kChannelThreads) {
+    const int d = i & (Dp - 1), t0 = (i >> shift) * (kC / 2);
+    if (d >= D) continue;
     const T* a = static_cast<const T*>(p.chan_a) + (static_cast<long long>(row0) * p.H + h) * D + d;
     const float bias = p.dt_bias[h * D + d];
-    float c = 0.f;
 #pragma unroll 8
-    for (int t = 0; t < kC; ++t) {
-      const float lg = t < m ? rate * softplus(to_f(a[static_cast<long long>(t) * p.H * D]) + bias) : 0.f;
-      c += lg;
-      cs[t * ld + d] = lg;
-    }
-    gc[d] = expf(c);
+    for (int t = t0; t < t0 + kC / 2; ++t)
+      cs[t * ld + d] = t < m ? rate * softplus(to_f(a[static_cast<long long>(t) * p.H * D]) + bias) : 0.f;
   }
-  for (int i = tid; i < 2 * kC * kGramLd; i += kChunkThreads) gram[i] = 0.f;
+  for (int i = tid; i < 2 * kC * kGramLd; i += kChannelThreads) gram[i] = 0.f;
   cp_wait<0>();
   __syncthreads();
-  for (int d = tid; d < D; d += kChunkThreads) {
-    float* dst = p.kq + (static_cast<long long>(row0) * p.H + h) * 3 * D + d;
-    const long long tok = static_cast<long long>(p.H) * 3 * D;
-    float c = 0.f, e = 0.f;                            // from the start up to t; after the t'th last to the end
-#pragma unroll 4
-    for (int t = 0; t < m; ++t) {
-      c += cs[t * ld + d];
-      const float f = expf(c);
-      dst[t * tok] = ks[t * ld + d] * f;
-      dst[t * tok + D] = qs[t * ld + d] * f;
-    }
-#pragma unroll 4
-    for (int t = m - 1; t >= 0; --t) {
-      dst[t * tok + 2 * D] = ks[t * ld + d] * expf(e);
-      e += cs[t * ld + d];
-    }
-  }
 #pragma unroll
   for (int half = kC / 2; half >= 4; half >>= 1) {
     // scaled vectors: first halves backwards from their last token, second halves forwards from there
-    for (int d = tid; d < Dp; d += kChunkThreads)
-      for (int blk = 0; blk < kC; blk += 2 * half) {
+    for (int i = tid; i < 2 * Dp; i += kChannelThreads) {
+      const int d = i & (Dp - 1), part = i >> shift;
+#pragma unroll
+      for (int j = 0; j < kC / 2 / half; ++j) {        // this thread's half blocks: every second one
+        const int blk = j * 2 * half, t0 = blk + part * half;
         float c = 0.f;
-#pragma unroll 4
-        for (int t = blk + half - 1; t >= blk; --t) {
-          sk[t * ld + d] = ks[t * ld + d] * expf(c);
-          c += cs[t * ld + d];
+        if (part == 0) {
+#pragma unroll 8
+          for (int t = t0 + half - 1; t >= t0; --t) {
+            sk[t * ld + d] = ks[t * ld + d] * ex2_approx(c);
+            c += cs[t * ld + d];
+          }
+        } else {
+#pragma unroll 8
+          for (int t = t0; t < t0 + half; ++t) {
+            c += cs[t * ld + d];
+            const float f = ex2_approx(c);
+            sk[t * ld + d] = ks[t * ld + d] * f;
+            sq[(t - half - blk / 2) * ld + d] = qs[t * ld + d] * f;
+          }
         }
-        c = 0.f;
-#pragma unroll 4
-        for (int t = blk + half; t < blk + 2 * half; ++t) {
-          c += cs[t * ld + d];
-          const float f = expf(c);
-          sk[t * ld + d] = ks[t * ld + d] * f;
-          sq[(t - half - blk / 2) * ld + d] = qs[t * ld + d] * f;
-        }
-      }
-    __syncthreads();
-    // kC / 2 second-half rows times `half` columns of their first half, for k and q; two rows per thread at the top
-    const int rows = half == kC / 2 ? 2 : 1, items = kC / 2 * half / rows;
-    if (tid < items) {
-      const int j = tid % half, r = tid / half * rows;           // r: place among the second-half rows
-      const int blk = r / half * 2 * half, t = blk + half + r % half;
-      const float* col = sk + (blk + j) * ld;
-      float kk[2] = {0.f, 0.f}, qk[2] = {0.f, 0.f};
-      for (int d = 0; d < Dp; d += 4) {
-        const float4 c = *reinterpret_cast<const float4*>(col + d);
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-          if (i >= rows) break;
-          const float4 a = *reinterpret_cast<const float4*>(sk + (t + i) * ld + d);
-          const float4 b = *reinterpret_cast<const float4*>(sq + (r + i) * ld + d);
-          kk[i] += a.x * c.x + a.y * c.y + a.z * c.z + a.w * c.w;
-          qk[i] += b.x * c.x + b.y * c.y + b.z * c.z + b.w * c.w;
-        }
-      }
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        if (i >= rows) break;
-        gram[(t + i) * kGramLd + blk + j] = kk[i];
-        gram[(kC + t + i) * kGramLd + blk + j] = qk[i];
       }
     }
     __syncthreads();
+    {
+      // kC / 2 second-half rows times `half` columns of their first half, for k and q; neighbouring lanes share the
+      // channels of one product
+      const int parts = kC / 2 / half, part = tid & (parts - 1), item = tid / parts;
+      const int j = item % half, r = item / half;                // r: place among the second-half rows
+      const int blk = r / half * 2 * half, t = blk + half + r % half;
+      const float *col = sk + (blk + j) * ld, *rk = sk + t * ld, *rq = sq + r * ld;
+      float kk = 0.f, qk = 0.f;
+#pragma unroll 4
+      for (int d = 4 * part; d < Dp; d += 4 * parts) {
+        const float4 c = *reinterpret_cast<const float4*>(col + d);
+        const float4 a = *reinterpret_cast<const float4*>(rk + d), b = *reinterpret_cast<const float4*>(rq + d);
+        kk += a.x * c.x + a.y * c.y + a.z * c.z + a.w * c.w;
+        qk += b.x * c.x + b.y * c.y + b.z * c.z + b.w * c.w;
+      }
+#pragma unroll
+      for (int o = parts / 2; o > 0; o >>= 1) {
+        kk += __shfl_xor_sync(0xffffffffu, kk, o);
+        qk += __shfl_xor_sync(0xffffffffu, qk, o);
+      }
+      if (part == 0) {
+        gram[t * kGramLd + blk + j] = kk;
+        gram[(kC + t) * kGramLd + blk + j] = qk;
+      }
+    }
+    if (half > 4) __syncthreads();
   }
-  // blocks of four tokens: one warp each, lanes share the channels
-  for (int blk = warp * 4; blk < kC; blk += kChunkThreads / 32 * 4) {
+  {
+    // blocks of four tokens: one warp each, lanes share the channels
+    const int blk = warp * 4;
     float kk[6], qk[10];
 #pragma unroll
     for (int i = 0; i < 6; ++i) kk[i] = 0.f;
@@ -536,7 +531,7 @@ __global__ void __launch_bounds__(kChunkThreads) delta_chunk_channel_kernel(cons
 #pragma unroll
         for (int j = t - 1; j >= 0; --j) {
           e += c[j + 1];
-          const float f = expf(e) * k[j];
+          const float f = ex2_approx(e) * k[j];
           kk[t * (t - 1) / 2 + j] += k[t] * f;
           qk[t * (t + 1) / 2 + j] += q[t] * f;
         }
@@ -544,40 +539,62 @@ __global__ void __launch_bounds__(kChunkThreads) delta_chunk_channel_kernel(cons
       }
     }
 #pragma unroll
-    for (int t = 0; t < 4; ++t)
+    for (int i = 0; i < 6; ++i) kk[i] = warp_sum(kk[i]);
 #pragma unroll
-      for (int j = 0; j <= t; ++j) {
-        const float b = warp_sum(qk[t * (t + 1) / 2 + j]);
-        const float a = j < t ? warp_sum(kk[t > 0 ? t * (t - 1) / 2 + (j < t ? j : 0) : 0]) : 0.f;
-        if (lane == 0) {
-          gram[(blk + t) * kGramLd + blk + j] = a;
-          gram[(kC + blk + t) * kGramLd + blk + j] = b;
+    for (int i = 0; i < 10; ++i) qk[i] = warp_sum(qk[i]);
+    if (lane == 0)
+#pragma unroll
+      for (int t = 0; t < 4; ++t)
+#pragma unroll
+        for (int j = 0; j <= t; ++j) {
+          if (j < t) gram[(blk + t) * kGramLd + blk + j] = kk[t * (t - 1) / 2 + j];
+          gram[(kC + blk + t) * kGramLd + blk + j] = qk[t * (t + 1) / 2 + j];
         }
-      }
+  }
+  __syncthreads();
+  float* out = p.coef + (static_cast<long long>(idx) * p.H + h) * kCoefs;
+  const float* betas = p.gb + (static_cast<long long>(row0) * p.H + h) * 2 + 1;
+  for (int i = tid; i < kC * kC; i += kChannelThreads) {
+    const int t = i / kC, j = i % kC;
+    out[kCoefB + i] = gram[(kC + t) * kGramLd + j];
+    gram[t * kGramLd + j] *= t < m ? betas[static_cast<long long>(t) * p.H * 2] : 0.f;
   }
   __syncthreads();
   if (warp == 0) {
-    const float beta = lane < m ? p.gb[(static_cast<long long>(row0 + lane) * p.H + h) * 2 + 1] : 0.f;
-    float* out = p.coef + (static_cast<long long>(idx) * p.H + h) * kCoefs;
+    const float beta = lane < m ? betas[static_cast<long long>(lane) * p.H * 2] : 0.f;
     float X[kC];                                       // lane c: column c of (I + A)^-1
 #pragma unroll
     for (int t = 0; t < kC; ++t) {
-      const float bt = __shfl_sync(0xffffffffu, beta, t);
-      __syncwarp();
-      line[lane] = lane < t ? bt * gram[t * kGramLd + lane] : 0.f;
-      out[kCoefB + t * kCoefRow + lane] = lane <= t ? gram[(kC + t) * kGramLd + lane] : 0.f;
-      __syncwarp();
-      float x = lane == t ? 1.f : 0.f;
+      float x[4] = {lane == t ? 1.f : 0.f, 0.f, 0.f, 0.f};
 #pragma unroll
       for (int j = 0; j < t; j += 4) {
-        const float4 c = *reinterpret_cast<const float4*>(line + j);
-        x -= c.x * X[j];
-        if (j + 1 < t) x -= c.y * X[j + 1];
-        if (j + 2 < t) x -= c.z * X[j + 2];
-        if (j + 3 < t) x -= c.w * X[j + 3];
+        const float4 c = *reinterpret_cast<const float4*>(gram + t * kGramLd + j);
+        x[0] -= c.x * X[j];
+        if (j + 1 < t) x[1] -= c.y * X[j + 1];
+        if (j + 2 < t) x[2] -= c.z * X[j + 2];
+        if (j + 3 < t) x[3] -= c.w * X[j + 3];
       }
-      X[t] = x;
-      out[t * kCoefRow + lane] = x * beta;
+      X[t] = (x[0] + x[1]) + (x[2] + x[3]);
+      out[t * kCoefRow + lane] = X[t] * beta;
+    }
+  } else if (warp >= 4) {
+    for (int d = tid - 128; d < D; d += 128) {
+      float* dst = p.kq + (static_cast<long long>(row0) * p.H + h) * 3 * D + d;
+      const long long tok = static_cast<long long>(p.H) * 3 * D;
+      float c = 0.f, e = 0.f;                          // from the start up to t; behind t to the end
+#pragma unroll 8
+      for (int t = 0; t < m; ++t) {
+        c += cs[t * ld + d];
+        const float f = ex2_approx(c);
+        dst[t * tok] = ks[t * ld + d] * f;
+        dst[t * tok + D] = qs[t * ld + d] * f;
+      }
+#pragma unroll 8
+      for (int t = m - 1; t >= 0; --t) {
+        dst[t * tok + 2 * D] = ks[t * ld + d] * ex2_approx(e);
+        e += cs[t * ld + d];
+      }
+      p.gc[(static_cast<long long>(idx) * p.H + h) * D + d] = ex2_approx(c);
     }
   }
 }
@@ -1060,7 +1077,7 @@ int launch_scan_channel(const DeltaParams& p, cudaStream_t s) {
   int e = set_smem(delta_chunk_channel_kernel<T>, ChannelShape::smem(ScanShape<16>::kDp), &cfg_chunk);
   if (e == 0) e = set_smem(delta_scan_kernel<T, RPT, true>, Sh::kSmem, &cfg);
   if (e != 0) return e;
-  launch_pdl(delta_chunk_channel_kernel<T>, dim3(chunk_base(p.T, p.B), p.H), dim3(kChunkThreads), chunk_smem, s, p,
+  launch_pdl(delta_chunk_channel_kernel<T>, dim3(chunk_base(p.T, p.B), p.H), dim3(kChannelThreads), chunk_smem, s, p,
              static_cast<int>(Sh::kDp));
   e = static_cast<int>(cudaGetLastError());
   if (e != 0) return e;

@@ -14,7 +14,7 @@ namespace sglb {
 namespace {
 
 constexpr int kMaxExperts = 512, kMaxTop = 16;
-constexpr int kRouteThreads = 256;
+constexpr int kRouteThreads = 512;
 
 __device__ __forceinline__ float to_f(float v) { return v; }
 __device__ __forceinline__ float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
@@ -22,26 +22,42 @@ template <typename T> __device__ __forceinline__ T from_f(float v);
 template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
 template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
 
-// dot product of one row pair over a warp's lanes
+// kAtOnce dot products with one vector over a warp's lanes: rows w, w + ld, ... (those below `rows`); every load of a step is
+// in flight at the same time
+constexpr int kAtOnce = 4;
+
 template <typename T>
-__device__ __forceinline__ float warp_dot(const T* __restrict__ w, const float* __restrict__ x, int K, int lane, bool wide) {
-  float a = 0.f;
+__device__ __forceinline__ void warp_dots(const T* __restrict__ w, long long ld, int rows, const float* __restrict__ x, int K,
+                                          int lane, bool wide, float (&a)[kAtOnce]) {
+#pragma unroll
+  for (int r = 0; r < kAtOnce; ++r) a[r] = 0.f;
   if (sizeof(T) == 2 && wide) {
+#pragma unroll 2
     for (int i = lane * 8; i < K; i += 256) {
-      const uint4 v = *reinterpret_cast<const uint4*>(w + i);
-      const uint32_t u[4] = {v.x, v.y, v.z, v.w};
+      uint4 v[kAtOnce];
+#pragma unroll
+      for (int r = 0; r < kAtOnce; ++r)
+        v[r] = r < rows ? *reinterpret_cast<const uint4*>(w + r * ld + i) : make_uint4(0, 0, 0, 0);
       const float4 p = *reinterpret_cast<const float4*>(x + i), q = *reinterpret_cast<const float4*>(x + i + 4);
       const float f[8] = {p.x, p.y, p.z, p.w, q.x, q.y, q.z, q.w};
 #pragma unroll
-      for (int e = 0; e < 4; ++e)
-        a += __uint_as_float(u[e] << 16) * f[2 * e] + __uint_as_float(u[e] & 0xffff0000u) * f[2 * e + 1];
+      for (int r = 0; r < kAtOnce; ++r) {
+        const uint32_t u[4] = {v[r].x, v[r].y, v[r].z, v[r].w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          a[r] += __uint_as_float(u[e] << 16) * f[2 * e] + __uint_as_float(u[e] & 0xffff0000u) * f[2 * e + 1];
+      }
     }
   } else {
-    for (int i = lane; i < K; i += 32) a += to_f(w[i]) * x[i];
+    for (int i = lane; i < K; i += 32)
+#pragma unroll
+      for (int r = 0; r < kAtOnce; ++r)
+        if (r < rows) a[r] += to_f(w[r * ld + i]) * x[i];
   }
 #pragma unroll
-  for (int o = 16; o > 0; o >>= 1) a += __shfl_xor_sync(0xffffffffu, a, o);
-  return a;
+  for (int r = 0; r < kAtOnce; ++r)
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) a[r] += __shfl_xor_sync(0xffffffffu, a[r], o);
 }
 
 // The k largest of z[0 .. E) by one warp (ties: the lower index), and their softmax.
@@ -100,9 +116,13 @@ route_token_kernel(const T* __restrict__ x, const T* __restrict__ w, const T* __
   const size_t t = blockIdx.x;
   for (int i = tid; i < K; i += kRouteThreads) xs[i] = to_f(x[t * K + i]);
   __syncthreads();
-  for (int e = warp; e < E; e += kRouteThreads / 32) {
-    const float a = warp_dot(w + static_cast<size_t>(e) * K, xs, K, lane, wide != 0);
-    if (lane == 0) z[e] = a + (bias != nullptr ? to_f(bias[e]) : 0.f);
+  for (int e = warp * kAtOnce; e < E; e += kRouteThreads / 32 * kAtOnce) {
+    float a[kAtOnce];
+    const int rows = min(kAtOnce, E - e);
+    warp_dots(w + static_cast<size_t>(e) * K, static_cast<long long>(K), rows, xs, K, lane, wide != 0, a);
+#pragma unroll
+    for (int r = 0; r < kAtOnce; ++r)
+      if (lane == r && r < rows) z[e + r] = a[r] + (bias != nullptr ? to_f(bias[e + r]) : 0.f);
   }
   __syncthreads();
   if (warp == 0) choose(z, E, k, out_w + t * k, out_ids + t * k, lane);

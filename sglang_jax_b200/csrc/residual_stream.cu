@@ -108,24 +108,34 @@ __global__ void postnorm_add_kernel(float* __restrict__ x, T* __restrict__ xt, c
   __shared__ float red[64];
   pdl_wait();
   const size_t row = static_cast<size_t>(blockIdx.x) * W;
-  float v[VPT][VEC];
+  constexpr bool kEarly = VPT <= 2;                  // rows that fit: everything is on its way before the first sum
+  float v[VPT][VEC], xs[kEarly ? VPT : 1][VEC];
   float ss = 0.f;
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int c = (threadIdx.x + i * blockDim.x) * VEC;
     if (c < W) {
       load_v<VEC>(y + row + c, v[i]);
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) ss += v[i][e] * v[i][e];
+      if constexpr (kEarly) load_v<VEC>(x + row + c, xs[i]);
     }
   }
+#pragma unroll
+  for (int i = 0; i < VPT; ++i)
+    if ((threadIdx.x + i * blockDim.x) * VEC < W)
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) ss += v[i][e] * v[i][e];
   const float inv = 1.f / sqrtf(block_sum(ss, red) / W + eps);
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int c = (threadIdx.x + i * blockDim.x) * VEC;
     if (c < W) {
       float xv[VEC], sv[VEC];
-      load_v<VEC>(x + row + c, xv);
+      if constexpr (kEarly) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) xv[e] = xs[i][e];
+      } else {
+        load_v<VEC>(x + row + c, xv);
+      }
       load_v<VEC>(s + c, sv);
 #pragma unroll
       for (int e = 0; e < VEC; ++e) xv[e] += v[i][e] * inv * sv[e];
@@ -158,6 +168,12 @@ __global__ void postnorm_add_kernel(float* __restrict__ x, T* __restrict__ xt, c
       }
     }
   }
+}
+
+// g / (1 + exp(-alpha g)): the accurate form, and one whose error is far below a bf16 step where the result is rounded to that
+__device__ __forceinline__ float swish(float g, float alpha, float) { return g / (1.f + expf(-alpha * g)); }
+__device__ __forceinline__ float swish(float g, float alpha, __nv_bfloat16) {
+  return __fdividef(g, 1.f + __expf(-alpha * g));
 }
 
 // One row per CTA.  `rows` (null: none) holds k result rows per token, negative where a result lives on another rank.
@@ -255,7 +271,7 @@ __global__ void clipped_swiglu_kernel(T* __restrict__ out, const T* __restrict__
 #pragma unroll
     for (int e = 0; e < VEC; ++e) {
       const float g = fminf(a[e], limit), u = fminf(fmaxf(b[e], -limit), limit);
-      a[e] = g / (1.f + expf(-alpha * g)) * (u + 1.f);
+      a[e] = swish(g, alpha, T()) * (u + 1.f);
     }
     store_v<VEC>(out + r * F + c, a);
   }
