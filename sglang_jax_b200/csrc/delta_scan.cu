@@ -411,7 +411,7 @@ constexpr int kChannelThreads = 256;
 
 struct ChannelShape {
   static constexpr int kRows = 3 * kC + kC + kC / 2;   // k, q, logs of the decays; scaled k, scaled q of second halves
-  static int smem(int Dp) { return (kRows * (Dp + 4) + 2 * kC * kGramLd) * 4; }
+  static int smem(int Dp) { return (kRows * (Dp + 4) + 2 * kC * kGramLd + kC) * 4; }
 };
 
 __device__ __forceinline__ float ex2_approx(float x) {
@@ -430,6 +430,7 @@ __global__ void __launch_bounds__(kChannelThreads, 2) delta_chunk_channel_kernel
   float* sk = cs + kC * ld;                            // [kC][ld]
   float* sq = sk + kC * ld;                            // [kC / 2][ld]
   float* gram = sq + kC / 2 * ld;                      // [beta k . k | q . k][kC][kGramLd]
+  float* betas = gram + 2 * kC * kGramLd;              // [kC]
   pdl_wait();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.y, hk = h / (p.H / p.Hk), D = p.D;
   const int idx = blockIdx.x;
@@ -440,6 +441,7 @@ __global__ void __launch_bounds__(kChannelThreads, 2) delta_chunk_channel_kernel
   stage_rows<kChannelThreads>(ks, ld, p, row0, hk, 1, m);
   stage_rows<kChannelThreads>(qs, ld, p, row0, hk, 0, m);
   cp_commit();
+  if (tid < kC) betas[tid] = tid < m ? p.gb[(static_cast<long long>(row0 + tid) * p.H + h) * 2 + 1] : 0.f;
   // a channel's 32 tokens are shared by two threads, one for each half
   const int shift = 31 - __clz(Dp);
   const float rate = -1.4426950408889634f * expf(p.a_log[h]);
@@ -448,9 +450,14 @@ __global__ void __launch_bounds__(kChannelThreads, 2) delta_chunk_channel_kernel
     if (d >= D) continue;
     const T* a = static_cast<const T*>(p.chan_a) + (static_cast<long long>(row0) * p.H + h) * D + d;
     const float bias = p.dt_bias[h * D + d];
-#pragma unroll 8
-    for (int t = t0; t < t0 + kC / 2; ++t)
-      cs[t * ld + d] = t < m ? rate * softplus(to_f(a[static_cast<long long>(t) * p.H * D]) + bias) : 0.f;
+#pragma unroll 1
+    for (int t = t0; t < t0 + kC / 2; t += 8) {
+      float in[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) in[e] = to_f(a[static_cast<long long>(min(t + e, m - 1)) * p.H * D]);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) cs[(t + e) * ld + d] = t + e < m ? rate * softplus(in[e] + bias) : 0.f;
+    }
   }
   for (int i = tid; i < 2 * kC * kGramLd; i += kChannelThreads) gram[i] = 0.f;
   cp_wait<0>();
@@ -553,15 +560,14 @@ __global__ void __launch_bounds__(kChannelThreads, 2) delta_chunk_channel_kernel
   }
   __syncthreads();
   float* out = p.coef + (static_cast<long long>(idx) * p.H + h) * kCoefs;
-  const float* betas = p.gb + (static_cast<long long>(row0) * p.H + h) * 2 + 1;
   for (int i = tid; i < kC * kC; i += kChannelThreads) {
     const int t = i / kC, j = i % kC;
     out[kCoefB + i] = gram[(kC + t) * kGramLd + j];
-    gram[t * kGramLd + j] *= t < m ? betas[static_cast<long long>(t) * p.H * 2] : 0.f;
+    gram[t * kGramLd + j] *= betas[t];
   }
   __syncthreads();
   if (warp == 0) {
-    const float beta = lane < m ? betas[static_cast<long long>(lane) * p.H * 2] : 0.f;
+    const float beta = betas[lane];
     float X[kC];                                       // lane c: column c of (I + A)^-1
 #pragma unroll
     for (int t = 0; t < kC; ++t) {
