@@ -62,6 +62,35 @@ def _zozopel(d: dict, shapes: dict) -> dict:
         tie_word_embeddings=False, torch_dtype="bfloat16", eos_token_id=None, bos_token_id=None)
 
 
+@native_format("Kunudra")
+def _kunudra(d: dict, shapes: dict) -> dict:
+    layers, known = d["layers"], ("attention", "latent_attention")
+    values = set()
+    for i, e in enumerate(layers):
+        if e["type"] not in known:
+            raise ValueError(f"layer {i}: unknown mixer {e['type']!r}; known: {sorted(known)}")
+        if e.get("mlp") is not None and e["mlp"]["kind"] not in ("dense", "moe"):
+            raise ValueError(f"layer {i}: unknown feed-forward {e['mlp']['kind']!r}")
+        m = e["mixer"]
+        if e["type"] == "latent_attention" and m["rot"]["dims"] != m["rot_dim"]:
+            raise ValueError(f"layer {i}: the whole rotary part of a head is rotated, {m['rot_dim']} lanes, not {m['rot']['dims']}")
+        if m.get("v_mix"):
+            values.add(m["kv_heads"] * m["vdim"])
+    if len(values) > 1:
+        raise ValueError(f"layers that mix values must have equally many: {sorted(values)}")
+    first = layers[0]["mixer"]
+    routers = [e["mlp"]["router"] for e in layers if e.get("mlp") is not None and e["mlp"]["kind"] == "moe"]
+    moe = dict(num_experts=max(r["experts"] for r in routers), num_experts_per_tok=max(r["top"] for r in routers)) \
+        if routers else {}
+    return dict(
+        architectures=["KunudraForCausalLM"], model_type="kunudra", hidden_size=d["width"], vocab_size=d["vocab"],
+        num_hidden_layers=len(layers), num_attention_heads=first["heads"],
+        num_key_value_heads=first.get("kv_heads", first["heads"]), head_dim=first["dim"], layers=layers,
+        norm_eps=d["norm"]["eps"], residual_alpha=d["postln_alpha"], pair_embedding=d["embedding"]["bigram"],
+        max_position_embeddings=DEFAULT_CONTEXT, unbounded_positions=True, tie_word_embeddings=True, torch_dtype="bfloat16",
+        eos_token_id=None, bos_token_id=None, **moe)
+
+
 @native_format("Zidivik")
 def _zidivik(d: dict, shapes: dict) -> dict:
     known = {"channel_delta": "linear_attention", "attention": "full_attention"}

@@ -34,6 +34,8 @@ KERNEL_SETS = {
                      "residual_stream.cu"],
     "window_delta": ["runtime.cu", "gemm_sm100.cu", "window_attn.cu", "window_extend.cu", "delta_scan.cu",
                      "residual_stream.cu", "moe.cu", "moe_any.cu"],
+    "window_latent": ["runtime.cu", "gemm_sm100.cu", "window_attn.cu", "window_extend.cu", "mla.cu", "latent_attn.cu",
+                      "latent_extend.cu", "residual_stream.cu", "moe.cu", "moe_any.cu"],
 }
 
 

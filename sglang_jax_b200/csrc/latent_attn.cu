@@ -2,10 +2,13 @@
 // the paged latent cache  [pages, P, row]  (row >= R + rotary lanes):
 //
 //   latent_prep       one pass over a step's fused projection: RMS-normalises the latent, rotates the shared key part
-//                     and the queries' rotary part (interleaved pairs, fp32 angles), writes the cache rows
+//                     and the queries' rotary part (interleaved pairs, fp32 angles), writes the cache rows; where queries
+//                     have a latent of their own, RMS-normalises that instead, and
+//   latent_rotate     rotates the queries that come out of it
 //   latent_attn_any   absorbed attention of single query tokens on the CUDA cores, everything in fp32: the fp32 mode,
-//                     and bf16 sizes that the tensor-core kernels (mla.cu, latent_extend.cu) do not take
-//   latent_gather     cache rows of whole sequences -> contiguous latents and key parts (input of the prefill kernel)
+//                     and bf16 sizes that the tensor-core kernels (mla.cu, latent_extend.cu) do not take; window, sink
+//   latent_gather     cache rows of whole sequences (or from a token on) -> contiguous latents and key parts (input of the
+//                     prefill kernel)
 //
 // Compiled without fast-math substitutions.
 #include <math.h>
@@ -23,14 +26,33 @@ template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float
 
 constexpr int kPrepThreads = 128;
 
+// A block's sum of `v` in every thread; `red` holds one value per warp.
+__device__ __forceinline__ float prep_sum(float v, float* red) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float tot = 0.f;
+#pragma unroll
+  for (int i = 0; i < kPrepThreads / 32; ++i) tot += red[i];
+  return tot;
+}
+
+// Queries that come from a latent: its columns in the projection, its norm's weight, the result [T, rank] (out null: none).
+struct QueryLatent {
+  int off, rank;
+  const float* norm_w;
+  void* out;
+};
+
 // One CTA per token.  `proj` is the fused projection [T, ld]: query heads at column q_off, [latent | key part] at dkv_off.
 template <typename T>
 __global__ void __launch_bounds__(kPrepThreads)
 latent_prep_kernel(T* __restrict__ proj, long long ld, int q_off, int dkv_off, int H, int dim, int rot, int R,
                    const float* __restrict__ norm_w, float eps, const float* __restrict__ cos_sin,
                    const int* __restrict__ positions, const int* __restrict__ loc, T* __restrict__ cache,
-                   int row_elems) {
-  __shared__ float red[kPrepThreads / 32];
+                   int row_elems, const QueryLatent ql) {
+  __shared__ float red[2][kPrepThreads / 32];
   pdl_wait();
   const int t = blockIdx.x, tid = threadIdx.x, half = rot / 2;
   T* row = proj + static_cast<long long>(t) * ld;
@@ -42,19 +64,24 @@ latent_prep_kernel(T* __restrict__ proj, long long ld, int q_off, int dkv_off, i
     const float v = to_f(lat[i]);
     ss += v * v;
   }
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-  if ((tid & 31) == 0) red[tid >> 5] = ss;
-  __syncthreads();
-  float tot = 0.f;
-#pragma unroll
-  for (int i = 0; i < kPrepThreads / 32; ++i) tot += red[i];
-  const float inv = 1.f / sqrtf(tot / R + eps);
+  const float inv = 1.f / sqrtf(prep_sum(ss, red[0]) / R + eps);
   for (int i = tid; i < R; i += kPrepThreads) dst[i] = from_f<T>(to_f(lat[i]) * inv * norm_w[i]);
   for (int i = tid; i < half; i += kPrepThreads) {
     const float u = to_f(lat[R + 2 * i]), v = to_f(lat[R + 2 * i + 1]), c = cs[i], s = cs[half + i];
     dst[R + 2 * i] = from_f<T>(u * c - v * s);
     dst[R + 2 * i + 1] = from_f<T>(v * c + u * s);
+  }
+  if (ql.out != nullptr) {
+    const T* c = row + ql.off;
+    T* o = static_cast<T*>(ql.out) + static_cast<long long>(t) * ql.rank;
+    float sq = 0.f;
+    for (int i = tid; i < ql.rank; i += kPrepThreads) {
+      const float v = to_f(c[i]);
+      sq += v * v;
+    }
+    const float qi = 1.f / sqrtf(prep_sum(sq, red[1]) / ql.rank + eps);
+    for (int i = tid; i < ql.rank; i += kPrepThreads) o[i] = from_f<T>(to_f(c[i]) * qi * ql.norm_w[i]);
+    return;
   }
   for (int j = tid; j < H * half; j += kPrepThreads) {
     const int h = j / half, i = j - h * half;
@@ -62,6 +89,37 @@ latent_prep_kernel(T* __restrict__ proj, long long ld, int q_off, int dkv_off, i
     const float u = to_f(q[0]), v = to_f(q[1]), c = cs[i], s = cs[half + i];
     q[0] = from_f<T>(u * c - v * s);
     q[1] = from_f<T>(v * c + u * s);
+  }
+}
+
+// Rotates the last `rot` of every head's `dim + rot` lanes in place, one pair per thread.
+template <typename T> struct Pair { T u, v; };
+template <> struct alignas(4) Pair<__nv_bfloat16> { __nv_bfloat16 u, v; };
+template <> struct alignas(8) Pair<float> { float u, v; };
+
+template <typename T, bool ALIGNED>
+__global__ void __launch_bounds__(256)
+latent_rotate_kernel(T* __restrict__ q, long long ld, long long pairs, int H, int dim, int rot,
+                     const float* __restrict__ cos_sin, const int* __restrict__ positions) {
+  pdl_wait();
+  const int half = rot / 2, per = H * half;
+  for (long long n = blockIdx.x * 256ll + threadIdx.x; n < pairs; n += gridDim.x * 256ll) {
+    const long long t = n / per;
+    const int j = static_cast<int>(n - t * per), h = j / half, i = j - h * half;
+    const float* cs = cos_sin + static_cast<long long>(positions[t]) * rot;
+    T* a = q + t * ld + static_cast<long long>(h) * (dim + rot) + dim + 2 * i;
+    Pair<T> p;
+    if constexpr (ALIGNED) p = *reinterpret_cast<const Pair<T>*>(a);
+    else p = Pair<T>{a[0], a[1]};
+    const float u = to_f(p.u), v = to_f(p.v), c = cs[i], s = cs[half + i];
+    p.u = from_f<T>(u * c - v * s);
+    p.v = from_f<T>(v * c + u * s);
+    if constexpr (ALIGNED) {
+      *reinterpret_cast<Pair<T>*>(a) = p;
+    } else {
+      a[0] = p.u;
+      a[1] = p.v;
+    }
   }
 }
 
@@ -76,7 +134,8 @@ __global__ void __launch_bounds__(kAnyThreads)
 latent_attn_any_kernel(const T* __restrict__ q_lat, const T* __restrict__ q_pe, long long pe_token_stride,
                        int pe_head_stride, const T* __restrict__ cache, int row_elems,
                        const int* __restrict__ page_table, int max_pages, int page_size, const int* __restrict__ rows,
-                       const int* __restrict__ kv_lens, T* __restrict__ out, int H, int R, int rot, float scale) {
+                       const int* __restrict__ kv_lens, T* __restrict__ out, int H, int R, int rot, float scale,
+                       int window, const float* __restrict__ sink) {
   extern __shared__ float sm[];
   float* qs = sm;                             // [R + rot]
   float* sc = sm + R + rot;                   // [kAnyTile]
@@ -93,8 +152,8 @@ latent_attn_any_kernel(const T* __restrict__ q_lat, const T* __restrict__ q_pe, 
 #pragma unroll
   for (int i = 0; i < kAnyMaxAcc; ++i) acc[i] = 0.f;
   float m = -INFINITY, l = 0.f;
-  const int D = R + rot;
-  for (int k0 = 0; k0 < len; k0 += kAnyTile) {
+  const int D = R + rot, first = window > 0 && len > window ? len - window : 0;
+  for (int k0 = first / kAnyTile * kAnyTile; k0 < len; k0 += kAnyTile) {
     const int nk = min(kAnyTile, len - k0);
     __syncthreads();                          // qs written / the previous tile's scores and slots read
     if (tid < nk) {
@@ -108,7 +167,7 @@ latent_attn_any_kernel(const T* __restrict__ q_lat, const T* __restrict__ q_pe, 
       for (int i = lane; i < D; i += 32) a += qs[i] * to_f(kr[i]);
 #pragma unroll
       for (int o = 16; o > 0; o >>= 1) a += __shfl_xor_sync(0xffffffffu, a, o);
-      if (lane == 0) sc[j] = a * scale;
+      if (lane == 0) sc[j] = k0 + j >= first ? a * scale : -INFINITY;
     }
     __syncthreads();
     float mx = m;
@@ -129,7 +188,11 @@ latent_attn_any_kernel(const T* __restrict__ q_lat, const T* __restrict__ q_pe, 
     }
     m = mx;
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  float inv = l > 0.f ? 1.f / l : 0.f;
+  if (sink != nullptr) {
+    const float mx = fmaxf(m, sink[h]), c = expf(m - mx);
+    inv = c / (l * c + expf(sink[h] - mx));
+  }
 #pragma unroll
   for (int i = 0; i < kAnyMaxAcc; ++i) {
     const int d = tid + i * kAnyThreads;
@@ -137,12 +200,13 @@ latent_attn_any_kernel(const T* __restrict__ q_lat, const T* __restrict__ q_pe, 
   }
 }
 
-// ctx row r of sequence b (ctx_start[b] <= r < ctx_start[b + 1]) is the sequence's token r - ctx_start[b].
+// ctx row r of sequence b (ctx_start[b] <= r < ctx_start[b + 1]) is the sequence's token r - ctx_start[b] + skip[b] (skip null:
+// none left out).
 __global__ void latent_gather_kernel(__nv_bfloat16* __restrict__ lat, __nv_bfloat16* __restrict__ pe,
                                      const __nv_bfloat16* __restrict__ cache, int row_elems,
                                      const int* __restrict__ page_table, int max_pages, int page_size,
-                                     const int* __restrict__ rows, const int* __restrict__ ctx_start, int B, int total,
-                                     int R, int rot) {
+                                     const int* __restrict__ rows, const int* __restrict__ ctx_start,
+                                     const int* __restrict__ skip, int B, int total, int R, int rot) {
   pdl_wait();
   const int lane = threadIdx.x & 31;
   const int r = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -153,7 +217,7 @@ __global__ void latent_gather_kernel(__nv_bfloat16* __restrict__ lat, __nv_bfloa
     if (ctx_start[mid] <= r) lo = mid;
     else hi = mid - 1;
   }
-  const int pos = r - ctx_start[lo], pg = pos / page_size;
+  const int pos = r - ctx_start[lo] + (skip != nullptr ? skip[lo] : 0), pg = pos / page_size;
   const int slot = page_table[static_cast<long long>(rows[lo]) * max_pages + pg] * page_size + (pos - pg * page_size);
   const uint4* src = reinterpret_cast<const uint4*>(cache + static_cast<long long>(slot) * row_elems);
   uint4* d0 = reinterpret_cast<uint4*>(lat + static_cast<long long>(r) * R);
@@ -167,11 +231,11 @@ __global__ void latent_gather_kernel(__nv_bfloat16* __restrict__ lat, __nv_bfloa
 template <typename T>
 int attn_any(const void* q_lat, const void* q_pe, long long pe_token_stride, int pe_head_stride, const void* cache,
              int row_elems, const int* page_table, int max_pages, int page_size, const int* rows, const int* kv_lens,
-             void* out, int N, int H, int R, int rot, float scale, cudaStream_t s) {
+             void* out, int N, int H, int R, int rot, float scale, int window, const float* sink, cudaStream_t s) {
   const size_t smem = (R + rot + 2 * kAnyTile) * sizeof(float);
   launch_pdl(latent_attn_any_kernel<T>, dim3(N, H), dim3(kAnyThreads), smem, s, static_cast<const T*>(q_lat),
              static_cast<const T*>(q_pe), pe_token_stride, pe_head_stride, static_cast<const T*>(cache), row_elems,
-             page_table, max_pages, page_size, rows, kv_lens, static_cast<T*>(out), H, R, rot, scale);
+             page_table, max_pages, page_size, rows, kv_lens, static_cast<T*>(out), H, R, rot, scale, window, sink);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -180,49 +244,73 @@ int attn_any(const void* q_lat, const void* q_pe, long long pe_token_stride, int
 
 extern "C" {
 
-// proj [T, ld] (queries rotated in place), cos_sin fp32 [positions, rot] = [cos | sin], cache rows of `row_elems`.
+// proj [T, ld] (queries rotated in place), cos_sin fp32 [positions, rot] = [cos | sin], cache rows of `row_elems`.  With
+// `q_latent` [T, q_rank] the projection holds no queries but their latent at column q_off, which is normalised (q_norm_w) into
+// it.
 int sglb_latent_prep(void* proj, long long ld, int q_off, int dkv_off, int T, int H, int dim, int rot, int R,
                      const float* norm_w, float eps, const float* cos_sin, const int* positions, const int* loc,
-                     void* cache, int row_elems, int is_f32, cudaStream_t s) {
+                     void* cache, int row_elems, void* q_latent, int q_rank, const float* q_norm_w, int is_f32,
+                     cudaStream_t s) {
   using namespace sglb;
   if (T <= 0) return 0;
-  if (rot % 2 != 0 || row_elems < R + rot) return -kBadArgument;
+  if (rot % 2 != 0 || row_elems < R + rot || (q_latent != nullptr && (q_rank < 1 || q_norm_w == nullptr)))
+    return -kBadArgument;
+  const QueryLatent ql{q_off, q_rank, q_norm_w, q_latent};
   if (is_f32)
     launch_pdl(latent_prep_kernel<float>, dim3(T), dim3(kPrepThreads), 0, s, static_cast<float*>(proj), ld, q_off, dkv_off,
-               H, dim, rot, R, norm_w, eps, cos_sin, positions, loc, static_cast<float*>(cache), row_elems);
+               H, dim, rot, R, norm_w, eps, cos_sin, positions, loc, static_cast<float*>(cache), row_elems, ql);
   else
     launch_pdl(latent_prep_kernel<__nv_bfloat16>, dim3(T), dim3(kPrepThreads), 0, s, static_cast<__nv_bfloat16*>(proj), ld,
                q_off, dkv_off, H, dim, rot, R, norm_w, eps, cos_sin, positions, loc, static_cast<__nv_bfloat16*>(cache),
-               row_elems);
+               row_elems, ql);
+  return static_cast<int>(cudaGetLastError());
+}
+
+// Head h of token t at q + t * ld + h * (dim + rot), rotated in place.
+int sglb_latent_rotate(void* q, long long ld, int T, int H, int dim, int rot, const float* cos_sin, const int* positions,
+                       int is_f32, cudaStream_t s) {
+  using namespace sglb;
+  if (T <= 0 || rot == 0) return 0;
+  if (rot % 2 != 0 || H < 1) return -kBadArgument;
+  const long long pairs = static_cast<long long>(T) * H * (rot / 2), blocks = (pairs + 255) / 256;
+  const dim3 grid(static_cast<unsigned>(blocks < 148LL * 32 ? blocks : 148LL * 32));
+  const bool aligned = dim % 2 == 0 && ld % 2 == 0 && reinterpret_cast<uintptr_t>(q) % 8 == 0;
+  if (is_f32) {
+    const auto kernel = aligned ? latent_rotate_kernel<float, true> : latent_rotate_kernel<float, false>;
+    launch_pdl(kernel, grid, dim3(256), 0, s, static_cast<float*>(q), ld, pairs, H, dim, rot, cos_sin, positions);
+  } else {
+    const auto kernel = aligned ? latent_rotate_kernel<__nv_bfloat16, true> : latent_rotate_kernel<__nv_bfloat16, false>;
+    launch_pdl(kernel, grid, dim3(256), 0, s, static_cast<__nv_bfloat16*>(q), ld, pairs, H, dim, rot, cos_sin, positions);
+  }
   return static_cast<int>(cudaGetLastError());
 }
 
 // q_lat [N, H, R]; q_pe addressed by strides; query n sees the first kv_lens[n] tokens of table row rows[n];
-// out [N, H, R].
+// out [N, H, R].  `window` (0: none): tokens a query sees, its own included; `sink` [H] or null.
 int sglb_latent_attn_any(const void* q_lat, const void* q_pe, long long pe_token_stride, int pe_head_stride,
                          const void* cache, int row_elems, const int* page_table, int max_pages, int page_size,
                          const int* rows, const int* kv_lens, void* out, int N, int H, int R, int rot, float scale,
-                         int is_f32, cudaStream_t s) {
+                         int window, const float* sink, int is_f32, cudaStream_t s) {
   using namespace sglb;
   if (N <= 0) return 0;
   if (R > kAnyMaxAcc * kAnyThreads || R + rot > 8192 || H > 65535) return -kBadArgument;
   return is_f32 ? attn_any<float>(q_lat, q_pe, pe_token_stride, pe_head_stride, cache, row_elems, page_table, max_pages,
-                                  page_size, rows, kv_lens, out, N, H, R, rot, scale, s)
+                                  page_size, rows, kv_lens, out, N, H, R, rot, scale, window, sink, s)
                 : attn_any<__nv_bfloat16>(q_lat, q_pe, pe_token_stride, pe_head_stride, cache, row_elems, page_table,
-                                          max_pages, page_size, rows, kv_lens, out, N, H, R, rot, scale, s);
+                                          max_pages, page_size, rows, kv_lens, out, N, H, R, rot, scale, window, sink, s);
 }
 
-// lat [total, R], pe [total, rot] <- cache rows of B sequences laid end to end at ctx_start (bf16; R and rot multiples
-// of 8).
+// lat [total, R], pe [total, rot] <- cache rows of B sequences, each from token skip[b] on (null: 0), laid end to end at
+// ctx_start (bf16; R and rot multiples of 8).
 int sglb_latent_gather(void* lat, void* pe, const void* cache, int row_elems, const int* page_table, int max_pages,
-                       int page_size, const int* rows, const int* ctx_start, int B, int total, int R, int rot,
-                       cudaStream_t s) {
+                       int page_size, const int* rows, const int* ctx_start, const int* skip, int B, int total, int R,
+                       int rot, cudaStream_t s) {
   using namespace sglb;
   if (B <= 0 || total <= 0) return 0;
   if (R % 8 != 0 || rot % 8 != 0 || row_elems % 8 != 0) return -kBadArgument;
   launch_pdl(latent_gather_kernel, dim3((total + 7) / 8), dim3(256), 0, s, static_cast<__nv_bfloat16*>(lat),
              static_cast<__nv_bfloat16*>(pe), static_cast<const __nv_bfloat16*>(cache), row_elems, page_table, max_pages,
-             page_size, rows, ctx_start, B, total, R, rot);
+             page_size, rows, ctx_start, skip, B, total, R, rot);
   return static_cast<int>(cudaGetLastError());
 }
 

@@ -3,7 +3,8 @@
 // Keys of a head are [unrotated | rotated]: the unrotated lanes and the values come from one [context, heads,
 // dim + vdim] buffer that a GEMM computed from the latents, the rotated lanes from one [context, rot] buffer shared by
 // all heads.  Queries are read in place from the fused projection.  A sequence's context rows start at ctx_start[b];
-// query i of the step sees the first prefix[b] + i + 1 of them.
+// query i of the step sees the first prefix[b] + i + 1 of them, under a window only the last ones of these (then the rows may
+// start at token skip[b], a multiple of 64, of the sequence).  A sink joins the softmax's denominator (score_terms.cuh).
 //
 // One CTA per (256 query rows of one sequence, head): two 128-row tiles that share every K / V tile of 64 keys.  Warp 0
 // drives TMA (two-stage ring), warp 1 issues tcgen05.mma, warps 2..5 and 6..9 do the softmax of the two tiles, one
@@ -20,6 +21,8 @@
 #include <math.h>
 
 #include "common.cuh"
+#include "score_terms.cuh"
+#include "window_mask.cuh"
 
 namespace sglb {
 namespace {
@@ -31,7 +34,6 @@ constexpr int kThreads = 64 + kTiles * 128;
 constexpr int kTmemCols = 512;                      // per tile: S 2 x 64 (P in place), O 128
 constexpr int kTmemTile = 256, kTmemO = 128;
 constexpr float kRescale = 8.f;
-constexpr float kLog2e = 1.4426950408889634f;
 constexpr int kMinSmem = 120 * 1024;                // one CTA per SM: it takes all of tensor memory
 
 struct Bars {
@@ -45,11 +47,13 @@ struct Params {
   __nv_bfloat16* out;            // [T, heads, vdim] by strides
   long long out_token_stride;
   int out_head_stride;
-  const int *q_start, *q_len, *prefix, *ctx_start;   // [B]
+  const int *q_start, *q_len, *prefix, *ctx_start, *skip;   // [B], skip may be null
   Status* status;
   int B, dim, rot, vdim;
   int nb_n, nb_r, nb_v;          // 64-lane blocks of the unrotated / rotated key part and of the values
   float scale;
+  Window win;
+  ScoreTerms terms;              // (the sink only)
 };
 
 __device__ __forceinline__ float ex2_approx(float x) {
@@ -89,15 +93,14 @@ latent_extend_kernel(const __grid_constant__ CUtensorMap map_qn, const __grid_co
   }
   const int head = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int q_len = p.q_len[b], prefix = p.prefix[b], seq = prefix + q_len, ctx0 = p.ctx_start[b];
+  const int q_len = p.q_len[b], prefix = p.prefix[b], seq = prefix + q_len, ctx0 = p.ctx_start[b] - (p.skip != nullptr ? p.skip[b] : 0);
   const int q0 = tile * kTiles * kTileQ;
-  int n_t[kTiles];                                                // key tiles of the two query tiles
+  const KeyTiles<kTileK> keys(p.win, prefix + q0, prefix + min(q0 + kTiles * kTileQ, q_len) - 1);
+  QueryTile qt[kTiles];
 #pragma unroll
-  for (int t = 0; t < kTiles; ++t) {
-    const int first = q0 + t * kTileQ;
-    n_t[t] = first >= q_len ? 0 : (prefix + min(first + kTileQ, q_len) + kTileK - 1) / kTileK;
-  }
-  const int n = max(n_t[0], n_t[1]);
+  for (int t = 0; t < kTiles; ++t)
+    qt[t] = query_tile(p.win, keys, prefix + q0 + t * kTileQ, prefix + min(q0 + (t + 1) * kTileQ, q_len) - 1);
+  const int n = max(qt[0].n, qt[1].n);
 
   if (threadIdx.x == 0) {
     prefetch_tmap(&map_qn);
@@ -152,7 +155,7 @@ latent_extend_kernel(const __grid_constant__ CUtensorMap map_qn, const __grid_co
         }
         const uint32_t fb = smem_u32(values ? &bars->v_full[st] : &bars->k_full[st]);
         const uint32_t dst = smem_u32(kv_s + st * stage_bytes) + (values ? nb_q * kBlkK : 0);
-        const int row = ctx0 + j * kTileK;
+        const int row = ctx0 + keys.tile(j) * kTileK;
         if (values) {
           mbar_expect_tx(fb, p.nb_v * kBlkK);
           for (int c = 0; c < p.nb_v; ++c) tma_load_3d(dst + c * kBlkK, &map_v, fb, c * 64, head, row);
@@ -185,21 +188,22 @@ latent_extend_kernel(const __grid_constant__ CUtensorMap map_qn, const __grid_co
         }
         const uint32_t v_addr = smem_u32(kv_s + (i & 1) * stage_bytes) + nb_q * kBlkK;
         for (int t = 0; t < kTiles; ++t) {
-          if (i >= n_t[t]) continue;
-          if (!mbar_wait(smem_u32(&bars->p_ready[t][i & 1]), (i >> 1) & 1)) {
+          if (!qt[t].takes(i)) continue;
+          const int li = qt[t].local(i);
+          if (!mbar_wait(smem_u32(&bars->p_ready[t][li & 1]), (li >> 1) & 1)) {
             report(p.status, kTimeoutTmemFull, b, 1000 + i);
             return false;
           }
           tc_fence_after_sync();
-          const uint32_t p_tm = tmem + t * kTmemTile + (i & 1) * kTileK, o_tm = tmem + t * kTmemTile + kTmemO;
+          const uint32_t p_tm = tmem + t * kTmemTile + (li & 1) * kTileK, o_tm = tmem + t * kTmemTile + kTmemO;
 #pragma unroll
           for (int term = 0; term < 2; ++term)
 #pragma unroll
             for (int kk = 0; kk < kTileK / 16; ++kk)
               umma_bf16_ts(o_tm, p_tm + term * (kTileK / 2) + kk * 8,
                            make_smem_desc_sw128_mn(v_addr + kk * 16 * 128, kBlkK), idesc_pv,
-                           (i > 0 || term > 0 || kk > 0) ? 1u : 0u);
-          umma_commit(smem_u32(&bars->pv_done[t][i & 1]));
+                           (li > 0 || term > 0 || kk > 0) ? 1u : 0u);
+          umma_commit(smem_u32(&bars->pv_done[t][li & 1]));
         }
         umma_commit(smem_u32(&bars->v_empty[i & 1]));
         return true;
@@ -213,22 +217,23 @@ latent_extend_kernel(const __grid_constant__ CUtensorMap map_qn, const __grid_co
         }
         const uint32_t k_addr = smem_u32(kv_s + st * stage_bytes);
         for (int t = 0; ok && t < kTiles; ++t) {
-          if (j >= n_t[t]) continue;
-          // this S buffer holds P of tile j - 2 until its product is done
-          if (j >= 2 && !mbar_wait(smem_u32(&bars->pv_done[t][st]), ((j - 2) >> 1) & 1)) {
+          if (!qt[t].takes(j)) continue;
+          const int lj = qt[t].local(j), sb = lj & 1;
+          // this S buffer holds P of the tile before last until its product is done
+          if (lj >= 2 && !mbar_wait(smem_u32(&bars->pv_done[t][sb]), ((lj - 2) >> 1) & 1)) {
             report(p.status, kTimeoutTmemEmpty, b, j);
             ok = false;
             break;
           }
           tc_fence_after_sync();
-          const uint32_t q_addr = smem_u32(q_s + t * nb_q * kBlkQ), s_tm = tmem + t * kTmemTile + st * kTileK;
+          const uint32_t q_addr = smem_u32(q_s + t * nb_q * kBlkQ), s_tm = tmem + t * kTmemTile + sb * kTileK;
           for (int s = 0; s < steps_n + steps_r; ++s) {
             const int blk = s < steps_n ? s >> 2 : p.nb_n + ((s - steps_n) >> 2);
             const int sub = s < steps_n ? s & 3 : (s - steps_n) & 3;
             umma_bf16(s_tm, make_smem_desc_sw128(q_addr + blk * kBlkQ) + 2 * sub,
                       make_smem_desc_sw128(k_addr + blk * kBlkK) + 2 * sub, idesc_s, s > 0 ? 1u : 0u);
           }
-          umma_commit(smem_u32(&bars->s_full[t][st]));
+          umma_commit(smem_u32(&bars->s_full[t][sb]));
         }
         if (!ok) break;
         umma_commit(smem_u32(&bars->k_empty[st]));
@@ -244,14 +249,16 @@ latent_extend_kernel(const __grid_constant__ CUtensorMap map_qn, const __grid_co
     const uint32_t tm = tmem + t * kTmemTile + (static_cast<uint32_t>(qd * 32) << 16);
     const int r_seq = q0 + t * kTileQ + row;                        // row within the sequence's new tokens
     const int kmax = r_seq >= q_len ? seq - 1 : prefix + r_seq;     // last visible key
-    const float scale_log2 = p.scale * kLog2e;
-    const int nt = n_t[t];
+    const int kmin = p.win.first(kmax);                             // first visible key
+    const float scale_log2 = p.scale * kLog2E;
+    const int nt = qt[t].count();
     float m_used = -INFINITY, l = 0.f;
     bool ok = nt > 0;
-    for (int j = 0; ok && j < nt; ++j) {
-      const int st = j & 1;
+    for (int j = 0, lj = 0; ok && j < qt[t].n; ++j) {
+      if (!qt[t].takes(j)) continue;
+      const int st = lj & 1;
       // (votes keep the warp's control flow uniform: one lane per warp arrives on the barriers below)
-      if (!__all_sync(0xffffffffu, mbar_wait(smem_u32(&bars->s_full[t][st]), (j >> 1) & 1))) {
+      if (!__all_sync(0xffffffffu, mbar_wait(smem_u32(&bars->s_full[t][st]), (lj >> 1) & 1))) {
         report(p.status, kTimeoutTmemFull, b, j);
         *abort_flag = 1;
         ok = false;
@@ -263,26 +270,31 @@ latent_extend_kernel(const __grid_constant__ CUtensorMap map_qn, const __grid_co
       tmem_ld32(s_addr, v0);
       tmem_ld32(s_addr + 32, v1);
       tmem_ld_wait();
-      const int nvalid = kmax - j * kTileK + 1;                     // keys of this tile below it are visible
+      // bit e: key e of this tile is visible
+      const int k0 = keys.tile(j) * kTileK;
+      auto below = [](int c) -> uint64_t { return c <= 0 ? 0ull : (c >= 64 ? ~0ull : (1ull << c) - 1); };
+      const uint64_t seen = below(kmax - k0 + 1) & ~below(kmin - k0);
+      const bool full = seen == ~0ull;
+      const uint32_t see0 = static_cast<uint32_t>(seen), see1 = static_cast<uint32_t>(seen >> 32);
       float mx = -INFINITY;
-      if (nvalid >= kTileK) {
+      if (full) {
 #pragma unroll
         for (int e = 0; e < 32; ++e) mx = fmaxf(mx, fmaxf(__uint_as_float(v0[e]), __uint_as_float(v1[e])));
       } else {
 #pragma unroll
         for (int e = 0; e < 32; ++e) {
-          if (e < nvalid) mx = fmaxf(mx, __uint_as_float(v0[e]));
-          if (e + 32 < nvalid) mx = fmaxf(mx, __uint_as_float(v1[e]));
+          if ((see0 >> e) & 1) mx = fmaxf(mx, __uint_as_float(v0[e]));
+          if ((see1 >> e) & 1) mx = fmaxf(mx, __uint_as_float(v1[e]));
         }
       }
       mx *= scale_log2;
-      const bool raise = j > 0 && mx > m_used + kRescale;
-      if (j == 0) {
+      const bool raise = lj > 0 && mx > m_used + kRescale;
+      if (lj == 0) {
         m_used = mx;
       } else if (__any_sync(0xffffffffu, raise)) {
         // rare: bring O and the row sum to the new maximum, after the product in flight; tcgen05.ld / .st are
         // warp-collective, rows that do not need it take part with a factor of one
-        if (!__all_sync(0xffffffffu, mbar_wait(smem_u32(&bars->pv_done[t][(j - 1) & 1]), ((j - 1) >> 1) & 1))) {
+        if (!__all_sync(0xffffffffu, mbar_wait(smem_u32(&bars->pv_done[t][(lj - 1) & 1]), ((lj - 1) >> 1) & 1))) {
           report(p.status, kTimeoutTmemFull, b, 2000 + j);
           *abort_flag = 1;
           ok = false;
@@ -304,16 +316,17 @@ latent_extend_kernel(const __grid_constant__ CUtensorMap map_qn, const __grid_co
         if (raise) m_used = mx;
       }
       float sum = 0.f;
-      const bool full = nvalid >= kTileK;
+      const float ref = m_used == -INFINITY ? 0.f : m_used;         // (nothing seen so far)
       uint32_t hi[32], lo[32];
 #pragma unroll
       for (int c = 0; c < 32; ++c) {
         const uint32_t a = c < 16 ? v0[2 * c] : v1[2 * c - 32], bb = c < 16 ? v0[2 * c + 1] : v1[2 * c - 31];
-        float x = ex2_approx(fmaf(__uint_as_float(a), scale_log2, -m_used));
-        float y = ex2_approx(fmaf(__uint_as_float(bb), scale_log2, -m_used));
+        float x = ex2_approx(fmaf(__uint_as_float(a), scale_log2, -ref));
+        float y = ex2_approx(fmaf(__uint_as_float(bb), scale_log2, -ref));
         if (!full) {
-          if (2 * c >= nvalid) x = 0.f;
-          if (2 * c + 1 >= nvalid) y = 0.f;
+          const uint32_t see = c < 16 ? see0 >> (2 * c) : see1 >> (2 * c - 32);
+          if (!(see & 1)) x = 0.f;
+          if (!(see & 2)) y = 0.f;
         }
         sum += x + y;
         hi[c] = pack_bf16(x, y);
@@ -326,6 +339,7 @@ latent_extend_kernel(const __grid_constant__ CUtensorMap map_qn, const __grid_co
       tc_fence_before_sync();
       __syncwarp();
       if (lane == 0) mbar_arrive(smem_u32(&bars->p_ready[t][st]));
+      ++lj;
     }
     if (ok) {
       if (!__all_sync(0xffffffffu, mbar_wait(smem_u32(&bars->pv_done[t][(nt - 1) & 1]), ((nt - 1) >> 1) & 1))) {
@@ -333,6 +347,7 @@ latent_extend_kernel(const __grid_constant__ CUtensorMap map_qn, const __grid_co
         *abort_flag = 1;
       } else {
         tc_fence_after_sync();
+        if (p.terms.sink != nullptr) l += exp2f(p.terms.sink_log2(head) - m_used);
         const float inv = l > 0.f ? 1.f / l : 0.f;
         __nv_bfloat16* orow = p.out + (p.q_start[b] + r_seq) * p.out_token_stride +
                               static_cast<long long>(head) * p.out_head_stride;
@@ -389,11 +404,14 @@ int sglb_latent_extend_supported(int dim, int rot, int vdim) {
 
 // q: head h of token t at t * q_token_stride + h * (dim + rot), [unrotated | rotated] (total_q tokens);
 // kv [ctx_total, heads, dim + vdim]; k_rot [ctx_total, rot]; out by strides.  B sequences with q_start / q_len (rows of q),
-// prefix (context tokens before them) and ctx_start (first context row).  num_tiles = sum_b ceil(q_len / 256).
+// prefix (tokens before them), ctx_start (first context row) and skip (tokens in front that have no context row, multiples of
+// 64; null: none).  num_tiles = sum_b ceil(q_len / 256).  `window` (0: none): tokens a query sees, its own included; `sink`
+// [heads] or null.
 int sglb_latent_extend(const void* q, long long q_token_stride, int total_q, const void* kv, const void* k_rot,
                        int ctx_total, void* out, long long out_token_stride, int out_head_stride, const int* q_start,
-                       const int* q_len, const int* prefix, const int* ctx_start, int B, int num_tiles, int heads, int dim,
-                       int rot, int vdim, float scale, cudaStream_t stream) {
+                       const int* q_len, const int* prefix, const int* ctx_start, const int* skip, int B, int num_tiles,
+                       int heads, int dim, int rot, int vdim, float scale, int window, const float* sink,
+                       cudaStream_t stream) {
   using namespace sglb;
   if (B <= 0 || num_tiles <= 0 || total_q <= 0 || heads <= 0) return 0;
   if (!sglb_latent_extend_supported(dim, rot, vdim) || q_token_stride % 8 != 0 || out_token_stride % 8 != 0 ||
@@ -418,12 +436,15 @@ int sglb_latent_extend(const void* q, long long q_token_stride, int total_q, con
   p.q_len = q_len;
   p.prefix = prefix;
   p.ctx_start = ctx_start;
+  p.skip = skip;
   p.status = device_status();
   p.B = B; p.dim = dim; p.rot = rot; p.vdim = vdim;
   p.nb_n = (dim + 63) / 64;
   p.nb_r = (rot + 63) / 64;
   p.nb_v = (vdim + 63) / 64;
   p.scale = scale;
+  p.win = Window{window, 0};
+  p.terms = ScoreTerms{0.f, nullptr, sink};
   const int smem = extend_smem(dim, rot, vdim);
   static int cfg = 0;
   if (cfg < smem) {

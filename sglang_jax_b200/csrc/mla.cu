@@ -1,4 +1,4 @@
-// Absorbed multi-head latent attention, decode step (DeepSeek-V2/V3, Kimi-K2, GLM-5, Zozopel).
+// Absorbed multi-head latent attention, decode step (DeepSeek-V2/V3, Kimi-K2, GLM-5, Zozopel, Kunudra).
 //
 // Every head attends over the same latent cache rows  [pages, P, R + rotary lanes]  (R = kv_lora_rank; 512 + 64
 // lanes in the DeepSeek family): logits = q_latent . c + q_pe . k_pe, output = softmax . c  (the caller applies
@@ -13,7 +13,8 @@
 // softmax statistics, and then accumulates its own share of the R output lanes of O += P V (NG groups of
 // 16 lanes).  No cross-warp merge is needed at the end.  With EXACT the weights enter that product as a sum of
 // two bf16 numbers (their rounding and its remainder) instead of being rounded to bf16.  A fifth warp issues the
-// TMA copies (page gathers through the device page table).  All barrier waits are bounded; no multicast is used.
+// TMA copies (page gathers through the device page table).  With a window only the tiles it reaches are read; a sink joins
+// the denominator once the splits are together.  All barrier waits are bounded; no multicast is used.
 //
 // Reference contract: python/sgl_jax/srt/kernels/mla/v2/kernel.py:1338 (oracle mla/v1/ref.py).
 #include <cstdlib>
@@ -22,6 +23,7 @@
 #include <unordered_map>
 
 #include "common.cuh"
+#include "score_terms.cuh"
 
 namespace sglb {
 namespace {
@@ -37,7 +39,6 @@ constexpr int smem_bytes(int blocks, int stages) {
   return stages * blocks * kChunkBytes + blocks * 16 * 128 + kSBytes + 128 + 1024;
 }
 constexpr int kMaxSmem = 227 * 1024;
-constexpr float kLog2e = 1.4426950408889634f;
 
 struct MlaParams {
   const __nv_bfloat16* q_lat;   // [B, H, R]
@@ -55,6 +56,8 @@ struct MlaParams {
   long long pe_token_stride;
   int pe_head_stride;
   float scale;
+  int window;                   // keys a query sees, its own included; 0: all
+  ScoreTerms terms;             // (the sink only)
 };
 
 __device__ __forceinline__ void ldsm_x4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
@@ -92,9 +95,10 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap, const MlaParams p) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int seq = p.seq_lens[b];
   const int* pt_row = p.page_table + static_cast<size_t>(p.req_pool_indices[b]) * p.max_pages;
-  const int n_tiles = (seq + TN - 1) / TN;
-  const int per = (n_tiles + p.num_splits - 1) / p.num_splits;
-  const int t0 = split * per;
+  const int first = p.window > 0 && seq > p.window ? seq - p.window : 0;      // first visible token
+  const int n_tiles = (seq + TN - 1) / TN, tb = first / TN;
+  const int per = (n_tiles - tb + p.num_splits - 1) / p.num_splits;
+  const int t0 = tb + split * per;
   const int t1 = min(t0 + per, n_tiles);
 
   if (threadIdx.x == 0) {
@@ -174,7 +178,7 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap, const MlaParams p) {
 #pragma unroll
     for (int i = 0; i < 2 * NG; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
-    const float scale_log2 = p.scale * kLog2e;
+    const float scale_log2 = p.scale * kLog2E;
     const uint32_t q_base = smem_u32(q_sm);
     int stage = 0;
     uint32_t phase = 0;
@@ -209,7 +213,7 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap, const MlaParams p) {
         for (int e = 0; e < 4; ++e) {
           const int col = warp * 16 + j * 8 + t4 * 2 + (e & 1);
           const int tok = t * TN + col;
-          sb[(g + 8 * (e >> 1)) * TN + col] = tok < seq ? s[j][e] * scale_log2 : -INFINITY;
+          sb[(g + 8 * (e >> 1)) * TN + col] = tok < seq && tok >= first ? s[j][e] * scale_log2 : -INFINITY;
         }
       }
       named_bar_sync(1, kConsumerWarps * 32);
@@ -301,7 +305,11 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap, const MlaParams p) {
     for (int i = 0; i < 2; ++i) {
       const int h = hg * 16 + g + 8 * i;
       if (h >= p.H) continue;
-      const float inv = l_run[i] > 0.f ? 1.f / l_run[i] : 0.f;
+      float inv = l_run[i] > 0.f ? 1.f / l_run[i] : 0.f;
+      if (p.num_splits == 1 && p.terms.sink != nullptr) {
+        const float sink = p.terms.sink_log2(h), m = fmaxf(m_run[i], sink), c = exp2f(m_run[i] - m);
+        inv = c / (l_run[i] * c + exp2f(sink - m));
+      }
       const size_t bh = static_cast<size_t>(b) * p.H + h;
       if (p.num_splits == 1) {
         __nv_bfloat16* dst = p.out + bh * R;
@@ -342,12 +350,14 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap, const MlaParams p) {
 }
 
 __global__ void mla_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_lse,
-                                   __nv_bfloat16* __restrict__ out, int num_splits, int R) {
+                                   __nv_bfloat16* __restrict__ out, int num_splits, int R, int H, const ScoreTerms terms) {
   const int row = blockIdx.x;   // b * H + h
   const float* lse = part_lse + static_cast<size_t>(row) * num_splits;
   float mmax = -INFINITY;
   for (int s = 0; s < num_splits; ++s) mmax = fmaxf(mmax, lse[s]);
-  float wsum = 0.f;
+  const float sink = terms.sink_log2(row % H);
+  mmax = fmaxf(mmax, sink);
+  float wsum = sink == -INFINITY ? 0.f : exp2f(sink - mmax);
   for (int s = 0; s < num_splits; ++s) wsum += (lse[s] == -INFINITY) ? 0.f : exp2f(lse[s] - mmax);
   const float inv = wsum > 0.f ? 1.f / wsum : 0.f;
   for (int d = threadIdx.x; d < R; d += blockDim.x) {
@@ -429,12 +439,13 @@ int sglb_mla_num_splits(int B, int groups, int max_seq_len) {
 // Absorbed-MLA decode.  `kv_buffer` is the latent cache [num_pages, page_size, row_elems] (bf16, rows of
 // kv_lora_rank + rope_dim lanes and padding, row_elems a multiple of 8); `q_lat` [B, H, kv_lora_rank], `q_pe` addressed
 // by strides; `out` [B, H, kv_lora_rank].  With `num_splits > 1` the partial buffers `part_o [B, H, splits, R]` and
-// `part_lse [B, H, splits]` (fp32) are required.  `exact`: attention weights are not rounded to bf16.
+// `part_lse [B, H, splits]` (fp32) are required.  `exact`: attention weights are not rounded to bf16.  `window` (0: none):
+// tokens a query sees, its own included; `sink` [H] or null.
 int sglb_mla_decode(const void* q_lat, const void* q_pe, long long pe_token_stride, int pe_head_stride, void* out,
                     const void* kv_buffer, long long num_pages, int row_elems, const int* page_table, int max_pages,
                     const int* req_pool_indices, const int* seq_lens, int B, int H, int kv_lora_rank, int rope_dim,
-                    int page_size, float scale, int num_splits, float* part_o, float* part_lse, int exact,
-                    cudaStream_t stream) {
+                    int page_size, float scale, int window, const float* sink, int num_splits, float* part_o,
+                    float* part_lse, int exact, cudaStream_t stream) {
   using namespace sglb;
   if (B <= 0) return 0;
   const int dk = kv_lora_rank + rope_dim;
@@ -468,9 +479,11 @@ int sglb_mla_decode(const void* q_lat, const void* q_pe, long long pe_token_stri
   p.R = kv_lora_rank; p.DK = dk;
   p.num_splits = num_splits < 1 ? 1 : num_splits;
   p.scale = scale;
+  p.window = window;
+  p.terms = ScoreTerms{0.f, nullptr, sink};
   cudaError_t e = exact ? launch_width<true>(tm, p, smem, stream) : launch_width<false>(tm, p, smem, stream);
   if (e == cudaSuccess && p.num_splits > 1) {
-    mla_combine_kernel<<<B * H, 128, 0, stream>>>(part_o, part_lse, p.out, p.num_splits, kv_lora_rank);
+    mla_combine_kernel<<<B * H, 128, 0, stream>>>(part_o, part_lse, p.out, p.num_splits, kv_lora_rank, H, p.terms);
     e = cudaGetLastError();
   }
   return e == cudaSuccess ? 0 : static_cast<int>(e);

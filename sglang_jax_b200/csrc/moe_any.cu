@@ -1,6 +1,8 @@
 // Routed experts beside the tensor-core kernels of moe.cu / gemm_sm100.cu, in bf16 or fp32, any sizes:
 //
 //   route_by_logit     z = W x + b in fp32 (or z given), the k largest, weights = softmax over those
+//   route_by_score     s = softmax(W x) in fp32 (or the logits given), the k largest s + correction, weights = scale * s;
+//                      one more row of W may give a gate per token, its sigmoid
 //   grouped_gemm_any   out[r] = x[row(r)] . w[group of r]^T on the CUDA cores with fp32 accumulation: the fp32 mode, and
 //                      bf16 sizes whose rows are not whole 16-byte units
 //
@@ -60,11 +62,10 @@ __device__ __forceinline__ void warp_dots(const T* __restrict__ w, long long ld,
     for (int o = 16; o > 0; o >>= 1) a[r] += __shfl_xor_sync(0xffffffffu, a[r], o);
 }
 
-// The k largest of z[0 .. E) by one warp (ties: the lower index), and their softmax.
-__device__ __forceinline__ void choose(float* z, int E, int k, float* __restrict__ out_w, int* __restrict__ out_ids,
-                                       int lane) {
-  float mine = -INFINITY;
-  int my_id = 0;
+// The k largest of z[0 .. E) by one warp (ties: the lower index); lane j < k holds the j-th and its index.
+__device__ __forceinline__ void largest(float* z, int E, int k, int lane, float& mine, int& my_id) {
+  mine = -INFINITY;
+  my_id = 0;
   for (int j = 0; j < k; ++j) {
     float best = -INFINITY;
     int bi = 0x7fffffff;
@@ -93,6 +94,14 @@ __device__ __forceinline__ void choose(float* z, int E, int k, float* __restrict
     if (lane == 0) z[bi] = -INFINITY;
     __syncwarp();
   }
+}
+
+// ... and their softmax.
+__device__ __forceinline__ void choose(float* z, int E, int k, float* __restrict__ out_w, int* __restrict__ out_ids,
+                                       int lane) {
+  float mine;
+  int my_id;
+  largest(z, E, k, lane, mine, my_id);
   const float top = __shfl_sync(0xffffffffu, mine, 0);
   float p = lane < k ? expf(mine - top) : 0.f, sum = p;
 #pragma unroll
@@ -103,45 +112,86 @@ __device__ __forceinline__ void choose(float* z, int E, int k, float* __restrict
   }
 }
 
+// Choice by score: the softmax over all logits, corrected for the choice only.  `gate` (or null): one per token, from logit E.
+struct ScoreRule {
+  int on;
+  const float* correction;         // [E] or null
+  float scale;
+  float* gate;                     // [T] or null
+  __host__ __device__ __forceinline__ int logits(int E) const { return E + (gate != nullptr); }
+};
+
+__device__ __forceinline__ void choose_by_score(float* z, float* s, int E, int k, const ScoreRule& r, size_t t,
+                                                float* __restrict__ out_w, int* __restrict__ out_ids, int lane) {
+  if (r.gate != nullptr && lane == 0) r.gate[t] = 1.f / (1.f + expf(-z[E]));
+  float mx = -INFINITY, sum = 0.f;
+  for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+  for (int e = lane; e < E; e += 32) {
+    s[e] = expf(z[e] - mx);
+    sum += s[e];
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+  for (int e = lane; e < E; e += 32) {
+    s[e] /= sum;
+    z[e] = s[e] + (r.correction != nullptr ? r.correction[e] : 0.f);
+  }
+  __syncwarp();
+  float mine;
+  int my_id;
+  largest(z, E, k, lane, mine, my_id);
+  if (lane < k) {
+    out_w[lane] = s[my_id] * r.scale;
+    out_ids[lane] = my_id;
+  }
+}
+
 // One CTA per token: the warps share the experts' dot products, the first one chooses.
 template <typename T>
 __global__ void __launch_bounds__(kRouteThreads)
 route_token_kernel(const T* __restrict__ x, const T* __restrict__ w, const T* __restrict__ bias, float* __restrict__ out_w,
-                   int* __restrict__ out_ids, int E, int K, int k, int wide) {
+                   int* __restrict__ out_ids, int E, int K, int k, int wide, const ScoreRule rule) {
   extern __shared__ float4 sm4[];
   float* xs = reinterpret_cast<float*>(sm4);           // [K]
-  float* z = xs + (K + 3) / 4 * 4;                     // [E]
+  float* z = xs + (K + 3) / 4 * 4;                     // [n], by score also [E]
+  const int n = rule.logits(E);
   pdl_wait();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const size_t t = blockIdx.x;
   for (int i = tid; i < K; i += kRouteThreads) xs[i] = to_f(x[t * K + i]);
   __syncthreads();
-  for (int e = warp * kAtOnce; e < E; e += kRouteThreads / 32 * kAtOnce) {
+  for (int e = warp * kAtOnce; e < n; e += kRouteThreads / 32 * kAtOnce) {
     float a[kAtOnce];
-    const int rows = min(kAtOnce, E - e);
+    const int rows = min(kAtOnce, n - e);
     warp_dots(w + static_cast<size_t>(e) * K, static_cast<long long>(K), rows, xs, K, lane, wide != 0, a);
 #pragma unroll
     for (int r = 0; r < kAtOnce; ++r)
       if (lane == r && r < rows) z[e + r] = a[r] + (bias != nullptr ? to_f(bias[e + r]) : 0.f);
   }
   __syncthreads();
-  if (warp == 0) choose(z, E, k, out_w + t * k, out_ids + t * k, lane);
+  if (warp != 0) return;
+  if (rule.on) choose_by_score(z, z + n, E, k, rule, t, out_w + t * k, out_ids + t * k, lane);
+  else choose(z, E, k, out_w + t * k, out_ids + t * k, lane);
 }
 
 // Logits given: one warp per token.
 template <typename T>
 __global__ void __launch_bounds__(128)
 route_logits_kernel(const float* __restrict__ logits, const T* __restrict__ bias, float* __restrict__ out_w,
-                    int* __restrict__ out_ids, int T_, int E, int k) {
+                    int* __restrict__ out_ids, int T_, int E, int k, const ScoreRule rule) {
   extern __shared__ float4 sm4[];
   pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const size_t t = blockIdx.x * 4ull + warp;
   if (t >= T_) return;
-  float* z = reinterpret_cast<float*>(sm4) + warp * E;
-  for (int e = lane; e < E; e += 32) z[e] = logits[t * E + e] + (bias != nullptr ? to_f(bias[e]) : 0.f);
+  const int n = rule.logits(E);
+  float* z = reinterpret_cast<float*>(sm4) + warp * (n + E);
+  for (int e = lane; e < n; e += 32) z[e] = logits[t * n + e] + (bias != nullptr ? to_f(bias[e]) : 0.f);
   __syncwarp();
-  choose(z, E, k, out_w + t * k, out_ids + t * k, lane);
+  if (rule.on) choose_by_score(z, z + n, E, k, rule, t, out_w + t * k, out_ids + t * k, lane);
+  else choose(z, E, k, out_w + t * k, out_ids + t * k, lane);
 }
 
 // ---------------------------------------------------------------------------------------------
@@ -203,13 +253,14 @@ grouped_gemm_any_kernel(const T* __restrict__ x, const int* __restrict__ row_tok
 
 template <typename T>
 int route(const float* z, const void* x, const void* w, const void* bias, float* out_w, int* out_ids, int T_, int E, int K,
-          int k, cudaStream_t s) {
+          int k, const ScoreRule& rule, cudaStream_t s) {
   const T* b = static_cast<const T*>(bias);
+  const int held = rule.logits(E) + E;                 // floats per token for the choice
   if (z != nullptr) {
-    launch_pdl(route_logits_kernel<T>, dim3((T_ + 3) / 4), dim3(128), 4 * E * sizeof(float), s, z, b, out_w, out_ids, T_, E,
-               k);
+    launch_pdl(route_logits_kernel<T>, dim3((T_ + 3) / 4), dim3(128), 4 * held * sizeof(float), s, z, b, out_w, out_ids, T_,
+               E, k, rule);
   } else {
-    const size_t smem = ((K + 3) / 4 * 4 + E) * sizeof(float);
+    const size_t smem = ((K + 3) / 4 * 4 + held) * sizeof(float);
     if (smem > 48 * 1024) {
       static size_t cfg = 0;
       if (cfg < smem) {
@@ -221,7 +272,7 @@ int route(const float* z, const void* x, const void* w, const void* bias, float*
     }
     const int wide = K % 8 == 0 && reinterpret_cast<uintptr_t>(w) % 16 == 0;
     launch_pdl(route_token_kernel<T>, dim3(T_), dim3(kRouteThreads), smem, s, static_cast<const T*>(x),
-               static_cast<const T*>(w), b, out_w, out_ids, E, K, k, wide);
+               static_cast<const T*>(w), b, out_w, out_ids, E, K, k, wide, rule);
   }
   return static_cast<int>(cudaGetLastError());
 }
@@ -237,8 +288,21 @@ int sglb_route_by_logit(const float* z, const void* x, const void* w, const void
   using namespace sglb;
   if (T <= 0) return 0;
   if (E < 1 || E > kMaxExperts || k < 1 || k > kMaxTop || k > E || K < 1 || K > 32768) return -kBadArgument;
-  return is_f32 ? route<float>(z, x, w, bias, out_w, out_ids, T, E, K, k, s)
-                : route<__nv_bfloat16>(z, x, w, bias, out_w, out_ids, T, E, K, k, s);
+  const ScoreRule rule{0, nullptr, 1.f, nullptr};
+  return is_f32 ? route<float>(z, x, w, bias, out_w, out_ids, T, E, K, k, rule, s)
+                : route<__nv_bfloat16>(z, x, w, bias, out_w, out_ids, T, E, K, k, rule, s);
+}
+
+// w [E, K], with `gate` [T] one row more, whose product's sigmoid goes there; z [T, rows of w] fp32: products computed
+// elsewhere, or null.  correction [E] or null.
+int sglb_route_by_score(const float* z, const void* x, const void* w, const float* correction, float* out_w, int* out_ids,
+                        float* gate, int T, int E, int K, int k, float scale, int is_f32, cudaStream_t s) {
+  using namespace sglb;
+  if (T <= 0) return 0;
+  if (E < 1 || E > kMaxExperts || k < 1 || k > kMaxTop || k > E || K < 1 || K > 32768) return -kBadArgument;
+  const ScoreRule rule{1, correction, scale, gate};
+  return is_f32 ? route<float>(z, x, w, nullptr, out_w, out_ids, T, E, K, k, rule, s)
+                : route<__nv_bfloat16>(z, x, w, nullptr, out_w, out_ids, T, E, K, k, rule, s);
 }
 
 // x rows of K, row_token [rows] or null (row r reads x row r), w [groups, N, K], out [rows, N]; lists from sglb_moe_align.

@@ -3,13 +3,19 @@
 // back:
 //
 //   embed_scaled       x = table[id] * scale (+ sinusoidal position)  -> x (fp32), x in T
+//   embed_pair         x = table[id] + pairs[hash(previous id, id)]  -> x (fp32), x in T.  A token's predecessor is the one
+//                      before it in the step or, for the first of a sequence's portion, the id kept with its cache slot
+//   sum_norm           x <- norm(alpha x + s * y)                     -> x (fp32, in place), x in T (or the next norm's
+//                      result); y may be gated per token and joined by weighted rows of routed experts and, for choices
+//                      beyond the experts, by x itself
 //   postnorm_add       x <- x + s * y / sqrt(mean(y^2) + eps)         -> x (fp32, in place), x in T
 //                      (s, fp32 per channel, holds norm weight, layer scale and residual multiplier), or, instead of x in
 //                      T, the next sublayer's input x / sqrt(mean(x^2) + eps') * w
 //   stream_add         x <- x + y (+ weighted rows of routed experts) -> x (fp32, in place), x in T
 //   rmsnorm_stream     y = x / sqrt(mean(x^2) + eps) * w              -> y in T
 //   gelu_mul           gelu_tanh(a) * b of a fused [a | b] projection
-//   clipped_swiglu     g sigmoid(alpha g) (u + 1) of a fused [a | b] projection, g = min(a, limit), u = clamp(b, +-limit)
+//   clipped_swiglu     g sigmoid(alpha g) (u + shift) of a fused [a | b] projection, g = min(a, limit), u = clamp(b, +-limit);
+//                      without limit and shift and with alpha 1 the plain SwiGLU
 //   side_gate          gelu_tanh(z) * a column range of table[id]
 //   sigmoid_gate       o * sigmoid(g), g a column range of a wider projection
 //
@@ -98,6 +104,151 @@ __global__ void embed_scaled_kernel(float* __restrict__ x, T* __restrict__ xt, c
     if (turns != nullptr) add_position<VEC>(f, turns, i, positions[t]);
     store_v<VEC>(x + t * W + i, f);
     if (xt != nullptr) store_v<VEC>(xt + t * W + i, f);
+  }
+}
+
+// Ids that belong to the cache slots, and how the table of pairs is addressed.
+struct PairTable {
+  const void* table;               // [buckets + 1, W]; the last row is for a sequence's first token
+  int buckets;
+  long long mul_prev, mul_cur;
+  int* slot_ids;                   // id of the token in every cache slot
+  const int *positions, *loc;      // [T]
+  const int *cu, *rows;            // first token of every sequence of the step [B + 1] (null: one token each), table rows [B]
+  const int* page_table;
+  int B, max_pages, page_size;
+  __device__ __forceinline__ int row(const int* __restrict__ ids, int t) const {
+    const int pos = positions[t];
+    if (pos <= 0) return buckets;
+    int b = t;
+    if (cu != nullptr) {
+      int hi = B - 1;
+      b = 0;
+      while (b < hi) {             // last sequence that starts at or before t
+        const int mid = (b + hi + 1) >> 1;
+        if (cu[mid] <= t) b = mid;
+        else hi = mid - 1;
+      }
+    }
+    int prev;
+    if (cu != nullptr && t > cu[b]) {
+      prev = ids[t - 1];
+    } else {
+      const int pg = (pos - 1) / page_size;
+      prev = slot_ids[page_table[static_cast<long long>(rows[b]) * max_pages + pg] * page_size + (pos - 1 - pg * page_size)];
+    }
+    const long long h = (prev * mul_prev + ids[t] * mul_cur) % buckets;
+    return static_cast<int>(h < 0 ? h + buckets : h);
+  }
+};
+
+template <typename T, int VEC>
+__global__ void embed_pair_kernel(float* __restrict__ x, T* __restrict__ xt, const int* __restrict__ ids,
+                                  const T* __restrict__ table, int W, int rows, const PairTable p) {
+  pdl_wait();
+  const size_t t = blockIdx.x;
+  const int id = min(max(ids[t], 0), rows - 1), pr = p.row(ids, static_cast<int>(t));
+  if (threadIdx.x == 0) p.slot_ids[p.loc[t]] = ids[t];               // (a slot of this step: no other token reads it here)
+  const T* src = table + static_cast<size_t>(id) * W;
+  const T* pair = static_cast<const T*>(p.table) + static_cast<size_t>(pr) * W;
+  for (int i = threadIdx.x * VEC; i < W; i += blockDim.x * VEC) {
+    float f[VEC], g[VEC];
+    load_v<VEC>(src + i, f);
+    load_v<VEC>(pair + i, g);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) f[e] += g[e];
+    store_v<VEC>(x + t * W + i, f);
+    if (xt != nullptr) store_v<VEC>(xt + t * W + i, f);
+  }
+}
+
+struct SumNorm {
+  float* x;
+  void* xt;
+  const void* y;
+  const float *scale, *weight;     // [W]: of y, of the norm
+  float alpha, eps;
+  const float* y_gate;             // [n] or null: factor of y per token
+  const void* expert;              // rows of routed experts, or null
+  const float* weights;            // [n, k]
+  const int *rows, *ids;           // [n, k]: their rows (negative: elsewhere), the choices
+  int k, experts;                  // choices from `experts` on stand for x itself
+  const float* next_weight;        // the norm that follows, or null
+  float next_eps;
+  int W;
+};
+
+template <typename T, int VEC, int VPT, bool NEXT>
+__global__ void sum_norm_kernel(const SumNorm p) {
+  __shared__ float red[64];
+  pdl_wait();
+  const size_t t = blockIdx.x, row = t * p.W;
+  const T* y = static_cast<const T*>(p.y);
+  const T* expert = static_cast<const T*>(p.expert);
+  T* xt = static_cast<T*>(p.xt);
+  const float gate = p.y_gate != nullptr ? p.y_gate[t] : 1.f;
+  float own = 0.f;
+  for (int j = 0; j < p.k; ++j) own += p.ids[t * p.k + j] >= p.experts ? p.weights[t * p.k + j] : 0.f;
+  float z[VPT][VEC];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * VEC;
+    if (c < p.W) {
+      float v[VEC], xv[VEC], s[VEC];
+      load_v<VEC>(y + row + c, v);
+      load_v<VEC>(p.x + row + c, xv);
+      load_v<VEC>(p.scale + c, s);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v[e] = v[e] * gate + own * xv[e];
+      if (expert != nullptr)
+        for (int j = 0; j < p.k; ++j) {
+          const int r = p.rows[t * p.k + j];
+          if (r < 0) continue;
+          const float w = p.weights[t * p.k + j];
+          float g[VEC];
+          load_v<VEC>(expert + static_cast<size_t>(r) * p.W + c, g);
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) v[e] += w * g[e];
+        }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        z[i][e] = p.alpha * xv[e] + s[e] * v[e];
+        ss += z[i][e] * z[i][e];
+      }
+    }
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / p.W + p.eps);
+  ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * VEC;
+    if (c < p.W) {
+      float w[VEC];
+      load_v<VEC>(p.weight + c, w);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        z[i][e] *= inv * w[e];
+        ss += z[i][e] * z[i][e];
+      }
+      store_v<VEC>(p.x + row + c, z[i]);
+      if constexpr (!NEXT)
+        if (xt != nullptr) store_v<VEC>(xt + row + c, z[i]);
+    }
+  }
+  if constexpr (NEXT) {
+    const float next_inv = 1.f / sqrtf(block_sum(ss, red + 32) / p.W + p.next_eps);
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = (threadIdx.x + i * blockDim.x) * VEC;
+      if (c < p.W) {
+        float w[VEC];
+        load_v<VEC>(p.next_weight + c, w);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) z[i][e] *= next_inv * w[e];
+        store_v<VEC>(xt + row + c, z[i]);
+      }
+    }
   }
 }
 
@@ -258,7 +409,7 @@ __global__ void gelu_mul_kernel(T* __restrict__ out, const T* __restrict__ in, l
 
 template <typename T, int VEC>
 __global__ void clipped_swiglu_kernel(T* __restrict__ out, const T* __restrict__ in, long long rows, int F, float limit,
-                                      float alpha) {
+                                      float alpha, float shift) {
   pdl_wait();
   const long long per = F / VEC, total = rows * per;
   for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < total;
@@ -271,7 +422,7 @@ __global__ void clipped_swiglu_kernel(T* __restrict__ out, const T* __restrict__
 #pragma unroll
     for (int e = 0; e < VEC; ++e) {
       const float g = fminf(a[e], limit), u = fminf(fmaxf(b[e], -limit), limit);
-      a[e] = swish(g, alpha, T()) * (u + 1.f);
+      a[e] = swish(g, alpha, T()) * (u + shift);
     }
     store_v<VEC>(out + r * F + c, a);
   }
@@ -359,6 +510,29 @@ int embed_scaled(float* x, void* xt, const int* ids, const void* table, long lon
 }
 
 template <typename T>
+int embed_pair(float* x, void* xt, const int* ids, const void* table, long long n, int W, int rows, const PairTable& p,
+               cudaStream_t s) {
+  T* o = static_cast<T*>(xt);
+  const T* tb = static_cast<const T*>(table);
+  auto threads = [](int groups) { return dim3(row_threads(groups) < 256 ? row_threads(groups) : 256); };
+  if (W % 4 == 0)
+    launch_pdl(embed_pair_kernel<T, 4>, dim3(n), threads(W / 4), 0, s, x, o, ids, tb, W, rows, p);
+  else
+    launch_pdl(embed_pair_kernel<T, 1>, dim3(n), threads(W), 0, s, x, o, ids, tb, W, rows, p);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T>
+int sum_norm(const SumNorm& p, long long n, cudaStream_t s) {
+  int threads = 0;
+  const bool ok = for_row(p.W, p.W % 4 == 0, &threads, [&]<int VEC, int VPT>() {
+    const auto kernel = p.next_weight != nullptr ? sum_norm_kernel<T, VEC, VPT, true> : sum_norm_kernel<T, VEC, VPT, false>;
+    launch_pdl(kernel, dim3(n), dim3(threads), 0, s, p);
+  });
+  return ok ? static_cast<int>(cudaGetLastError()) : -kBadArgument;
+}
+
+template <typename T>
 int postnorm_add(float* x, void* xt, const void* y, const float* sc, long long n, int W, float eps, const float* next_s,
                  float next_eps, cudaStream_t s) {
   int threads = 0;
@@ -406,15 +580,15 @@ int stream_add(float* x, void* xt, const void* y, const void* expert, const floa
 }
 
 template <typename T>
-int clipped_swiglu(void* out, const void* in, long long rows, int F, float limit, float alpha, cudaStream_t s) {
+int clipped_swiglu(void* out, const void* in, long long rows, int F, float limit, float alpha, float shift, cudaStream_t s) {
   T* o = static_cast<T*>(out);
   const T* i = static_cast<const T*>(in);
   constexpr int kWide = sizeof(T) == 2 ? 8 : 4;
   if (F % kWide == 0)
     launch_pdl(clipped_swiglu_kernel<T, kWide>, dim3(grid_for(rows * (F / kWide))), dim3(256), 0, s, o, i, rows, F, limit,
-               alpha);
+               alpha, shift);
   else
-    launch_pdl(clipped_swiglu_kernel<T, 1>, dim3(grid_for(rows * F)), dim3(256), 0, s, o, i, rows, F, limit, alpha);
+    launch_pdl(clipped_swiglu_kernel<T, 1>, dim3(grid_for(rows * F)), dim3(256), 0, s, o, i, rows, F, limit, alpha, shift);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -465,6 +639,35 @@ int sglb_embed_scaled(float* x, void* xt, const int* ids, const void* table, lon
                 : sglb::embed_scaled<__nv_bfloat16>(x, xt, ids, table, n, W, rows, scale, positions, turns, s);
 }
 
+// pairs [buckets + 1, W]; slot_ids: id kept with every cache slot (read, and written at loc); cu [B + 1] / rows [B] / page_table:
+// the step's sequences (cu null: one token each).
+int sglb_embed_pair(float* x, void* xt, const int* ids, const void* table, long long n, int W, int rows, const void* pairs,
+                    int buckets, long long mul_prev, long long mul_cur, int* slot_ids, const int* positions, const int* loc,
+                    const int* cu, const int* req_rows, const int* page_table, int B, int max_pages, int page_size,
+                    int is_f32, cudaStream_t s) {
+  if (n <= 0) return 0;
+  if (buckets < 1 || page_size < 1 || (cu == nullptr && B != n)) return -sglb::kBadArgument;
+  const sglb::PairTable p{pairs, buckets, mul_prev, mul_cur, slot_ids, positions, loc, cu, req_rows, page_table, B, max_pages,
+                          page_size};
+  return is_f32 ? sglb::embed_pair<float>(x, xt, ids, table, n, W, rows, p, s)
+                : sglb::embed_pair<__nv_bfloat16>(x, xt, ids, table, n, W, rows, p, s);
+}
+
+// x <- weight * z / sqrt(mean(z^2) + eps) with z = alpha x + scale * (y_gate y + sum_j weights[t, j] * c_j), c_j being row
+// rows[t, j] of `expert`, nothing where that is negative, and x where ids[t, j] >= experts (k = 0: none of these).  With
+// next_weight, xt (then required in either type) receives next_weight * x / sqrt(mean(x^2) + next_eps).
+int sglb_sum_norm(float* x, void* xt, const void* y, const float* scale, const float* weight, float alpha, float eps,
+                  const float* y_gate, const void* expert, const float* weights, const int* rows, const int* ids, int k,
+                  int experts, const float* next_weight, float next_eps, long long n, int W, int is_f32, cudaStream_t s) {
+  if (n <= 0) return 0;
+  if ((next_weight != nullptr && xt == nullptr) || (k > 0 && (weights == nullptr || ids == nullptr)) ||
+      (expert != nullptr && rows == nullptr))
+    return -sglb::kBadArgument;
+  const sglb::SumNorm p{x, xt, y, scale, weight, alpha, eps, y_gate, expert, weights, rows, ids, k, experts, next_weight,
+                        next_eps, W};
+  return is_f32 ? sglb::sum_norm<float>(p, n, s) : sglb::sum_norm<__nv_bfloat16>(p, n, s);
+}
+
 // With `next_scale`, `xt` (then required in either type) receives next_scale * x / sqrt(mean(x^2) + next_eps).
 int sglb_postnorm_add(float* x, void* xt, const void* y, const float* scale, long long n, int W, float eps,
                       const float* next_scale, float next_eps, int is_f32, cudaStream_t s) {
@@ -482,11 +685,11 @@ int sglb_stream_add(float* x, void* xt, const void* y, const void* expert, const
                 : sglb::stream_add<__nv_bfloat16>(x, xt, y, expert, weights, rows, k, n, W, s);
 }
 
-int sglb_clipped_swiglu(void* out, const void* in, long long rows, int F, float limit, float alpha, int is_f32,
+int sglb_clipped_swiglu(void* out, const void* in, long long rows, int F, float limit, float alpha, float shift, int is_f32,
                         cudaStream_t s) {
   if (rows <= 0) return 0;
-  return is_f32 ? sglb::clipped_swiglu<float>(out, in, rows, F, limit, alpha, s)
-                : sglb::clipped_swiglu<__nv_bfloat16>(out, in, rows, F, limit, alpha, s);
+  return is_f32 ? sglb::clipped_swiglu<float>(out, in, rows, F, limit, alpha, shift, s)
+                : sglb::clipped_swiglu<__nv_bfloat16>(out, in, rows, F, limit, alpha, shift, s);
 }
 
 // out [rows, F] = gelu_tanh(z) * table[ids, offset : offset + F], table rows of `ld` elements.

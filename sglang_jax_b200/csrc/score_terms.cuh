@@ -1,0 +1,34 @@
+// What an attention does to its scores beside scaling them, all of it optional: a soft cap  c tanh(s / c),  a bias that falls
+// with the distance to the key  (- slope of the head * distance),  and a sink, an entry of the softmax's denominator per head
+// that has neither key nor value.  Cap and bias come in this order, the sink is neither scaled, capped nor biased.
+#pragma once
+#include <math.h>
+
+namespace sglb {
+
+constexpr float kLog2E = 1.4426950408889634f;
+
+struct ScoreTerms {
+  float cap;             // 0: none
+  const float* slope;    // [heads] or null
+  const float* sink;     // [heads] or null
+  __device__ __forceinline__ bool shaped() const { return cap > 0.f || slope != nullptr; }
+  __device__ __forceinline__ float slope_of(int h) const { return slope != nullptr ? slope[h] : 0.f; }
+  // the scaled score of a key at this distance
+  __device__ __forceinline__ float apply(float s, float slope_h, int distance) const {
+    if (cap > 0.f) s = cap * tanhf(s / cap);
+    return s - slope_h * static_cast<float>(distance);
+  }
+  // the sink in log2 units; -infinity without one
+  __device__ __forceinline__ float sink_log2(int h) const { return sink != nullptr ? sink[h] * kLog2E : -INFINITY; }
+};
+
+// tanh through one exponential and one division: its absolute error, which is what counts in a score, stays near 2^-22.
+__device__ __forceinline__ float tanh_by_exp(float z) {
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(fminf(z, 20.f) * (2.f * kLog2E)));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + e));
+  return fmaf(-2.f, r, 1.f);
+}
+
+}  // namespace sglb

@@ -3,16 +3,19 @@
 //
 //   attn_prep          one pass over a step's fused projection: divides queries and keys by their root mean square per head,
 //                      writes queries (padded with zeros) and cache rows
+//   attn_prep_rows     the same with norms over the whole query and key projections (and weights), and values mixed with those
+//                      of another layer
 //   window_decode      every query token on its own (bf16): the heads of one KV head fill the 16 rows of an MMA, 64-key
 //                      tiles stream through a TMA ring straight out of the pages, KV split over CTAs + combine.  The
 //                      attention weights enter the value product as two bf16 terms (rounding and remainder)
 //   window_attn_any    the same on the CUDA cores in fp32: the fp32 mode and sizes the above does not take
 //
-// Both finish with the gate per head, if there is one: out * sigmoid(gate).  Waits are bounded, no multicast.  Compiled
-// without fast-math substitutions.
+// Scores may be capped, biased by distance and joined by a sink (score_terms.cuh).  Attention finishes with the gate per
+// head, if there is one: out * sigmoid(gate).  Waits are bounded, no multicast.  Compiled without fast-math substitutions.
 #include <math.h>
 
 #include "common.cuh"
+#include "score_terms.cuh"
 #include "window_mask.cuh"
 
 namespace sglb {
@@ -23,8 +26,6 @@ __device__ __forceinline__ float to_f(__nv_bfloat16 v) { return __bfloat162float
 template <typename T> __device__ __forceinline__ T from_f(float v);
 template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
 template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
-
-constexpr float kLog2e = 1.4426950408889634f;
 
 // ------------------------------------------------------------------------------------------- prep
 template <typename T, int VEC> struct Pack { T v[VEC]; };
@@ -88,6 +89,90 @@ attn_prep_kernel(const T* __restrict__ proj, T* __restrict__ q, T* __restrict__ 
   }
 }
 
+// Norms over all heads at once: one CTA per token.  `sq` (else computed here): the sums of squares of the whole query and key
+// projections, of which a rank may hold a part; the means are over nq and nk elements.
+struct RowPrepParams {
+  PrepParams b;
+  const float *q_w, *k_w, *sq;
+  int nq, nk;
+  const void* v_mix;               // [T, ld] value rows to mix in, or null
+  long long v_mix_ld;
+  const float* share;              // their share
+};
+
+constexpr int kRowThreads = 256;
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(kRowThreads)
+attn_prep_rows_kernel(const T* __restrict__ proj, T* __restrict__ q, T* __restrict__ cache, const int* __restrict__ loc,
+                      const RowPrepParams r) {
+  __shared__ float red[2][kRowThreads / 32];
+  const PrepParams& p = r.b;
+  pdl_wait();
+  const long long t = blockIdx.x;
+  const int tid = threadIdx.x;
+  const T* row = proj + t * p.ld;
+  float sq = 0.f, sk = 0.f;
+  if (r.sq != nullptr) {
+    sq = r.sq[2 * t];
+    sk = r.sq[2 * t + 1];
+  } else {
+    auto squares = [&](const T* src, int n) {
+      float a = 0.f;
+      for (int i = tid * VEC; i < n; i += kRowThreads * VEC) {
+        const Pack<T, VEC> v = *reinterpret_cast<const Pack<T, VEC>*>(src + i);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) a += to_f(v.v[e]) * to_f(v.v[e]);
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) a += __shfl_xor_sync(0xffffffffu, a, o);
+      return a;
+    };
+    const float a = squares(row + p.q_off, p.H * p.D), b = squares(row + p.k_off, p.G * p.D);
+    if ((tid & 31) == 0) {
+      red[0][tid >> 5] = a;
+      red[1][tid >> 5] = b;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < kRowThreads / 32; ++i) {
+      sq += red[0][i];
+      sk += red[1][i];
+    }
+  }
+  const float iq = 1.f / sqrtf(sq / r.nq + p.eps), ik = 1.f / sqrtf(sk / r.nk + p.eps);
+  // n heads of `width` values each to rows of `padded`, the rest of a row zero
+  auto write = [&](const T* src, const float* w, float inv, const T* mix, float share, int n, int width, int padded, T* dst,
+                   long long stride) {
+    for (int i = tid * VEC; i < n * padded; i += kRowThreads * VEC) {
+      const int h = i / padded, c = i - h * padded;
+      Pack<T, VEC> a;
+      if (c < width) {
+        a = *reinterpret_cast<const Pack<T, VEC>*>(src + h * width + c);
+        if (w != nullptr) {
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) a.v[e] = from_f<T>(to_f(a.v[e]) * inv * w[h * width + c + e]);
+        } else if (mix != nullptr) {
+          const Pack<T, VEC> m = *reinterpret_cast<const Pack<T, VEC>*>(mix + h * width + c);
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) a.v[e] = from_f<T>((1.f - share) * to_f(a.v[e]) + share * to_f(m.v[e]));
+        }
+      } else {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) a.v[e] = from_f<T>(0.f);
+      }
+      *reinterpret_cast<Pack<T, VEC>*>(dst + h * stride + c) = a;
+    }
+  };
+  const int slot = loc[t], page = slot / p.P;
+  const long long width = p.Dp + p.Vp, head = width * p.P;       // cache row, and from one head's rows to the next one's
+  T* dst = cache + static_cast<long long>(page) * p.G * head + (slot - page * p.P) * width;
+  write(row + p.q_off, r.q_w, iq, nullptr, 0.f, p.H, p.D, p.Dp, q + t * p.H * p.Dp, p.Dp);
+  write(row + p.k_off, r.k_w, ik, nullptr, 0.f, p.G, p.D, p.Dp, dst, head);
+  const T* mix = r.v_mix != nullptr ? static_cast<const T*>(r.v_mix) + t * r.v_mix_ld : nullptr;
+  write(row + p.v_off, nullptr, 0.f, mix, mix != nullptr ? *r.share : 0.f, p.G, p.V, p.Vp, dst + p.Dp, head);
+}
+
 // ------------------------------------------------------------------------------------------- decode
 constexpr int kTile = 64;                    // keys per tile
 constexpr int kConsumers = 4;                // warps, 16 keys of a tile each
@@ -106,7 +191,8 @@ struct DecodeParams {
   Status* status;
   int H, G, Dp, V, max_pages, page_size, splits, m_blocks;
   Window win;
-  float scale_log2;
+  ScoreTerms terms;
+  float scale_log2, scale;
 };
 
 __device__ __forceinline__ void ldsm_x4(uint32_t addr, uint32_t (&r)[4]) {
@@ -158,6 +244,8 @@ window_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
   const int pos = p.lens[n] - 1;
   const int* pt = p.page_table + static_cast<size_t>(p.rows[n]) * p.max_pages;
   const int lo = p.win.first(pos);
+  const bool shaped = p.terms.shaped();
+  const float inv_cap = p.terms.cap > 0.f ? 1.f / p.terms.cap : 0.f;
   const KeyTiles<kTile> tiles(p.win, pos, pos);
   const int per = (tiles.count + p.splits - 1) / p.splits, i0 = split * per, i1 = min(i0 + per, tiles.count);
   __syncthreads();
@@ -207,6 +295,7 @@ window_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
       qf[kk][2] = gr < nh && c + 8 < p.Dp ? *reinterpret_cast<const uint32_t*>(qa + c + 8) : 0u;
       qf[kk][3] = gr + 8 < nh && c + 8 < p.Dp ? *reinterpret_cast<const uint32_t*>(qb + c + 8) : 0u;
     }
+    const float slope[2] = {gr < nh ? p.terms.slope_of(h0 + gr) : 0.f, gr + 8 < nh ? p.terms.slope_of(h0 + gr + 8) : 0.f};
     for (int i = i0, c = 0; i < i1 && !*abort_flag; ++i, ++c) {
       const int st = c % kStages;
       if (!mbar_wait(smem_u32(&full_bar[st]), (c / kStages) & 1)) {
@@ -234,7 +323,15 @@ window_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             const int key = tok0 + j * 8 + t4 * 2 + (e & 1);
-            s[j][e] = key <= pos && (key >= lo || key < p.win.keep) ? s[j][e] * p.scale_log2 : -INFINITY;
+            float a;
+            if (shaped) {
+              a = s[j][e] * p.scale;
+              if (inv_cap > 0.f) a = p.terms.cap * tanh_by_exp(a * inv_cap);
+              a = (a - slope[e >> 1] * static_cast<float>(pos - key)) * kLog2E;
+            } else {
+              a = s[j][e] * p.scale_log2;
+            }
+            s[j][e] = key <= pos && (key >= lo || key < p.win.keep) ? a : -INFINITY;
             mx[e >> 1] = fmaxf(mx[e >> 1], s[j][e]);
           }
         float corr[2], ref[2], sum[2] = {0.f, 0.f};
@@ -315,7 +412,9 @@ window_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
     float mm = -INFINITY;
 #pragma unroll
     for (int w = 0; w < kConsumers; ++w) mm = fmaxf(mm, m_s[w * 16 + r]);
-    float ls = 0.f, acc = 0.f;
+    const float sink = p.splits == 1 ? p.terms.sink_log2(h0 + r) : -INFINITY;    // (several splits: in the combine step)
+    mm = fmaxf(mm, sink);
+    float ls = sink == -INFINITY ? 0.f : exp2f(sink - mm), acc = 0.f;
 #pragma unroll
     for (int w = 0; w < kConsumers; ++w) {
       const float f = m_s[w * 16 + r] == -INFINITY ? 0.f : exp2f(m_s[w * 16 + r] - mm);
@@ -339,7 +438,9 @@ __global__ void window_combine_kernel(const DecodeParams p) {
   const float* lse = p.part_lse + row * p.splits;
   float mm = -INFINITY;
   for (int s = 0; s < p.splits; ++s) mm = fmaxf(mm, lse[s]);
-  float ws = 0.f;
+  const float sink = p.terms.sink_log2(static_cast<int>(row % p.H));
+  mm = fmaxf(mm, sink);
+  float ws = sink == -INFINITY ? 0.f : exp2f(sink - mm);
   for (int s = 0; s < p.splits; ++s) ws += lse[s] == -INFINITY ? 0.f : exp2f(lse[s] - mm);
   const float f = (ws > 0.f ? 1.f / ws : 0.f) * gate_of(p.gate, p.gate_ld, row / p.H, static_cast<int>(row % p.H));
   for (int d = threadIdx.x; d < p.V; d += blockDim.x) {
@@ -387,6 +488,7 @@ struct AnyParams {
   const int *page_table, *rows, *lens;
   int H, G, D, V, Dp, Vp, max_pages, page_size;
   Window win;
+  ScoreTerms terms;
   float scale;
 };
 
@@ -408,6 +510,7 @@ window_attn_any_kernel(const T* __restrict__ q, const T* __restrict__ gate, cons
 #pragma unroll
   for (int i = 0; i < kAnyMaxAcc; ++i) acc[i] = 0.f;
   float m = -INFINITY, l = 0.f;
+  const float slope = p.terms.slope_of(h);
   const KeyTiles<kTile> tiles(p.win, pos, pos);
   for (int t = 0; t < tiles.count; ++t) {
     const int k0 = tiles.tile(t) * kTile, nk = min(kTile, pos + 1 - k0);
@@ -423,7 +526,7 @@ window_attn_any_kernel(const T* __restrict__ q, const T* __restrict__ gate, cons
       for (int i = lane; i < p.D; i += 32) a += qs[i] * to_f(kr[i]);
 #pragma unroll
       for (int o = 16; o > 0; o >>= 1) a += __shfl_xor_sync(0xffffffffu, a, o);
-      if (lane == 0) sc[j] = p.win.sees(pos, k0 + j) ? a * p.scale : -INFINITY;
+      if (lane == 0) sc[j] = p.win.sees(pos, k0 + j) ? p.terms.apply(a * p.scale, slope, pos - k0 - j) : -INFINITY;
     }
     __syncthreads();
     float mx = m;
@@ -445,7 +548,13 @@ window_attn_any_kernel(const T* __restrict__ q, const T* __restrict__ gate, cons
     }
     m = mx;
   }
-  float f = l > 0.f ? 1.f / l : 0.f;
+  float f = 0.f;
+  if (p.terms.sink != nullptr) {
+    const float sink = p.terms.sink[h], mx = fmaxf(m, sink), c = expf(m - mx);
+    f = c / (l * c + expf(sink - mx));
+  } else if (l > 0.f) {
+    f = 1.f / l;
+  }
   if (gate != nullptr) f *= 1.f / (1.f + expf(-to_f(gate[n * p.gate_ld + h])));
 #pragma unroll
   for (int i = 0; i < kAnyMaxAcc; ++i) {
@@ -464,6 +573,19 @@ int prep(const void* proj, void* q, void* cache, const int* loc, long long token
   const auto kernel = vec ? attn_prep_kernel<T, 4> : attn_prep_kernel<T, 1>;
   launch_pdl(kernel, grid, dim3(128), 0, s, static_cast<const T*>(proj), static_cast<T*>(q), static_cast<T*>(cache), loc,
              tokens, p);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T>
+int prep_rows(const void* proj, void* q, void* cache, const int* loc, long long tokens, const RowPrepParams& r,
+              cudaStream_t s) {
+  const PrepParams& p = r.b;
+  const bool vec = p.D % 4 == 0 && p.V % 4 == 0 && p.ld % 4 == 0 && p.q_off % 4 == 0 && p.k_off % 4 == 0 &&
+                   p.v_off % 4 == 0 && r.v_mix_ld % 4 == 0 && reinterpret_cast<uintptr_t>(proj) % (4 * sizeof(T)) == 0 &&
+                   reinterpret_cast<uintptr_t>(r.v_mix) % (4 * sizeof(T)) == 0;
+  const auto kernel = vec ? attn_prep_rows_kernel<T, 4> : attn_prep_rows_kernel<T, 1>;
+  launch_pdl(kernel, dim3(static_cast<unsigned>(tokens)), dim3(kRowThreads), 0, s, static_cast<const T*>(proj),
+             static_cast<T*>(q), static_cast<T*>(cache), loc, r);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -492,6 +614,23 @@ int sglb_attn_prep(const void* proj, long long ld, int q_off, int k_off, int v_o
   return is_f32 ? prep<float>(proj, q, cache, loc, T, p, s) : prep<__nv_bfloat16>(proj, q, cache, loc, T, p, s);
 }
 
+// The same with norms over all H * D query and all G * D key values of a token (weights q_w [H * D], k_w [G * D]); the means
+// are over nq and nk values, whose sums of squares are sq [T, 2] where this rank holds only a part of them (else null).
+// v_mix (or null): rows of G * V values, by v_mix_ld, that replace `share` of the layer's own.
+int sglb_attn_prep_rows(const void* proj, long long ld, int q_off, int k_off, int v_off, void* q, void* cache,
+                        const int* loc, long long T, int H, int G, int D, int V, int P, const float* q_w, const float* k_w,
+                        const float* sq, int nq, int nk, float eps, const void* v_mix, long long v_mix_ld,
+                        const float* share, int is_f32, cudaStream_t s) {
+  using namespace sglb;
+  if (T <= 0) return 0;
+  if (H < 1 || G < 1 || D < 1 || P < 1 || nq < 1 || nk < 1 || q_w == nullptr || k_w == nullptr || k_off < 0 ||
+      (v_mix != nullptr && share == nullptr))
+    return -kBadArgument;
+  const RowPrepParams r{{ld, q_off, k_off, v_off, H, G, D, V, pad8(D), pad8(V), P, 1, eps}, q_w, k_w, sq, nq, nk, v_mix,
+                        v_mix_ld, share};
+  return is_f32 ? prep_rows<float>(proj, q, cache, loc, T, r, s) : prep_rows<__nv_bfloat16>(proj, q, cache, loc, T, r, s);
+}
+
 // Whether window_decode takes these sizes.
 int sglb_window_decode_supported(int D, int V, int page_size) {
   return D > 0 && V > 0 && D <= 256 && V <= 256 && (page_size < 64 ? page_size >= 8 && 64 % page_size == 0 : page_size % 64 == 0);
@@ -504,11 +643,12 @@ int sglb_window_num_splits(int N, int groups, int visible) {
   return splits < 1 ? 1 : (splits > 32 ? 32 : splits);
 }
 
-// Query n sees, of the first lens[n] tokens of table row rows[n], the last `window` (0: all) and the first `keep`.
+// Query n sees, of the first lens[n] tokens of table row rows[n], the last `window` (0: all) and the first `keep`.  softcap (0:
+// none), slope and sink ([H] or null): score_terms.cuh.
 int sglb_window_decode(const void* q, const void* gate, long long gate_ld, const void* cache, long long num_pages,
                        const int* page_table, int max_pages, int page_size, const int* rows, const int* lens, void* out,
-                       int N, int H, int G, int D, int V, float scale, int window, int keep, int splits, float* part_o,
-                       float* part_lse, cudaStream_t s) {
+                       int N, int H, int G, int D, int V, float scale, int window, int keep, float softcap,
+                       const float* slope, const float* sink, int splits, float* part_o, float* part_lse, cudaStream_t s) {
   using namespace sglb;
   if (N <= 0) return 0;
   if (!sglb_window_decode_supported(D, V, page_size) || H % G != 0 || (splits > 1 && (!part_o || !part_lse)))
@@ -536,7 +676,9 @@ int sglb_window_decode(const void* q, const void* gate, long long gate_ld, const
   p.m_blocks = (H / G + 15) / 16;
   if (static_cast<long long>(G) * p.m_blocks > 65535) return -kBadArgument;
   p.win = Window{window, keep};
-  p.scale_log2 = scale * kLog2e;
+  p.terms = ScoreTerms{softcap, slope, sink};
+  p.scale = scale;
+  p.scale_log2 = scale * kLog2E;
   const int nv = (Vp + 63) / 64;
   switch ((Dp + 63) / 64) {
     case 1: return launch_decode_v<1>(nv, mk, mv, p, N, s);
@@ -548,12 +690,13 @@ int sglb_window_decode(const void* q, const void* gate, long long gate_ld, const
 
 int sglb_window_attn_any(const void* q, const void* gate, long long gate_ld, const void* cache, const int* page_table,
                          int max_pages, int page_size, const int* rows, const int* lens, void* out, int N, int H, int G,
-                         int D, int V, float scale, int window, int keep, int is_f32, cudaStream_t s) {
+                         int D, int V, float scale, int window, int keep, float softcap, const float* slope,
+                         const float* sink, int is_f32, cudaStream_t s) {
   using namespace sglb;
   if (N <= 0) return 0;
   if (V > kAnyMaxAcc * kAnyThreads || D > 8192 || H > 65535 || H % G != 0) return -kBadArgument;
   const AnyParams p{gate_ld, page_table, rows, lens, H, G, D, V, pad8(D), pad8(V), max_pages, page_size,
-                    Window{window, keep}, scale};
+                    Window{window, keep}, ScoreTerms{softcap, slope, sink}, scale};
   return is_f32 ? attn_any<float>(q, gate, cache, out, N, p, s) : attn_any<__nv_bfloat16>(q, gate, cache, out, N, p, s);
 }
 

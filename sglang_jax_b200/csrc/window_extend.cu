@@ -13,11 +13,13 @@
 //
 // While one tile's exponentials run, the tensor pipe works on the other tile.  The running maximum is only raised when it
 // grows by more than 2^8.  Lanes past the widths arrive as zeros and whole zero steps are skipped.  The result is
-// multiplied by sigmoid(gate) per head, if there is one.  All waits are bounded; a timeout unwinds through the normal
+// multiplied by sigmoid(gate) per head, if there is one.  Scores may be capped, biased by distance and joined by a sink
+// (score_terms.cuh).  All waits are bounded; a timeout unwinds through the normal
 // teardown.  No multicast.
 #include <math.h>
 
 #include "common.cuh"
+#include "score_terms.cuh"
 #include "window_mask.cuh"
 
 namespace sglb {
@@ -30,7 +32,6 @@ constexpr int kThreads = 64 + kTiles * 128;
 constexpr int kTmemCols = 512;                      // per tile: S 2 x 64 (P in place), O 128
 constexpr int kTmemTile = 256, kTmemO = 128;
 constexpr float kRescale = 8.f;
-constexpr float kLog2e = 1.4426950408889634f;
 constexpr int kMinSmem = 120 * 1024;                // one CTA per SM: it takes all of tensor memory
 
 struct Bars {
@@ -50,16 +51,8 @@ struct Params {
   int B, H, G, Dp, V, max_pages, page_size;
   int nb_k, nb_v;                // 64-lane blocks of a key / value
   Window win;
-  float scale_log2;
-};
-
-// The key tiles of one CTA, and of each of its query tiles.  Tiles are numbered as KeyTiles orders them.  Query tile t
-// leaves out [gap, gap + skip) and everything from n on; local(j) counts the tiles it takes.
-struct QueryTile {
-  int n, gap, skip;
-  __device__ __forceinline__ bool takes(int j) const { return j < n && (j < gap || j >= gap + skip); }
-  __device__ __forceinline__ int local(int j) const { return j < gap ? j : j - skip; }
-  __device__ __forceinline__ int count() const { return n > 0 ? n - skip : 0; }
+  ScoreTerms terms;
+  float scale_log2, cap_arg, cap_log2;   // scale log2 e; 2 scale log2 e / cap and cap log2 e
 };
 
 __device__ __forceinline__ float ex2_approx(float x) {
@@ -68,6 +61,15 @@ __device__ __forceinline__ float ex2_approx(float x) {
   return y;
 }
 
+// cap tanh(s scale / cap) + bias in log2 units: c2 = cap log2 e, a = 2 scale log2 e / cap
+__device__ __forceinline__ float capped(float s, float a, float c2, float bias) {
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + ex2_approx(fminf(s * a, 60.f))));
+  return fmaf(-2.f * c2, r, c2 + bias);
+}
+
+// SHAPED: scores are capped or biased
+template <bool SHAPED>
 __global__ void __launch_bounds__(kThreads, 1)
 window_extend_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                      const __grid_constant__ CUtensorMap map_v, const Params p) {
@@ -103,21 +105,9 @@ window_extend_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
   const int* pt_row = p.page_table + static_cast<size_t>(p.rows[b]) * p.max_pages;
   const KeyTiles<kTileK> keys(p.win, prefix + q0, prefix + min(q0 + kTiles * kTileQ, q_len) - 1);
   QueryTile qt[kTiles];
-  {
-    // tiles of kept tokens reach this far; beyond, a query tile starts at its own window
-    const int kept_end = keys.kept + max(0, (p.win.keep + kTileK - 1) / kTileK - keys.begin);
 #pragma unroll
-    for (int t = 0; t < kTiles; ++t) {
-      const int first = q0 + t * kTileQ;
-      if (first >= q_len) {
-        qt[t] = {0, 0, 0};
-        continue;
-      }
-      const int own = keys.kept + p.win.first(prefix + first) / kTileK - keys.begin;
-      qt[t] = {keys.kept + (prefix + min(first + kTileQ, q_len) - 1) / kTileK + 1 - keys.begin, kept_end,
-               max(0, own - kept_end)};
-    }
-  }
+  for (int t = 0; t < kTiles; ++t)
+    qt[t] = query_tile(p.win, keys, prefix + q0 + t * kTileQ, prefix + min(q0 + (t + 1) * kTileQ, q_len) - 1);
   const int n = max(qt[0].n, qt[1].n);
 
   if (threadIdx.x == 0) {
@@ -260,7 +250,8 @@ window_extend_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
     const int r_seq = q0 + t * kTileQ + row;                        // row within the sequence's new tokens
     const int pos = min(prefix + r_seq, seq - 1);                   // rows past the end: anything finite
     const int kmin = p.win.first(pos);
-    const float scale_log2 = p.scale_log2;
+    const float scale_log2 = SHAPED ? 1.f : p.scale_log2;
+    const float slope = SHAPED ? p.terms.slope_of(head) * kLog2E : 0.f;
     const int nt = qt[t].count();
     float m_used = -INFINITY, l = 0.f;
     bool ok = nt > 0;
@@ -285,6 +276,22 @@ window_extend_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
       auto below = [](int c) -> uint64_t { return c <= 0 ? 0ull : (c >= 64 ? ~0ull : (1ull << c) - 1); };
       const uint64_t seen = below(pos - k0 + 1) & (~below(kmin - k0) | below(p.win.keep - k0));
       const bool full = seen == ~0ull;
+      if constexpr (SHAPED) {                                       // capped and biased scores, in log2 units
+        const float base = slope * static_cast<float>(k0 - pos);
+        if (p.terms.cap > 0.f) {
+#pragma unroll
+          for (int e = 0; e < 32; ++e) {
+            v0[e] = __float_as_uint(capped(__uint_as_float(v0[e]), p.cap_arg, p.cap_log2, fmaf(slope, e, base)));
+            v1[e] = __float_as_uint(capped(__uint_as_float(v1[e]), p.cap_arg, p.cap_log2, fmaf(slope, e + 32, base)));
+          }
+        } else {
+#pragma unroll
+          for (int e = 0; e < 32; ++e) {
+            v0[e] = __float_as_uint(fmaf(__uint_as_float(v0[e]), p.scale_log2, fmaf(slope, e, base)));
+            v1[e] = __float_as_uint(fmaf(__uint_as_float(v1[e]), p.scale_log2, fmaf(slope, e + 32, base)));
+          }
+        }
+      }
       const uint32_t see0 = static_cast<uint32_t>(seen), see1 = static_cast<uint32_t>(seen >> 32);
       float mx = -INFINITY;
       if (full) {
@@ -358,6 +365,7 @@ window_extend_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
       } else {
         tc_fence_after_sync();
         const long long tok = p.q_start[b] + r_seq;
+        if (p.terms.sink != nullptr) l += exp2f(p.terms.sink_log2(head) - m_used);
         float inv = l > 0.f ? 1.f / l : 0.f;
         if (p.gate != nullptr && r_seq < q_len)
           inv *= 1.f / (1.f + expf(-__bfloat162float(p.gate[tok * p.gate_ld + head])));
@@ -409,6 +417,19 @@ int extend_smem(int nb_k, int nb_v) {
 
 int pad8(int n) { return (n + 7) / 8 * 8; }
 
+template <bool SHAPED>
+int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const Params& p, dim3 grid, int smem,
+           cudaStream_t stream) {
+  static int cfg = 0;
+  if (cfg < smem) {
+    const cudaError_t e = cudaFuncSetAttribute(window_extend_kernel<SHAPED>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    cfg = smem;
+  }
+  window_extend_kernel<SHAPED><<<grid, kThreads, smem, stream>>>(mq, mk, mv, p);
+  return static_cast<int>(cudaGetLastError());
+}
+
 }  // namespace
 }  // namespace sglb
 
@@ -422,10 +443,12 @@ int sglb_window_extend_supported(int D, int V, int page_size) {
 
 // q [total_q, H, pad8(D)]; cache [num_pages, G, page_size, pad8(D) + pad8(V)]; out [total_q, H, V].  B sequences: rows
 // q_start .. q_start + q_len of q, `prefix` tokens before them, page-table row `rows`.  num_tiles = sum_b ceil(q_len / 256).
+// softcap (0: none), slope and sink ([H] or null): score_terms.cuh.
 int sglb_window_extend(const void* q, int total_q, const void* gate, long long gate_ld, const void* cache,
                        long long num_pages, const int* page_table, int max_pages, int page_size, const int* rows,
                        const int* q_start, const int* q_len, const int* prefix, int B, int num_tiles, void* out, int H,
-                       int G, int D, int V, float scale, int window, int keep, cudaStream_t stream) {
+                       int G, int D, int V, float scale, int window, int keep, float softcap, const float* slope,
+                       const float* sink, cudaStream_t stream) {
   using namespace sglb;
   if (B <= 0 || num_tiles <= 0 || total_q <= 0) return 0;
   if (!sglb_window_extend_supported(D, V, page_size) || H < 1 || H > 65535 || H % G != 0) return -kBadArgument;
@@ -451,16 +474,14 @@ int sglb_window_extend(const void* q, int total_q, const void* gate, long long g
   p.nb_k = (Dp + 63) / 64;
   p.nb_v = (Vp + 63) / 64;
   p.win = Window{window, keep};
-  p.scale_log2 = scale * kLog2e;
+  p.terms = ScoreTerms{softcap, slope, sink};
+  p.scale_log2 = scale * kLog2E;
+  p.cap_arg = softcap > 0.f ? 2.f * kLog2E * scale / softcap : 0.f;
+  p.cap_log2 = softcap * kLog2E;
   const int smem = extend_smem(p.nb_k, p.nb_v);
-  static int cfg = 0;
-  if (cfg < smem) {
-    const cudaError_t e = cudaFuncSetAttribute(window_extend_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-    if (e != cudaSuccess) return static_cast<int>(e);
-    cfg = smem;
-  }
-  window_extend_kernel<<<dim3(num_tiles, H), kThreads, smem, stream>>>(mq, mk, mv, p);
-  return static_cast<int>(cudaGetLastError());
+  const dim3 grid(num_tiles, H);
+  return softcap > 0.f || slope != nullptr ? launch<true>(mq, mk, mv, p, grid, smem, stream)
+                                           : launch<false>(mq, mk, mv, p, grid, smem, stream);
 }
 
 }  // extern "C"

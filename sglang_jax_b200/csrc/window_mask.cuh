@@ -24,4 +24,23 @@ struct KeyTiles {
   __device__ __forceinline__ int tile(int i) const { return i < kept ? i : begin + (i - kept); }
 };
 
+// What one of several query tiles takes of the key tiles that a CTA walks for all of them (numbered as KeyTiles orders them):
+// it leaves out [gap, gap + skip) and everything from n on; local(j) counts the tiles it takes.
+struct QueryTile {
+  int n, gap, skip;
+  __device__ __forceinline__ bool takes(int j) const { return j < n && (j < gap || j >= gap + skip); }
+  __device__ __forceinline__ int local(int j) const { return j < gap ? j : j - skip; }
+  __device__ __forceinline__ int count() const { return n > 0 ? n - skip : 0; }
+};
+
+// The query tile with positions lo .. hi; lo > hi: none.
+template <int TILE>
+__device__ __forceinline__ QueryTile query_tile(const Window& w, const KeyTiles<TILE>& keys, int lo, int hi) {
+  if (lo > hi) return {0, 0, 0};
+  // tiles of kept tokens reach this far; beyond, the query tile starts at its own window
+  const int kept_end = keys.kept + max(0, (w.keep + TILE - 1) / TILE - keys.begin);
+  const int own = keys.kept + w.first(lo) / TILE - keys.begin;
+  return {keys.kept + hi / TILE + 1 - keys.begin, kept_end, max(0, own - kept_end)};
+}
+
 }  // namespace sglb

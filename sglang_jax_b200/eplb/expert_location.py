@@ -169,7 +169,8 @@ class ExpertDistributionRecorder:
         ids = topk_ids.reshape(-1).long()
         if ids.device != self.counts.device:
             ids = ids.to(self.counts.device)
-        self.counts[layer_id].scatter_add_(0, ids.clamp_(0, self.counts.shape[1] - 1), torch.ones_like(ids))
+        hit = (ids >= 0).to(self.counts.dtype)             # negative: a choice without an expert
+        self.counts[layer_id].scatter_add_(0, ids.clamp_(0, self.counts.shape[1] - 1), hit)
 
     def step(self):
         self.forwards += 1

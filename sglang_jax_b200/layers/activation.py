@@ -9,6 +9,13 @@ class SiluAndMul(nn.Module):
         return ops.silu_and_mul(x)
 
 
+class SwiGLU(nn.Module):
+    """As `SiluAndMul` for every width, in bf16 and fp32."""
+
+    def forward(self, x):
+        return ops.swiglu(x)
+
+
 class GeluAndMul(nn.Module):
     def __init__(self, approximate="tanh"):
         super().__init__()

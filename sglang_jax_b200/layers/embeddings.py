@@ -58,6 +58,25 @@ class VocabParallelEmbedding(nn.Module):
         return out if out.dtype == self.out_dtype else out.to(self.out_dtype)
 
 
+class PairEmbedding(nn.Module):
+    """Adds to a token's embedding a row of a second table, chosen by a hash of the token and its predecessor: row
+    `(previous * mul_prev + token * mul_cur) mod buckets`, and the last row for a sequence's first token.  The predecessor of a
+    portion's first token comes out of the KV pool, which keeps every slot's token id (`PackedKVPool(token_ids=True)`), so
+    portions, decoding, shared prefixes and moved pages need nothing else.  Replicated over tensor ranks."""
+
+    def __init__(self, buckets: int, embedding_dim: int, mul_prev: int, mul_cur: int, dtype=torch.bfloat16):
+        super().__init__()
+        self.mul_prev, self.mul_cur = int(mul_prev), int(mul_cur)
+        self.weight = nn.Parameter(torch.zeros(buckets + 1, embedding_dim, dtype=dtype), requires_grad=False)
+
+    def weight_loader(self, param, w, shard_id=None):
+        param.data.copy_(w)
+
+    def forward(self, ids, embed: "VocabParallelEmbedding", fb):
+        """`(fp32 sum, the same in the table's type)`."""
+        return ops.embed_pair(ids, embed.weight, self.weight, self.mul_prev, self.mul_cur, fb.token_to_kv_pool.token_ids, fb)
+
+
 class ParallelLMHead(nn.Module):
     """Vocab-parallel output projection; each rank holds `[vocab/tp, hidden]`."""
 

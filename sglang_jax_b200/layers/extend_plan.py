@@ -2,6 +2,8 @@
 
 from __future__ import annotations
 
+from typing import NamedTuple
+
 import numpy as np
 import torch
 
@@ -9,6 +11,16 @@ import torch
 MIN_TILE_TOKENS = 32
 # query rows per CTA of the prefill kernels (`csrc/latent_extend.cu`, `csrc/window_extend.cu`)
 TILE_ROWS = 256
+# keys per tile of the prefill kernels
+KEY_TILE = 64
+
+
+class Context(NamedTuple):
+    """The tokens that the long sequences of a step attend to, laid end to end: first row of each (and the end), how many of a
+    sequence's tokens are left out in front (None: of none), rows in all."""
+    start: torch.Tensor
+    skip: torch.Tensor | None
+    total: int
 
 
 class ExtendPlan:
@@ -28,14 +40,12 @@ class ExtendPlan:
         self.token_lens = fb.positions + 1
         self.short_tokens = None
         if self.long:
-            ctx = (pre + n)[long]
-            ctx_start = np.concatenate([[0], np.cumsum(ctx)])
-            self.ctx_total = int(ctx_start[-1])
+            self._prefix, self._end, self._contexts = pre[long], (pre + n)[long], {}
             self.num_tiles = int(((n[long] + TILE_ROWS - 1) // TILE_ROWS).sum())
             rows = fb.req_pool_indices[torch.from_numpy(long).to(dev)]
-            meta = torch.from_numpy(np.concatenate([start[long], n[long], pre[long], ctx_start]).astype(np.int32)).to(dev)
+            meta = torch.from_numpy(np.concatenate([start[long], n[long], pre[long]]).astype(np.int32)).to(dev)
             L = self.long
-            self.q_start, self.q_len, self.prefix, self.ctx_start = meta[:L], meta[L:2 * L], meta[2 * L:3 * L], meta[3 * L:]
+            self.q_start, self.q_len, self.prefix = meta[:L], meta[L:2 * L], meta[2 * L:]
             self.rows = rows
             if L < len(n):
                 keep = np.ones(len(n), bool)
@@ -43,6 +53,16 @@ class ExtendPlan:
                 short = np.concatenate([np.arange(start[i], start[i] + n[i]) for i in np.nonzero(keep)[0]])
                 if len(short):
                     self.short_tokens = torch.from_numpy(short).to(dev)
+
+
+    def context(self, window: int = 0) -> Context:
+        """What the long sequences see under a window (0: everything), from a multiple of `KEY_TILE` on."""
+        if window not in self._contexts:
+            skip = np.maximum(self._prefix - window + 1, 0) // KEY_TILE * KEY_TILE if window else np.zeros_like(self._prefix)
+            start = np.concatenate([[0], np.cumsum(self._end - skip)])
+            meta = torch.from_numpy(np.concatenate([start, skip]).astype(np.int32)).to(self.rows.device)
+            self._contexts[window] = Context(meta[:len(start)], meta[len(start):] if skip.any() else None, int(start[-1]))
+        return self._contexts[window]
 
 
 def extend_plan(fb, tiles: bool) -> ExtendPlan:

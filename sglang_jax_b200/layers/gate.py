@@ -16,9 +16,11 @@ class GateLogit(nn.Module):
     rounding); the optional selection bias (`e_score_correction_bias`) lives here too."""
 
     def __init__(self, hidden_size: int, num_experts: int, dtype=torch.bfloat16, use_bias: bool = False,
-                 score_func: str = "softmax", correction_bias: bool = False):
+                 score_func: str = "softmax", correction_bias: bool = False, token_gate: bool = False):
+        """`token_gate`: one more row behind the experts', whose product gates something per token (`route_by_score`)."""
         super().__init__()
-        self.weight = nn.Parameter(torch.empty(num_experts, hidden_size, dtype=dtype), requires_grad=False)
+        self.token_gate = token_gate
+        self.weight = nn.Parameter(torch.empty(num_experts + token_gate, hidden_size, dtype=dtype), requires_grad=False)
         self.bias = nn.Parameter(torch.zeros(num_experts, dtype=dtype), requires_grad=False) if use_bias else None
         self.e_score_correction_bias = nn.Parameter(torch.zeros(num_experts, dtype=torch.float32),
                                                     requires_grad=False) if correction_bias else None
@@ -34,6 +36,12 @@ class GateLogit(nn.Module):
         """The experts with the largest logits, weights the softmax over the chosen logits only: `(weights fp32, ids int32)`,
         `[T, top_k]` each."""
         return ops.route_by_logit(x, self.weight, self.bias, top_k)
+
+
+    def route_by_score(self, x: torch.Tensor, top_k: int, scale: float):
+        """The experts with the largest corrected softmax scores, weights their scores times `scale`, not renormalised: `(weights
+        fp32, ids int32, gate)`; `gate` fp32 `[T]`: sigmoid of the gate row's product, or None."""
+        return ops.route_by_score(x, self.weight, self.e_score_correction_bias, top_k, scale, self.token_gate)
 
 
 class TopK(nn.Module):

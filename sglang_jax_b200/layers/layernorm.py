@@ -98,18 +98,46 @@ class PostNormResidual(nn.Module):
         return ops.postnorm_add_norm(y, x, self.channel_scale, self.eps, norm.channel_scale, norm.eps)
 
 
+class SumNorm(nn.Module):
+    """`x <- rms-normalised (alpha x + layer_scale * y) * (1 + weight)` on an fp32 residual stream, y a sublayer's output: the
+    norm sits behind the sum, its weight is stored around zero.  Returns x in y's type, the input of the next projections, or
+    with `then` that norm of x."""
+
+    def __init__(self, hidden_size: int, eps: float, alpha: float, dtype=torch.bfloat16):
+        super().__init__()
+        self.weight = nn.Parameter(torch.zeros(hidden_size, dtype=dtype), requires_grad=False)
+        self.layer_scale = nn.Parameter(torch.ones(hidden_size, dtype=dtype), requires_grad=False)
+        self.eps, self.alpha = float(eps), float(alpha)
+        for name in ("sum_scale", "norm_scale"):
+            self.register_buffer(name, torch.ones(hidden_size, dtype=torch.float32), persistent=False)
+
+    def fold(self):
+        self.sum_scale.copy_(self.layer_scale.float())
+        self.norm_scale.copy_(1 + self.weight.float())
+
+    def weight_loader(self, param, w, shard_id=None):
+        param.data.copy_(w)
+
+    def forward(self, y: torch.Tensor, x: torch.Tensor, then: "StreamRMSNorm | None" = None, **parts) -> torch.Tensor:
+        """`parts`: what joins y in the sum (`ops.sum_norm`)."""
+        if then is not None:
+            parts.update(next_weight=then.channel_scale, next_eps=then.eps)
+        return ops.sum_norm(y, x, self.alpha, self.sum_scale, self.norm_scale, self.eps, **parts)
+
+
 class StreamRMSNorm(nn.Module):
     """RMSNorm of an fp32 residual stream, result in the model's type.  `multiplier` scales the result (a logit scale
-    in front of a linear head)."""
+    in front of a linear head); `one_plus`: the weight is stored around zero."""
 
-    def __init__(self, hidden_size: int, eps: float, multiplier: float = 1.0, dtype=torch.bfloat16):
+    def __init__(self, hidden_size: int, eps: float, multiplier: float = 1.0, dtype=torch.bfloat16, one_plus: bool = False):
         super().__init__()
-        self.weight = nn.Parameter(torch.ones(hidden_size, dtype=dtype), requires_grad=False)
-        self.eps, self.multiplier = eps, multiplier
+        fill = torch.zeros if one_plus else torch.ones
+        self.weight = nn.Parameter(fill(hidden_size, dtype=dtype), requires_grad=False)
+        self.eps, self.multiplier, self.one_plus = eps, multiplier, one_plus
         self.register_buffer("channel_scale", torch.ones(hidden_size, dtype=torch.float32), persistent=False)
 
     def fold(self):
-        self.channel_scale.copy_(self.weight.float() * self.multiplier)
+        self.channel_scale.copy_((self.weight.float() + int(self.one_plus)) * self.multiplier)
 
     def weight_loader(self, param, w, shard_id=None):
         param.data.copy_(w)

@@ -76,11 +76,12 @@ class FusedMoE(nn.Module):
     def __init__(self, num_experts: int, hidden_size: int, intermediate_size: int, dtype=torch.bfloat16,
                  ep_size: int | None = None, tp_size=None, tp_rank=None, layer_id: int = 0,
                  activation: str = "silu", act_limit: float = 0.0, act_alpha: float = 1.702):
-        """`activation`: "silu", "gelu", or "clipped_swiglu" with its `act_limit` and `act_alpha`
-        (`ops.clipped_swiglu`)."""
+        """`activation`: "silu", "gelu", "swiglu" (SiLU for every width, bf16 and fp32), or "clipped_swiglu" with its `act_limit`
+        and `act_alpha` (`ops.clipped_swiglu`)."""
         super().__init__()
         self.activation = activation
         self.act_limit, self.act_alpha = float(act_limit), float(act_alpha)
+        self.extra_choices = 0           # routed ids from the number of experts on: outputs that own no weights here
         self.tp_size = tp_size if tp_size is not None else ps.tp_size()
         self.tp_rank = tp_rank if tp_rank is not None else ps.tp_rank()
         ep = ep_size if ep_size is not None else ps.ep_size()
@@ -256,12 +257,17 @@ class FusedMoE(nn.Module):
                 (self.w2_weight.float() * self.w2_scale[..., None]).to(self.dtype))
 
     def _observe(self, topk_ids):
-        """Report the chosen experts to whoever listens; physical ids where experts have replicas."""
+        """Report the chosen experts to whoever listens; physical ids where experts have replicas.  Choices beyond the experts
+        (outputs without weights) are -1 to both."""
         if self.routed_experts_capturer is not None:
             self.routed_experts_capturer.capture(self.layer_id, topk_ids)
         if self.recorder is not None:
-            self.recorder.record(self.layer_id, topk_ids)
-        return topk_ids if self.expert_location is None else self.expert_location.logical_to_physical(topk_ids)
+            kept = torch.where(topk_ids < self.num_logical_experts, topk_ids, -1) if self.extra_choices else topk_ids
+            self.recorder.record(self.layer_id, kept)
+        if self.expert_location is None:
+            return topk_ids
+        phys = self.expert_location.logical_to_physical(topk_ids.clamp_max(self.num_logical_experts - 1))
+        return torch.where(topk_ids < self.num_logical_experts, phys, -1) if self.extra_choices else phys
 
     def _workspace(self, pairs: int, device):
         from ..ops import moe_native
@@ -275,18 +281,28 @@ class FusedMoE(nn.Module):
         """Gated activation of `[gate | up]` rows by this layer's kind."""
         if self.activation == "clipped_swiglu":
             return ops.clipped_swiglu(h, self.act_limit, self.act_alpha)
+        if self.activation == "swiglu":
+            return ops.swiglu(h)
         return ops.silu_and_mul(h) if self.activation == "silu" else ops.gelu_and_mul(h)
+
+    def sorted_outputs(self, x: torch.Tensor, topk_ids: torch.Tensor):
+        """`(outputs, pair_row)` of the chosen experts, one row per (token, choice) in the workspace's order, negative for choices
+        that are not this rank's; None where the kernels that produce them do not run."""
+        if not ops.use_native_wide(x) or self.tp_size != 1 or self.fp8:
+            return None
+        from ..ops import moe_native
+        topk_ids = self._observe(topk_ids)
+        ws = self._workspace(topk_ids.numel(), x.device)
+        return moe_native.sorted_experts(x, self.w13_weight, self.w2_weight, topk_ids, self.expert_start, ws,
+                                         self._act), ws.pair_row
 
     def forward_stream(self, x: torch.Tensor, topk_weights: torch.Tensor, topk_ids: torch.Tensor, mixed: torch.Tensor,
                        stream: torch.Tensor) -> torch.Tensor:
         """`stream += mixed + sum of the chosen experts' outputs` on an fp32 residual stream, `mixed` another sublayer's
         output (a partial sum, like the experts', under tensor parallelism); returns the stream in x's type."""
-        if ops.use_native_wide(x) and self.tp_size == 1 and not self.fp8:
-            from ..ops import moe_native
-            topk_ids = self._observe(topk_ids)
-            ws = self._workspace(topk_ids.numel(), x.device)
-            y = moe_native.sorted_experts(x, self.w13_weight, self.w2_weight, topk_ids, self.expert_start, ws, self._act)
-            return ops.stream_add(mixed, stream, y, topk_weights, ws.pair_row)
+        made = self.sorted_outputs(x, topk_ids)
+        if made is not None:
+            return ops.stream_add(mixed, stream, made[0], topk_weights, made[1])
         y = self.forward(x, topk_weights, topk_ids, add=mixed)
         return ops.stream_add(ps.all_reduce(y) if self.tp_size > 1 else y, stream)
 
@@ -308,7 +324,7 @@ class FusedMoE(nn.Module):
                                                     out)
             return moe_native.fused_experts(x, self.w13_weight, self.w2_weight, topk_weights, topk_ids,
                                             self.expert_start, self.workspace, add, out)
-        if self.activation == "clipped_swiglu" and not self.fp8 and ops.use_native(x) and x.shape[1] % 8 == 0:
+        if self.activation in ("clipped_swiglu", "swiglu") and not self.fp8 and ops.use_native(x) and x.shape[1] % 8 == 0:
             from ..ops import moe_native
             ws = self._workspace(topk_ids.numel(), x.device)
             y = moe_native.sorted_experts(x, self.w13_weight, self.w2_weight, topk_ids, self.expert_start, ws, self._act)
@@ -322,7 +338,7 @@ class FusedMoE(nn.Module):
                                   add)
         else:
             from ..ops import reference
-            act = self._act if self.activation == "clipped_swiglu" else self.activation
+            act = self._act if self.activation in ("clipped_swiglu", "swiglu") else self.activation
             y = reference.moe_forward(x, self.w13_weight, self.w2_weight, topk_weights, topk_ids, self.expert_start, act=act)
             if add is not None:
                 y = (y.float() + add.float()).to(y.dtype)
@@ -396,6 +412,59 @@ class RoutedFeedForward(nn.Module):
     def forward(self, h: torch.Tensor, mixed: torch.Tensor, stream: torch.Tensor) -> torch.Tensor:
         weights, ids = self.gate.route_by_logit(h, self.top_k)
         return self.experts.forward_stream(h, weights, ids, mixed, stream)
+
+
+class ScoredFeedForward(nn.Module):
+    """Feed-forward of experts chosen by their corrected softmax scores, weighted by the scores themselves (times `scale`).  The
+    last `identity` outputs of the router stand for the input itself.  A shared expert (`shared` wide, 0: none) runs for every
+    token, gated by one number per token.  The whole sum enters a norm behind the residual sum (`SumNorm`)."""
+
+    def __init__(self, hidden_size: int, num_experts: int, identity: int, top_k: int, intermediate_size: int, scale: float,
+                 shared: int, dtype, layer_id: int = 0):
+        super().__init__()
+        from ..models.llama import DenseMLP
+        from .activation import SwiGLU
+        from .gate import GateLogit
+        self.top_k, self.scale = top_k, float(scale)
+        self.gate = GateLogit(hidden_size, num_experts + identity, dtype, correction_bias=True, token_gate=bool(shared))
+        self.experts = FusedMoE(num_experts, hidden_size, intermediate_size, dtype, layer_id=layer_id, activation="swiglu")
+        self.experts.extra_choices = identity
+        self.shared = None
+        if shared:
+            self.shared = DenseMLP(hidden_size, shared, dtype)
+            self.shared.act_fn = SwiGLU()
+            self.shared.down_proj.reduce_results = False      # reduced together with the experts
+
+    def load(self, name: str, w: torch.Tensor):
+        """One checkpoint tensor: `router`, `correction`, `e<i>.gate` / `.up` / `.down`, `shared.gate` / `.up` / `.down` / `.sg`."""
+        if name == "router":
+            return self.gate.weight.data[:w.shape[0]].copy_(w)
+        if name == "correction":
+            return self.gate.e_score_correction_bias.data.copy_(w)
+        expert, shard = name.split(".")
+        if expert != "shared":
+            param = self.experts.w2_weight if shard == "down" else self.experts.w13_weight
+            return self.experts.weight_loader(param, w, shard, int(expert[1:]))
+        if shard == "sg":
+            return self.gate.weight.data[-1].copy_(w.view(-1))
+        if shard == "down":
+            return self.shared.down_proj.weight_loader(self.shared.down_proj.weight, w)
+        up = self.shared.gate_up_proj
+        up.weight_loader(up.weight, w, 0 if shard == "gate" else 1)
+
+    def forward(self, h: torch.Tensor, stream: torch.Tensor, norm, then=None) -> torch.Tensor:
+        """`norm(...)` of the stream and this layer's output, both in one launch where the experts' rows are at hand."""
+        weights, ids, gate = self.gate.route_by_score(h, self.top_k, self.scale)
+        y = self.shared(h) if self.shared is not None else None
+        made = self.experts.sorted_outputs(h, ids)
+        own = dict(weights=weights, ids=ids, experts=self.experts.num_logical_experts)
+        if made is not None:
+            y = torch.zeros_like(h) if y is None else y
+            return norm(y, stream, then, y_gate=gate, expert_out=made[0], pair_row=made[1], **own)
+        if y is not None:
+            y = (y.float() * gate[:, None]).to(y.dtype)
+        y = self.experts(h, weights, ids, add=y)
+        return norm(ps.all_reduce(y) if self.experts.tp_size > 1 else y, stream, then, **own)
 
 
 EPMoE = FusedMoE

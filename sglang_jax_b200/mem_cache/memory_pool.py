@@ -324,6 +324,8 @@ class MLATokenToKVPool(KVCache):
     def get_kv_buffer(self, layer_id):
         return self.kv_buffer[layer_id - self.start_layer]
 
+    get_latent_buffer = get_kv_buffer
+
     def set_kv_buffer(self, layer_id, loc, kv_c: torch.Tensor, k_pe: torch.Tensor):
         buf = self.get_kv_buffer(layer_id).flatten(0, 1)
         rank, rope = self.layer_dims[layer_id - self.start_layer]
@@ -338,28 +340,45 @@ class MLATokenToKVPool(KVCache):
 class PackedKVPool(KVCache):
     """Keys and values of unequal widths, every layer with sizes of its own: per layer `[num_pages, heads, page_size, row]`,
     a row being `[key | value]` of one head and token, both parts padded to whole 16-byte units (of bf16), so that either
-    part of a page is a strided 2-D block that a tensor copy can fetch.  `layer_shapes`: `(heads, key width, value width)`."""
+    part of a page is a strided 2-D block that a tensor copy can fetch.  `layer_shapes`: `(heads, key width, value width)`; a
+    latent layer is one head of `latent + rotary` lanes without values.  `token_ids`: also keep the id of the token in every
+    slot, one more page-wise buffer that moves with the others."""
 
-    def __init__(self, size, page_size, dtype, layer_shapes: list[tuple[int, int, int]], device, start_layer: int = 0):
+    def __init__(self, size, page_size, dtype, layer_shapes: list[tuple[int, int, int]], device, start_layer: int = 0,
+                 token_ids: bool = False):
         super().__init__(size, page_size, dtype, len(layer_shapes), device, start_layer)
         self.layer_shapes = list(layer_shapes)
+        self.token_ids = None
         self.kv_buffer = [torch.zeros((self.num_pages, h, page_size, self.padded(k) + self.padded(v)), dtype=dtype,
                                       device=device) for h, k, v in layer_shapes]
+        if token_ids:
+            ids = torch.zeros((self.num_pages, page_size), dtype=torch.int32, device=device)
+            self.kv_buffer.append(ids)
+            self.token_ids = ids.view(-1)
 
     @staticmethod
     def padded(width: int) -> int:
         return -(-width // 8) * 8
 
     @staticmethod
-    def cell_size(layer_shapes, dtype) -> int:
+    def cell_size(layer_shapes, dtype, token_ids: bool = False) -> int:
         return sum(h * (PackedKVPool.padded(k) + PackedKVPool.padded(v)) for h, k, v in layer_shapes) * \
-            torch.finfo(dtype).bits // 8
+            torch.finfo(dtype).bits // 8 + 4 * token_ids
 
     def get_kv_size_bytes(self):
         return sum(b.numel() * b.element_size() for b in self.kv_buffer)
 
     def get_kv_buffer(self, layer_id):
         return self.kv_buffer[layer_id - self.start_layer]
+
+    def get_latent_buffer(self, layer_id):
+        """`[pages, page_size, row]` of a layer with one head."""
+        return self.get_kv_buffer(layer_id).squeeze(1)
+
+    def move_kv_cache(self, tgt_loc: torch.Tensor, src_loc: torch.Tensor):
+        super().move_kv_cache(tgt_loc, src_loc)
+        if self.token_ids is not None:
+            self.token_ids[tgt_loc.long()] = self.token_ids[src_loc.long()]
 
     def set_kv_buffer(self, layer_id, loc, k: torch.Tensor, v: torch.Tensor):
         """`k [T, heads, key width]`, `v [T, heads, value width]` into slots `loc [T]`."""

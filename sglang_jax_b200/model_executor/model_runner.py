@@ -170,7 +170,7 @@ class ModelRunner:
         kv_dtype = self.kv_cache_dtype
         n_layers = getattr(self.model, "num_kv_layers", None) or mc.num_hidden_layers
         if getattr(self.model, "kv_layer_shapes", None):
-            return PackedKVPool.cell_size(self.model.kv_layer_shapes, kv_dtype)
+            return PackedKVPool.cell_size(self.model.kv_layer_shapes, kv_dtype, getattr(self.model, "kv_token_ids", False))
         if mc.attention_arch == AttentionArch.MLA:
             return MLATokenToKVPool.cell_size(mc.kv_lora_rank, mc.qk_rope_head_dim, n_layers, kv_dtype,
                                               getattr(self.model, "index_head_dim", 0),
@@ -254,7 +254,8 @@ class ModelRunner:
         n_layers = getattr(self.model, "num_kv_layers", None) or mc.num_hidden_layers
         if getattr(self.model, "kv_layer_shapes", None):
             self.token_to_kv_pool = PackedKVPool(self.max_total_num_tokens, self.page_size, self.kv_cache_dtype,
-                                                 self.model.kv_layer_shapes, str(self.device))
+                                                 self.model.kv_layer_shapes, str(self.device),
+                                                 token_ids=getattr(self.model, "kv_token_ids", False))
         elif mc.attention_arch == AttentionArch.MLA:
             self.token_to_kv_pool = MLATokenToKVPool(self.max_total_num_tokens, self.page_size, self.kv_cache_dtype,
                                                      mc.kv_lora_rank, mc.qk_rope_head_dim, n_layers, str(self.device),

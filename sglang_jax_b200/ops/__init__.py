@@ -79,9 +79,14 @@ def sigmoid_gate(o, gate):
     return (_native() if use_native_wide(o) else reference).sigmoid_gate(o, gate)
 
 
-def clipped_swiglu(x, limit: float, alpha: float = 1.702):
-    """`g * sigmoid(alpha g) * (u + 1)` of `x = [gate | up]`, `g = min(gate, limit)`, `u = clamp(up, -limit, limit)`."""
-    return (_native() if use_native_wide(x) else reference).clipped_swiglu(x, limit, alpha)
+def clipped_swiglu(x, limit: float, alpha: float = 1.702, shift: float = 1.0):
+    """`g * sigmoid(alpha g) * (u + shift)` of `x = [gate | up]`, `g = min(gate, limit)`, `u = clamp(up, -limit, limit)`."""
+    return (_native() if use_native_wide(x) else reference).clipped_swiglu(x, limit, alpha, shift)
+
+
+def swiglu(x):
+    """`silu(gate) * up` of `x = [gate | up]`, any width, bf16 or fp32."""
+    return clipped_swiglu(x, float("inf"), 1.0, 0.0)
 
 
 def token_side_gate(z, table, ids, offset: int):
@@ -94,6 +99,22 @@ def embed_scaled(ids, table, scale, positions=None, turns=None):
     """`table[ids] * scale` as `(fp32 stream, the same in the table's type)`.  `turns` (double, `[ceil(width / 2)]`): adds
     the sinusoidal vector of `positions`, channels 2i and 2i + 1 being sine and cosine of `turns[i]` turns a position."""
     return (_native() if use_native_wide(table) else reference).embed_scaled(ids, table, scale, positions, turns)
+
+
+def embed_pair(ids, table, pairs, mul_prev: int, mul_cur: int, slot_ids, fb):
+    """`table[ids] + pairs[(previous id * mul_prev + id * mul_cur) mod buckets]` as `(fp32 stream, the same in the table's
+    type)`; `pairs [buckets + 1, W]`, the last row is for a sequence's first token.  `slot_ids` int32: the id of the token in
+    every slot of the KV pool, read for the predecessor of a portion's first token and written at the step's slots."""
+    args = (ids, table, pairs, mul_prev, mul_cur, slot_ids, fb.positions, fb.out_cache_loc,
+            None if fb.forward_mode.is_decode() else fb.cu_q_lens, fb.req_pool_indices, fb.page_table, fb.page_size)
+    return (_native() if use_native_wide(table) else reference).embed_pair(*args)
+
+
+def sum_norm(y, x, alpha, scale, weight, eps, **kw):
+    """`x <- weight * z / rms(z)` in place on the fp32 stream with `z = alpha x + scale * (y_gate y + sum_j weights[t, j] c_j)`;
+    `c_j` is row `pair_row[t, j]` of `expert_out` (negative: nothing), or x itself where `ids[t, j] >= experts`.  Returns x in
+    y's type, or with `next_weight` (and `next_eps`) `next_weight * x / rms(x)`."""
+    return (_native() if use_native_wide(y) else reference).sum_norm(y, x, alpha, scale, weight, eps, **kw)
 
 
 def stream_add(y, x, expert_out=None, weights=None, pair_row=None):
@@ -132,22 +153,27 @@ def attn_prep(proj, *a, **kw):
     return (_native() if use_native_wide(proj) else reference).attn_prep(proj, *a, **kw)
 
 
-def window_attention(q, gate, cache, fb, rows, lens, dim, v_dim, scale, window, keep_first):
+def attn_prep_rows(proj, *a, **kw):
+    return (_native() if use_native_wide(proj) else reference).attn_prep_rows(proj, *a, **kw)
+
+
+def window_attention(q, gate, cache, fb, rows, lens, dim, v_dim, scale, window, keep_first, **terms):
     """Every query token on its own: query n sees the first `lens[n]` tokens of page-table row `rows[n]`, of those the last
-    `window` (0: all) and the first `keep_first`."""
+    `window` (0: all) and the first `keep_first`.  `softcap` (0: none), `slope` and `sink` (fp32 per head, or None): scores are
+    `softcap * tanh(score / softcap) - slope * distance`, and `exp(sink)` joins the denominator."""
     n = _native()
     args = (q, gate, cache, fb.page_table, rows, lens, dim, v_dim, fb.page_size, scale, window, keep_first)
     if n.window_decode_supported(q, cache, dim, v_dim, fb.page_size):
-        return n.window_decode(*args, max_seq_len=fb.max_seq_len)
-    return n.window_attn_any(*args)
+        return n.window_decode(*args, max_seq_len=fb.max_seq_len, **terms)
+    return n.window_attn_any(*args, **terms)
 
 
 def window_extend_supported(q, cache, dim, v_dim) -> bool:
     return use_native(q) and _native().window_extend_supported(q, cache, dim, v_dim)
 
 
-def window_extend(q, gate, cache, fb, plan, out, dim, v_dim, scale, window, keep_first):
-    return _native().window_extend(q, gate, cache, fb.page_table, plan, out, dim, v_dim, scale, window, keep_first)
+def window_extend(q, gate, cache, fb, plan, out, dim, v_dim, scale, window, keep_first, **terms):
+    return _native().window_extend(q, gate, cache, fb.page_table, plan, out, dim, v_dim, scale, window, keep_first, **terms)
 
 
 def low_rank_up(x, w):
@@ -163,22 +189,37 @@ def route_by_logit(x, weight, bias, top_k):
     return reference.route_by_logit(x, weight, bias, top_k)
 
 
+def route_by_score(x, weight, correction, top_k, scale, gated: bool = False):
+    """`s = softmax(x weight^T)` (fp32), the `top_k` choices with the largest `s + correction`, weighted by `scale * s`; `gated`:
+    the last row of `weight` is no choice but a gate per token, whose sigmoid comes third (else None)."""
+    if use_native_wide(x) and weight.shape[0] <= 512 and top_k <= 16 and weight.dtype == x.dtype:
+        from . import moe_native
+        return moe_native.route_by_score(x, weight, correction, top_k, scale, gated)
+    return reference.route_by_score(x, weight, correction, top_k, scale, gated)
+
+
 # ---- latent attention (see `native.latent_prep`)
 def latent_prep(proj, *a, **kw):
     return (_native() if use_native_wide(proj) else reference).latent_prep(proj, *a, **kw)
 
 
-def latent_attention(q_lat, q_pe, cache, fb, scale, rows=None, lens=None):
+def latent_rotate(q, *a):
+    (_native() if use_native_wide(q) else reference).latent_rotate(q, *a)
+
+
+def latent_attention(q_lat, q_pe, cache, fb, scale, rows=None, lens=None, window: int = 0, sink=None):
     """Absorbed attention of every query token over the cache rows it sees: `q_lat [T, H, R]`, `q_pe [T, H, rot]`,
     `cache [pages, P, >= R + rot]` -> `[T, H, R]`.  `rows`, `lens` (int32 `[T]`): page-table row and number of visible
-    tokens of each query; None = the step's own tokens."""
+    tokens of each query; None = the step's own tokens.  `window` (0: all): of those only the last; `sink` fp32 `[H]`: joins
+    the softmax's denominator."""
     R = q_lat.shape[-1]
     if not use_native_wide(q_lat):
         assert rows is None
         decode = fb.forward_mode.is_decode()
         return reference.mla_paged_attention(q_lat, q_pe, cache[..., :R + q_pe.shape[-1]], fb.page_table,
                                              fb.req_pool_indices, fb.seq_lens, fb.page_size, scale, R,
-                                             None if decode else fb.cu_q_lens, None if decode else fb.extend_prefix_lens)
+                                             None if decode else fb.cu_q_lens, None if decode else fb.extend_prefix_lens,
+                                             window=window, sink=sink)
     native = _native()
     if rows is None:
         if fb.forward_mode.is_decode():
@@ -189,8 +230,8 @@ def latent_attention(q_lat, q_pe, cache, fb, scale, rows=None, lens=None):
             rows, lens = plan.token_rows, plan.token_lens
     if native.mla_decode_supported(q_lat, q_pe, cache, R, fb.page_size):
         return native.mla_decode(q_lat, q_pe, cache, fb.page_table, rows, lens, fb.page_size, scale, fb.max_seq_len,
-                                 exact=True)
-    return native.latent_attn_any(q_lat, q_pe, cache, fb.page_table, rows, lens, fb.page_size, scale)
+                                 exact=True, window=window, sink=sink)
+    return native.latent_attn_any(q_lat, q_pe, cache, fb.page_table, rows, lens, fb.page_size, scale, window, sink)
 
 
 def latent_extend_supported(q, dim, rot, v_dim, rank) -> bool:
@@ -201,8 +242,8 @@ def latent_gather(*a):
     return _native().latent_gather(*a)
 
 
-def latent_extend(*a):
-    return _native().latent_extend(*a)
+def latent_extend(*a, **kw):
+    return _native().latent_extend(*a, **kw)
 
 
 def linear(x, w, bias=None):

@@ -84,43 +84,54 @@ def lib():
     sig("sglb_conv1d_update", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
                                      c_void_p])
     sig("sglb_mla_decode", [c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_longlong, c_int, c_void_p,
-                            c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p,
-                            c_void_p, c_int, c_void_p])
+                            c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int,
+                            c_void_p, c_void_p, c_int, c_void_p])
     sig("sglb_mla_num_splits", [c_int, c_int, c_int])
     sig("sglb_embed_scaled", [c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_float, c_void_p,
                               c_void_p, c_int, c_void_p])
+    sig("sglb_embed_pair", [c_void_p] * 4 + [c_longlong, c_int, c_int, c_void_p, c_int, c_longlong, c_longlong]
+        + [c_void_p] * 6 + [c_int] * 4 + [c_void_p])
+    sig("sglb_sum_norm", [c_void_p] * 5 + [c_float, c_float] + [c_void_p] * 5 + [c_int, c_int, c_void_p, c_float, c_longlong,
+                                                                             c_int, c_int, c_void_p])
     sig("sglb_postnorm_add", [c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_float, c_void_p, c_float, c_int,
                               c_void_p])
     sig("sglb_stream_add", [c_void_p] * 6 + [c_int, c_longlong, c_int, c_int, c_void_p])
-    sig("sglb_clipped_swiglu", [c_void_p, c_void_p, c_longlong, c_int, c_float, c_float, c_int, c_void_p])
+    sig("sglb_clipped_swiglu", [c_void_p, c_void_p, c_longlong, c_int, c_float, c_float, c_float, c_int, c_void_p])
     sig("sglb_side_gate", [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_int, c_longlong, c_int, c_int,
                            c_void_p])
     sig("sglb_rmsnorm_stream", [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_float, c_int, c_void_p])
     sig("sglb_gelu_tanh_and_mul", [c_void_p, c_void_p, c_longlong, c_int, c_int, c_void_p])
     sig("sglb_sigmoid_gate", [c_void_p, c_void_p, c_void_p, c_longlong, c_longlong, c_int, c_int, c_void_p])
     sig("sglb_latent_prep", [c_void_p, c_longlong] + [c_int] * 7 + [c_void_p, c_float, c_void_p, c_void_p, c_void_p,
-                                                                    c_void_p, c_int, c_int, c_void_p])
+                                                                    c_void_p, c_int, c_void_p, c_int, c_void_p, c_int,
+                                                                    c_void_p])
+    sig("sglb_latent_rotate", [c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p])
     sig("sglb_latent_attn_any", [c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p,
-                                 c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p])
-    sig("sglb_latent_gather", [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int,
-                               c_int, c_int, c_int, c_void_p])
+                                 c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_void_p])
+    sig("sglb_latent_gather", [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p,
+                               c_int, c_int, c_int, c_int, c_void_p])
     sig("sglb_latent_extend_supported", [c_int, c_int, c_int])
     sig("sglb_latent_extend", [c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_int]
-        + [c_void_p] * 4 + [c_int] * 6 + [c_float, c_void_p])
+        + [c_void_p] * 5 + [c_int] * 6 + [c_float, c_int, c_void_p, c_void_p])
     sig("sglb_delta_scan", [c_void_p, c_longlong, c_int, c_int, c_int] + [c_void_p] * 18 + [c_int] * 9 + [c_void_p])
     sig("sglb_delta_gate", [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_int, c_int, c_float, c_int,
                             c_int, c_void_p])
     sig("sglb_attn_prep", [c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_longlong]
         + [c_int] * 6 + [c_float, c_int, c_void_p])
+    sig("sglb_attn_prep_rows", [c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_longlong]
+        + [c_int] * 5 + [c_void_p] * 3 + [c_int, c_int, c_float, c_void_p, c_longlong, c_void_p, c_int, c_void_p])
     sig("sglb_window_decode_supported", [c_int, c_int, c_int])
     sig("sglb_window_num_splits", [c_int, c_int, c_int])
     sig("sglb_window_decode", [c_void_p, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_int, c_int, c_void_p,
-                               c_void_p, c_void_p] + [c_int] * 5 + [c_float, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p])
+                               c_void_p, c_void_p] + [c_int] * 5 + [c_float, c_int, c_int, c_float, c_void_p, c_void_p, c_int,
+                                                                    c_void_p, c_void_p, c_void_p])
     sig("sglb_window_attn_any", [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p,
-                                 c_void_p] + [c_int] * 5 + [c_float, c_int, c_int, c_int, c_void_p])
+                                 c_void_p] + [c_int] * 5 + [c_float, c_int, c_int, c_float, c_void_p, c_void_p, c_int,
+                                                            c_void_p])
     sig("sglb_window_extend_supported", [c_int, c_int, c_int])
     sig("sglb_window_extend", [c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_int, c_int]
-        + [c_void_p] * 4 + [c_int, c_int, c_void_p] + [c_int] * 4 + [c_float, c_int, c_int, c_void_p])
+        + [c_void_p] * 4 + [c_int, c_int, c_void_p] + [c_int] * 4 + [c_float, c_int, c_int, c_float, c_void_p, c_void_p,
+                                                                       c_void_p])
     sig("sglb_paged_decode", [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p,
                                     c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_float, c_int, c_void_p,
                                     c_void_p, c_void_p])
@@ -567,6 +578,11 @@ def conv1d_update(x, state_pool, weight, slots, silu=True):
     return y
 
 
+def _per_head(t, heads: int):
+    assert t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.numel() == heads)
+    return _p(t)
+
+
 def mla_decode_supported(q_latent, q_pe, kv_buffer, kv_lora_rank, page_size) -> bool:
     return (q_latent.dtype == torch.bfloat16 and kv_buffer.dtype == torch.bfloat16 and kv_lora_rank <= 512
             and q_pe.shape[-1] <= 64 and q_pe.stride(-1) == 1 and kv_buffer.shape[-1] % 8 == 0
@@ -575,15 +591,17 @@ def mla_decode_supported(q_latent, q_pe, kv_buffer, kv_lora_rank, page_size) -> 
 
 
 def mla_decode(q_latent, q_pe, kv_buffer, page_table, req_pool_indices, seq_lens, page_size, scale, max_seq_len=0,
-               num_splits=None, exact=False):
+               num_splits=None, exact=False, window=0, sink=None):
     """Absorbed-MLA decode: `q_latent [B, H, R]`, `q_pe [B, H, rotary lanes]` (any strides, unit innermost), latent
     cache `[pages, P, row]` with `row >= R + rotary lanes` -> latent output `[B, H, R]` (the caller applies W_UV).
-    `exact`: the attention weights enter the value product unrounded."""
+    `exact`: the attention weights enter the value product unrounded.  `window` (0: none): tokens a query sees, its own
+    included; `sink` fp32 `[H]`: joins the softmax's denominator."""
     B, H, R = q_latent.shape
     q_latent = q_latent.contiguous()
     out = torch.empty_like(q_latent)
     if num_splits is None:
-        num_splits = lib().sglb_mla_num_splits(B, (H + 15) // 16, max(max_seq_len or page_table.shape[1] * page_size, 1))
+        seen = max_seq_len or page_table.shape[1] * page_size
+        num_splits = lib().sglb_mla_num_splits(B, (H + 15) // 16, max(min(seen, window + 63) if window else seen, 1))
     part_o = part_lse = None
     if num_splits > 1:
         part_o = torch.empty((B, H, num_splits, R), dtype=torch.float32, device=q_latent.device)
@@ -591,7 +609,8 @@ def mla_decode(q_latent, q_pe, kv_buffer, page_table, req_pool_indices, seq_lens
     _check(lib().sglb_mla_decode(_p(q_latent), q_pe.data_ptr(), q_pe.stride(0), q_pe.stride(1), _p(out), _p(kv_buffer),
                                  kv_buffer.shape[0], kv_buffer.shape[-1], _p(page_table), page_table.shape[1],
                                  _p(req_pool_indices), _p(seq_lens), B, H, R, q_pe.shape[-1], page_size, scale,
-                                 num_splits, _p(part_o), _p(part_lse), int(exact), _stream()), "mla_decode")
+                                 int(window), _per_head(sink, H), num_splits, _p(part_o), _p(part_lse), int(exact), _stream()),
+           "mla_decode")
     return out
 
 
@@ -616,6 +635,45 @@ def embed_scaled(ids, table, scale, positions=None, turns=None):
     _check(lib().sglb_embed_scaled(_p(x), _p(xt), _p(ids), _p(table), n, W, table.shape[0], float(scale), _p(positions),
                                    _p(turns), f32, _stream()), "embed_scaled")
     return x, (x if f32 else xt)
+
+
+def embed_pair(ids, table, pairs, mul_prev, mul_cur, slot_ids, positions, loc, cu, rows, page_table, page_size):
+    """`table[ids] + pairs[hash of a token's predecessor and itself]` as `embed_scaled` returns it; see `ops.embed_pair`."""
+    ids = ids.contiguous()
+    assert table.is_contiguous() and pairs.is_contiguous() and pairs.dtype == table.dtype and pairs.shape[1] == table.shape[1]
+    ints = [ids, slot_ids, positions, loc, rows, page_table] + ([cu] if cu is not None else [])
+    assert all(t.dtype == torch.int32 and t.is_contiguous() for t in ints)
+    n, W = ids.numel(), table.shape[1]
+    x = torch.empty((n, W), dtype=torch.float32, device=table.device)
+    f32 = _f32(table)
+    xt = None if f32 else torch.empty((n, W), dtype=table.dtype, device=table.device)
+    _check(lib().sglb_embed_pair(_p(x), _p(xt), _p(ids), _p(table), n, W, table.shape[0], _p(pairs), pairs.shape[0] - 1,
+                                 mul_prev, mul_cur, _p(slot_ids), _p(positions), _p(loc), _p(cu), _p(rows), _p(page_table),
+                                 rows.numel(), page_table.shape[1], page_size, f32, _stream()), "embed_pair")
+    return x, (x if f32 else xt)
+
+
+def sum_norm(y, x, alpha, scale, weight, eps, y_gate=None, expert_out=None, weights=None, pair_row=None, ids=None, experts=0,
+             next_weight=None, next_eps=0.0):
+    """See `ops.sum_norm`."""
+    y = y.contiguous()
+    n, W = x.shape
+    assert x.dtype == scale.dtype == weight.dtype == torch.float32 and x.is_contiguous() and y.shape == x.shape
+    k = 0
+    if weights is not None:
+        k = weights.shape[1]
+        assert weights.dtype == torch.float32 and weights.is_contiguous() and ids.dtype == torch.int32 and ids.is_contiguous()
+        assert ids.shape == weights.shape == (n, k)
+    if expert_out is not None:
+        assert expert_out.is_contiguous() and expert_out.dtype == y.dtype and expert_out.shape[1] == W
+        assert pair_row.dtype == torch.int32 and pair_row.numel() >= n * k
+    assert y_gate is None or (y_gate.dtype == torch.float32 and y_gate.is_contiguous() and y_gate.numel() == n)
+    f32 = _f32(y)
+    xt = torch.empty_like(y) if next_weight is not None or not f32 else None
+    _check(lib().sglb_sum_norm(_p(x), _p(xt), _p(y), _p(scale), _p(weight), float(alpha), float(eps), _p(y_gate),
+                               _p(expert_out), _p(weights), _p(pair_row), _p(ids), k, experts, _p(next_weight),
+                               float(next_eps), n, W, f32, _stream()), "sum_norm")
+    return x if xt is None else xt
 
 
 def postnorm_add(y, x, channel_scale, eps):
@@ -658,12 +716,12 @@ def stream_add(y, x, expert_out=None, weights=None, pair_row=None):
     return x if f32 else xt
 
 
-def clipped_swiglu(x, limit, alpha=1.702):
+def clipped_swiglu(x, limit, alpha=1.702, shift=1.0):
     x = x.contiguous()
     F = x.shape[-1] // 2
     out = torch.empty((*x.shape[:-1], F), dtype=x.dtype, device=x.device)
-    _check(lib().sglb_clipped_swiglu(_p(out), _p(x), out.numel() // F, F, float(limit), float(alpha), _f32(x), _stream()),
-           "clipped_swiglu")
+    _check(lib().sglb_clipped_swiglu(_p(out), _p(x), out.numel() // F, F, float(limit), float(alpha), float(shift), _f32(x),
+                                     _stream()), "clipped_swiglu")
     return out
 
 
@@ -705,38 +763,55 @@ def sigmoid_gate(o, gate):
 
 
 # ---- latent attention of any sizes (csrc/latent_attn.cu, latent_extend.cu)
-def latent_prep(proj, q_off, dkv_off, heads, dim, rot, rank, norm_w, eps, cos_sin, positions, loc, cache):
+def latent_prep(proj, q_off, dkv_off, heads, dim, rot, rank, norm_w, eps, cos_sin, positions, loc, cache, q_norm_w=None):
     """Rotates the queries of `proj [T, ld]` in place and writes the normalised latent and the rotated key part of its
-    rows into `cache [pages, P, row]` at slots `loc`."""
+    rows into `cache [pages, P, row]` at slots `loc`.  With `q_norm_w [q_rank]` the projection holds the queries' latent at
+    `q_off` instead, and its normalised form `[T, q_rank]` is returned."""
     assert proj.stride(1) == 1 and cache.is_contiguous() and cache.dtype == proj.dtype
     assert positions.dtype == loc.dtype == torch.int32 and norm_w.dtype == cos_sin.dtype == torch.float32
     assert cos_sin.device == norm_w.device == cache.device == proj.device and cos_sin.is_contiguous()
+    q_latent, q_rank = None, 0
+    if q_norm_w is not None:
+        q_rank = q_norm_w.numel()
+        assert q_norm_w.dtype == torch.float32
+        q_latent = torch.empty((proj.shape[0], q_rank), dtype=proj.dtype, device=proj.device)
     _check(lib().sglb_latent_prep(_p(proj), proj.stride(0), q_off, dkv_off, proj.shape[0], heads, dim, rot, rank,
                                   _p(norm_w), float(eps), _p(cos_sin), _p(positions), _p(loc), _p(cache),
-                                  cache.shape[-1], _f32(proj), _stream()), "latent_prep")
+                                  cache.shape[-1], _p(q_latent), q_rank, _p(q_norm_w), _f32(proj), _stream()),
+           "latent_prep")
+    return q_latent
 
 
-def latent_attn_any(q_lat, q_pe, cache, page_table, rows, kv_lens, page_size, scale):
+def latent_rotate(q, dim, cos_sin, positions):
+    """Rotates the lanes from `dim` on of every head of `q [T, H, dim + rot]` (any token stride) in place."""
+    T, H, lanes = q.shape
+    assert q.stride(2) == 1 and q.stride(1) == lanes and positions.dtype == torch.int32 and cos_sin.dtype == torch.float32
+    _check(lib().sglb_latent_rotate(q.data_ptr(), q.stride(0), T, H, dim, lanes - dim, _p(cos_sin), _p(positions), _f32(q),
+                                    _stream()), "latent_rotate")
+
+
+def latent_attn_any(q_lat, q_pe, cache, page_table, rows, kv_lens, page_size, scale, window=0, sink=None):
     """Absorbed attention of single query tokens, fp32 arithmetic: `q_lat [N, H, R]`, query n sees the first
-    `kv_lens[n]` tokens of page-table row `rows[n]`."""
+    `kv_lens[n]` tokens of page-table row `rows[n]`, of those the last `window` (0: all); `sink` as in `mla_decode`."""
     N, H, R = q_lat.shape
     q_lat = q_lat.contiguous()
     assert q_pe.stride(-1) == 1 and rows.dtype == kv_lens.dtype == torch.int32 and cache.dtype == q_lat.dtype
     out = torch.empty_like(q_lat)
     _check(lib().sglb_latent_attn_any(_p(q_lat), q_pe.data_ptr(), q_pe.stride(0), q_pe.stride(1), _p(cache),
                                       cache.shape[-1], _p(page_table), page_table.shape[1], page_size, _p(rows),
-                                      _p(kv_lens), _p(out), N, H, R, q_pe.shape[-1], float(scale), _f32(q_lat),
-                                      _stream()), "latent_attn_any")
+                                      _p(kv_lens), _p(out), N, H, R, q_pe.shape[-1], float(scale), int(window),
+                                      _per_head(sink, H), _f32(q_lat), _stream()), "latent_attn_any")
     return out
 
 
-def latent_gather(cache, page_table, rows, ctx_start, total, rank, rot, page_size):
-    """Cache rows of whole sequences, laid end to end -> `(latents [total, rank], key parts [total, rot])`."""
+def latent_gather(cache, page_table, rows, ctx_start, total, rank, rot, page_size, skip=None):
+    """Cache rows of whole sequences (or, with `skip`, from that token on), laid end to end -> `(latents [total, rank], key
+    parts [total, rot])`."""
     lat = torch.empty((total, rank), dtype=cache.dtype, device=cache.device)
     pe = torch.empty((total, rot), dtype=cache.dtype, device=cache.device)
     _check(lib().sglb_latent_gather(_p(lat), _p(pe), _p(cache), cache.shape[-1], _p(page_table), page_table.shape[1],
-                                    page_size, _p(rows), _p(ctx_start), rows.numel(), total, rank, rot, _stream()),
-           "latent_gather")
+                                    page_size, _p(rows), _p(ctx_start), _p(skip), rows.numel(), total, rank, rot,
+                                    _stream()), "latent_gather")
     return lat, pe
 
 
@@ -747,15 +822,18 @@ def latent_extend_supported(q, dim, rot, v_dim, rank) -> bool:
             and bool(lib().sglb_latent_extend_supported(dim, rot, v_dim)))
 
 
-def latent_extend(q, kv, k_rot, out, plan, dim, v_dim, scale):
+def latent_extend(q, kv, k_rot, out, plan, dim, v_dim, scale, window=0, sink=None):
     """Causal attention of the sequences of `plan` (`layers/extend_plan.ExtendPlan`) over expanded keys and values:
     `q [T, H, dim + rot]` (strided view), `kv [ctx, H * (dim + v_dim)]`, `k_rot [ctx, rot]`, result into the rows of
-    those sequences of `out [T, H, v_dim]` (strided view)."""
+    those sequences of `out [T, H, v_dim]` (strided view).  Context rows as `plan.context(window)` lays them out; `sink` as in
+    `mla_decode`."""
     assert kv.is_contiguous() and k_rot.is_contiguous() and out.stride(2) == 1 and out.dtype == q.dtype
+    ctx = plan.context(window)
     _check(lib().sglb_latent_extend(q.data_ptr(), q.stride(0), q.shape[0], _p(kv), _p(k_rot), k_rot.shape[0],
                                     out.data_ptr(), out.stride(0), out.stride(1), _p(plan.q_start), _p(plan.q_len),
-                                    _p(plan.prefix), _p(plan.ctx_start), plan.long, plan.num_tiles, q.shape[1], dim,
-                                    k_rot.shape[1], v_dim, float(scale), _stream()), "latent_extend")
+                                    _p(plan.prefix), _p(ctx.start), _p(ctx.skip), plan.long, plan.num_tiles, q.shape[1], dim,
+                                    k_rot.shape[1], v_dim, float(scale), int(window), _per_head(sink, q.shape[1]), _stream()),
+           "latent_extend")
 
 
 # ---- gated delta rule over ragged batches (csrc/delta_scan.cu)
@@ -819,6 +897,29 @@ def attn_prep(proj, q_off, k_off, v_off, heads, kv_heads, dim, v_dim, eps, qk_no
     return q
 
 
+def attn_prep_rows(proj, q_off, k_off, v_off, heads, kv_heads, dim, v_dim, eps, q_norm_w, k_norm_w, loc, cache, squares=None,
+                   totals=None, mix=None, share=None):
+    """As `attn_prep`, but queries and keys are divided by the root mean square of all heads at once and multiplied by
+    `q_norm_w [heads * dim]` / `k_norm_w [kv_heads * dim]`.  `squares` fp32 `[T, 2]`, `totals`: sums of squares of the whole
+    projections and their widths where this rank holds a part of them.  `mix [T, kv_heads * v_dim]` (any row stride): values
+    that replace `share` (fp32, one number on the device) of the layer's own."""
+    T = proj.shape[0]
+    assert proj.stride(1) == 1 and cache.is_contiguous() and cache.dtype == proj.dtype and loc.dtype == torch.int32
+    assert cache.shape[1] == kv_heads and cache.shape[3] == _pad8(dim) + _pad8(v_dim)
+    assert q_norm_w.dtype == k_norm_w.dtype == torch.float32
+    assert q_norm_w.numel() == heads * dim and k_norm_w.numel() == kv_heads * dim
+    assert squares is None or (squares.dtype == torch.float32 and squares.is_contiguous() and squares.shape == (T, 2))
+    assert mix is None or (mix.dtype == proj.dtype and mix.stride(1) == 1 and mix.shape == (T, kv_heads * v_dim)
+                           and share.dtype == torch.float32)
+    nq, nk = totals or (heads * dim, kv_heads * dim)
+    q = torch.empty((T, heads, _pad8(dim)), dtype=proj.dtype, device=proj.device)
+    _check(lib().sglb_attn_prep_rows(_p(proj), proj.stride(0), q_off, k_off, v_off, _p(q), _p(cache), _p(loc), T, heads,
+                                     kv_heads, dim, v_dim, cache.shape[2], _p(q_norm_w), _p(k_norm_w), _p(squares), nq, nk,
+                                     float(eps), None if mix is None else mix.data_ptr(), 0 if mix is None else mix.stride(0),
+                                     None if mix is None else _p(share), _f32(proj), _stream()), "attn_prep_rows")
+    return q
+
+
 def _check_window_args(q, gate, cache, rows, lens, dim, v_dim):
     assert q.is_contiguous() and q.shape[2] == _pad8(dim) and cache.is_contiguous() and cache.dtype == q.dtype
     assert cache.shape[3] == _pad8(dim) + _pad8(v_dim) and q.shape[1] % cache.shape[1] == 0
@@ -832,7 +933,7 @@ def window_decode_supported(q, cache, dim, v_dim, page_size) -> bool:
 
 
 def window_decode(q, gate, cache, page_table, rows, lens, dim, v_dim, page_size, scale, window, keep_first, max_seq_len=0,
-                  num_splits=None):
+                  num_splits=None, softcap=0.0, slope=None, sink=None):
     """Attention of single query tokens (`ops.window_attention`), times `sigmoid(gate)` per head -> `[N, heads, v_dim]`."""
     _check_window_args(q, gate, cache, rows, lens, dim, v_dim)
     N, H, _ = q.shape
@@ -850,19 +951,20 @@ def window_decode(q, gate, cache, page_table, rows, lens, dim, v_dim, page_size,
     _check(lib().sglb_window_decode(_p(q), None if gate is None else gate.data_ptr(), 0 if gate is None else gate.stride(0),
                                     _p(cache), cache.shape[0], _p(page_table), page_table.shape[1], page_size, _p(rows),
                                     _p(lens), _p(out), N, H, G, dim, v_dim, float(scale), int(window), int(keep_first),
-                                    num_splits, _p(part_o), _p(part_lse), _stream()), "window_decode")
+                                    float(softcap), _per_head(slope, H), _per_head(sink, H), num_splits, _p(part_o), _p(part_lse), _stream()), "window_decode")
     return out
 
 
-def window_attn_any(q, gate, cache, page_table, rows, lens, dim, v_dim, page_size, scale, window, keep_first):
+def window_attn_any(q, gate, cache, page_table, rows, lens, dim, v_dim, page_size, scale, window, keep_first, softcap=0.0,
+                    slope=None, sink=None):
     """The same in fp32 arithmetic for any sizes, bf16 or fp32."""
     _check_window_args(q, gate, cache, rows, lens, dim, v_dim)
     N, H, _ = q.shape
     out = torch.empty((N, H, v_dim), dtype=q.dtype, device=q.device)
     _check(lib().sglb_window_attn_any(_p(q), None if gate is None else gate.data_ptr(), 0 if gate is None else gate.stride(0),
                                       _p(cache), _p(page_table), page_table.shape[1], page_size, _p(rows), _p(lens), _p(out),
-                                      N, H, cache.shape[1], dim, v_dim, float(scale), int(window), int(keep_first), _f32(q),
-                                      _stream()), "window_attn_any")
+                                      N, H, cache.shape[1], dim, v_dim, float(scale), int(window), int(keep_first),
+                                      float(softcap), _per_head(slope, H), _per_head(sink, H), _f32(q), _stream()), "window_attn_any")
     return out
 
 
@@ -871,7 +973,8 @@ def window_extend_supported(q, cache, dim, v_dim) -> bool:
         bool(lib().sglb_window_extend_supported(dim, v_dim, cache.shape[2]))
 
 
-def window_extend(q, gate, cache, page_table, plan, out, dim, v_dim, scale, window, keep_first):
+def window_extend(q, gate, cache, page_table, plan, out, dim, v_dim, scale, window, keep_first, softcap=0.0, slope=None,
+                  sink=None):
     """Prefill attention of the sequences of `plan` (`layers/extend_plan.ExtendPlan`) into their rows of
     `out [T, heads, v_dim]`."""
     _check_window_args(q, gate, cache, plan.rows, plan.prefix, dim, v_dim)
@@ -880,7 +983,8 @@ def window_extend(q, gate, cache, page_table, plan, out, dim, v_dim, scale, wind
                                     0 if gate is None else gate.stride(0), _p(cache), cache.shape[0], _p(page_table),
                                     page_table.shape[1], cache.shape[2], _p(plan.rows), _p(plan.q_start), _p(plan.q_len),
                                     _p(plan.prefix), plan.long, plan.num_tiles, _p(out), q.shape[1], cache.shape[1], dim,
-                                    v_dim, float(scale), int(window), int(keep_first), _stream()), "window_extend")
+                                    v_dim, float(scale), int(window), int(keep_first), float(softcap),
+                                    _per_head(slope, q.shape[1]), _per_head(sink, q.shape[1]), _stream()), "window_extend")
 
 
 def lora_bgmv(x, y, a_buf, b_bufs, out_offsets, token_slots, scalings):

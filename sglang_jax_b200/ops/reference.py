@@ -315,11 +315,13 @@ def grouped_gemm(x, w, group_sizes):
 
 # ----------------------------------------------------------------------------- MLA
 def mla_paged_attention(q_nope_latent, q_pe, kv_buffer, page_table, req_pool_indices, seq_lens,
-                        page_size, scale, kv_lora_rank, cu_q_lens=None, prefix_lens=None, allowed=None):
+                        page_size, scale, kv_lora_rank, cu_q_lens=None, prefix_lens=None, allowed=None, window=0,
+                        sink=None):
     """Absorbed MLA: every head attends over the shared latent cache
     `[pages, P, kv_lora_rank + rope_dim]`; logits = q_latent·c + q_pe·k_pe; output stays
     latent `[T, H, kv_lora_rank]` (caller applies W_UV).  `allowed[b]` (bool `[n_b, S_b]`) restricts
-    request b's queries to the keys a sparse-attention indexer selected."""
+    request b's queries to the keys a sparse-attention indexer selected, `window` (0: all) to the last keys; `sink [H]` joins
+    the softmax's denominator."""
     T, H, R = q_nope_latent.shape
     out = torch.empty_like(q_nope_latent)
     B = len(req_pool_indices)
@@ -342,8 +344,10 @@ def mla_paged_attention(q_nope_latent, q_pe, kv_buffer, page_table, req_pool_ind
         keep = kpos <= qpos
         if allowed is not None and allowed[b] is not None:      # sparse attention: [n, S] selected keys
             keep = keep & allowed[b]
+        if window:
+            keep = keep & (qpos - kpos < window)
         logits = logits.masked_fill(~keep.view(1, n, S), float("-inf"))
-        p = torch.softmax(logits, dim=-1)
+        p = softmax_with_sink(logits, sink)
         out[q0:q1] = torch.einsum("hns,sr->nhr", p, c).to(out.dtype)
     return out
 
@@ -353,10 +357,10 @@ def sigmoid_gate(o, gate):
     return (o.float() * torch.sigmoid(gate.float())).to(o.dtype)
 
 
-def clipped_swiglu(x, limit, alpha=1.702):
+def clipped_swiglu(x, limit, alpha=1.702, shift=1.0):
     g, u = x.float().chunk(2, -1)
     g, u = g.clamp(max=limit), u.clamp(-limit, limit)
-    return (g * torch.sigmoid(alpha * g) * (u + 1)).to(x.dtype)
+    return (g * torch.sigmoid(alpha * g) * (u + shift)).to(x.dtype)
 
 
 def token_side_gate(z, table, ids, offset):
@@ -375,6 +379,54 @@ def stream_add(y, x, expert_out=None, weights=None, pair_row=None):
 def postnorm_add_norm(y, x, channel_scale, eps, next_scale, next_eps):
     postnorm_add(y, x, channel_scale, eps)
     return rmsnorm_stream(x, next_scale, next_eps, y.dtype)
+
+
+def softmax_with_sink(logits, sink=None):
+    """Softmax over the last axis of `[H, n, S]`; `sink [H]` joins the denominator."""
+    if sink is None:
+        return torch.softmax(logits, dim=-1)
+    s = sink.float()[:, None, None].expand(-1, logits.shape[1], 1)
+    return torch.softmax(torch.cat([logits, s], -1), dim=-1)[..., :-1]
+
+
+def sum_norm(y, x, alpha, scale, weight, eps, y_gate=None, expert_out=None, weights=None, pair_row=None, ids=None, experts=0,
+             next_weight=None, next_eps=0.0):
+    v = y.float() if y_gate is None else y.float() * y_gate[:, None]
+    if expert_out is not None:
+        rows = pair_row[:weights.numel()].view(weights.shape).long()
+        v = v + ((weights * (rows >= 0)).unsqueeze(-1) * expert_out[rows.clamp_min(0)].float()).sum(1)
+    if weights is not None:
+        v = v + (weights * (ids >= experts)).sum(1, keepdim=True) * x
+    z = alpha * x + scale * v
+    x.copy_(z * torch.rsqrt(z.pow(2).mean(-1, keepdim=True) + eps) * weight)
+    if next_weight is not None:
+        return rmsnorm_stream(x, next_weight, next_eps, y.dtype)
+    return x if y.dtype == torch.float32 else x.to(y.dtype)
+
+
+def embed_pair(ids, table, pairs, mul_prev, mul_cur, slot_ids, positions, loc, cu, rows, page_table, page_size):
+    ids64, pos = ids.long(), positions.long()
+    start = torch.arange(ids.numel(), device=ids.device) if cu is None else cu[:-1].long()
+    seen = start < ids.numel()
+    if cu is not None:
+        seen &= cu[1:] > cu[:-1]
+    start, row = start[seen], rows.long()[seen]
+    before = (pos[start] - 1).clamp_min(0)                   # in front of a portion: kept with the slot
+    prev = ids64.roll(1)
+    prev[start] = slot_ids[page_table[row, before // page_size].long() * page_size + before % page_size].long()
+    buckets = pairs.shape[0] - 1
+    at = torch.where(pos > 0, (prev * mul_prev + ids64 * mul_cur) % buckets, buckets)
+    slot_ids[loc.long()] = ids.to(slot_ids.dtype)
+    x = F.embedding(ids64, table).float() + pairs[at].float()
+    return x, (x if table.dtype == torch.float32 else x.to(table.dtype))
+
+
+def route_by_score(x, weight, correction, top_k, scale, gated=False):
+    z = F.linear(x.float(), weight.float())
+    gate = torch.sigmoid(z[:, -1]) if gated else None
+    s = torch.softmax(z[:, :-1] if gated else z, -1)
+    ids = (s if correction is None else s + correction).topk(top_k, dim=-1).indices
+    return s.gather(1, ids) * scale, ids.to(torch.int32), gate
 
 
 def route_by_logit(x, weight, bias, top_k):
@@ -398,7 +450,24 @@ def attn_prep(proj, q_off, k_off, v_off, heads, kv_heads, dim, v_dim, eps, qk_no
     return unit(part(q_off, heads, dim)).to(proj.dtype)
 
 
-def window_attention(q, gate, cache, fb, dim, v_dim, scale, window, keep_first):
+def attn_prep_rows(proj, q_off, k_off, v_off, heads, kv_heads, dim, v_dim, eps, q_norm_w, k_norm_w, loc, cache, squares=None,
+                   totals=None, mix=None, share=None):
+    def normed(off, n, w, i):
+        t = proj[:, off:off + n * dim].float()
+        ms = t.pow(2).mean(-1, keepdim=True) if squares is None else squares[:, i:i + 1] / totals[i]
+        return (t * torch.rsqrt(ms + eps) * w).unflatten(-1, (n, dim))
+
+    P, at = cache.shape[2], -(-dim // 8) * 8
+    page, off = (loc // P).long(), (loc % P).long()
+    v = proj[:, v_off:v_off + kv_heads * v_dim].float()
+    if mix is not None:
+        v = (1 - share) * v + share * mix.float()
+    cache[page, :, off, :dim] = normed(k_off, kv_heads, k_norm_w, 1).to(cache.dtype)
+    cache[page, :, off, at:at + v_dim] = v.unflatten(-1, (kv_heads, v_dim)).to(cache.dtype)
+    return normed(q_off, heads, q_norm_w, 0).to(proj.dtype)
+
+
+def window_attention(q, gate, cache, fb, dim, v_dim, scale, window, keep_first, softcap=0.0, slope=None, sink=None):
     """Statement of the windowed attention of a whole step; `q [T, heads, >= dim]`, `cache [pages, kv heads, P, row]`."""
     decode = fb.forward_mode.is_decode()
     B, at = fb.batch_size, -(-dim // 8) * 8
@@ -418,8 +487,12 @@ def window_attention(q, gate, cache, fb, dim, v_dim, scale, window, keep_first):
         see = j <= i
         if window > 0:
             see &= (i - j < window) | (j < keep_first)
-        s = torch.einsum("nghd,sgd->ghns", qb, k) * scale
-        p = torch.softmax(s.masked_fill(~see, float("-inf")), -1)
+        s = (torch.einsum("nghd,sgd->ghns", qb, k) * scale).flatten(0, 1)
+        if softcap:
+            s = softcap * torch.tanh(s / softcap)
+        if slope is not None:
+            s = s - slope[:, None, None] * (i - j)
+        p = softmax_with_sink(s.masked_fill(~see, float("-inf")), sink).unflatten(0, (k.shape[1], -1))
         o = torch.einsum("ghns,sgd->nghd", p, v).flatten(1, 2)
         if gate is not None:
             o = o * torch.sigmoid(gate[cu[b]:cu[b + 1]].float())[..., None]
@@ -498,10 +571,19 @@ def delta_gate(o, gate, weight, eps, act="silu"):
     return y.view(T, H * V).to(gate.dtype)
 
 
-def latent_prep(proj, q_off, dkv_off, heads, dim, rot, rank, norm_w, eps, cos_sin, positions, loc, cache):
-    q = proj[:, q_off:q_off + heads * (dim + rot)].unflatten(-1, (heads, dim + rot))[..., dim:]
-    q.copy_(apply_rope(q, positions, cos_sin, False))
+def latent_rotate(q, dim, cos_sin, positions):
+    q[..., dim:].copy_(apply_rope(q[..., dim:], positions, cos_sin, False))
+
+
+def latent_prep(proj, q_off, dkv_off, heads, dim, rot, rank, norm_w, eps, cos_sin, positions, loc, cache, q_norm_w=None):
+    c_q = None
+    if q_norm_w is not None:
+        c_q = proj[:, q_off:q_off + q_norm_w.numel()].float()
+        c_q = (c_q * torch.rsqrt(c_q.pow(2).mean(-1, keepdim=True) + eps) * q_norm_w).to(proj.dtype)
+    else:
+        latent_rotate(proj[:, q_off:q_off + heads * (dim + rot)].unflatten(-1, (heads, dim + rot)), dim, cos_sin, positions)
     c = proj[:, dkv_off:dkv_off + rank].float()
     c = c * torch.rsqrt(c.pow(2).mean(-1, keepdim=True) + eps) * norm_w
     pe = apply_rope(proj[:, dkv_off + rank:dkv_off + rank + rot].unsqueeze(1), positions, cos_sin, False).squeeze(1)
     cache.view(-1, cache.shape[-1])[loc.long(), :rank + rot] = torch.cat([c, pe.float()], -1).to(cache.dtype)
+    return c_q

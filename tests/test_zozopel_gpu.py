@@ -195,7 +195,8 @@ def test_expanded_latent_prefill(native, H, dim, rot, v, lens, pres, gain):
     kv, pe = rnd(sum(ctx), H * (dim + v)), rnd(sum(ctx), rot)
     out = torch.zeros(T, H, v, device="cuda", dtype=torch.bfloat16)
     qs, cs = np.concatenate([[0], np.cumsum(lens)]), np.concatenate([[0], np.cumsum(ctx)])
-    plan = SimpleNamespace(q_start=_i32(qs[:-1]), q_len=_i32(lens), prefix=_i32(pres), ctx_start=_i32(cs), long=len(lens),
+    plan = SimpleNamespace(q_start=_i32(qs[:-1]), q_len=_i32(lens), prefix=_i32(pres), long=len(lens),
+                           context=lambda window: SimpleNamespace(start=_i32(cs), skip=None),
                            num_tiles=sum((n + 255) // 256 for n in lens))
     assert native.latent_extend_supported(q, dim, rot, v, 64)
     native.latent_extend(q, kv, pe, out, plan, dim, v, (dim + rot) ** -0.5)
