@@ -102,8 +102,8 @@ def parse_args():
     ap.add_argument("--device", default=None)
     ap.add_argument("--log-level", default="error")
     ap.add_argument("--hybrid", action="store_true",
-                    help="instead of the headline workload: prefill / decode throughput of the hybrid recurrent "
-                         "decoders at equal sizes (sglang_jax_b200/bench_hybrid.py), one JSON line per size")
+                    help="instead of the headline workload: prefill / decode throughput of the decoders with mixed "
+                         "layers at equal sizes (sglang_jax_b200/bench_hybrid.py), one JSON line per size")
     ap.add_argument("--hybrid-size", nargs="*", default=None)
     ap.add_argument("--hybrid-models", nargs="*", default=None)
     ap.add_argument("--hang-timeout", type=float, default=float(os.environ.get("SGLB_BENCH_HANG_TIMEOUT", "300")),

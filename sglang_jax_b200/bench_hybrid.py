@@ -1,9 +1,10 @@
-"""Prefill and decode throughput of hybrid recurrent decoders at equal sizes, random weights: Zozopel (dense feed-forward)
-and Zidivik (routed experts) beside the framework's closest other models, Kimi-Linear (per-channel delta rule + latent
-attention) and Qwen3-Next (gated delta rule + grouped attention), with the feed-forward of the size.  Runs on the model
-runner, decode through its CUDA graphs.
+"""Prefill and decode throughput of decoders that mix kinds of layers at equal sizes, random weights: Zozopel (dense
+feed-forward) and Zidivik (routed experts) beside the framework's closest other models, Kimi-Linear (per-channel delta rule +
+latent attention) and Qwen3-Next (gated delta rule + grouped attention), and Kunudra (latent and grouped attention, routed and
+shared experts) beside DeepSeek-V3 (latent attention, routed and shared experts) and Qwen3-MoE (grouped attention, routed
+experts), with the feed-forward of the size.  Runs on the model runner, decode through its CUDA graphs.
 
-    python bench.py --hybrid [--hybrid-size base large moe moe-large] [--hybrid-models zozopel zidivik kimi_linear ...]
+    python bench.py --hybrid [--hybrid-size base large moe moe-large latent-moe ...] [--hybrid-models zozopel kunudra ...]
 
 One JSON line per size.  Times are CUDA events around the forward, median over the repetitions; a step streams the
 weights of all layers, more than the L2 holds."""
@@ -25,8 +26,21 @@ SIZES = {
     "moe": dict(width=2048, ff=768, experts=64, top=8, heads=16, kv_heads=8, rank=512, side=128, layers=8, vocab=32768),
     "moe-large": dict(width=4096, ff=1536, experts=64, top=4, heads=32, kv_heads=16, rank=512, side=256, layers=8,
                       vocab=32768),
+    # no recurrent layers: latent and grouped attention in turn, routed experts and a shared one; whole context as above
+    "latent-moe": dict(width=2048, ff=768, experts=64, top=8, identity=16, shared=768, heads=16, kv_heads=4, rank=512, q_rank=768,
+                       layers=8, vocab=32768),
+    "latent-moe-large": dict(width=4096, ff=1536, experts=64, top=4, identity=16, shared=1536, heads=32, kv_heads=8, rank=512,
+                             q_rank=1536, layers=8, vocab=32768),
 }
-MODELS = {False: ["zozopel", "kimi_linear", "qwen3_next"], True: ["zidivik", "kimi_linear", "qwen3_next"]}
+
+
+def models_of(size: dict) -> list[str]:
+    if "q_rank" in size:
+        return ["kunudra", "deepseek_v3", "qwen3_moe"]
+    return ["zidivik" if "experts" in size else "zozopel", "kimi_linear", "qwen3_next"]
+
+
+METRIC = "hybrid decoders, prefill and decode tokens/s"
 PREFILL = [(1, 4096), (4, 2048), (16, 512)]        # (sequences, new tokens each)
 DECODE = [(1, 2048), (32, 2048), (128, 2048)]      # (sequences, cached tokens each)
 
@@ -50,11 +64,31 @@ def model_config(name: str, s: dict) -> dict:
                  "mixer": dict(heads=s["heads"], kv_heads=s["kv_heads"], dim=128, vdim=128, conv=4)}
         return dict(architecture="Zidivik", vocab=s["vocab"], width=w, norm={"eps": 1e-6}, token_side={"dim": s["side"]},
                     layers=[attn if i % 2 else delta for i in range(n)])
+    if name == "kunudra":
+        mlp = {"kind": "moe", "expert": {"ff": s["ff"]}, "shared": {"ff": s["shared"]},
+               "router": {"experts": s["experts"], "top": s["top"], "identity": s["identity"], "scale": 1.0}}
+        lat = {"type": "latent_attention", "mlp": mlp,
+               "mixer": dict(heads=s["heads"], dim=128, rot_dim=64, vdim=128, kv_rank=s["rank"], q_rank=s["q_rank"],
+                             scale=192 ** -0.5, rot={"base": 10000.0, "dims": 64}, mask={"size": 8192})}
+        attn = {"type": "attention", "mlp": mlp,
+                "mixer": dict(heads=s["heads"], kv_heads=s["kv_heads"], dim=128, vdim=128, scale=128 ** -0.5, softcap=30.0,
+                              v_mix=True, mask={"size": 8192})}
+        return dict(architecture="Kunudra", vocab=s["vocab"], width=w, norm={"eps": 1e-6}, postln_alpha=2.0,
+                    embedding={"bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 7}},
+                    layers=[attn if i % 2 else lat for i in range(n)])
     experts = dict(num_experts=s["experts"], num_experts_per_tok=s["top"], moe_intermediate_size=s["ff"],
                    norm_topk_prob=True) if "experts" in s else dict(num_experts=0)
     common = dict(hidden_size=w, intermediate_size=s["ff"], num_hidden_layers=n, rms_norm_eps=1e-6,
                   vocab_size=s["vocab"], max_position_embeddings=32768, tie_word_embeddings=False,
                   torch_dtype="bfloat16", num_attention_heads=s["heads"])
+    if name == "deepseek_v3":
+        return dict(common, architectures=["DeepseekV3ForCausalLM"], model_type="deepseek_v3", num_key_value_heads=s["heads"],
+                    kv_lora_rank=s["rank"], q_lora_rank=s["q_rank"], qk_nope_head_dim=128, qk_rope_head_dim=64, v_head_dim=128,
+                    n_routed_experts=s["experts"], n_shared_experts=1, scoring_func="softmax", topk_method="noaux_tc",
+                    routed_scaling_factor=1.0, first_k_dense_replace=0, rope_theta=10000.0, **experts)
+    if name == "qwen3_moe":
+        return dict(common, architectures=["Qwen3MoeForCausalLM"], model_type="qwen3_moe", head_dim=128,
+                    num_key_value_heads=s["kv_heads"], rope_theta=10000.0, decoder_sparse_step=1, mlp_only_layers=[], **experts)
     if name == "kimi_linear":
         return dict(common, architectures=["KimiLinearForCausalLM"], model_type="kimi_linear",
                     num_key_value_heads=s["heads"], kv_lora_rank=s["rank"], q_lora_rank=None, qk_nope_head_dim=128,
@@ -180,14 +214,14 @@ def main(sizes=None, models=None) -> int:
 
     from .parallel import state as ps
     if not torch.cuda.is_available():
-        print(json.dumps({"metric": "hybrid decoders, prefill and decode tokens/s", "unavailable": "needs a CUDA device"}))
+        print(json.dumps({"metric": METRIC, "unavailable": "needs a CUDA device"}))
         return 0
     if not ps.get_state().initialized:
         ps.init_distributed(0, 1, "cuda")
     for s in sizes or list(SIZES):
-        out = {"metric": "hybrid decoders, prefill and decode tokens/s", "size": s, **SIZES[s], "dtype": "bf16",
+        out = {"metric": METRIC, "size": s, **SIZES[s], "dtype": "bf16",
                "data": "synthetic token ids, random weights", "models": {}}
-        for m in models or MODELS["experts" in SIZES[s]]:
+        for m in models or models_of(SIZES[s]):
             out["models"][m] = run_model(m, SIZES[s])
         print(json.dumps(out), flush=True)
     return 0

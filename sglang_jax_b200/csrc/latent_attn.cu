@@ -13,6 +13,8 @@
 // Compiled without fast-math substitutions.
 #include <math.h>
 
+#include <type_traits>
+
 #include "common.cuh"
 
 namespace sglb {
@@ -26,18 +28,6 @@ template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float
 
 constexpr int kPrepThreads = 128;
 
-// A block's sum of `v` in every thread; `red` holds one value per warp.
-__device__ __forceinline__ float prep_sum(float v, float* red) {
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
-  __syncthreads();
-  float tot = 0.f;
-#pragma unroll
-  for (int i = 0; i < kPrepThreads / 32; ++i) tot += red[i];
-  return tot;
-}
-
 // Queries that come from a latent: its columns in the projection, its norm's weight, the result [T, rank] (out null: none).
 struct QueryLatent {
   int off, rank;
@@ -45,81 +35,121 @@ struct QueryLatent {
   void* out;
 };
 
+// VEC consecutive values as one access (8 of bf16 or 4 of fp32: 16 bytes; 2: a rotary pair; 1: any alignment)
+template <typename T, int VEC> struct Vec { T v[VEC]; };
+template <> struct alignas(16) Vec<__nv_bfloat16, 8> { __nv_bfloat16 v[8]; };
+template <> struct alignas(16) Vec<float, 4> { float v[4]; };
+template <> struct alignas(4) Vec<__nv_bfloat16, 2> { __nv_bfloat16 v[2]; };
+template <> struct alignas(8) Vec<float, 2> { float v[2]; };
+
+// A warp's sum of squares of what its lanes read of src
+template <typename T, int VEC>
+__device__ __forceinline__ float squares(const T* __restrict__ src, int n) {
+  float ss = 0.f;
+  for (int i = threadIdx.x * VEC; i < n; i += kPrepThreads * VEC) {
+    const Vec<T, VEC> a = *reinterpret_cast<const Vec<T, VEC>*>(src + i);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) ss += to_f(a.v[e]) * to_f(a.v[e]);
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  return ss;
+}
+
+// dst = src * inv * w over n values
+template <typename T, int VEC>
+__device__ __forceinline__ void scaled_row(const T* __restrict__ src, T* __restrict__ dst, const float* __restrict__ w, int n,
+                                           float inv) {
+  for (int i = threadIdx.x * VEC; i < n; i += kPrepThreads * VEC) {
+    Vec<T, VEC> a = *reinterpret_cast<const Vec<T, VEC>*>(src + i);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) a.v[e] = from_f<T>(to_f(a.v[e]) * inv * w[i + e]);
+    *reinterpret_cast<Vec<T, VEC>*>(dst + i) = a;
+  }
+}
+
+// VEC / 2 interleaved pairs from pair i on; cs = [cos | sin] of the position, `half` each
+template <typename T, int VEC>
+__device__ __forceinline__ void rotate_pairs(const T* src, T* dst, const float* __restrict__ cs, int half, int i) {
+  constexpr int N = VEC < 2 ? 2 : VEC;
+  Vec<T, N> a;
+  if constexpr (VEC < 2) {
+    a.v[0] = src[0];
+    a.v[1] = src[1];
+  } else {
+    a = *reinterpret_cast<const Vec<T, N>*>(src);
+  }
+#pragma unroll
+  for (int e = 0; e < N; e += 2) {
+    const float u = to_f(a.v[e]), v = to_f(a.v[e + 1]), c = cs[i + e / 2], s = cs[half + i + e / 2];
+    a.v[e] = from_f<T>(u * c - v * s);
+    a.v[e + 1] = from_f<T>(v * c + u * s);
+  }
+  if constexpr (VEC < 2) {
+    dst[0] = a.v[0];
+    dst[1] = a.v[1];
+  } else {
+    *reinterpret_cast<Vec<T, N>*>(dst) = a;
+  }
+}
+
 // One CTA per token.  `proj` is the fused projection [T, ld]: query heads at column q_off, [latent | key part] at dkv_off.
-template <typename T>
+template <typename T, int VEC>
 __global__ void __launch_bounds__(kPrepThreads)
 latent_prep_kernel(T* __restrict__ proj, long long ld, int q_off, int dkv_off, int H, int dim, int rot, int R,
                    const float* __restrict__ norm_w, float eps, const float* __restrict__ cos_sin,
                    const int* __restrict__ positions, const int* __restrict__ loc, T* __restrict__ cache,
                    int row_elems, const QueryLatent ql) {
   __shared__ float red[2][kPrepThreads / 32];
+  constexpr int kPairs = VEC < 2 ? 1 : VEC / 2;
   pdl_wait();
   const int t = blockIdx.x, tid = threadIdx.x, half = rot / 2;
   T* row = proj + static_cast<long long>(t) * ld;
   const float* cs = cos_sin + static_cast<long long>(positions[t]) * rot;
   T* dst = cache + static_cast<long long>(loc[t]) * row_elems;
   const T* lat = row + dkv_off;
-  float ss = 0.f;
-  for (int i = tid; i < R; i += kPrepThreads) {
-    const float v = to_f(lat[i]);
-    ss += v * v;
+  for (int i = tid * kPairs; i < half; i += kPrepThreads * kPairs)
+    rotate_pairs<T, VEC>(lat + R + 2 * i, dst + R + 2 * i, cs, half, i);
+  const float s0 = squares<T, VEC>(lat, R), s1 = ql.out != nullptr ? squares<T, VEC>(row + ql.off, ql.rank) : 0.f;
+  if ((tid & 31) == 0) {
+    red[0][tid >> 5] = s0;
+    red[1][tid >> 5] = s1;
   }
-  const float inv = 1.f / sqrtf(prep_sum(ss, red[0]) / R + eps);
-  for (int i = tid; i < R; i += kPrepThreads) dst[i] = from_f<T>(to_f(lat[i]) * inv * norm_w[i]);
-  for (int i = tid; i < half; i += kPrepThreads) {
-    const float u = to_f(lat[R + 2 * i]), v = to_f(lat[R + 2 * i + 1]), c = cs[i], s = cs[half + i];
-    dst[R + 2 * i] = from_f<T>(u * c - v * s);
-    dst[R + 2 * i + 1] = from_f<T>(v * c + u * s);
+  __syncthreads();
+  float tot = 0.f, tot_q = 0.f;
+#pragma unroll
+  for (int i = 0; i < kPrepThreads / 32; ++i) {
+    tot += red[0][i];
+    tot_q += red[1][i];
   }
+  scaled_row<T, VEC>(lat, dst, norm_w, R, 1.f / sqrtf(tot / R + eps));
   if (ql.out != nullptr) {
-    const T* c = row + ql.off;
-    T* o = static_cast<T*>(ql.out) + static_cast<long long>(t) * ql.rank;
-    float sq = 0.f;
-    for (int i = tid; i < ql.rank; i += kPrepThreads) {
-      const float v = to_f(c[i]);
-      sq += v * v;
-    }
-    const float qi = 1.f / sqrtf(prep_sum(sq, red[1]) / ql.rank + eps);
-    for (int i = tid; i < ql.rank; i += kPrepThreads) o[i] = from_f<T>(to_f(c[i]) * qi * ql.norm_w[i]);
+    scaled_row<T, VEC>(row + ql.off, static_cast<T*>(ql.out) + static_cast<long long>(t) * ql.rank, ql.norm_w, ql.rank,
+                       1.f / sqrtf(tot_q / ql.rank + eps));
     return;
   }
-  for (int j = tid; j < H * half; j += kPrepThreads) {
-    const int h = j / half, i = j - h * half;
+  const int per = half / kPairs;
+  for (int j = tid; j < H * per; j += kPrepThreads) {
+    const int h = j / per, i = (j - h * per) * kPairs;
     T* q = row + q_off + static_cast<long long>(h) * (dim + rot) + dim + 2 * i;
-    const float u = to_f(q[0]), v = to_f(q[1]), c = cs[i], s = cs[half + i];
-    q[0] = from_f<T>(u * c - v * s);
-    q[1] = from_f<T>(v * c + u * s);
+    rotate_pairs<T, VEC>(q, q, cs, half, i);
   }
 }
 
-// Rotates the last `rot` of every head's `dim + rot` lanes in place, one pair per thread.
-template <typename T> struct Pair { T u, v; };
-template <> struct alignas(4) Pair<__nv_bfloat16> { __nv_bfloat16 u, v; };
-template <> struct alignas(8) Pair<float> { float u, v; };
-
-template <typename T, bool ALIGNED>
+// Rotates the last `rot` of every head's `dim + rot` lanes in place.
+template <typename T, int VEC>
 __global__ void __launch_bounds__(256)
-latent_rotate_kernel(T* __restrict__ q, long long ld, long long pairs, int H, int dim, int rot,
-                     const float* __restrict__ cos_sin, const int* __restrict__ positions) {
+latent_rotate_kernel(T* __restrict__ q, long long ld, int H, int dim, int rot, const float* __restrict__ cos_sin,
+                     const int* __restrict__ positions) {
+  constexpr int kPairs = VEC < 2 ? 1 : VEC / 2;
   pdl_wait();
-  const int half = rot / 2, per = H * half;
-  for (long long n = blockIdx.x * 256ll + threadIdx.x; n < pairs; n += gridDim.x * 256ll) {
-    const long long t = n / per;
-    const int j = static_cast<int>(n - t * per), h = j / half, i = j - h * half;
-    const float* cs = cos_sin + static_cast<long long>(positions[t]) * rot;
-    T* a = q + t * ld + static_cast<long long>(h) * (dim + rot) + dim + 2 * i;
-    Pair<T> p;
-    if constexpr (ALIGNED) p = *reinterpret_cast<const Pair<T>*>(a);
-    else p = Pair<T>{a[0], a[1]};
-    const float u = to_f(p.u), v = to_f(p.v), c = cs[i], s = cs[half + i];
-    p.u = from_f<T>(u * c - v * s);
-    p.v = from_f<T>(v * c + u * s);
-    if constexpr (ALIGNED) {
-      *reinterpret_cast<Pair<T>*>(a) = p;
-    } else {
-      a[0] = p.u;
-      a[1] = p.v;
-    }
+  const int half = rot / 2, per = half / kPairs;
+  const float* cs = cos_sin + static_cast<long long>(positions[blockIdx.x]) * rot;
+  T* row = q + blockIdx.x * ld + dim;
+  for (int j = threadIdx.x; j < H * per; j += blockDim.x) {
+    const int h = j / per, i = (j - h * per) * kPairs;
+    T* a = row + static_cast<long long>(h) * (dim + rot) + 2 * i;
+    rotate_pairs<T, VEC>(a, a, cs, half, i);
   }
 }
 
@@ -256,13 +286,18 @@ int sglb_latent_prep(void* proj, long long ld, int q_off, int dkv_off, int T, in
   if (rot % 2 != 0 || row_elems < R + rot || (q_latent != nullptr && (q_rank < 1 || q_norm_w == nullptr)))
     return -kBadArgument;
   const QueryLatent ql{q_off, q_rank, q_norm_w, q_latent};
-  if (is_f32)
-    launch_pdl(latent_prep_kernel<float>, dim3(T), dim3(kPrepThreads), 0, s, static_cast<float*>(proj), ld, q_off, dkv_off,
-               H, dim, rot, R, norm_w, eps, cos_sin, positions, loc, static_cast<float*>(cache), row_elems, ql);
-  else
-    launch_pdl(latent_prep_kernel<__nv_bfloat16>, dim3(T), dim3(kPrepThreads), 0, s, static_cast<__nv_bfloat16*>(proj), ld,
-               q_off, dkv_off, H, dim, rot, R, norm_w, eps, cos_sin, positions, loc, static_cast<__nv_bfloat16*>(cache),
-               row_elems, ql);
+  const int n = is_f32 ? 4 : 8;
+  auto whole = [&](long long v) { return v % n == 0; };
+  const bool wide = whole(ld) && whole(dkv_off) && whole(R) && whole(rot) && whole(row_elems) && whole(q_off) &&
+                    (q_latent != nullptr ? whole(q_rank) : whole(dim)) && reinterpret_cast<uintptr_t>(proj) % 16 == 0;
+  auto run = [&](auto kernel, auto* p) {
+    using T_ = std::remove_pointer_t<decltype(p)>;
+    launch_pdl(kernel, dim3(T), dim3(kPrepThreads), 0, s, p, ld, q_off, dkv_off, H, dim, rot, R, norm_w, eps, cos_sin,
+               positions, loc, static_cast<T_*>(cache), row_elems, ql);
+  };
+  if (is_f32) run(wide ? latent_prep_kernel<float, 4> : latent_prep_kernel<float, 1>, static_cast<float*>(proj));
+  else run(wide ? latent_prep_kernel<__nv_bfloat16, 8> : latent_prep_kernel<__nv_bfloat16, 1>,
+           static_cast<__nv_bfloat16*>(proj));
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -272,16 +307,20 @@ int sglb_latent_rotate(void* q, long long ld, int T, int H, int dim, int rot, co
   using namespace sglb;
   if (T <= 0 || rot == 0) return 0;
   if (rot % 2 != 0 || H < 1) return -kBadArgument;
-  const long long pairs = static_cast<long long>(T) * H * (rot / 2), blocks = (pairs + 255) / 256;
-  const dim3 grid(static_cast<unsigned>(blocks < 148LL * 32 ? blocks : 148LL * 32));
-  const bool aligned = dim % 2 == 0 && ld % 2 == 0 && reinterpret_cast<uintptr_t>(q) % 8 == 0;
-  if (is_f32) {
-    const auto kernel = aligned ? latent_rotate_kernel<float, true> : latent_rotate_kernel<float, false>;
-    launch_pdl(kernel, grid, dim3(256), 0, s, static_cast<float*>(q), ld, pairs, H, dim, rot, cos_sin, positions);
-  } else {
-    const auto kernel = aligned ? latent_rotate_kernel<__nv_bfloat16, true> : latent_rotate_kernel<__nv_bfloat16, false>;
-    launch_pdl(kernel, grid, dim3(256), 0, s, static_cast<__nv_bfloat16*>(q), ld, pairs, H, dim, rot, cos_sin, positions);
-  }
+  const int n = is_f32 ? 4 : 8;
+  const uintptr_t at = reinterpret_cast<uintptr_t>(q);
+  const bool wide = ld % n == 0 && dim % n == 0 && rot % n == 0 && at % 16 == 0;
+  const bool pairs = ld % 2 == 0 && dim % 2 == 0 && at % 8 == 0;
+  auto run = [&](auto kernel, auto* p) {
+    launch_pdl(kernel, dim3(T), dim3(256), 0, s, p, ld, H, dim, rot, cos_sin, positions);
+  };
+  if (is_f32)
+    run(wide ? latent_rotate_kernel<float, 4> : (pairs ? latent_rotate_kernel<float, 2> : latent_rotate_kernel<float, 1>),
+        static_cast<float*>(q));
+  else
+    run(wide ? latent_rotate_kernel<__nv_bfloat16, 8>
+             : (pairs ? latent_rotate_kernel<__nv_bfloat16, 2> : latent_rotate_kernel<__nv_bfloat16, 1>),
+        static_cast<__nv_bfloat16*>(q));
   return static_cast<int>(cudaGetLastError());
 }
 

@@ -24,26 +24,24 @@ template <typename T> __device__ __forceinline__ T from_f(float v);
 template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
 template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
 
-// kAtOnce dot products with one vector over a warp's lanes: rows w, w + ld, ... (those below `rows`); every load of a step is
-// in flight at the same time
-constexpr int kAtOnce = 4;
-
-template <typename T>
+// N dot products with one vector over a warp's lanes: rows w, w + ld, ... (those below `rows`); every load of a step is in flight
+// at the same time
+template <typename T, int N>
 __device__ __forceinline__ void warp_dots(const T* __restrict__ w, long long ld, int rows, const float* __restrict__ x, int K,
-                                          int lane, bool wide, float (&a)[kAtOnce]) {
+                                          int lane, bool wide, float (&a)[N]) {
 #pragma unroll
-  for (int r = 0; r < kAtOnce; ++r) a[r] = 0.f;
+  for (int r = 0; r < N; ++r) a[r] = 0.f;
   if (sizeof(T) == 2 && wide) {
 #pragma unroll 2
     for (int i = lane * 8; i < K; i += 256) {
-      uint4 v[kAtOnce];
+      uint4 v[N];
 #pragma unroll
-      for (int r = 0; r < kAtOnce; ++r)
+      for (int r = 0; r < N; ++r)
         v[r] = r < rows ? *reinterpret_cast<const uint4*>(w + r * ld + i) : make_uint4(0, 0, 0, 0);
       const float4 p = *reinterpret_cast<const float4*>(x + i), q = *reinterpret_cast<const float4*>(x + i + 4);
       const float f[8] = {p.x, p.y, p.z, p.w, q.x, q.y, q.z, q.w};
 #pragma unroll
-      for (int r = 0; r < kAtOnce; ++r) {
+      for (int r = 0; r < N; ++r) {
         const uint32_t u[4] = {v[r].x, v[r].y, v[r].z, v[r].w};
 #pragma unroll
         for (int e = 0; e < 4; ++e)
@@ -53,11 +51,11 @@ __device__ __forceinline__ void warp_dots(const T* __restrict__ w, long long ld,
   } else {
     for (int i = lane; i < K; i += 32)
 #pragma unroll
-      for (int r = 0; r < kAtOnce; ++r)
+      for (int r = 0; r < N; ++r)
         if (r < rows) a[r] += to_f(w[r * ld + i]) * x[i];
   }
 #pragma unroll
-  for (int r = 0; r < kAtOnce; ++r)
+  for (int r = 0; r < N; ++r)
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) a[r] += __shfl_xor_sync(0xffffffffu, a[r], o);
 }
@@ -149,7 +147,7 @@ __device__ __forceinline__ void choose_by_score(float* z, float* s, int E, int k
 }
 
 // One CTA per token: the warps share the experts' dot products, the first one chooses.
-template <typename T>
+template <typename T, int kAtOnce>
 __global__ void __launch_bounds__(kRouteThreads)
 route_token_kernel(const T* __restrict__ x, const T* __restrict__ w, const T* __restrict__ bias, float* __restrict__ out_w,
                    int* __restrict__ out_ids, int E, int K, int k, int wide, const ScoreRule rule) {
@@ -180,7 +178,7 @@ route_token_kernel(const T* __restrict__ x, const T* __restrict__ w, const T* __
 template <typename T>
 __global__ void __launch_bounds__(128)
 route_logits_kernel(const float* __restrict__ logits, const T* __restrict__ bias, float* __restrict__ out_w,
-                    int* __restrict__ out_ids, int T_, int E, int k, const ScoreRule rule) {
+                    int* __restrict__ out_ids, int T_, int E, int k, int ld, const ScoreRule rule) {
   extern __shared__ float4 sm4[];
   pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -188,7 +186,7 @@ route_logits_kernel(const float* __restrict__ logits, const T* __restrict__ bias
   if (t >= T_) return;
   const int n = rule.logits(E);
   float* z = reinterpret_cast<float*>(sm4) + warp * (n + E);
-  for (int e = lane; e < n; e += 32) z[e] = logits[t * n + e] + (bias != nullptr ? to_f(bias[e]) : 0.f);
+  for (int e = lane; e < n; e += 32) z[e] = logits[t * ld + e] + (bias != nullptr ? to_f(bias[e]) : 0.f);
   __syncwarp();
   if (rule.on) choose_by_score(z, z + n, E, k, rule, t, out_w + t * k, out_ids + t * k, lane);
   else choose(z, E, k, out_w + t * k, out_ids + t * k, lane);
@@ -251,29 +249,37 @@ grouped_gemm_any_kernel(const T* __restrict__ x, const int* __restrict__ row_tok
         out[static_cast<size_t>(r0 + tr + i) * N + n0 + tc + j] = from_f<T>(acc[i][j]);
 }
 
+template <typename T, int kAtOnce>
+int route_token(const void* x, const void* w, const T* bias, float* out_w, int* out_ids, int T_, int E, int K, int k,
+                const ScoreRule& rule, cudaStream_t s) {
+  const size_t smem = ((K + 3) / 4 * 4 + rule.logits(E) + E) * sizeof(float);
+  if (smem > 48 * 1024) {
+    static size_t cfg = 0;
+    if (cfg < smem) {
+      const cudaError_t e = cudaFuncSetAttribute(route_token_kernel<T, kAtOnce>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                                 static_cast<int>(smem));
+      if (e != cudaSuccess) return static_cast<int>(e);
+      cfg = smem;
+    }
+  }
+  const int wide = K % 8 == 0 && reinterpret_cast<uintptr_t>(w) % 16 == 0;
+  launch_pdl(route_token_kernel<T, kAtOnce>, dim3(T_), dim3(kRouteThreads), smem, s, static_cast<const T*>(x),
+             static_cast<const T*>(w), bias, out_w, out_ids, E, K, k, wide, rule);
+  return static_cast<int>(cudaGetLastError());
+}
+
+// ld: row stride of the given logits
 template <typename T>
 int route(const float* z, const void* x, const void* w, const void* bias, float* out_w, int* out_ids, int T_, int E, int K,
-          int k, const ScoreRule& rule, cudaStream_t s) {
+          int k, int ld, const ScoreRule& rule, cudaStream_t s) {
   const T* b = static_cast<const T*>(bias);
-  const int held = rule.logits(E) + E;                 // floats per token for the choice
-  if (z != nullptr) {
-    launch_pdl(route_logits_kernel<T>, dim3((T_ + 3) / 4), dim3(128), 4 * held * sizeof(float), s, z, b, out_w, out_ids, T_,
-               E, k, rule);
-  } else {
-    const size_t smem = ((K + 3) / 4 * 4 + held) * sizeof(float);
-    if (smem > 48 * 1024) {
-      static size_t cfg = 0;
-      if (cfg < smem) {
-        const cudaError_t e = cudaFuncSetAttribute(route_token_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                                   static_cast<int>(smem));
-        if (e != cudaSuccess) return static_cast<int>(e);
-        cfg = smem;
-      }
-    }
-    const int wide = K % 8 == 0 && reinterpret_cast<uintptr_t>(w) % 16 == 0;
-    launch_pdl(route_token_kernel<T>, dim3(T_), dim3(kRouteThreads), smem, s, static_cast<const T*>(x),
-               static_cast<const T*>(w), b, out_w, out_ids, E, K, k, wide, rule);
-  }
+  const int n = rule.logits(E);
+  // one round of the warps over the rows where that is possible
+  if (z == nullptr)
+    return n <= kRouteThreads / 32 * 4 ? route_token<T, 4>(x, w, b, out_w, out_ids, T_, E, K, k, rule, s)
+                                       : route_token<T, 8>(x, w, b, out_w, out_ids, T_, E, K, k, rule, s);
+  launch_pdl(route_logits_kernel<T>, dim3((T_ + 3) / 4), dim3(128), 4 * (n + E) * sizeof(float), s, z, b, out_w, out_ids, T_, E,
+             k, ld, rule);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -289,20 +295,20 @@ int sglb_route_by_logit(const float* z, const void* x, const void* w, const void
   if (T <= 0) return 0;
   if (E < 1 || E > kMaxExperts || k < 1 || k > kMaxTop || k > E || K < 1 || K > 32768) return -kBadArgument;
   const ScoreRule rule{0, nullptr, 1.f, nullptr};
-  return is_f32 ? route<float>(z, x, w, bias, out_w, out_ids, T, E, K, k, rule, s)
-                : route<__nv_bfloat16>(z, x, w, bias, out_w, out_ids, T, E, K, k, rule, s);
+  return is_f32 ? route<float>(z, x, w, bias, out_w, out_ids, T, E, K, k, E, rule, s)
+                : route<__nv_bfloat16>(z, x, w, bias, out_w, out_ids, T, E, K, k, E, rule, s);
 }
 
-// w [E, K], with `gate` [T] one row more, whose product's sigmoid goes there; z [T, rows of w] fp32: products computed
-// elsewhere, or null.  correction [E] or null.
+// w [rows, K], of which the first E are the choices', with `gate` [T] the next one's product's sigmoid goes there (rows beyond:
+// padding); z [T, rows] fp32: products computed elsewhere, or null.  correction [E] or null.
 int sglb_route_by_score(const float* z, const void* x, const void* w, const float* correction, float* out_w, int* out_ids,
-                        float* gate, int T, int E, int K, int k, float scale, int is_f32, cudaStream_t s) {
+                        float* gate, int T, int rows, int E, int K, int k, float scale, int is_f32, cudaStream_t s) {
   using namespace sglb;
   if (T <= 0) return 0;
-  if (E < 1 || E > kMaxExperts || k < 1 || k > kMaxTop || k > E || K < 1 || K > 32768) return -kBadArgument;
+  if (rows < E + (gate != nullptr) || E < 1 || E > kMaxExperts || k < 1 || k > kMaxTop || k > E || K < 1 || K > 32768) return -kBadArgument;
   const ScoreRule rule{1, correction, scale, gate};
-  return is_f32 ? route<float>(z, x, w, nullptr, out_w, out_ids, T, E, K, k, rule, s)
-                : route<__nv_bfloat16>(z, x, w, nullptr, out_w, out_ids, T, E, K, k, rule, s);
+  return is_f32 ? route<float>(z, x, w, nullptr, out_w, out_ids, T, E, K, k, rows, rule, s)
+                : route<__nv_bfloat16>(z, x, w, nullptr, out_w, out_ids, T, E, K, k, rows, rule, s);
 }
 
 // x rows of K, row_token [rows] or null (row r reads x row r), w [groups, N, K], out [rows, N]; lists from sglb_moe_align.

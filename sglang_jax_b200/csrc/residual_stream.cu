@@ -28,7 +28,11 @@ namespace {
 
 // VEC consecutive elements: 8 (bf16 only, 16 bytes), 4 (8 / 16 bytes) or 1 (any alignment)
 template <int VEC> __device__ __forceinline__ void load_v(const float* p, float (&f)[VEC]) {
-  if constexpr (VEC == 4) {
+  if constexpr (VEC == 8) {
+    const float4 v = *reinterpret_cast<const float4*>(p), w = *reinterpret_cast<const float4*>(p + 4);
+    f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+    f[4] = w.x; f[5] = w.y; f[6] = w.z; f[7] = w.w;
+  } else if constexpr (VEC == 4) {
     const float4 v = *reinterpret_cast<const float4*>(p);
     f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
   } else {
@@ -54,8 +58,14 @@ template <int VEC> __device__ __forceinline__ void load_v(const __nv_bfloat16* p
   }
 }
 template <int VEC> __device__ __forceinline__ void store_v(float* p, const float (&f)[VEC]) {
-  if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
-  else *p = f[0];
+  if constexpr (VEC == 8) {
+    *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+    *reinterpret_cast<float4*>(p + 4) = make_float4(f[4], f[5], f[6], f[7]);
+  } else if constexpr (VEC == 4) {
+    *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  } else {
+    *p = f[0];
+  }
 }
 template <int VEC> __device__ __forceinline__ void store_v(__nv_bfloat16* p, const float (&f)[VEC]) {
   if constexpr (VEC == 8)
@@ -178,8 +188,14 @@ struct SumNorm {
   int W;
 };
 
-template <typename T, int VEC, int VPT, bool NEXT>
-__global__ void sum_norm_kernel(const SumNorm p) {
+constexpr int kRowsAtOnce = 4, kSumThreads = 512;
+
+// VEC elements as they lie in memory
+template <typename T, int VEC> struct alignas(sizeof(T) * VEC) Raw { T v[VEC]; };
+
+template <typename T, int VEC, int VPT, bool NEXT, bool EXPERTS>
+__global__ void __launch_bounds__(kSumThreads, VPT == 1 ? 2 : 1)
+sum_norm_kernel(const SumNorm p) {
   __shared__ float red[64];
   pdl_wait();
   const size_t t = blockIdx.x, row = t * p.W;
@@ -195,22 +211,32 @@ __global__ void sum_norm_kernel(const SumNorm p) {
   for (int i = 0; i < VPT; ++i) {
     const int c = (threadIdx.x + i * blockDim.x) * VEC;
     if (c < p.W) {
-      float v[VEC], xv[VEC], s[VEC];
+      float v[VEC], xv[VEC];
       load_v<VEC>(y + row + c, v);
       load_v<VEC>(p.x + row + c, xv);
-      load_v<VEC>(p.scale + c, s);
 #pragma unroll
       for (int e = 0; e < VEC; ++e) v[e] = v[e] * gate + own * xv[e];
-      if (expert != nullptr)
-        for (int j = 0; j < p.k; ++j) {
-          const int r = p.rows[t * p.k + j];
-          if (r < 0) continue;
-          const float w = p.weights[t * p.k + j];
-          float g[VEC];
-          load_v<VEC>(expert + static_cast<size_t>(r) * p.W + c, g);
+      if constexpr (EXPERTS) {
+        for (int j0 = 0; j0 < p.k; j0 += kRowsAtOnce) {
+          Raw<T, VEC> g[kRowsAtOnce] = {};
+          float w[kRowsAtOnce];
 #pragma unroll
-          for (int e = 0; e < VEC; ++e) v[e] += w * g[e];
+          for (int u = 0; u < kRowsAtOnce; ++u) {        // all on their way before the first is used
+            const int j = j0 + u, r = j < p.k ? p.rows[t * p.k + j] : -1;
+            w[u] = 0.f;
+            if (r >= 0) {
+              w[u] = p.weights[t * p.k + j];
+              g[u] = *reinterpret_cast<const Raw<T, VEC>*>(expert + static_cast<size_t>(r) * p.W + c);
+            }
+          }
+#pragma unroll
+          for (int u = 0; u < kRowsAtOnce; ++u)
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) v[e] += w[u] * static_cast<float>(g[u].v[e]);
         }
+      }
+      float s[VEC];
+      load_v<VEC>(p.scale + c, s);
 #pragma unroll
       for (int e = 0; e < VEC; ++e) {
         z[i][e] = p.alpha * xv[e] + s[e] * v[e];
@@ -232,8 +258,9 @@ __global__ void sum_norm_kernel(const SumNorm p) {
         ss += z[i][e] * z[i][e];
       }
       store_v<VEC>(p.x + row + c, z[i]);
-      if constexpr (!NEXT)
+      if constexpr (!NEXT) {
         if (xt != nullptr) store_v<VEC>(xt + row + c, z[i]);
+      }
     }
   }
   if constexpr (NEXT) {
@@ -524,12 +551,26 @@ int embed_pair(float* x, void* xt, const int* ids, const void* table, long long 
 
 template <typename T>
 int sum_norm(const SumNorm& p, long long n, cudaStream_t s) {
-  int threads = 0;
-  const bool ok = for_row(p.W, p.W % 4 == 0, &threads, [&]<int VEC, int VPT>() {
-    const auto kernel = p.next_weight != nullptr ? sum_norm_kernel<T, VEC, VPT, true> : sum_norm_kernel<T, VEC, VPT, false>;
+  constexpr int kWide = sizeof(T) == 2 ? 8 : 4;
+  const int groups = p.W % kWide == 0 ? p.W / kWide : p.W;
+  const int threads = row_threads(groups) < kSumThreads ? row_threads(groups) : kSumThreads;
+  const int vpt = (groups + threads - 1) / threads;
+  if (vpt > 16) return -kBadArgument;
+  auto run = [&]<int VEC, int VPT>() {
+    const bool next = p.next_weight != nullptr, experts = p.expert != nullptr;
+    const auto kernel = next ? (experts ? sum_norm_kernel<T, VEC, VPT, true, true> : sum_norm_kernel<T, VEC, VPT, true, false>)
+                             : (experts ? sum_norm_kernel<T, VEC, VPT, false, true> : sum_norm_kernel<T, VEC, VPT, false, false>);
     launch_pdl(kernel, dim3(n), dim3(threads), 0, s, p);
-  });
-  return ok ? static_cast<int>(cudaGetLastError()) : -kBadArgument;
+  };
+  auto rows = [&]<int VEC>() {
+    if (vpt <= 1) run.template operator()<VEC, 1>();
+    else if (vpt <= 2) run.template operator()<VEC, 2>();
+    else if (vpt <= 4) run.template operator()<VEC, 4>();
+    else run.template operator()<VEC, 16>();
+  };
+  if (p.W % kWide == 0) rows.template operator()<kWide>();
+  else rows.template operator()<1>();
+  return static_cast<int>(cudaGetLastError());
 }
 
 template <typename T>

@@ -30,6 +30,7 @@ template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float
 // ------------------------------------------------------------------------------------------- prep
 template <typename T, int VEC> struct Pack { T v[VEC]; };
 template <> struct alignas(8) Pack<__nv_bfloat16, 4> { __nv_bfloat16 v[4]; };
+template <> struct alignas(16) Pack<__nv_bfloat16, 8> { __nv_bfloat16 v[8]; };
 template <> struct alignas(16) Pack<float, 4> { float v[4]; };
 
 struct PrepParams {
@@ -112,6 +113,8 @@ attn_prep_rows_kernel(const T* __restrict__ proj, T* __restrict__ q, T* __restri
   const long long t = blockIdx.x;
   const int tid = threadIdx.x;
   const T* row = proj + t * p.ld;
+  const int slot = loc[t], page = slot / p.P;
+  const float v_share = r.v_mix != nullptr ? *r.share : 0.f;
   float sq = 0.f, sk = 0.f;
   if (r.sq != nullptr) {
     sq = r.sq[2 * t];
@@ -164,13 +167,12 @@ attn_prep_rows_kernel(const T* __restrict__ proj, T* __restrict__ q, T* __restri
       *reinterpret_cast<Pack<T, VEC>*>(dst + h * stride + c) = a;
     }
   };
-  const int slot = loc[t], page = slot / p.P;
   const long long width = p.Dp + p.Vp, head = width * p.P;       // cache row, and from one head's rows to the next one's
   T* dst = cache + static_cast<long long>(page) * p.G * head + (slot - page * p.P) * width;
   write(row + p.q_off, r.q_w, iq, nullptr, 0.f, p.H, p.D, p.Dp, q + t * p.H * p.Dp, p.Dp);
   write(row + p.k_off, r.k_w, ik, nullptr, 0.f, p.G, p.D, p.Dp, dst, head);
   const T* mix = r.v_mix != nullptr ? static_cast<const T*>(r.v_mix) + t * r.v_mix_ld : nullptr;
-  write(row + p.v_off, nullptr, 0.f, mix, mix != nullptr ? *r.share : 0.f, p.G, p.V, p.Vp, dst + p.Dp, head);
+  write(row + p.v_off, nullptr, 0.f, mix, v_share, p.G, p.V, p.Vp, dst + p.Dp, head);
 }
 
 // ------------------------------------------------------------------------------------------- decode
@@ -580,10 +582,12 @@ template <typename T>
 int prep_rows(const void* proj, void* q, void* cache, const int* loc, long long tokens, const RowPrepParams& r,
               cudaStream_t s) {
   const PrepParams& p = r.b;
-  const bool vec = p.D % 4 == 0 && p.V % 4 == 0 && p.ld % 4 == 0 && p.q_off % 4 == 0 && p.k_off % 4 == 0 &&
-                   p.v_off % 4 == 0 && r.v_mix_ld % 4 == 0 && reinterpret_cast<uintptr_t>(proj) % (4 * sizeof(T)) == 0 &&
-                   reinterpret_cast<uintptr_t>(r.v_mix) % (4 * sizeof(T)) == 0;
-  const auto kernel = vec ? attn_prep_rows_kernel<T, 4> : attn_prep_rows_kernel<T, 1>;
+  constexpr int kWide = sizeof(T) == 2 ? 8 : 4;
+  auto whole = [](long long v) { return v % kWide == 0; };
+  const bool vec = whole(p.D) && whole(p.V) && whole(p.ld) && whole(p.q_off) && whole(p.k_off) && whole(p.v_off) &&
+                   whole(r.v_mix_ld) && reinterpret_cast<uintptr_t>(proj) % 16 == 0 &&
+                   reinterpret_cast<uintptr_t>(r.v_mix) % 16 == 0;
+  const auto kernel = vec ? attn_prep_rows_kernel<T, kWide> : attn_prep_rows_kernel<T, 1>;
   launch_pdl(kernel, dim3(static_cast<unsigned>(tokens)), dim3(kRowThreads), 0, s, static_cast<const T*>(proj),
              static_cast<T*>(q), static_cast<T*>(cache), loc, r);
   return static_cast<int>(cudaGetLastError());

@@ -39,6 +39,7 @@ struct Bars {
   uint64_t s_full[kTiles][2], p_ready[kTiles][2], pv_done[kTiles][2];
   uint32_t tmem_slot;
   int abort_flag;
+  alignas(16) float bias[kTileK];       // slope of the head times the key's place in its tile, in log2 units
 };
 
 struct Params {
@@ -61,11 +62,11 @@ __device__ __forceinline__ float ex2_approx(float x) {
   return y;
 }
 
-// cap tanh(s scale / cap) + bias in log2 units: c2 = cap log2 e, a = 2 scale log2 e / cap
+// cap tanh(s scale / cap) - cap + bias in log2 units: c2 = 2 cap log2 e, a = 2 scale log2 e / cap
 __device__ __forceinline__ float capped(float s, float a, float c2, float bias) {
   float r;
-  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + ex2_approx(fminf(s * a, 60.f))));
-  return fmaf(-2.f * c2, r, c2 + bias);
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + ex2_approx(s * a)));
+  return fmaf(-c2, r, bias);
 }
 
 // SHAPED: scores are capped or biased
@@ -128,6 +129,9 @@ window_extend_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
     }
     bars->abort_flag = 0;
     fence_barrier_init();
+  }
+  if constexpr (SHAPED) {
+    if (threadIdx.x < kTileK) bars->bias[threadIdx.x] = p.terms.slope_of(head) * kLog2E * static_cast<float>(threadIdx.x);
   }
   if (warp == 1) {
     tmem_alloc(smem_u32(&bars->tmem_slot), kTmemCols);
@@ -276,19 +280,31 @@ window_extend_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
       auto below = [](int c) -> uint64_t { return c <= 0 ? 0ull : (c >= 64 ? ~0ull : (1ull << c) - 1); };
       const uint64_t seen = below(pos - k0 + 1) & (~below(kmin - k0) | below(p.win.keep - k0));
       const bool full = seen == ~0ull;
+      float base = 0.f;                                             // what all keys of the tile have in common is added late
       if constexpr (SHAPED) {                                       // capped and biased scores, in log2 units
-        const float base = slope * static_cast<float>(k0 - pos);
+        base = slope * static_cast<float>(k0 - pos);
+        const float4* bias = reinterpret_cast<const float4*>(bars->bias);
         if (p.terms.cap > 0.f) {
+          base += p.cap_log2;
+          const float c2 = 2.f * p.cap_log2;
 #pragma unroll
-          for (int e = 0; e < 32; ++e) {
-            v0[e] = __float_as_uint(capped(__uint_as_float(v0[e]), p.cap_arg, p.cap_log2, fmaf(slope, e, base)));
-            v1[e] = __float_as_uint(capped(__uint_as_float(v1[e]), p.cap_arg, p.cap_log2, fmaf(slope, e + 32, base)));
+          for (int e = 0; e < 64; e += 4) {
+            const float4 t4 = bias[e / 4];
+            uint32_t* v = e < 32 ? v0 + e : v1 + (e - 32);
+            v[0] = __float_as_uint(capped(__uint_as_float(v[0]), p.cap_arg, c2, t4.x));
+            v[1] = __float_as_uint(capped(__uint_as_float(v[1]), p.cap_arg, c2, t4.y));
+            v[2] = __float_as_uint(capped(__uint_as_float(v[2]), p.cap_arg, c2, t4.z));
+            v[3] = __float_as_uint(capped(__uint_as_float(v[3]), p.cap_arg, c2, t4.w));
           }
         } else {
 #pragma unroll
-          for (int e = 0; e < 32; ++e) {
-            v0[e] = __float_as_uint(fmaf(__uint_as_float(v0[e]), p.scale_log2, fmaf(slope, e, base)));
-            v1[e] = __float_as_uint(fmaf(__uint_as_float(v1[e]), p.scale_log2, fmaf(slope, e + 32, base)));
+          for (int e = 0; e < 64; e += 4) {
+            const float4 t4 = bias[e / 4];
+            uint32_t* v = e < 32 ? v0 + e : v1 + (e - 32);
+            v[0] = __float_as_uint(fmaf(__uint_as_float(v[0]), p.scale_log2, t4.x));
+            v[1] = __float_as_uint(fmaf(__uint_as_float(v[1]), p.scale_log2, t4.y));
+            v[2] = __float_as_uint(fmaf(__uint_as_float(v[2]), p.scale_log2, t4.z));
+            v[3] = __float_as_uint(fmaf(__uint_as_float(v[3]), p.scale_log2, t4.w));
           }
         }
       }
@@ -304,7 +320,7 @@ window_extend_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
           if ((see1 >> e) & 1) mx = fmaxf(mx, __uint_as_float(v1[e]));
         }
       }
-      mx *= scale_log2;
+      mx = SHAPED ? mx + base : mx * scale_log2;
       const bool raise = lj > 0 && mx > m_used + kRescale;
       if (lj == 0) {
         m_used = mx;
@@ -333,7 +349,7 @@ window_extend_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
         if (raise) m_used = mx;
       }
       float sum = 0.f;
-      const float ref = m_used == -INFINITY ? 0.f : m_used;         // (nothing seen so far)
+      const float ref = (m_used == -INFINITY ? 0.f : m_used) - base;         // (nothing seen so far)
       uint32_t hi[32], lo[32];
 #pragma unroll
       for (int c = 0; c < 32; ++c) {
@@ -411,7 +427,7 @@ window_extend_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
 }
 
 int extend_smem(int nb_k, int nb_v) {
-  const int need = kTiles * nb_k * kBlkQ + 2 * (nb_k + nb_v) * kBlkK + 256 + 1024;
+  const int need = kTiles * nb_k * kBlkQ + 2 * (nb_k + nb_v) * kBlkK + 512 + 1024;
   return need > kMinSmem ? need : kMinSmem;
 }
 

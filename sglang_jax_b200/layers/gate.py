@@ -17,10 +17,13 @@ class GateLogit(nn.Module):
 
     def __init__(self, hidden_size: int, num_experts: int, dtype=torch.bfloat16, use_bias: bool = False,
                  score_func: str = "softmax", correction_bias: bool = False, token_gate: bool = False):
-        """`token_gate`: one more row behind the experts', whose product gates something per token (`route_by_score`)."""
+        """`token_gate`: one more row behind the experts', whose product gates something per token (`route_by_score`); then the
+        rows are padded with zeros to whole 16-byte units of a product's row."""
         super().__init__()
-        self.token_gate = token_gate
-        self.weight = nn.Parameter(torch.empty(num_experts + token_gate, hidden_size, dtype=dtype), requires_grad=False)
+        self.num_experts, self.token_gate = num_experts, token_gate
+        rows = -(-(num_experts + 1) // 8) * 8 if token_gate else num_experts
+        fill = torch.zeros if token_gate else torch.empty
+        self.weight = nn.Parameter(fill(rows, hidden_size, dtype=dtype), requires_grad=False)
         self.bias = nn.Parameter(torch.zeros(num_experts, dtype=dtype), requires_grad=False) if use_bias else None
         self.e_score_correction_bias = nn.Parameter(torch.zeros(num_experts, dtype=torch.float32),
                                                     requires_grad=False) if correction_bias else None
@@ -41,7 +44,8 @@ class GateLogit(nn.Module):
     def route_by_score(self, x: torch.Tensor, top_k: int, scale: float):
         """The experts with the largest corrected softmax scores, weights their scores times `scale`, not renormalised: `(weights
         fp32, ids int32, gate)`; `gate` fp32 `[T]`: sigmoid of the gate row's product, or None."""
-        return ops.route_by_score(x, self.weight, self.e_score_correction_bias, top_k, scale, self.token_gate)
+        return ops.route_by_score(x, self.weight, self.e_score_correction_bias, top_k, scale, self.num_experts,
+                                  self.token_gate)
 
 
 class TopK(nn.Module):

@@ -446,7 +446,7 @@ class ScoredFeedForward(nn.Module):
             param = self.experts.w2_weight if shard == "down" else self.experts.w13_weight
             return self.experts.weight_loader(param, w, shard, int(expert[1:]))
         if shard == "sg":
-            return self.gate.weight.data[-1].copy_(w.view(-1))
+            return self.gate.weight.data[self.gate.num_experts].copy_(w.view(-1))
         if shard == "down":
             return self.shared.down_proj.weight_loader(self.shared.down_proj.weight, w)
         up = self.shared.gate_up_proj

@@ -189,13 +189,13 @@ def route_by_logit(x, weight, bias, top_k):
     return reference.route_by_logit(x, weight, bias, top_k)
 
 
-def route_by_score(x, weight, correction, top_k, scale, gated: bool = False):
-    """`s = softmax(x weight^T)` (fp32), the `top_k` choices with the largest `s + correction`, weighted by `scale * s`; `gated`:
-    the last row of `weight` is no choice but a gate per token, whose sigmoid comes third (else None)."""
-    if use_native_wide(x) and weight.shape[0] <= 512 and top_k <= 16 and weight.dtype == x.dtype:
+def route_by_score(x, weight, correction, top_k, scale, choices: int, gated: bool = False):
+    """`s = softmax(x weight[:choices]^T)` (fp32), the `top_k` choices with the largest `s + correction`, weighted by `scale * s`;
+    `gated`: the row behind them is a gate per token, whose sigmoid comes third (else None); further rows are padding."""
+    if use_native_wide(x) and choices <= 512 and top_k <= 16 and weight.dtype == x.dtype:
         from . import moe_native
-        return moe_native.route_by_score(x, weight, correction, top_k, scale, gated)
-    return reference.route_by_score(x, weight, correction, top_k, scale, gated)
+        return moe_native.route_by_score(x, weight, correction, top_k, scale, choices, gated)
+    return reference.route_by_score(x, weight, correction, top_k, scale, choices, gated)
 
 
 # ---- latent attention (see `native.latent_prep`)

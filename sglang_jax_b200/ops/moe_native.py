@@ -26,7 +26,7 @@ def _lib():
         L.sglb_route_by_logit.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                                           c_int, c_int, c_void_p]
         L.sglb_route_by_score.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
-                                          c_int, c_int, c_float, c_int, c_void_p]
+                                          c_int, c_int, c_int, c_float, c_int, c_void_p]
         L.sglb_grouped_gemm_any.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                             c_int, c_int, c_int, c_int, c_int, c_void_p]
         L.sglb_grouped_gemm_fp8.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
@@ -225,11 +225,11 @@ def route_by_logit(x, weight, bias, top_k):
     return w, ids
 
 
-def route_by_score(x, weight, correction, top_k, scale, gated: bool = False):
-    """`s = softmax(x weight^T)` in fp32, the `top_k` largest `s + correction` (ties: the lower index) and `scale * s` of
-    those; `gated`: the last row of `weight` is no choice, the sigmoid of its product is returned too (`[T]`, else None)."""
+def route_by_score(x, weight, correction, top_k, scale, choices, gated: bool = False):
+    """`s = softmax(x weight[:choices]^T)` in fp32, the `top_k` largest `s + correction` (ties: the lower index) and `scale * s`
+    of those; `gated`: the sigmoid of the next row's product is returned too (`[T]`, else None)."""
     T, K = x.shape
-    E = weight.shape[0] - gated
+    E = choices
     x = x.contiguous()
     assert weight.is_contiguous() and weight.dtype == x.dtype
     assert correction is None or (correction.dtype == torch.float32 and correction.numel() == E)
@@ -237,11 +237,11 @@ def route_by_score(x, weight, correction, top_k, scale, gated: bool = False):
     ids = torch.empty((T, top_k), dtype=torch.int32, device=x.device)
     gate = torch.empty(T, dtype=torch.float32, device=x.device) if gated else None
     z = None
-    if T > ROUTE_FUSED_TOKENS:
+    if T > ROUTE_FUSED_TOKENS or (K % 8 == 0 and weight.shape[0] % 8 == 0):     # (a split product beats one CTA per token)
         z = torch.mm(x, weight.t()) if x.dtype == torch.float32 else torch.mm(x, weight.t(), out_dtype=torch.float32)
     p = native._p
-    native._check(_lib().sglb_route_by_score(p(z), p(x), p(weight), p(correction), p(w), p(ids), p(gate), T, E, K, top_k,
-                                             float(scale), native._f32(x), native._stream()), "route_by_score")
+    native._check(_lib().sglb_route_by_score(p(z), p(x), p(weight), p(correction), p(w), p(ids), p(gate), T, weight.shape[0], E, K,
+                                             top_k, float(scale), native._f32(x), native._stream()), "route_by_score")
     return w, ids, gate
 
 

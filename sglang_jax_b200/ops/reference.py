@@ -421,10 +421,10 @@ def embed_pair(ids, table, pairs, mul_prev, mul_cur, slot_ids, positions, loc, c
     return x, (x if table.dtype == torch.float32 else x.to(table.dtype))
 
 
-def route_by_score(x, weight, correction, top_k, scale, gated=False):
+def route_by_score(x, weight, correction, top_k, scale, choices, gated=False):
     z = F.linear(x.float(), weight.float())
-    gate = torch.sigmoid(z[:, -1]) if gated else None
-    s = torch.softmax(z[:, :-1] if gated else z, -1)
+    gate = torch.sigmoid(z[:, choices]) if gated else None
+    s = torch.softmax(z[:, :choices], -1)
     ids = (s if correction is None else s + correction).topk(top_k, dim=-1).indices
     return s.gather(1, ids) * scale, ids.to(torch.int32), gate
 

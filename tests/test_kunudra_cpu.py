@@ -87,7 +87,7 @@ def test_router_chooses_by_corrected_score_and_weighs_by_the_score():
     from sglang_jax_b200.layers.gate import GateLogit
     gate = GateLogit(8, 6, torch.float32, correction_bias=True, token_gate=True)
     g = torch.Generator().manual_seed(0)
-    gate.weight.data.copy_(torch.randn(7, 8, generator=g))
+    gate.weight.data[:7] = torch.randn(7, 8, generator=g)
     gate.e_score_correction_bias.data.copy_(torch.randn(6, generator=g) * 0.3)
     x = torch.randn(20, 8, generator=g)
     w = {"router": gate.weight[:6], "correction": gate.e_score_correction_bias}
@@ -97,6 +97,7 @@ def test_router_chooses_by_corrected_score_and_weighs_by_the_score():
         assert torch.equal(ids.long(), want_ids) and torch.allclose(got, want_w, atol=1e-6)
         assert torch.allclose(own, torch.sigmoid(x @ gate.weight[6]), atol=1e-6)
     plain = torch.topk(torch.softmax(x @ w["router"].T, -1), 3).indices
+    assert gate.weight.shape[0] == 8 and not gate.weight[7].any()
     assert not torch.equal(plain, gate.route_by_score(x, 3, 1.0)[1].long())               # the correction matters here
 
 

@@ -121,12 +121,12 @@ def test_gated_activation(native, dtype, F):
 def test_routing_by_score(native, dtype, T, E, k, K):
     from sglang_jax_b200.ops import moe_native
     g = torch.Generator().manual_seed(E + T)
-    x, w = torch.randn(T, K, generator=g).to(dtype), (torch.randn(E + 1, K, generator=g) * 2 * K ** -0.5).to(dtype)
+    x, w = torch.randn(T, K, generator=g).to(dtype), (torch.randn(E + 4, K, generator=g) * 2 * K ** -0.5).to(dtype)
     c = torch.randn(E, generator=g) * 0.05
     for gated in (False, True):
         s = torch.softmax(x.double() @ w[:E].double().T, -1)
         best = torch.topk(s + c.double(), k, -1)
-        weights, ids, gate = moe_native.route_by_score(x.cuda(), (w if gated else w[:E]).cuda(), c.cuda(), k, 1.6, gated)
+        weights, ids, gate = moe_native.route_by_score(x.cuda(), (w if gated else w[:E]).cuda(), c.cuda(), k, 1.6, E, gated)
         chosen = ids.cpu().long()
         assert torch.allclose((s + c.double()).gather(1, chosen), best.values, atol=2e-6)
         assert torch.allclose(weights.cpu().double(), 1.6 * s.gather(1, chosen), atol=2e-6)
@@ -217,14 +217,14 @@ def test_latent_rows_and_queries_from_their_latent(native, H, dim, rot, R, Rq, d
     assert torch.allclose(c_q.cpu().double(), oracle.rms(proj[:, :Rq].double(), 1e-4) * qw.double(), atol=tol, rtol=tol)
     rows = cache.cpu().flatten(0, 1)[loc.long()].double()
     assert torch.allclose(rows[:, :R], oracle.rms(proj[:, at:at + R].double(), 1e-4) * cw.double(), atol=tol, rtol=tol)
-    want = oracle.rotate(proj[:, at + R:at + R + rot].double(), pos, base)
-    assert torch.allclose(rows[:, R:R + rot], want, atol=20 * tol * 1e-1, rtol=tol)
+    want, turned = oracle.rotate(proj[:, at + R:at + R + rot].double(), pos, base), max(tol, 5e-4)      # (fp32 angles)
+    assert torch.allclose(rows[:, R:R + rot], want, atol=turned, rtol=tol)
     q = (torch.randn(T, H * (dim + rot) + 4, generator=g) * 2).to(dtype)
     qc = q.cuda()[:, :H * (dim + rot)].unflatten(-1, (H, dim + rot))
     native.latent_rotate(qc, dim, cs, pos.cuda())
     q = q[:, :H * (dim + rot)].double().unflatten(-1, (H, dim + rot))
     want = torch.cat([q[..., :dim], oracle.rotate(q[..., dim:], pos, base)], -1)
-    assert torch.allclose(qc.cpu().double(), want, atol=tol, rtol=tol)
+    assert torch.allclose(qc.cpu().double(), want, atol=turned, rtol=tol)
 
 
 # ------------------------------------------------------------------ attention
@@ -466,24 +466,24 @@ def _engine(path, dtype, **kw):
                   **{"page_size": 64, "max_total_tokens": 4096, "max_running_requests": 8, "cuda_graph_max_bs": 8, **kw})
 
 
-def _near_greedy(prompt, out, w, cfg, slack):
-    """Every generated token is the oracle's best one, or as good within `slack` of the logits' spread."""
+def _near_greedy(prompt, out, w, cfg, dtype):
+    """Every generated token is the oracle's best one, or nearly as good."""
     logits = oracle.forward(prompt + out, w, cfg)[len(prompt) - 1:-1]
     best = logits.max(-1).values - logits[torch.arange(len(out)), torch.tensor(out)]
-    return bool((best <= slack * logits.std()).all())
+    return bool((best <= (1e-4 if dtype == "float32" else 0.2) * logits.std()).all())
 
 
 @pytest.mark.parametrize("kw", [dict(), dict(disable_cuda_graph=True), dict(chunked_prefill_size=64, enable_mixed_chunk=True)])
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_greedy_generation_through_the_engine(models, dtype, kw):
-    path, cfg, w = models["plain"]
+    path, cfg, w = models["plain" if dtype == "float32" else "dense"]
     prompts = [cases.tokens(n, cfg["vocab"], n) for n in (29, 7, 170, 64, 65)]
     eng = _engine(path, dtype, **kw)
     try:
         got = eng.generate(input_ids=prompts, sampling_params={"max_new_tokens": 12, "temperature": 0, "ignore_eos": True})
         for p, o in zip(prompts, got):
             assert len(o["output_ids"]) == 12
-            assert _near_greedy(p, o["output_ids"], w, cfg, 1e-4 if dtype == "float32" else 0.3)
+            assert _near_greedy(p, o["output_ids"], w, cfg, dtype)
         info = eng.get_server_info()["internal_states"][0]
         assert (info["cuda_graph_replays"] > 5) != bool(kw.get("disable_cuda_graph")) and info["cuda_graph_recaptures"] == 0
         eng.scheduler.check_memory()
@@ -501,6 +501,6 @@ def test_shared_prefixes(models):
         again = base[:128] + cases.tokens(20, cfg["vocab"], 2)
         out = eng.generate(input_ids=again, sampling_params=sp)
         assert out["meta_info"]["cached_tokens"] == 128
-        assert _near_greedy(again, out["output_ids"], w, cfg, 1e-4)
+        assert _near_greedy(again, out["output_ids"], w, cfg, "float32")
     finally:
         eng.shutdown()
