@@ -274,7 +274,7 @@ int route(const float* z, const void* x, const void* w, const void* bias, float*
           int k, int ld, const ScoreRule& rule, cudaStream_t s) {
   const T* b = static_cast<const T*>(bias);
   const int n = rule.logits(E);
-  // one round of the warps over the rows where that is possible
+  // one pass of the warps over the rows where that is possible
   if (z == nullptr)
     return n <= kRouteThreads / 32 * 4 ? route_token<T, 4>(x, w, b, out_w, out_ids, T_, E, K, k, rule, s)
                                        : route_token<T, 8>(x, w, b, out_w, out_ids, T_, E, K, k, rule, s);

@@ -38,13 +38,13 @@ def config(layers, width, vocab, buckets=97, mul_prev=13, mul_cur=5, eps=1e-6, a
 CONFIGS = {
     # sizes that the tensor-core kernels take; two readers of the first values; identity choices and a shared expert
     "plain": config([attention(4, 2, 32, 32, 24, 9.0, True, mlp=moe(48, 6, 2, 2, 1.3, 40)),
-                     latent(4, 32, 16, 32, 64, 48, 24, mlp=dense(160)),
+                     latent(4, 40, 16, 48, 72, 56, 24, mlp=dense(160)),
                      attention(4, 2, 32, 32, 50, 4.0, True, mlp=moe(48, 6, 3, 3, 0.8, 40)),
-                     latent(4, 32, 16, 32, 64, 48, 9, 500.0, mlp=moe(48, 6, 2, 2, 2.0, 24)),
+                     latent(4, 40, 24, 32, 80, 48, 9, 500.0, mlp=moe(48, 6, 2, 2, 2.0, 24)),
                      attention(4, 2, 32, 32, 9, 30.0, True)], 128, 200),
     # no routers, whose choices may hang on a rounding
     "dense": config([attention(6, 2, 64, 64, 70, 5.0, True, mlp=dense(200)), latent(6, 48, 32, 64, 96, 80, 40, 1000.0, mlp=dense(144)),
-                     attention(2, 2, 64, 64, 20, 2.0, True), latent(3, 32, 16, 32, 64, 48, 100, mlp=dense(96))], 192, 150, alpha=2.2),
+                     attention(2, 2, 64, 64, 20, 2.0, True), latent(3, 32, 24, 40, 64, 48, 100, mlp=dense(96))], 192, 150, alpha=2.2),
     # every size another one, values wider or narrower than keys, a layer that keeps its values to itself, no cap, no window, no
     # feed-forward in places, no identity choice, no shared expert, one expert of one, all of all, other hash and constants
     "mixed": config([latent(6, 24, 8, 40, 56, 40, 17, 300.0, mlp=moe(40, 5, 3, 1, 0.7, 32)),

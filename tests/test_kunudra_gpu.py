@@ -202,7 +202,7 @@ def test_norms_over_whole_projections_and_mixed_values(native, D, V, H, G, dtype
 
 
 @pytest.mark.parametrize("dtype", BOTH)
-@pytest.mark.parametrize("H,dim,rot,R,Rq", [(4, 32, 16, 64, 48), (3, 10, 6, 21, 19), (2, 7, 2, 9, 5), (16, 128, 64, 512, 768)])
+@pytest.mark.parametrize("H,dim,rot,R,Rq", [(4, 40, 16, 72, 56), (3, 10, 6, 21, 19), (2, 7, 2, 9, 5), (16, 128, 64, 512, 768)])
 def test_latent_rows_and_queries_from_their_latent(native, H, dim, rot, R, Rq, dtype):
     from sglang_jax_b200.layers.embeddings import get_rope
     g = torch.Generator().manual_seed(R)
